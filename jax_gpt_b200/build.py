@@ -26,6 +26,11 @@ NVCC_FLAGS = [
 ]
 
 
+# Sources whose fp32 instances are exact to rounding: no approximate division, square root, exponential or denormal
+# flush (kernels in them that want the fast intrinsics name them).
+PRECISE_SOURCES = {"serve_kernels.cu", "ssm_kernels.cu", "ssd_scan_sm100.cu"}
+
+
 def _cuda_home() -> str:
     return os.environ.get("CUDA_HOME", "/usr/local/cuda")
 
@@ -72,7 +77,8 @@ def build(verbose: bool = False, force: bool = False, debug: bool = False) -> st
         obj = os.path.join(OBJ, f[:-3] + ".o")
         objs.append(obj)
         if force or _stale(src, obj, hdr_m):
-            jobs.append([nvcc, *NVCC_FLAGS, "-I", CSRC, "-c", src, "-o", obj])
+            flags = [x for x in NVCC_FLAGS if x != "--use_fast_math"] if f in PRECISE_SOURCES else NVCC_FLAGS
+            jobs.append([nvcc, *flags, "-I", CSRC, "-c", src, "-o", obj])
     # host-side bindings
     inc = []
     for p in ce.include_paths():
@@ -93,10 +99,12 @@ def build(verbose: bool = False, force: bool = False, debug: bool = False) -> st
             list(ex.map(_run, jobs))
     if jobs or not os.path.exists(LIB):
         torch_lib = os.path.join(os.path.dirname(torch.__file__), "lib")
-        cmd = ["g++", "-shared", "-o", LIB, *objs, f"-L{torch_lib}", "-lc10", "-lc10_cuda", "-ltorch_cpu",
+        tmp = f"{LIB}.{os.getpid()}.tmp"
+        cmd = ["g++", "-shared", "-o", tmp, *objs, f"-L{torch_lib}", "-lc10", "-lc10_cuda", "-ltorch_cpu",
                "-ltorch_cuda", "-ltorch", f"-L{os.path.join(_cuda_home(), 'lib64')}", "-lcudart", "-lpthread",
                f"-Wl,-rpath,{torch_lib}"]
         _run(cmd)
+        os.replace(tmp, LIB)                      # readers never see a half-written library
         if verbose:
             print(f"[b200 build] linked {LIB}", file=sys.stderr)
     return LIB

@@ -42,6 +42,7 @@ struct FwdArgs {
   int64_t ldo;
   float* lse;
   int* status;
+  const float* sink;        // [H] or nullptr: extra term exp(sink[h]) of the softmax denominator
 };
 
 // D: width of q and k heads; DV: width of v heads (MLA prefill uses 192 / 128).
@@ -298,6 +299,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       if (ok) l += lsum[(half ^ 1) * 128 + r];
     }
     if (ok && qi < a.T) {
+      if (a.sink != nullptr) l += exp2f(a.sink[h] * kLog2e - m);   // m: row maximum in log2 units
       const float inv = (l > 0.f) ? 1.f / l : 0.f;
       __nv_bfloat16* orow = a.out + static_cast<int64_t>(b * a.T + qi) * a.ldo + h * DV + half * DH;
 #pragma unroll
@@ -749,7 +751,7 @@ cudaError_t fwd_launch(const AttnTensors& t, const AttnShape& s, const AttnKvLay
     configured = true;
   }
   FwdArgs a{s.B, s.T, kv.Tk, s.H, s.Hkv, kv.q_pos0, kv.rows_b, kv.rows_h, kv.k_col_h, kv.v_col_h,
-            s.scale * kLog2e, s.causal, out, ldo, lse, status};
+            s.scale * kLog2e, s.causal, out, ldo, lse, status, s.sink};
   dim3 grid(s.H, s.B, (s.T + 127) / 128);
   kernel<<<grid, kThreads, C::kSmem, stream>>>(tq, tk, tv, a);
   return cudaGetLastError();
@@ -808,7 +810,7 @@ cudaError_t launch_attn_fwd_kv(const AttnTensors& t, const AttnShape& s, const A
       const char* e = getenv("B200_ATTN_FWD");
       return e != nullptr && e[0] == '1';
     }();
-    if (!one_tile) return launch_attn_fwd2_d64(t, s, kv, out, ldo, lse, status, stream);
+    if (!one_tile && s.sink == nullptr) return launch_attn_fwd2_d64(t, s, kv, out, ldo, lse, status, stream);
     return fwd_launch<64, 64>(t, s, kv, out, ldo, lse, status, stream);
   }
   if (s.D == 128 && dv == 128) return fwd_launch<128, 128>(t, s, kv, out, ldo, lse, status, stream);

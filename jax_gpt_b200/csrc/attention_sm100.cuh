@@ -20,6 +20,7 @@ struct AttnShape {
   float scale;          // softmax scale (1/sqrt(D) by default)
   int causal;
   int Dv;               // v head width when it differs from D (forward only: 192/128 for MLA); 0 = D
+  const float* sink = nullptr;  // forward: [H] fp32, exp(sink[h]) joins every denominator of head h (no key, no value, not scaled)
 };
 
 // Where the keys and values of (batch b, kv head hkv) live. Token-major activations: K and V are [B*Tk, Hkv*D]

@@ -316,7 +316,7 @@ void adamw_bf16_state(Tensor p, Tensor g, Tensor m, Tensor v, const Tensor& hp, 
 
 // q/k/v: 2-D bf16 views [B*T, H*D] (possibly column slices of one fused buffer).
 void attn_fwd(const Tensor& q, const Tensor& k, const Tensor& v, Tensor out, Tensor lse, int64_t B, int64_t T,
-              int64_t H, int64_t Hkv, int64_t D, double scale, bool causal, int64_t Dv) {
+              int64_t H, int64_t Hkv, int64_t D, double scale, bool causal, int64_t Dv, const c10::optional<Tensor>& sink) {
   c10::cuda::CUDAGuard guard(q.device());
   check_bf16_2d(q, "q");
   check_bf16_2d(k, "k");
@@ -325,6 +325,10 @@ void attn_fwd(const Tensor& q, const Tensor& k, const Tensor& v, Tensor out, Ten
   b200::AttnTensors t{bf16_ptr(q), bf16_ptr(k), bf16_ptr(v), q.stride(0), k.stride(0), v.stride(0)};
   b200::AttnShape s{static_cast<int>(B), static_cast<int>(T), static_cast<int>(H), static_cast<int>(Hkv),
                     static_cast<int>(D), static_cast<float>(scale), causal ? 1 : 0, static_cast<int>(Dv)};
+  if (sink.has_value()) {
+    TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == at::kFloat && sink->numel() == H, "attn_fwd: sink is [H] fp32");
+    s.sink = sink->data_ptr<float>();
+  }
   B200_CHECK_CUDA(b200::launch_attn_fwd(t, s, bf16_mut(out), out.stride(0), lse.data_ptr<float>(), status_ptr(q),
                                         cur_stream()));
 }
@@ -498,6 +502,7 @@ void cast_rows(const Tensor& src, Tensor dst) {
 }  // namespace
 
 #include "bindings_extra.inc"
+#include "bindings_serve.inc"
 
 void b200_register_runtime(torch::Library& m);
 
@@ -539,7 +544,7 @@ TORCH_LIBRARY(b200, m) {
       &adamw);
   m.def(
       "attn_fwd(Tensor q, Tensor k, Tensor v, Tensor(a!) out, Tensor(b!) lse, int B, int T, int H, int Hkv, int D, "
-      "float scale, bool causal, int Dv) -> ()",
+      "float scale, bool causal, int Dv, Tensor? sink=None) -> ()",
       &attn_fwd);
   m.def(
       "attn_bwd(Tensor q, Tensor k, Tensor v, Tensor out, Tensor dout, Tensor lse, Tensor(a!) delta, Tensor(b!) "
@@ -577,5 +582,6 @@ TORCH_LIBRARY(b200, m) {
     return b200::gemm_pair_wanted(a);
   });
   b200_register_extra(m);
+  b200_register_serve(m);
   b200_register_runtime(m);
 }

@@ -95,6 +95,13 @@ _Pragma("unroll") for (int j = 0; j < 32; ++j)
       }
     }
   }
+  if (args.epilogue == kEpiRelu2) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+      const float r = fmaxf(f[j], 0.f);
+      f[j] = r * r;
+    }
+  }
   if (args.residual != nullptr && ks == 0) {
     const __nv_bfloat16* res = args.residual + static_cast<int64_t>(row) * args.ldr + col0;
     if (full && (args.ldr & 7) == 0) {
@@ -179,7 +186,7 @@ __device__ __forceinline__ bool gemm_epilogue_staged_ok(const GemmArgs& args, in
     return false;
   const bool has_res = args.residual != nullptr && ks == 0;
   if (has_res && (args.epilogue == kEpiGeluGrad || (args.ldr & 7) != 0)) return false;
-  if (args.epilogue != kEpiNone && (args.ldaux & 7) != 0) return false;
+  if ((args.epilogue == kEpiGelu || args.epilogue == kEpiGeluGrad) && (args.ldaux & 7) != 0) return false;
   if (args.bias != nullptr && (reinterpret_cast<uintptr_t>(args.bias) & 15) != 0) return false;
   return true;
 }
@@ -250,6 +257,13 @@ __device__ __forceinline__ void gemm_epilogue_group64(const GemmArgs& args, uint
         f[j + 5] += a2.y;
         f[j + 6] += a3.x;
         f[j + 7] += a3.y;
+      }
+    }
+    if (args.epilogue == kEpiRelu2) {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) {
+        const float r = fmaxf(f[j], 0.f);
+        f[j] = r * r;
       }
     }
 #pragma unroll

@@ -12,6 +12,7 @@ enum GemmEpilogue : int {
   kEpiGelu = 1,      // pre = acc + bias; aux_out = pre; out = gelu_tanh(pre)
   kEpiGeluGrad = 2,  // out = acc * gelu_tanh'(aux_in)
   kEpiSiluMul = 3,   // reserved for SwiGLU-style epilogues
+  kEpiRelu2 = 4,     // out = max(acc + bias, 0)^2
 };
 enum GemmOut : int {
   kOutBf16 = 0,       // store bf16

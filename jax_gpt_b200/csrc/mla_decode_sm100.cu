@@ -373,15 +373,17 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap t_pool, const __grid_const
   }
 }
 
-// out[b, h, :] = sum_s w_s part[b, s, h, :] / sum_s w_s,  w_s = 2^(lse_s - max lse)
+// out[b, h, :] = sum_s w_s part[b, s, h, :] / (sum_s w_s + sink term),  w_s = 2^(lse_s - max lse)
 __global__ void mla_merge_kernel(const float* __restrict__ part_out, const float* __restrict__ part_lse,
-                                 __nv_bfloat16* __restrict__ out, int heads, int n_splits) {
+                                 __nv_bfloat16* __restrict__ out, int heads, int n_splits,
+                                 const float* __restrict__ sink) {
   const int bh = blockIdx.x;  // b * heads + h
   const int b = bh / heads, h = bh % heads;
-  float mx = -INFINITY;
+  const float sk = sink != nullptr ? sink[h] * 1.4426950408889634f : -INFINITY;
+  float mx = sk;
   for (int s = 0; s < n_splits; ++s) mx = fmaxf(mx, part_lse[(static_cast<int64_t>(b) * n_splits + s) * heads + h]);
   float acc[4] = {0.f, 0.f, 0.f, 0.f};
-  float wsum = 0.f;
+  float wsum = sk != -INFINITY ? exp2f(sk - mx) : 0.f;
   for (int s = 0; s < n_splits; ++s) {
     const int64_t idx = (static_cast<int64_t>(b) * n_splits + s) * heads + h;
     const float lse = part_lse[idx];
@@ -451,7 +453,7 @@ cudaError_t launch_mla_paged_decode(const __nv_bfloat16* q, const __nv_bfloat16*
   e = hpc == 16 ? launch_decode_t<16>(t_pool, t_q, a2, stream) : launch_decode_t<32>(t_pool, t_q, a2, stream);
   if (e != cudaSuccess) return e;
   mla_merge_kernel<<<args.batch * args.heads, kMlaLatent / 4, 0, stream>>>(args.part_out, args.part_lse, out, args.heads,
-                                                                          2 * args.n_splits);
+                                                                          2 * args.n_splits, args.sink);
   return cudaGetLastError();
 }
 

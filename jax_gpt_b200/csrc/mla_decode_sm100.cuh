@@ -24,6 +24,7 @@ struct MlaDecodeArgs {
   float* part_out;                // [batch, 2 * n_splits, heads, 512] normalised partials (two softmax groups per split)
   float* part_lse;                // [batch, 2 * n_splits, heads] log2-sum-exp of each partial (-inf when empty)
   int* status;
+  const float* sink = nullptr;    // [heads] fp32 or nullptr: exp(sink[h]) joins the softmax denominator of head h
 };
 
 // q [batch * heads, 576] bf16 (absorbed nope part | rotated rope part); pool: one layer of the page pool,

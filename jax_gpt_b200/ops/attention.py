@@ -44,8 +44,9 @@ def _as2d(t):
     return t.as_strided((B * T, H * D), (t.stride(1), 1))
 
 
-def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None):
-    """Raw CUDA forward. Returns (out [B,T,H,D] bf16, lse [B,H,T] fp32 in log2 units)."""
+def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None, sink=None):
+    """Raw CUDA forward. Returns (out [B,T,H,D] bf16, lse [B,H,T] fp32 in log2 units). ``sink`` (H,) fp32 adds
+    exp(sink) to every softmax denominator of its head (and to lse)."""
     B, T, H, D = q.shape
     Hkv, Dv = k.shape[2], v.shape[3]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -53,7 +54,7 @@ def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None):
         out = torch.empty(B, T, H, Dv, device=q.device, dtype=torch.bfloat16)
     if lse is None:
         lse = torch.empty(B, H, T, device=q.device, dtype=torch.float32)
-    _ext.ops().attn_fwd(_as2d(q), _as2d(k), _as2d(v), _as2d(out), lse, B, T, H, Hkv, D, scale, causal, Dv)
+    _ext.ops().attn_fwd(_as2d(q), _as2d(k), _as2d(v), _as2d(out), lse, B, T, H, Hkv, D, scale, causal, Dv, sink)
     return out, lse
 
 

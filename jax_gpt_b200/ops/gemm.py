@@ -14,7 +14,7 @@ import torch
 
 from .. import _ext
 
-EPI_NONE, EPI_GELU, EPI_GELU_GRAD = 0, 1, 2
+EPI_NONE, EPI_GELU, EPI_GELU_GRAD, EPI_RELU2 = 0, 1, 2, 4
 OUT_BF16, OUT_F32, OUT_F32_ATOMIC = 0, 1, 2
 
 
@@ -44,6 +44,8 @@ def gemm_ref(a, b, *, a_mn_major=False, b_mn_major=False, out=None, bias=None, r
         acc = gelu_tanh(pre.float())
     elif epilogue == EPI_GELU_GRAD:
         acc = acc * gelu_tanh_grad(aux.float())
+    elif epilogue == EPI_RELU2:
+        acc = acc.clamp_min(0).square()
     if residual is not None:
         acc = acc + residual.float()
     if out is None:
@@ -114,6 +116,35 @@ def linear_f32out(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
             and w.shape[0] % 8 == 0 and w.is_contiguous()):
         return _LinearF32OutFn.apply(x, w)
     return x.float() @ w.float()
+
+
+ROWS_KERNEL_MAX = 8      # rows up to which a linear layer streams its weights through the few-row kernel
+
+
+def linear_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *, act: Optional[str] = None,
+                accumulate: bool = False, f32_out: bool = False) -> torch.Tensor:
+    """Inference linear layer with ``w`` stored (out, in) as checkpoints have it: ``act(x @ w.T)``; ``act`` is None or
+    "relu2" (the square of relu). ``accumulate`` adds into ``out`` (fp32: a 32-bit residual), ``f32_out`` returns fp32.
+    x (M, in), bf16 or fp32, unit inner stride. On CUDA up to ``ROWS_KERNEL_MAX`` rows run on the few-row kernel
+    (weights streamed once), more rows on the tcgen05 GEMM in bf16 and on the library's fp32 GEMM in fp32."""
+    M, N = x.shape[0], w.shape[0]
+    if out is None:
+        assert not accumulate
+        out = torch.empty(M, N, device=x.device, dtype=torch.float32 if f32_out else x.dtype)
+    mode = 2 if accumulate else (1 if out.dtype == torch.float32 and x.dtype != torch.float32 else 0)
+    if x.is_cuda and M <= ROWS_KERNEL_MAX:
+        _ext.ops().rows_linear(x, w, out, 1 if act == "relu2" else 0, mode)
+        return out
+    if x.is_cuda and x.dtype == torch.bfloat16 and w.shape[1] % 8 == 0 and w.stride(0) % 8 == 0 and w.data_ptr() % 16 == 0:
+        if x.stride(0) % 8 != 0 or x.data_ptr() % 16 != 0:
+            x = x.contiguous()
+        if act is None or mode == 0:
+            return gemm(x, w, out=out, epilogue=EPI_RELU2 if act == "relu2" else EPI_NONE,
+                        out_mode=(OUT_BF16, OUT_F32, OUT_F32_ATOMIC)[mode])
+    y = x @ w.t() if mode == 0 else x.float() @ w.float().t()
+    if act == "relu2":
+        y = y.clamp_min(0).square()
+    return out.add_(y) if accumulate else out.copy_(y)
 
 
 class _LinearFn(torch.autograd.Function):

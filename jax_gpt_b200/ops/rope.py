@@ -62,3 +62,42 @@ def rmsnorm_rope(x, norm_w, freqs, rope_dim: int, pos0: int = 0, eps: float = 1e
     y = torch.empty_like(xc)
     _ext.ops().rmsnorm_rope(xc, norm_w, freqs.contiguous() if freqs is not None else None, y, T, rope_dim, pos0, eps, one_plus)
     return y.view(B, T, H, dh)
+
+
+# ---- interleaved rotation with optional YaRN scaling ---------------------------------------------------------------
+def yarn_frequencies(dims: int, base: float, scaling=None):
+    """(frequencies [dims / 2] as Python floats, factor of cos and sin). ``scaling`` is None or a mapping with
+    ``factor``, ``original``, ``fast``, ``slow``: pairs that turn more than ``fast`` times over ``original`` positions
+    keep their frequency, pairs that turn fewer than ``slow`` times are slowed by ``factor``, a linear ramp in between
+    (Peng et al., "YaRN: Efficient Context Window Extension of Large Language Models")."""
+    import math
+    freqs = [base ** (-2.0 * i / dims) for i in range(dims // 2)]
+    if not scaling:
+        return freqs, 1.0
+    factor = float(scaling["factor"])
+    edge = lambda turns: dims * math.log(scaling["original"] / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo = max(math.floor(edge(scaling["fast"])), 0)
+    hi = min(math.ceil(edge(scaling["slow"])), dims - 1)
+    width = max(hi - lo, 0.001)
+    ramp = [min(max((i - lo) / width, 0.0), 1.0) for i in range(dims // 2)]
+    return [f / factor * r + f * (1.0 - r) for f, r in zip(freqs, ramp)], 0.1 * math.log(factor) + 1.0
+
+
+def rope_tables(dims: int, base: float, n_pos: int, scaling=None, device="cpu"):
+    """(cos, sin) [n_pos, dims / 2] fp32 with the YaRN amplitude folded in; angles are taken in fp64 before rounding."""
+    freqs, amp = yarn_frequencies(dims, base, scaling)
+    ang = torch.arange(n_pos, dtype=torch.float64)[:, None] * torch.tensor(freqs, dtype=torch.float64)[None, :]
+    return (ang.cos() * amp).float().to(device).contiguous(), (ang.sin() * amp).float().to(device).contiguous()
+
+
+def rotate_interleaved(x: torch.Tensor, pos: torch.Tensor, tables) -> torch.Tensor:
+    """x (N, ..., d): the first ``dims`` features turn in pairs (2i, 2i + 1) by the angles of position ``pos[n]``."""
+    cos, sin = tables
+    dims = 2 * cos.shape[1]
+    if dims == 0:
+        return x
+    shape = [x.shape[0]] + [1] * (x.dim() - 2) + [dims // 2]
+    c, s = cos[pos.long()].reshape(shape), sin[pos.long()].reshape(shape)
+    u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+    turned = torch.stack([u * c - v * s, v * c + u * s], dim=-1).flatten(-2)
+    return torch.cat([turned, x[..., dims:]], dim=-1)
