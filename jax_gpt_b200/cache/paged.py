@@ -15,7 +15,7 @@ by the ``paged_kv_write`` kernel and read by the paged decode kernel (csrc/mla_d
 """
 from __future__ import annotations
 
-from typing import List, Optional
+from typing import List, Optional, Sequence, Union
 
 import torch
 
@@ -125,14 +125,22 @@ class _NativeTable:
 
 
 class PagedCache:
-    """``pool``: (n_layers, n_pages, page_size, width). ``block_table``: (max_seqs, max_pages_per_seq)
+    """``pool``: (n_layers, n_pages, page_size, width), or with ``width`` a sequence of ``n_layers`` widths a list of
+    (n_pages, page_size, width) pools, one per layer. ``block_table``: (max_seqs, max_pages_per_seq)
     int32 page ids (-1 = unassigned). ``seq_lens``: (max_seqs,) int32 tokens stored per sequence."""
 
-    def __init__(self, n_layers: int, width: int, n_pages: int, page_size: int = 64, max_seqs: int = 64,
+    def __init__(self, n_layers: int, width: Union[int, Sequence[int]], n_pages: int, page_size: int = 64, max_seqs: int = 64,
                  max_pages_per_seq: int = 64, dtype=torch.bfloat16, device="cpu", native: Optional[bool] = None):
-        self.page_size, self.width, self.n_layers = page_size, width, n_layers
+        self.page_size, self.n_layers, self.dtype = page_size, n_layers, dtype
         self.device = torch.device(device)
-        self.pool = torch.zeros(n_layers, n_pages, page_size, width, dtype=dtype, device=device)
+        if isinstance(width, int):
+            self.widths = [width] * n_layers
+            self.pool = torch.zeros(n_layers, n_pages, page_size, width, dtype=dtype, device=device)
+        else:
+            self.widths = [int(w) for w in width]
+            assert len(self.widths) == n_layers, "one width per layer"
+            self.pool = [torch.zeros(n_pages, page_size, w, dtype=dtype, device=device) for w in self.widths]
+        self.width = width
         on_gpu = self.device.type == "cuda"
         ops = None
         if native is not False:
@@ -197,14 +205,14 @@ class PagedCache:
         starts = [self._tab.length(s) for s in seq_ids]
         self._tab.reserve(seq_ids, [s + T for s in starts])
         self._sync()
-        if rows.is_cuda and self.pool.dtype == torch.bfloat16 and self.width % 8 == 0:
+        if rows.is_cuda and self.dtype == torch.bfloat16 and self.widths[layer] % 8 == 0:
             ids = self.seq_id_tensor(seq_ids)
             start = self.seq_lens[ids.long()]   # device lengths equal the host ones after _sync
             self._ops.paged_kv_write(rows.to(torch.bfloat16).contiguous(), self.pool[layer], self.block_table, ids, start)
         else:
             for b, sid in enumerate(seq_ids):
                 pages, offs = self.slots(sid, starts[b], T)
-                self.pool[layer, pages, offs] = rows[b].to(self.pool.dtype)
+                self.pool[layer][pages, offs] = rows[b].to(self.dtype)
         if commit:
             self.commit(seq_ids, T)
 
@@ -212,11 +220,25 @@ class PagedCache:
         self._tab.advance(list(seq_ids), n_new)
         self._sync()
 
+    def begin_step(self, seq_ids, n_new) -> None:
+        """Reserves pages for ``n_new[i]`` more tokens of every listed sequence and uploads what changed. For steps
+        whose kernels write the rows and advance ``seq_lens`` on the device; ``end_step`` mirrors that on the host."""
+        self._tab.reserve(list(seq_ids), [self._tab.length(s) + n for s, n in zip(seq_ids, n_new)])
+        self._sync()
+
+    def end_step(self, seq_ids, n_new) -> None:
+        by_n = {}
+        for s, n in zip(seq_ids, n_new):
+            by_n.setdefault(int(n), []).append(s)
+        for n, ids in by_n.items():
+            self._tab.advance(ids, n)
+        self._synced = self._tab.version          # the device lengths were advanced by the step itself
+
     def gather(self, layer: int, seq_id: int, length: Optional[int] = None) -> torch.Tensor:
         """Dense (length, width) view of one sequence (reference path and tests)."""
         length = self._tab.length(seq_id) if length is None else length
         pages, offs = self.slots(seq_id, 0, length)
-        return self.pool[layer, pages, offs]
+        return self.pool[layer][pages, offs]
 
     def length(self, seq_id: int) -> int:
         return self._tab.length(seq_id)
