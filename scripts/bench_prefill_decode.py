@@ -9,7 +9,7 @@ that fits (doubling then bisection on out-of-memory, ``--max-batch`` caps it), t
 
 Timing is on the device with CUDA events, maximum over ranks (the reference uses host
 perf_counter and means only, scripts/bench_prefill_decode.py:246-264). ``--model`` selects the
-Qwen3.5 hybrid (``--config`` preset) or the DeepSeek-V3 shape with its paged latent cache.
+Qwen3.5 hybrid (``--config`` preset), the DeepSeek-V3 shape with its paged latent cache or Vobunex on its step engine.
 Results are printed and written as JSON to ``--out``.
 """
 from __future__ import annotations
@@ -19,7 +19,7 @@ import json
 import statistics
 import time
 
-from utils import fake_quant_w8a8, init_distributed, load_hf_dir, make_tp_dp_groups, qwen_config
+from utils import fake_quant_w8a8, init_distributed, load_hf_dir, make_tp_dp_groups, qwen_config, vobunex_config
 
 import torch
 
@@ -118,6 +118,32 @@ def make_runner(args, device):
             logits, cache = forward(params, nxt[:, None], cfg, cache=cache, is_decode=True, ep_group=ep, tp_group=tp_group)
             return logits[:, -1].argmax(-1), cache
         return prefill, decode, cfg
+    if args.model == "vobunex":
+        if args.tp > 1 or args.dp > 1 or args.w8a8 or args.fp8:
+            raise SystemExit("--tp / --dp / --w8a8 / --fp8 do not apply to --model vobunex")
+        from jax_gpt_b200.models.registry import load_model
+        from jax_gpt_b200.models.vobunex import VobunexEngine, init_params, make_cache
+        if args.model_dir and not args.random_weights:
+            _, cfg, params = load_model(args.model_dir, dtype, device)
+        else:
+            cfg = vobunex_config(args.config if args.config != "mini" else "serving")
+            params = init_params(cfg, 0, dtype=dtype, device=device, on_device=device.type == "cuda")
+        plen, dlen = SCENARIOS[args.scenario]
+        live = {}
+
+        def prefill(B):
+            live.clear()
+            per = (plen + dlen + cfg.page_size - 1) // cfg.page_size
+            eng = VobunexEngine(params, cfg, make_cache(cfg, B * per, B, per, dtype, device), use_cuda_graph=not args.no_graph)
+            gen = torch.Generator().manual_seed(1234)
+            tok = torch.randint(0, cfg.vocab_size, (B, plen), generator=gen)
+            live["eng"] = eng
+            return eng.step(list(range(B)), tok.tolist()).argmax(-1), eng
+
+        def decode(state):
+            nxt, eng = state
+            return eng.decode(list(range(nxt.shape[0])), nxt).argmax(-1), eng
+        return prefill, decode, cfg
     if args.tp > 1 or args.dp > 1 or args.model_dir or args.w8a8:
         raise SystemExit("--tp / --dp / --sharding / --model-dir / --w8a8 apply to --model qwen35; the DeepSeek-V3 shape "
                          "runs data-parallel attention with expert-parallel MoE over all ranks of the launch")
@@ -195,7 +221,7 @@ def find_max_batch(prefill, decode, cap):
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--model", default="qwen35", choices=["qwen35", "deepseek_v3"])
+    ap.add_argument("--model", default="qwen35", choices=["qwen35", "deepseek_v3", "vobunex"])
     ap.add_argument("--model-dir", default="", help="HF safetensors directory (random weights when empty)")
     ap.add_argument("--scenario", default="1k1k", choices=sorted(SCENARIOS))
     ap.add_argument("--tp", type=int, default=1)

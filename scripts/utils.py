@@ -50,39 +50,12 @@ def make_tp_dp_groups(tp: int, dp: int):
 
 
 def load_hf_dir(model_dir: str):
-    """All ``*.safetensors`` shards of a Hugging Face directory as one lazy name -> tensor mapping."""
-    import glob
-    from safetensors import safe_open
-    files = sorted(glob.glob(os.path.join(model_dir, "*.safetensors")))
-    if not files:
-        raise SystemExit(f"no *.safetensors files in {model_dir}")
-
-    class _Lazy(dict):
-        def __init__(self):
-            super().__init__()
-            self._where = {}
-            self._open = {}
-            for f in files:
-                h = safe_open(f, framework="pt", device="cpu")
-                self._open[f] = h
-                for k in h.keys():
-                    self._where[k] = f
-
-        def __contains__(self, k):
-            return k in self._where
-
-        def keys(self):
-            return self._where.keys()
-
-        def __iter__(self):
-            return iter(self._where)
-
-        def __len__(self):
-            return len(self._where)
-
-        def __getitem__(self, k):
-            return self._open[self._where[k]].get_tensor(k)
-    return _Lazy()
+    """All ``*.safetensors`` shards of a model folder as one lazy name -> tensor mapping."""
+    from jax_gpt_b200.utils.safetensors_dir import SafetensorsDir
+    try:
+        return SafetensorsDir(model_dir)
+    except FileNotFoundError as e:
+        raise SystemExit(str(e)) from None
 
 
 def fake_quant_w8a8(params):
@@ -110,6 +83,12 @@ def qwen_config(name: str):
     from jax_gpt_b200.models.qwen35 import Qwen35Config
     return {"mini": Qwen35Config.mini, "mid": Qwen35Config.mid, "mid_large": Qwen35Config.mid_large,
             "full": Qwen35Config.full, "ns": Qwen35Config.ns, "tiny": Qwen35Config.tiny}[name]()
+
+
+def vobunex_config(name: str):
+    from jax_gpt_b200.models.vobunex import VobunexConfig
+    return {"tiny": VobunexConfig.tiny, "serving": VobunexConfig.serving,
+            "serving_wide": lambda: VobunexConfig.serving(width=4096, heads=32, ff=1536)}[name]()
 
 
 class ByteTokenizer:
