@@ -158,6 +158,17 @@ class ClockSampler:
                 "reasons": sorted(reasons), "samples": len(sm), "power_w_max": max(power) if power else None}
 
 
+def serve_bench(args) -> int:
+    """One JSON line with the serving tables (utils/serve_bench.py), clocks sampled meanwhile."""
+    from jax_gpt_b200.utils.serve_bench import run
+    sampler = ClockSampler(0)
+    sampler.start()
+    res = run(args.serve_part)
+    res["clocks"] = sampler.stop()
+    print(json.dumps({"bench": "serve", "n_gpus": 1, **res}), flush=True)
+    return 0
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -175,12 +186,17 @@ def main():
     ap.add_argument("--no-extra", action="store_true",
                     help="2+ GPUs: skip the expert-parallel extras (fused EP-MoE layer, Qwen3.5-style MoE training step)")
     ap.add_argument("--extra-budget-s", type=float, default=420.0, help="wall-clock limit of the extras; past it the line is printed without them")
+    ap.add_argument("--serve", action="store_true",
+                    help="instead of the training benchmark: prefill / decode throughput and kernel rooflines of Vobunex beside the closest families")
+    ap.add_argument("--serve-part", default="all", choices=["kernels", "models", "all"])
     ap.add_argument("--extras-child", default="", help=argparse.SUPPRESS)   # internal: run only the extras, write them to this file
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)
     if args.extras_child:
         return extras_child(args.extras_child)
+    if args.serve:
+        return serve_bench(args)
 
     import torch
     import torch.distributed as dist
