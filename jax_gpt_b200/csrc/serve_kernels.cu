@@ -84,6 +84,65 @@ __global__ void norm_rows_kernel(int mode, const float* __restrict__ x, const fl
   }
 }
 
+// The same with the row in registers: D a multiple of 4, at most 1024 * kIt; a warp per row up to 1024, else a block.
+template <typename TO, int kIt, int kThr>
+__global__ void __launch_bounds__(256)
+norm_rows_vec_kernel(int mode, const float* __restrict__ x, const float* __restrict__ gamma, const float* __restrict__ beta,
+                     TO* __restrict__ out, int rows, int D, float eps) {
+  __shared__ float red[33];
+  constexpr int kPer = 256 / kThr;   // rows per block
+  const int row = blockIdx.x * kPer + threadIdx.x / kThr, t = threadIdx.x % kThr;
+  if (kThr == 32 && row >= rows) return;
+  auto total = [&](float v) { return kThr == 32 ? warp_sum(v) : block_sum(v, red); };
+  const float* xr = x + static_cast<int64_t>(row) * D;
+  float4 v[kIt];
+  float s = 0.f;
+#pragma unroll
+  for (int k = 0; k < kIt; ++k) {
+    const int i = (k * kThr + t) * 4;
+    v[k] = i < D ? *reinterpret_cast<const float4*>(xr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    s += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+  }
+  const float mu = mode == 0 ? total(s) / D : 0.f;
+  float q = 0.f;
+#pragma unroll
+  for (int k = 0; k < kIt; ++k) {
+    if ((k * kThr + t) * 4 < D) {
+      v[k].x -= mu; v[k].y -= mu; v[k].z -= mu; v[k].w -= mu;
+      q += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+    }
+  }
+  const float inv = 1.f / sqrtf(total(q) / D + eps);
+  TO* o = out + static_cast<int64_t>(row) * D;
+#pragma unroll
+  for (int k = 0; k < kIt; ++k) {
+    const int i = (k * kThr + t) * 4;
+    if (i < D) {
+      const float4 g = *reinterpret_cast<const float4*>(gamma + i);
+      float4 r = make_float4(v[k].x * inv * g.x, v[k].y * inv * g.y, v[k].z * inv * g.z, v[k].w * inv * g.w);
+      if (mode == 0 && beta != nullptr) {
+        const float4 b = *reinterpret_cast<const float4*>(beta + i);
+        r.x += b.x; r.y += b.y; r.z += b.z; r.w += b.w;
+      }
+      if constexpr (sizeof(TO) == 2) *reinterpret_cast<uint2*>(o + i) = make_uint2(pack_bf16x2(r.x, r.y), pack_bf16x2(r.z, r.w));
+      else *reinterpret_cast<float4*>(o + i) = r;
+    }
+  }
+}
+
+template <typename TO>
+void norm_rows_go(int mode, const float* x, const float* gamma, const float* beta, TO* out, int rows, int D, float eps,
+                  cudaStream_t st) {
+  const bool vec = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gamma) |
+                                   reinterpret_cast<uintptr_t>(beta) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+  if (vec && D <= 512 && rows >= 64) norm_rows_vec_kernel<TO, 4, 32><<<(rows + 7) / 8, 256, 0, st>>>(mode, x, gamma, beta, out, rows, D, eps);
+  else if (vec && D <= 1024) norm_rows_vec_kernel<TO, 1, 256><<<rows, 256, 0, st>>>(mode, x, gamma, beta, out, rows, D, eps);
+  else if (vec && D <= 2048) norm_rows_vec_kernel<TO, 2, 256><<<rows, 256, 0, st>>>(mode, x, gamma, beta, out, rows, D, eps);
+  else if (vec && D <= 4096) norm_rows_vec_kernel<TO, 4, 256><<<rows, 256, 0, st>>>(mode, x, gamma, beta, out, rows, D, eps);
+  else if (vec && D <= 8192) norm_rows_vec_kernel<TO, 8, 256><<<rows, 256, 0, st>>>(mode, x, gamma, beta, out, rows, D, eps);
+  else norm_rows_kernel<TO><<<rows, D >= 1024 ? 256 : (D >= 256 ? 128 : 64), 0, st>>>(mode, x, gamma, beta, out, D, eps);
+}
+
 // ---- few-row linear ------------------------------------------------------------------------------------------------
 constexpr int kLinWarps = 8;
 
@@ -169,6 +228,85 @@ void rows_linear_go(bool vec, const T* x, int64_t ldx, const T* w, int64_t ldw, 
     rows_linear_kernel<T, MR, NR, false><<<grid, kLinWarps * 32, 0, st>>>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode);
 }
 
+// bf16, up to 8 * MT rows: weights are the A operand of mma.sync m16n8k16 (16 output features), activation rows the B
+// operand. Every lane loads 16 contiguous bytes of a weight row and of an activation row; the products' k index is
+// permuted the same way on both sides, which leaves the sums unchanged. The warps of a block split the contraction.
+// Bound by the stream of weights: tcgen05 tiles would be 94 % padding here.
+__device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                          uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int MT, int kW>   // kW warps per block
+__global__ void __launch_bounds__(kW * 32)
+rows_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx, const __nv_bfloat16* __restrict__ w, int64_t ldw,
+                       void* __restrict__ y, int64_t ldy, int M, int N, int K, int act, int out_mode) {
+  __shared__ float red[kW][MT][32][4];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int n0 = blockIdx.x * 16;
+  const __nv_bfloat16* w0 = w + static_cast<int64_t>(min(n0 + g, N - 1)) * ldw;
+  const __nv_bfloat16* w1 = w + static_cast<int64_t>(min(n0 + g + 8, N - 1)) * ldw;
+  const __nv_bfloat16* xr[MT];
+#pragma unroll
+  for (int m = 0; m < MT; ++m) xr[m] = x + static_cast<int64_t>(min(m * 8 + g, M - 1)) * ldx;
+  float acc[MT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[m][j] = 0.f;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  constexpr int kU = MT == 1 ? 4 : 2;
+  for (int kb = warp * 32; kb < K; kb += kW * 32 * kU) {
+    uint4 a[kU], c[kU], b[kU][MT];
+#pragma unroll
+    for (int u = 0; u < kU; ++u) {
+      const int k = kb + u * kW * 32 + t * 8;
+      const bool in = k < K;   // K is a multiple of 8
+      a[u] = in ? __ldg(reinterpret_cast<const uint4*>(w0 + k)) : zero;
+      c[u] = in ? __ldg(reinterpret_cast<const uint4*>(w1 + k)) : zero;
+#pragma unroll
+      for (int m = 0; m < MT; ++m) b[u][m] = in ? __ldg(reinterpret_cast<const uint4*>(xr[m] + k)) : zero;
+    }
+#pragma unroll
+    for (int u = 0; u < kU; ++u)
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        mma_16816(acc[m], a[u].x, c[u].x, a[u].y, c[u].y, b[u][m].x, b[u][m].y);
+        mma_16816(acc[m], a[u].z, c[u].z, a[u].w, c[u].w, b[u][m].z, b[u][m].w);
+      }
+  }
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) red[warp][m][lane][j] = acc[m][j];
+  __syncthreads();
+  // accumulator j of lane (g, t): feature g + 8 * (j / 2), row 2 t + j % 2
+  for (int i = threadIdx.x; i < MT * 128; i += kW * 32) {
+    const int m = i / 128, f = i % 16, r = (i / 16) % 8;
+    const int src = (f % 8) * 4 + r / 2, j = (f / 8) * 2 + r % 2;
+    float v = 0.f;
+#pragma unroll
+    for (int q = 0; q < kW; ++q) v += red[q][m][src][j];
+    if (m * 8 + r < M && n0 + f < N) {
+      v = row_act(v, act);
+      const int64_t o = static_cast<int64_t>(m * 8 + r) * ldy + n0 + f;
+      if (out_mode == 0) static_cast<__nv_bfloat16*>(y)[o] = __float2bfloat16(v);
+      else if (out_mode == 1) static_cast<float*>(y)[o] = v;
+      else static_cast<float*>(y)[o] += v;
+    }
+  }
+}
+
+template <int MT>
+void rows_linear_mma_go(const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16* w, int64_t ldw, void* y, int64_t ldy, int M,
+                        int N, int K, int act, int out_mode, cudaStream_t st) {
+  const int grid = (N + 15) / 16;   // wide outputs: small blocks, so that all of them are resident at once
+  if (grid >= 296) rows_linear_mma_kernel<MT, 4><<<grid, 128, 0, st>>>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode);
+  else rows_linear_mma_kernel<MT, 8><<<grid, 256, 0, st>>>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode);
+}
+
 template <typename T>
 cudaError_t rows_linear_t(const void* x, int64_t ldx, const void* w, int64_t ldw, void* y, int64_t ldy, int M, int N, int K,
                           int act, int out_mode, cudaStream_t st) {
@@ -177,6 +315,14 @@ cudaError_t rows_linear_t(const void* x, int64_t ldx, const void* w, int64_t ldw
   const T* xt = static_cast<const T*>(x);
   const T* wt = static_cast<const T*>(w);
   // narrow outputs take fewer features per warp so that the grid still covers the SMs
+  if constexpr (sizeof(T) == 2) {
+    if (vec && M > 1 && M <= 32) {
+      if (M <= 8) rows_linear_mma_go<1>(xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st);
+      else if (M <= 16) rows_linear_mma_go<2>(xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st);
+      else rows_linear_mma_go<4>(xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st);
+      return cudaGetLastError();
+    }
+  }
   const bool wide = N >= 148 * kLinWarps * 4;
 #define B200_GO(MR)                                                                                       \
   (wide ? rows_linear_go<T, MR, 4>(vec, xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st)             \
@@ -279,30 +425,77 @@ __global__ void mla_rope_qk_kernel(const SeqBatch sb, T* __restrict__ q, const T
   }
 }
 
-constexpr int kAbsTok = 8;   // tokens per block of the absorption kernels
+constexpr int kAbsTok = 8;    // tokens per block of the absorption kernels
+constexpr int kAbsCols = 64;  // latent columns per block of the query absorption
 
-template <typename T>
-__global__ void mla_absorb_q_kernel(const SeqBatch sb, const T* __restrict__ q, const T* __restrict__ w_uk,
-                                    T* __restrict__ qf, int H, int dn, int dr, int R, const RopeTable rope) {
-  extern __shared__ float sm[];   // [kAbsTok][dn + dr]
+// Block: 8 tokens, one head, 64 columns. Lanes 0..7 of every eight own eight columns each, the other lane bits and
+// the warps split the contraction over dn; partial sums meet in shuffles and in shared memory.
+template <typename T, bool kVec>
+__global__ void __launch_bounds__(256)
+mla_absorb_q_kernel(const SeqBatch sb, const T* __restrict__ q, const T* __restrict__ w_uk, T* __restrict__ qf, int H, int dn,
+                    int dr, int R, const RopeTable rope) {
+  extern __shared__ float sm[];   // [kAbsTok][dn + dr], then [8 warps][kAbsTok][kAbsCols]
   const int D = dn + dr, h = blockIdx.y, n0 = blockIdx.x * kAbsTok;
+  float* red = sm + kAbsTok * D;
   const int cnt = min(kAbsTok, sb.n_tok - n0);
-  for (int i = threadIdx.x; i < cnt * D; i += blockDim.x)
-    sm[i] = ldf(q + (static_cast<int64_t>(n0 + i / D) * H + h) * D + i % D);
-  for (int i = threadIdx.x + cnt * D; i < kAbsTok * D; i += blockDim.x) sm[i] = 0.f;
+  for (int i = threadIdx.x; i < kAbsTok * D; i += blockDim.x)
+    sm[i] = i < cnt * D ? ldf(q + (static_cast<int64_t>(n0 + i / D) * H + h) * D + i % D) : 0.f;
   __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int c0 = blockIdx.z * kAbsCols + (lane & 7) * 8, dg = warp * 4 + (lane >> 3);   // 32 slices of dn
   const T* w = w_uk + static_cast<int64_t>(h) * dn * R;
-  for (int r = blockIdx.z * blockDim.x + threadIdx.x; r < R; r += gridDim.z * blockDim.x) {
-    float acc[kAbsTok];
+  float acc[kAbsTok][8];
 #pragma unroll
-    for (int t = 0; t < kAbsTok; ++t) acc[t] = 0.f;
-#pragma unroll 4
-    for (int d = 0; d < dn; ++d) {
-      const float wv = ldf(w + static_cast<int64_t>(d) * R + r);
+  for (int t = 0; t < kAbsTok; ++t)
 #pragma unroll
-      for (int t = 0; t < kAbsTok; ++t) acc[t] = fmaf(sm[t * D + d], wv, acc[t]);
+    for (int j = 0; j < 8; ++j) acc[t][j] = 0.f;
+#pragma unroll 2
+  for (int d = dg; d < dn; d += 32) {
+    float wv[8];
+    if constexpr (kVec) {
+      if (c0 < R) {
+        if constexpr (sizeof(T) == 2) {
+          Vec16<T>::load(w + static_cast<int64_t>(d) * R + c0, wv);
+        } else {
+          float f[4];
+          Vec16<T>::load(w + static_cast<int64_t>(d) * R + c0, f);
+          wv[0] = f[0]; wv[1] = f[1]; wv[2] = f[2]; wv[3] = f[3];
+          Vec16<T>::load(w + static_cast<int64_t>(d) * R + c0 + 4, f);
+          wv[4] = f[0]; wv[5] = f[1]; wv[6] = f[2]; wv[7] = f[3];
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) wv[j] = 0.f;
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) wv[j] = c0 + j < R ? ldf(w + static_cast<int64_t>(d) * R + c0 + j) : 0.f;
     }
-    for (int t = 0; t < cnt; ++t) stf(qf + (static_cast<int64_t>(n0 + t) * H + h) * (R + dr) + r, acc[t]);
+#pragma unroll
+    for (int t = 0; t < kAbsTok; ++t) {
+      const float x = sm[t * D + d];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc[t][j] = fmaf(x, wv[j], acc[t][j]);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < kAbsTok; ++t)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      float v = acc[t][j];
+      v += __shfl_xor_sync(0xffffffffu, v, 8);
+      v += __shfl_xor_sync(0xffffffffu, v, 16);
+      if ((lane >> 3) == (t & 3)) red[(warp * kAbsTok + t) * kAbsCols + (lane & 7) * 8 + j] = v;
+    }
+  __syncthreads();
+  for (int i = threadIdx.x; i < cnt * kAbsCols; i += blockDim.x) {
+    const int t = i / kAbsCols, c = i % kAbsCols, r = blockIdx.z * kAbsCols + c;
+    if (r < R) {
+      float v = 0.f;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v += red[(k * kAbsTok + t) * kAbsCols + c];
+      stf(qf + (static_cast<int64_t>(n0 + t) * H + h) * (R + dr) + r, v);
+    }
   }
   if (blockIdx.z == 0)
     for (int i = threadIdx.x; i < cnt * dr; i += blockDim.x) {
@@ -313,15 +506,26 @@ __global__ void mla_absorb_q_kernel(const SeqBatch sb, const T* __restrict__ q, 
     }
 }
 
-template <typename T>
-__global__ void mla_absorb_out_kernel(const T* __restrict__ o_lat, const T* __restrict__ w_uv, T* __restrict__ o, int n_tok,
-                                      int H, int dv, int R) {
+// A warp computes one value feature of a head for up to 8 tokens; lanes stride the latent.
+template <typename T, bool kVec>
+__global__ void __launch_bounds__(256)
+mla_absorb_out_kernel(const T* __restrict__ o_lat, const T* __restrict__ w_uv, T* __restrict__ o, int n_tok, int H, int dv,
+                      int R) {
   extern __shared__ float sm[];   // [kAbsTok][R]
   const int h = blockIdx.y, n0 = blockIdx.x * kAbsTok;
   const int cnt = min(kAbsTok, n_tok - n0);
-  for (int i = threadIdx.x; i < cnt * R; i += blockDim.x)
-    sm[i] = ldf(o_lat + (static_cast<int64_t>(n0 + i / R) * H + h) * R + i % R);
-  for (int i = threadIdx.x + cnt * R; i < kAbsTok * R; i += blockDim.x) sm[i] = 0.f;
+  if constexpr (kVec) {
+    constexpr int V = Vec16<T>::n;
+    for (int i = threadIdx.x * V; i < kAbsTok * R; i += blockDim.x * V) {
+      float f[V];
+      if (i < cnt * R) Vec16<T>::load(o_lat + (static_cast<int64_t>(n0 + i / R) * H + h) * R + i % R, f);
+#pragma unroll
+      for (int j = 0; j < V; ++j) sm[i + j] = i < cnt * R ? f[j] : 0.f;
+    }
+  } else {
+    for (int i = threadIdx.x; i < kAbsTok * R; i += blockDim.x)
+      sm[i] = i < cnt * R ? ldf(o_lat + (static_cast<int64_t>(n0 + i / R) * H + h) * R + i % R) : 0.f;
+  }
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   for (int v = blockIdx.z * nw + warp; v < dv; v += gridDim.z * nw) {
@@ -329,11 +533,27 @@ __global__ void mla_absorb_out_kernel(const T* __restrict__ o_lat, const T* __re
     float acc[kAbsTok];
 #pragma unroll
     for (int t = 0; t < kAbsTok; ++t) acc[t] = 0.f;
-#pragma unroll 4
-    for (int r = lane; r < R; r += 32) {
-      const float wv = ldf(w + r);
+    if constexpr (kVec) {
+      constexpr int V = Vec16<T>::n;
+#pragma unroll 2
+      for (int r = lane * V; r < R; r += 32 * V) {
+        float wv[V];
+        Vec16<T>::load(w + r, wv);
 #pragma unroll
-      for (int t = 0; t < kAbsTok; ++t) acc[t] = fmaf(sm[t * R + r], wv, acc[t]);
+        for (int t = 0; t < kAbsTok; ++t)
+#pragma unroll
+          for (int j = 0; j < V; j += 4) {
+            const float4 x = *reinterpret_cast<const float4*>(sm + t * R + r + j);
+            acc[t] = fmaf(x.x, wv[j], fmaf(x.y, wv[j + 1], fmaf(x.z, wv[j + 2], fmaf(x.w, wv[j + 3], acc[t]))));
+          }
+      }
+    } else {
+#pragma unroll 4
+      for (int r = lane; r < R; r += 32) {
+        const float wv = ldf(w + r);
+#pragma unroll
+        for (int t = 0; t < kAbsTok; ++t) acc[t] = fmaf(sm[t * R + r], wv, acc[t]);
+      }
     }
 #pragma unroll
     for (int t = 0; t < kAbsTok; ++t) {
@@ -343,10 +563,11 @@ __global__ void mla_absorb_out_kernel(const T* __restrict__ o_lat, const T* __re
   }
 }
 
-// Latent attention, any sizes. A block owns up to kLaQ consecutive queries of one sequence and one head; it walks
-// the keys in tiles of 32 rows staged in shared memory as fp32. Warp w scores queries w, w + 4, ... with one key per
-// lane and keeps their running maxima and sums; outputs are accumulated in shared memory.
-constexpr int kLaQ = 8, kLaK = 32, kLaWarps = 4;
+// Latent attention, any sizes. The heads of a token share the cached rows, so the work items of a sequence are its
+// (token, head) pairs with the head running fastest; a block owns kLaQ consecutive pairs and walks the keys in tiles of
+// 32 rows staged in shared memory as fp32. Warp w scores pairs w and w + 4 with one key per lane, keeps their running
+// maxima and sums and accumulates their outputs in shared memory.
+constexpr int kLaQ = 8, kLaK = 32, kLaWarps = 4, kLaMine = kLaQ / kLaWarps;
 
 template <typename T>
 __global__ void __launch_bounds__(kLaWarps * 32)
@@ -359,79 +580,99 @@ latent_attn_kernel(const SeqBatch sb, const T* __restrict__ qf, const PagedRows 
   float* sq = sk + kLaK * WS;              // [kLaQ][W]
   float* so = sq + kLaQ * W;               // [kLaQ][R]
   float* sp = so + kLaQ * R;               // [kLaQ][kLaK]
-  const int h = blockIdx.y, split = blockIdx.z, S = gridDim.z;
+  const int split = blockIdx.y, S = gridDim.y;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  // tile -> (sequence, first query)
-  int tile = blockIdx.x, b = 0, n0 = -1, cnt = 0;
+  // tile -> (sequence, first pair)
+  int tile = blockIdx.x, b = 0, r0 = -1, cnt = 0;
   for (; b < sb.n_seq; ++b) {
-    const int len = sb.cu[b + 1] - sb.cu[b], tiles = (len + kLaQ - 1) / kLaQ;
+    const int pairs = (sb.cu[b + 1] - sb.cu[b]) * H, tiles = (pairs + kLaQ - 1) / kLaQ;
     if (tile < tiles) {
-      n0 = sb.cu[b] + tile * kLaQ;
-      cnt = min(kLaQ, len - tile * kLaQ);
+      r0 = tile * kLaQ;
+      cnt = min(kLaQ, pairs - r0);
       break;
     }
     tile -= tiles;
   }
-  if (n0 < 0) return;
-  const int slot = sb.ids[b];
-  const int pos0 = sb.start[b] + n0 - sb.cu[b];
-  const int n_keys = pos0 + cnt;
+  if (r0 < 0) return;
+  const int slot = sb.ids[b], start = sb.start[b];
+  const int64_t g0 = static_cast<int64_t>(sb.cu[b]) * H + r0;   // first pair in the packed arrays
+  const int n_keys = start + (r0 + cnt - 1) / H + 1;
   const int tiles_k = (n_keys + kLaK - 1) / kLaK, per = (tiles_k + S - 1) / S;
   const int kt0 = split * per, kt1 = min(tiles_k, kt0 + per);
-  for (int i = threadIdx.x; i < kLaQ * W; i += blockDim.x) {
-    const int q = i / W;
-    sq[i] = q < cnt ? ldf(qf + (static_cast<int64_t>(n0 + q) * H + h) * W + i % W) : 0.f;
-  }
+  for (int i = threadIdx.x; i < kLaQ * W; i += blockDim.x) sq[i] = i < cnt * W ? ldf(qf + g0 * W + i) : 0.f;
   for (int i = threadIdx.x; i < kLaQ * R; i += blockDim.x) so[i] = 0.f;
-  constexpr int kMine = kLaQ / kLaWarps;
-  float m[kMine], l[kMine];
+  float m[kLaMine], l[kLaMine];
+  int pos[kLaMine];                        // position of the pair's token; -1: no pair
 #pragma unroll
-  for (int j = 0; j < kMine; ++j) { m[j] = -INFINITY; l[j] = 0.f; }
+  for (int j = 0; j < kLaMine; ++j) {
+    const int q = warp + j * kLaWarps;
+    m[j] = -INFINITY;
+    l[j] = 0.f;
+    pos[j] = q < cnt ? start + (r0 + q) / H : -1;
+  }
   for (int kt = kt0; kt < kt1; ++kt) {
     __syncthreads();
     for (int k = warp; k < kLaK; k += kLaWarps) {
-      const int pos = kt * kLaK + k;
-      const int64_t row = pos < n_keys ? page_row(pages, slot, pos) : -1;
+      const int p = kt * kLaK + k;
+      const int64_t row = p < n_keys ? page_row(pages, slot, p) : -1;
       const T* src = static_cast<const T*>(pages.pool) + (row < 0 ? 0 : row) * W;
-      for (int i = lane; i < W; i += 32) sk[k * WS + i] = row < 0 ? 0.f : ldf(src + i);
+      if (row >= 0 && W % Vec16<T>::n == 0) {
+        for (int i = lane * Vec16<T>::n; i < W; i += 32 * Vec16<T>::n) {
+          float f[Vec16<T>::n];
+          Vec16<T>::load(src + i, f);
+#pragma unroll
+          for (int j = 0; j < Vec16<T>::n; ++j) sk[k * WS + i + j] = f[j];
+        }
+      } else {
+        for (int i = lane; i < W; i += 32) sk[k * WS + i] = row < 0 ? 0.f : ldf(src + i);
+      }
     }
     __syncthreads();
+    float s[kLaMine];
 #pragma unroll
-    for (int j = 0; j < kMine; ++j) {
-      const int q = warp + j * kLaWarps;
-      if (q >= cnt) continue;   // warp-uniform
-      float s = 0.f;
-      const float* qv = sq + q * W;
-      const float* kv = sk + lane * WS;
+    for (int j = 0; j < kLaMine; ++j) s[j] = 0.f;
+    const float* kv = sk + lane * WS;
+    const float* qv = sq + warp * W;
 #pragma unroll 4
-      for (int i = 0; i < W; ++i) s = fmaf(qv[i], kv[i], s);
-      s = (kt * kLaK + lane <= pos0 + q) ? s * scale : -INFINITY;
-      const float mn = fmaxf(m[j], warp_max(s));
-      if (mn == -INFINITY) {
-        sp[q * kLaK + lane] = 0.f;
-        __syncwarp();
-        continue;
-      }
-      const float p = expf(s - mn), a = expf(m[j] - mn);
-      l[j] = l[j] * a + warp_sum(p);
+    for (int i = 0; i < W; ++i) {
+      const float kk = kv[i];
+#pragma unroll
+      for (int j = 0; j < kLaMine; ++j) s[j] = fmaf(qv[j * kLaWarps * W + i], kk, s[j]);
+    }
+    float a[kLaMine];
+#pragma unroll
+    for (int j = 0; j < kLaMine; ++j) {
+      const float sc = kt * kLaK + lane <= pos[j] ? s[j] * scale : -INFINITY;
+      const float mn = fmaxf(m[j], warp_max(sc));
+      const float ref = mn == -INFINITY ? 0.f : mn;   // nothing seen yet: every weight below is 0
+      const float p = expf(sc - ref);
+      a[j] = expf(m[j] - ref);
+      l[j] = l[j] * a[j] + warp_sum(p);
       m[j] = mn;
-      sp[q * kLaK + lane] = p;
-      __syncwarp();
-      for (int c = lane; c < R; c += 32) {
-        float o = so[q * R + c] * a;
+      sp[(warp + j * kLaWarps) * kLaK + lane] = p;
+    }
+    __syncwarp();
+    for (int c = lane; c < R; c += 32) {
+      float o[kLaMine];
+#pragma unroll
+      for (int j = 0; j < kLaMine; ++j) o[j] = so[(warp + j * kLaWarps) * R + c] * a[j];
 #pragma unroll 8
-        for (int k = 0; k < kLaK; ++k) o = fmaf(sp[q * kLaK + k], sk[k * WS + c], o);
-        so[q * R + c] = o;
+      for (int k = 0; k < kLaK; ++k) {
+        const float v = sk[k * WS + c];
+#pragma unroll
+        for (int j = 0; j < kLaMine; ++j) o[j] = fmaf(sp[(warp + j * kLaWarps) * kLaK + k], v, o[j]);
       }
-      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < kLaMine; ++j) so[(warp + j * kLaWarps) * R + c] = o[j];
     }
   }
 #pragma unroll
-  for (int j = 0; j < kMine; ++j) {
+  for (int j = 0; j < kLaMine; ++j) {
     const int q = warp + j * kLaWarps;
     if (q >= cnt) continue;
-    const int64_t nh = static_cast<int64_t>(n0 + q) * H + h;
+    const int64_t nh = g0 + q;
     if (S == 1) {
+      const int h = (r0 + q) % H;
       float mm = m[j];
       if (sink != nullptr) mm = fmaxf(mm, sink[h]);
       const float f = expf(m[j] - mm);
@@ -627,7 +868,7 @@ cudaError_t latent_attention_t(const SeqBatch& sb, const T* qf, const PagedRows&
   const int smem = 4 * (kLaK * (pages.width + 1) + kLaQ * pages.width + kLaQ * R + kLaQ * kLaK);
   cudaError_t e = want_smem(latent_attn_kernel<T>, smem, have);
   if (e != cudaSuccess) return e;
-  const dim3 grid(sb.n_tok / kLaQ + sb.n_seq, H, n_splits);
+  const dim3 grid(static_cast<unsigned>(static_cast<int64_t>(sb.n_tok) * H / kLaQ + sb.n_seq), n_splits);
   latent_attn_kernel<T><<<grid, kLaWarps * 32, smem, st>>>(sb, qf, pages, R, sink, scale, H, part_o, part_ml, o_lat);
   if (n_splits > 1) latent_merge_kernel<T><<<sb.n_tok * H, 128, 0, st>>>(part_o, part_ml, sink, H, R, n_splits, o_lat);
   return cudaGetLastError();
@@ -636,25 +877,29 @@ cudaError_t latent_attention_t(const SeqBatch& sb, const T* qf, const PagedRows&
 template <typename T>
 cudaError_t absorb_q_t(const SeqBatch& sb, const T* q, const T* w_uk, T* qf, int H, int dn, int dr, int R,
                        const RopeTable& rope, cudaStream_t st) {
-  static int have = 0;
-  const int smem = 4 * kAbsTok * (dn + dr);
-  cudaError_t e = want_smem(mla_absorb_q_kernel<T>, smem, have);
+  static int have_v = 0, have_s = 0;
+  const int smem = 4 * (kAbsTok * (dn + dr) + 8 * kAbsTok * kAbsCols);
+  const bool vec = R % 8 == 0 && (reinterpret_cast<uintptr_t>(w_uk) & 15) == 0;
+  cudaError_t e = vec ? want_smem(mla_absorb_q_kernel<T, true>, smem, have_v) : want_smem(mla_absorb_q_kernel<T, false>, smem, have_s);
   if (e != cudaSuccess) return e;
-  const int tiles = (sb.n_tok + kAbsTok - 1) / kAbsTok;
-  const int z = tiles * H < 296 ? min(4, (R + 127) / 128) : 1;
-  mla_absorb_q_kernel<T><<<dim3(tiles, H, z), 128, smem, st>>>(sb, q, w_uk, qf, H, dn, dr, R, rope);
+  const dim3 grid((sb.n_tok + kAbsTok - 1) / kAbsTok, H, (R + kAbsCols - 1) / kAbsCols);
+  if (vec) mla_absorb_q_kernel<T, true><<<grid, 256, smem, st>>>(sb, q, w_uk, qf, H, dn, dr, R, rope);
+  else mla_absorb_q_kernel<T, false><<<grid, 256, smem, st>>>(sb, q, w_uk, qf, H, dn, dr, R, rope);
   return cudaGetLastError();
 }
 
 template <typename T>
 cudaError_t absorb_out_t(const T* o_lat, const T* w_uv, T* o, int n_tok, int H, int dv, int R, cudaStream_t st) {
-  static int have = 0;
+  static int have_v = 0, have_s = 0;
   const int smem = 4 * kAbsTok * R;
-  cudaError_t e = want_smem(mla_absorb_out_kernel<T>, smem, have);
+  const bool vec = R % Vec16<T>::n == 0 && ((reinterpret_cast<uintptr_t>(w_uv) | reinterpret_cast<uintptr_t>(o_lat)) & 15) == 0;
+  cudaError_t e = vec ? want_smem(mla_absorb_out_kernel<T, true>, smem, have_v) : want_smem(mla_absorb_out_kernel<T, false>, smem, have_s);
   if (e != cudaSuccess) return e;
   const int tiles = (n_tok + kAbsTok - 1) / kAbsTok;
-  const int z = tiles * H < 296 ? min(8, (dv + 7) / 8) : 1;
-  mla_absorb_out_kernel<T><<<dim3(tiles, H, z), 256, smem, st>>>(o_lat, w_uv, o, n_tok, H, dv, R);
+  const int per = (dv + 7) / 8, z = tiles * H < 148 ? (per < 16 ? per : 16) : 1;
+  const dim3 grid(tiles, H, z);
+  if (vec) mla_absorb_out_kernel<T, true><<<grid, 256, smem, st>>>(o_lat, w_uv, o, n_tok, H, dv, R);
+  else mla_absorb_out_kernel<T, false><<<grid, 256, smem, st>>>(o_lat, w_uv, o, n_tok, H, dv, R);
   return cudaGetLastError();
 }
 
@@ -682,8 +927,8 @@ cudaError_t launch_embed_bigram(bool f32, const SeqBatch& sb, const int* tokens,
 
 cudaError_t launch_norm_rows(bool f32_out, int mode, const float* x, const float* gamma, const float* beta, void* out,
                              int rows, int D, float eps, cudaStream_t st) {
-  if (f32_out) norm_rows_kernel<float><<<rows, threads_for(D), 0, st>>>(mode, x, gamma, beta, static_cast<float*>(out), D, eps);
-  else norm_rows_kernel<__nv_bfloat16><<<rows, threads_for(D), 0, st>>>(mode, x, gamma, beta, static_cast<__nv_bfloat16*>(out), D, eps);
+  if (f32_out) norm_rows_go(mode, x, gamma, beta, static_cast<float*>(out), rows, D, eps, st);
+  else norm_rows_go(mode, x, gamma, beta, static_cast<__nv_bfloat16*>(out), rows, D, eps, st);
   return cudaGetLastError();
 }
 

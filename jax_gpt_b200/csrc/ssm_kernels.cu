@@ -35,7 +35,7 @@ __global__ void ssm_conv_kernel(const SeqBatch sb, const T* __restrict__ x, int6
 }
 
 // bf16, 8 channels per thread and a strip of tokens: the window slides through registers. taps <= 4.
-constexpr int kStrip = 16;
+constexpr int kStrip = 32;
 __global__ void ssm_conv_strip_kernel(const SeqBatch sb, const __nv_bfloat16* __restrict__ x, int64_t ldx,
                                       const float* __restrict__ w, const float* __restrict__ bias,
                                       const float* __restrict__ ring, __nv_bfloat16* __restrict__ y, int C, int taps) {
@@ -47,14 +47,20 @@ __global__ void ssm_conv_strip_kernel(const SeqBatch sb, const __nv_bfloat16* __
 #pragma unroll
   for (int j = 0; j < 8; ++j) {
     bs[j] = bias[c0 + j];
+    if (taps == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(w + static_cast<int64_t>(c0 + j) * 4);
+      wt[j][0] = v.x; wt[j][1] = v.y; wt[j][2] = v.z; wt[j][3] = v.w;
+    } else {
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
-      const int kk = k - (4 - taps);
-      wt[j][k] = kk >= 0 ? w[static_cast<int64_t>(c0 + j) * taps + kk] : 0.f;
+      for (int k = 0; k < 4; ++k) {
+        const int kk = k - (4 - taps);
+        wt[j][k] = kk >= 0 ? w[static_cast<int64_t>(c0 + j) * taps + kk] : 0.f;
+      }
     }
   }
   float win[3][8];
   int b = -1, seq_end = -1;
+#pragma unroll 4
   for (; n < n_end; ++n) {
     if (n >= seq_end) {   // a new sequence starts in this strip, or the strip itself starts: reload the window
       b = sb.tok_seq[n];
@@ -75,7 +81,7 @@ __global__ void ssm_conv_strip_kernel(const SeqBatch sb, const __nv_bfloat16* __
       }
     }
     float cur[8];
-    Vec16<__nv_bfloat16>::load(x + static_cast<int64_t>(n) * ldx + c0, cur);
+    Vec16<__nv_bfloat16>::load(x + static_cast<int64_t>(n) * ldx + c0, cur);   // independent of the window: loads run ahead
     uint32_t o[4];
     float r[8];
 #pragma unroll
@@ -85,7 +91,7 @@ __global__ void ssm_conv_strip_kernel(const SeqBatch sb, const __nv_bfloat16* __
       a = fmaf(wt[j][1], win[1][j], a);
       a = fmaf(wt[j][2], win[2][j], a);
       a = fmaf(wt[j][3], cur[j], a);
-      r[j] = a / (1.f + __expf(-a));
+      r[j] = __fdividef(a, 1.f + __expf(-a));
       win[0][j] = win[1][j];
       win[1][j] = win[2][j];
       win[2][j] = cur[j];
@@ -304,33 +310,37 @@ __global__ void gated_group_norm_kernel(const TY* __restrict__ y, const T* __res
     stf(out + static_cast<int64_t>(n) * D + c0 + i, buf[i] * inv * gamma[c0 + i]);
 }
 
-// bf16 y and z, eight features per thread and step, kIt steps: part <= 8 * 256 * kIt
-template <int kIt>
+// bf16 y and z, part <= 8 * kThr * kIt:
+// eight features per thread and step; kThr threads (a warp or the block) own one piece of one row
+template <int kIt, int kThr>
 __global__ void __launch_bounds__(256)
 gated_group_norm_vec_kernel(const __nv_bfloat16* __restrict__ y, const __nv_bfloat16* __restrict__ z, int64_t ldz,
-                            const float* __restrict__ gamma, __nv_bfloat16* __restrict__ out, int D, int part, float eps) {
+                            const float* __restrict__ gamma, __nv_bfloat16* __restrict__ out, int pieces, int parts, int D,
+                            int part, float eps) {
   __shared__ float red[33];
-  const int n = blockIdx.x, c0 = blockIdx.y * part;
+  const int piece = blockIdx.x * (256 / kThr) + threadIdx.x / kThr, tid = threadIdx.x % kThr;
+  if (kThr == 32 && piece >= pieces) return;
+  const int n = piece / parts, c0 = (piece % parts) * part;
   float v[kIt][8];
   float ss = 0.f;
 #pragma unroll
   for (int k = 0; k < kIt; ++k) {
-    const int i = (k * 256 + threadIdx.x) * 8;
+    const int i = (k * kThr + tid) * 8;
     if (i < part) {
       float zv[8];
       Vec16<__nv_bfloat16>::load(y + static_cast<int64_t>(n) * D + c0 + i, v[k]);
       Vec16<__nv_bfloat16>::load(z + static_cast<int64_t>(n) * ldz + c0 + i, zv);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        v[k][j] *= zv[j] / (1.f + __expf(-zv[j]));
+        v[k][j] *= __fdividef(zv[j], 1.f + __expf(-zv[j]));
         ss += v[k][j] * v[k][j];
       }
     }
   }
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / part + eps);
+  const float inv = 1.f / sqrtf((kThr == 32 ? warp_sum(ss) : block_sum(ss, red)) / part + eps);
 #pragma unroll
   for (int k = 0; k < kIt; ++k) {
-    const int i = (k * 256 + threadIdx.x) * 8;
+    const int i = (k * kThr + tid) * 8;
     if (i < part) {
       const float4 g0 = *reinterpret_cast<const float4*>(gamma + c0 + i), g1 = *reinterpret_cast<const float4*>(gamma + c0 + i + 4);
       *reinterpret_cast<uint4*>(out + static_cast<int64_t>(n) * D + c0 + i) =
@@ -420,10 +430,15 @@ cudaError_t launch_gated_group_norm(bool f32, bool y_f32, const void* y, const v
   if (y_f32) return gated_norm_t<float, __nv_bfloat16>(static_cast<const float*>(y), zb, ldz, gamma, o, rows, D, parts, eps, st);
   const __nv_bfloat16* yb = static_cast<const __nv_bfloat16*>(y);
   if (zb != nullptr && part % 8 == 0 && ldz % 8 == 0 && (reinterpret_cast<uintptr_t>(zb) & 15) == 0 && part <= 16384) {
-    const dim3 grid(rows, parts);
-    if (part <= 2048) gated_group_norm_vec_kernel<1><<<grid, 256, 0, st>>>(yb, zb, ldz, gamma, o, D, part, eps);
-    else if (part <= 4096) gated_group_norm_vec_kernel<2><<<grid, 256, 0, st>>>(yb, zb, ldz, gamma, o, D, part, eps);
-    else gated_group_norm_vec_kernel<8><<<grid, 256, 0, st>>>(yb, zb, ldz, gamma, o, D, part, eps);
+    const int pieces = rows * parts;
+#define B200_GN(IT, THR) \
+  gated_group_norm_vec_kernel<IT, THR><<<(pieces + 256 / THR - 1) / (256 / THR), 256, 0, st>>>(yb, zb, ldz, gamma, o, pieces, parts, D, part, eps)
+    if (part <= 512) B200_GN(2, 32);
+    else if (part <= 1024) B200_GN(4, 32);
+    else if (part <= 2048) B200_GN(1, 256);
+    else if (part <= 4096) B200_GN(2, 256);
+    else B200_GN(8, 256);
+#undef B200_GN
     return cudaGetLastError();
   }
   return gated_norm_t<__nv_bfloat16, __nv_bfloat16>(yb, zb, ldz, gamma, o, rows, D, parts, eps, st);

@@ -118,7 +118,7 @@ def linear_f32out(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return x.float() @ w.float()
 
 
-ROWS_KERNEL_MAX = 8      # rows up to which a linear layer streams its weights through the few-row kernel
+ROWS_KERNEL_MAX = {torch.bfloat16: 32, torch.float32: 8}   # rows up to which linear layers run on the few-row kernel
 
 
 def linear_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *, act: Optional[str] = None,
@@ -126,13 +126,13 @@ def linear_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = 
     """Inference linear layer with ``w`` stored (out, in) as checkpoints have it: ``act(x @ w.T)``; ``act`` is None or
     "relu2" (the square of relu). ``accumulate`` adds into ``out`` (fp32: a 32-bit residual), ``f32_out`` returns fp32.
     x (M, in), bf16 or fp32, unit inner stride. On CUDA up to ``ROWS_KERNEL_MAX`` rows run on the few-row kernel
-    (weights streamed once), more rows on the tcgen05 GEMM in bf16 and on the library's fp32 GEMM in fp32."""
+    (weights streamed once where the rows are 16-byte aligned), more rows on the tcgen05 GEMM in bf16 and on the library's fp32 GEMM in fp32."""
     M, N = x.shape[0], w.shape[0]
     if out is None:
         assert not accumulate
         out = torch.empty(M, N, device=x.device, dtype=torch.float32 if f32_out else x.dtype)
     mode = 2 if accumulate else (1 if out.dtype == torch.float32 and x.dtype != torch.float32 else 0)
-    if x.is_cuda and M <= ROWS_KERNEL_MAX:
+    if x.is_cuda and M <= ROWS_KERNEL_MAX.get(x.dtype, 0):
         _ext.ops().rows_linear(x, w, out, 1 if act == "relu2" else 0, mode)
         return out
     if x.is_cuda and x.dtype == torch.bfloat16 and w.shape[1] % 8 == 0 and w.stride(0) % 8 == 0 and w.data_ptr() % 16 == 0:

@@ -71,7 +71,7 @@ def key_splits(batch: PackedBatch, n_heads: int) -> int:
     """Key ranges per query of the any-size kernel: decode steps spread a long cache over the SMs."""
     if not batch.single:
         return 1
-    return max(1, min(296 // max(1, batch.n_seq * n_heads), (batch.max_len + 63) // 64, 16))
+    return max(1, min(592 // max(1, batch.n_seq * ((n_heads + 7) // 8)), (batch.max_len + 63) // 64, 32))
 
 
 def latent_attention(batch: PackedBatch, qf, cache, layer: int, R: int, scale: float, sink=None, n_splits: int = 0):

@@ -4,6 +4,7 @@
     python -m jax_gpt_b200.utils.kernel_bench --op attn_fwd --B 16 --T 1024 --H 12 --D 64
     python -m jax_gpt_b200.utils.kernel_bench --op attn_bwd | norm_fwd | norm_bwd | adamw | ce
     python -m jax_gpt_b200.utils.kernel_bench --op mla_decode --B 32 --T 2304 --H 16
+    python -m jax_gpt_b200.utils.kernel_bench --op ssd_scan --B 2 --T 4096 --H 64
     python -m jax_gpt_b200.utils.kernel_bench --op gdn_prep_fwd | gdn_prep_bwd | gdn_prefill --B 1 --T 4096
 
 Each run does ``--warmup`` untimed launches, then times ``--iters`` launches with CUDA events on
@@ -200,6 +201,19 @@ def main(argv=None):
                 DN._GdnGatedNormFn.apply(o, z, w, Hv, 1e-6).backward(dy)
             flops = 0.0
             bytes_ = 0.0
+    elif args.op == "ssd_scan":
+        # --B sequences of --T tokens, --H heads of 64 with state 128 in 8 groups
+        from ..ops import ssm
+        from .serve_bench import _start_batch
+        B, T, H, G = args.B, args.T, args.H, 8
+        batch = _start_batch(list(range(B)), [T] * B, 0, dev, T)
+        C = H * 64 + 2 * G * 128
+        xbc, dt = torch.randn(B * T, C, device=dev).to(torch.bfloat16), torch.randn(B * T, H, device=dev).to(torch.bfloat16)
+        al, db, dk = torch.rand(H, device=dev), torch.rand(H, device=dev) - 4, torch.randn(H, device=dev)
+        state = torch.zeros(B, H, 128, 64, device=dev)
+        fn = lambda: ssm.ssd_scan(batch, xbc, dt, db, al, dk, state, G)
+        bytes_ = 2.0 * B * T * (C + H * 64 + H) + 4.0 * state.numel()
+        flops = B * T / 128 * H * 2.0 * 128 * (128 * 128 + 3 * 128 * 64)
     elif args.op == "mla_decode":
         # --B sequences of --T cached tokens each, --H heads (16 = DeepSeek-V3 with 8-way head sharding)
         from ..cache.paged import PagedCache

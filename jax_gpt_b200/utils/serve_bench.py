@@ -35,7 +35,6 @@ class _KernelTimer:
     def __init__(self, device, n: int = 10):
         self.flush = torch.empty(64 * 1024 * 1024, dtype=torch.float32, device=device)
         self.n, self.peaks = n, R.load_peaks()
-        self.base = min(self._run(None) for _ in range(2))
 
     def _run(self, fn):
         if fn is not None:
@@ -63,7 +62,7 @@ class _KernelTimer:
         return statistics.median(times)
 
     def __call__(self, fn, bytes_: float = 0.0, flops: float = 0.0) -> dict:
-        ms = max(self._run(fn) - self.base, 1e-4)
+        ms = max(self._run(fn) - self._run(None), 1e-4)
         roof = max(bytes_ / (self.peaks["hbm_gbs"] * 1e6), flops / (self.peaks["bf16_tflops"] * 1e9))
         return {"us": round(ms * 1e3, 2), "roofline_us": round(roof * 1e3, 2), "frac": round(roof / ms, 3)}
 
@@ -379,7 +378,7 @@ def model_table(dev, sizes=((2048, 16), (4096, 32)), shapes=((1, 4096), (8, 1024
     rows = []
     for width, heads in sizes:
         hybrid = VobunexConfig.serving(width=width, n_mamba=6, n_attention=2, experts=E, top=top, ff=ff, heads=heads, vocab=V)
-        qwen = Qwen35Config(d_model=width, vocab_size=V, n_layers=8, max_position_embeddings=8192, gqa_n_q_heads=heads, gqa_n_kv_heads=2,
+        qwen = Qwen35Config(d_model=width, vocab_size=V, n_layers=8, max_position_embeddings=8192, gqa_n_q_heads=heads, gqa_n_kv_heads=heads // 8,
                             gqa_head_dim=256, delta_n_qk_heads=16, delta_n_v_heads=2 * width // 128, delta_qk_head_dim=128,
                             delta_v_head_dim=128, delta_chunk_size=64, n_routed_experts=E, n_experts_per_token=top,
                             moe_intermediate_size=ff, shared_expert_intermediate_size=128)
@@ -413,4 +412,8 @@ def run(part: str = "all") -> dict:
         out["models"] = model_table(dev)
     from .. import _ext
     _ext.check_status(dev)
+    _sync_free()
+    import torch.distributed as dist
+    if dist.is_initialized():
+        dist.destroy_process_group()
     return out

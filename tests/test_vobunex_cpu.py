@@ -159,3 +159,24 @@ def test_presets():
     c = VobunexConfig.tiny()
     lg = forward(init_params(c, 0), torch.arange(12)[None], c)
     assert lg.shape == (1, 12, c.vocab_size) and torch.isfinite(lg).all()
+
+
+def test_sample_script_continues_token_ids(tmp_path):
+    import subprocess
+    from safetensors.torch import save_file
+    cfg = K.CONFIGS["aligned"]
+    w = K.weights(cfg, 50)
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    save_file({k: v.contiguous() for k, v in w.items()}, str(tmp_path / "model.safetensors"))
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    prompts = [K.tokens(cfg, 7, 1), K.tokens(cfg, 3, 2)]
+    args = [sys.executable, "scripts/sample.py", "--model-dir", str(tmp_path), "--dtype", "float32", "--temperature", "0", "--new_tokens", "5"]
+    for p in prompts:
+        args += ["--prompt-ids", ",".join(map(str, p))]
+    r = subprocess.run(args, cwd=root, capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr
+    rows = [list(map(int, l.split(","))) for l in r.stdout.splitlines() if l and not l.startswith("---")]
+    for p, got in zip(prompts, rows):
+        for n, t in enumerate(got):
+            lg = O.forward(p + got[:n], cfg, w)[-1]
+            assert float(lg.max() - lg[t]) < 1e-3
