@@ -105,7 +105,7 @@ struct SsdShape {
 cudaError_t launch_ssd_scan(bool f32, const SeqBatch& sb, const void* xbc, const void* dt_raw, int64_t ld_dt,
                             const float* dt_bias, const float* a_log, const float* d_skip, float* state, void* y,
                             const SsdShape& s, cudaStream_t st);
-// The same on tensor cores, 128-token chunks: bf16, N = 128, P in {64, 128}.
+// The same on tensor cores, 128-token chunks: bf16, N = 128, P a multiple of 64.
 bool ssd_scan_sm100_ok(const SsdShape& s);
 cudaError_t launch_ssd_scan_sm100(const SeqBatch& sb, const __nv_bfloat16* xbc, const __nv_bfloat16* dt_raw, int64_t ld_dt,
                                   const float* dt_bias, const float* a_log, const float* d_skip, float* state,

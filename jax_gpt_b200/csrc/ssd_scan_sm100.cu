@@ -1,16 +1,20 @@
 // Chunked state-space recurrence (Mamba-2, "state-space duality") on tcgen05 tensor cores, bf16 activations with
 // fp32 state:
 //   S_t = exp(-exp(A_log) dt_t) S_(t-1) + dt_t B_t x_t^T,   y_t = S_t^T C_t + D x_t      (S is N x P, N = 128)
-// One CTA per (head, sequence) walks chunks of 128 tokens with S in the registers of 256 threads (fp32). With
-// c_i = the running sum of -exp(A_log) dt inside the chunk and L_ij = exp(c_i - c_j) dt_j for j <= i, else 0:
-//   1. G = C B^T,  Yo = C S          (S the state the chunk starts from)
-//   2. Y = (G * L) X,  T = B^T X'    (X'_j = exp(c_end - c_j) dt_j x_j)
-//   3. y_i = Y_i + exp(c_i) Yo_i + D x_i,   S <- exp(c_end) S + T
-// B, C and X enter the products as the bf16 values they are; the fp32 operands (G * L, S, X') are split into a
-// high and a low bf16 part and multiplied twice, so the products carry about 16 mantissa bits of them and the sums
-// are fp32. G * L goes back to TMEM as the A operand; S and X' are B operands in shared memory. Chunk tiles arrive by
-// TMA (double-buffered at P = 64). A tail chunk reads rows of the next sequence (or the zero fill): their step sizes
-// count as 0, so they neither decay nor feed the state, and their outputs are not stored.
+// One CTA per (64 columns of a head, sequence) walks chunks of 128 tokens. With c_i = the running sum of
+// -exp(A_log) dt inside the chunk and L_ij = exp(c_i - c_j) dt_j for j <= i, else 0:
+//   G = C B^T,  M = G * L + D I,  Y = M X                              (inside the chunk, skip term included)
+//   Yo = C S                                                           (S the state the chunk starts from)
+//   T = B^T X'  with X'_j = exp(c_end - c_j) dt_j x_j
+//   y_i = Y_i + exp(c_i) Yo_i,   S <- exp(c_end) S + T
+// B, C and X enter the products as the bf16 values they are; the fp32 operands (M, S, X') are split into a high and a
+// low bf16 part, so the products carry about 16 mantissa bits of them and the sums are fp32. M goes back to TMEM over
+// G as the A operand; S and X' are B operands in shared memory (S high | low side by side as one 128-wide operand).
+//
+// Only S links the chunks, so the work is a pipeline over chunks: warp 0 loads tiles by TMA (two stages), warp 1 issues
+// the MMAs, eight "chunk" warps turn G(n + 1) into M and X into X' while eight "state" warps finish chunk n (outputs,
+// state update, next S operand); G is double-buffered in TMEM. A tail chunk reads rows of the next sequence (or the
+// zero fill): their step sizes count as 0, so they neither decay nor feed the state, and their outputs are not stored.
 // Step sizes, decays and exponentials are fp32 (this file is built without fast-math).
 #include "serve_kernels.cuh"
 
@@ -21,29 +25,29 @@ namespace b200 {
 
 namespace {
 
-constexpr int kL = 128, kN = 128;
-constexpr int kTileBytes = kL * kN * 2;   // 32 KB: 128 x 128 bf16 as two 64-column blocks of 16 KB
-constexpr int kThreads = 320;             // TMA warp, MMA warp, eight compute warps
-constexpr int kCompute = 256;
+constexpr int kL = 128, kN = 128, kP = 64;
+constexpr int kTileBytes = kL * kN * 2;            // 32 KB: 128 x 128 bf16 as two 64-column blocks of 16 KB
+constexpr int kXBytes = kL * kP * 2;               // 16 KB
+constexpr int kStages = 2;
+constexpr int kStageBytes = 2 * kTileBytes + kXBytes;   // C | B | X
+constexpr int kGroup = 256;                        // threads of the chunk warps, and of the state warps
+constexpr int kThreads = 64 + 2 * kGroup;
+constexpr int kCd = 4;                             // chunks whose c_j are kept
+constexpr int kOffXp = kStages * kStageBytes;      // X' high, X' low
+constexpr int kOffS = kOffXp + 2 * kXBytes;        // S high, S low
+constexpr int kOffBar = kOffS + 2 * kXBytes;
+constexpr uint32_t kColG = 0, kColY = 256, kColT = 320, kColYo = 384;   // G: two buffers of 128 columns
 
-template <int P>
-struct SsdCfg {
-  static constexpr int kStages = P == 64 ? 2 : 1;
-  static constexpr int kXBytes = kL * P * 2;
-  static constexpr int kStageBytes = 2 * kTileBytes + kXBytes;   // C | B | X
-  static constexpr int kOffXp = kStages * kStageBytes;           // X' high, X' low
-  static constexpr int kOffS = kOffXp + 2 * kXBytes;             // S high, S low (128 x P each)
-  static constexpr int kOffCd = kOffS + 2 * kXBytes;             // float2 [128]: (c_j in log2 units, dt_j)
-  static constexpr int kOffBar = kOffCd + kL * 8;
-  static constexpr int kSmem = 1024 + kOffBar + 192;
-};
-
-struct SsdBars {
-  uint64_t full[2], empty[2], g_full, m_ready, y_full, s_ready;
+struct SsdShared {
+  uint64_t full[kStages], empty[kStages], g_full[2], m_ready[2], c_full[kCd], xp_ready, y_full, s_ready;
   uint32_t tmem_base;
   int abort_flag;
   float part[4];
+  alignas(16) float e[kL];                         // c_j - log2(dt_j) of the chunk in work: L_ij = 2^(c_i - e_j)
+  alignas(16) float c[kCd][kL];                    // c_j in log2 units; the chunk warps run ahead of the state warps
 };
+constexpr int kSmem = kOffBar + ((sizeof(SsdShared) + 15) & ~15);   // the window starts 1024-byte aligned (checked)
+static_assert(kSmem <= 227 * 1024, "shared memory");
 
 struct SsdArgs {
   SeqBatch sb;
@@ -63,12 +67,20 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ void compute_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kCompute) : "memory"); }
+__device__ __forceinline__ void chunk_sync() { asm volatile("bar.sync 1, %0;" ::"n"(kGroup) : "memory"); }
 
-// byte offset of (row r, column c) in a bf16 tile of 64-column blocks (16 KB each) with 128-byte swizzled rows
-__device__ __forceinline__ uint32_t swz(int r, int c) {
-  return (c >> 6) * 16384 + r * 128 + ((((c & 63) >> 3) ^ (r & 7)) << 4) + (c & 7) * 2;
+__device__ __forceinline__ void tmem_ld_x16(uint32_t taddr, uint32_t (&v)[16]) {
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
+      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]),
+        "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+      : "r"(taddr)
+      : "memory");
 }
+
+// byte offset of (row r, column c < 64) in a bf16 tile of 128-byte swizzled rows
+__device__ __forceinline__ uint32_t swz(int r, int c) { return r * 128 + (((c >> 3) ^ (r & 7)) << 4) + (c & 7) * 2; }
 
 // v[0..7] as a high bf16 part and the bf16 rounding of the remainder
 __device__ __forceinline__ void split8(const float* v, uint4& hi, uint4& lo) {
@@ -83,131 +95,262 @@ __device__ __forceinline__ void split8(const float* v, uint4& hi, uint4& lo) {
   lo = make_uint4(l[0], l[1], l[2], l[3]);
 }
 
-template <int P>
 __global__ void __launch_bounds__(kThreads, 1)
 ssd_scan_sm100_kernel(const __grid_constant__ CUtensorMap t_xbc, const __grid_constant__ SsdArgs a) {
-  using C = SsdCfg<P>;
-  constexpr int kHalf = P / 2;
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  SsdBars* bars = reinterpret_cast<SsdBars*>(smem + C::kOffBar);
-  volatile int* abort_flag = &bars->abort_flag;
+  extern __shared__ __align__(1024) uint8_t smem[];
+  SsdShared* sh = reinterpret_cast<SsdShared*>(smem + kOffBar);
+  volatile int* abort_flag = &sh->abort_flag;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int h = blockIdx.x, b = blockIdx.y;
+  const int halves = a.s.P / kP;
+  const int h = blockIdx.x / halves, p0 = (blockIdx.x % halves) * kP, b = blockIdx.y;
   const int first = a.sb.cu[b], len = a.sb.cu[b + 1] - first;
   const int n_chunks = (len + kL - 1) / kL;
-  const int inner = a.s.H * P;
+  const int inner = a.s.H * a.s.P;
+  if ((smem_u32(smem) & 1023) != 0) {
+    if (threadIdx.x == 0) report_status(a.status, kBadArgument, 315, smem_u32(smem));
+    return;
+  }
 
   if (threadIdx.x == 0) {
-    for (int s = 0; s < 2; ++s) {
-      mbar_init(&bars->full[s], 1);
-      mbar_init(&bars->empty[s], 1);
+    for (int s = 0; s < kStages; ++s) {
+      mbar_init(&sh->full[s], 1);
+      mbar_init(&sh->empty[s], 1);
+      mbar_init(&sh->g_full[s], 1);
+      mbar_init(&sh->m_ready[s], kGroup);   // per buffer: the chunk warps may be a chunk ahead of the MMA warp
     }
-    mbar_init(&bars->g_full, 1);
-    mbar_init(&bars->m_ready, kCompute);
-    mbar_init(&bars->y_full, 1);
-    mbar_init(&bars->s_ready, kCompute);
-    bars->abort_flag = 0;
+    for (int s = 0; s < kCd; ++s) mbar_init(&sh->c_full[s], kL);
+    mbar_init(&sh->xp_ready, kGroup);
+    mbar_init(&sh->y_full, 1);
+    mbar_init(&sh->s_ready, kGroup);
+    sh->abort_flag = 0;
     fence_mbar_init();
   }
   if (warp == 1) {
-    tmem_alloc(&bars->tmem_base, 512);
+    tmem_alloc(&sh->tmem_base, 512);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = bars->tmem_base;
-  constexpr uint32_t kColG = 0, kColY = 128, kColYo = 256, kColT = 384;   // G is overwritten by (G * L) high | low
+  const uint32_t tmem = sh->tmem_base;
 
   if (warp == 0) {
     if (lane == 0) {
       const int g = h / (a.s.H / a.s.G);
-      const int col_b = inner + g * kN, col_c = inner + a.s.G * kN + g * kN;
+      const int col_b = inner + g * kN, col_c = inner + a.s.G * kN + g * kN, col_x = h * a.s.P + p0;
       int issued = 0;
       bool ok = true;
       for (int n = 0; n < n_chunks; ++n, ++issued) {
-        const int st = n % C::kStages;
-        if (n >= C::kStages && !mbar_wait(&bars->empty[st], ((n / C::kStages) - 1) & 1, abort_flag)) {
+        const int st = n & 1;
+        if (n >= kStages && !mbar_wait(&sh->empty[st], ((n >> 1) - 1) & 1, abort_flag)) {
           report_status(a.status, kWaitEmptyTimeout, 310, h, n);
           ok = false;
           break;
         }
-        uint8_t* base = smem + st * C::kStageBytes;
+        uint8_t* base = smem + st * kStageBytes;
         const int row = first + n * kL;
-        mbar_arrive_expect_tx(&bars->full[st], C::kStageBytes);
-        tma_load_2d(base, &t_xbc, &bars->full[st], col_c, row);
-        tma_load_2d(base + 16384, &t_xbc, &bars->full[st], col_c + 64, row);
-        tma_load_2d(base + kTileBytes, &t_xbc, &bars->full[st], col_b, row);
-        tma_load_2d(base + kTileBytes + 16384, &t_xbc, &bars->full[st], col_b + 64, row);
-#pragma unroll
-        for (int k = 0; k < P / 64; ++k)
-          tma_load_2d(base + 2 * kTileBytes + k * 16384, &t_xbc, &bars->full[st], h * P + k * 64, row);
+        mbar_arrive_expect_tx(&sh->full[st], kStageBytes);
+        tma_load_2d(base, &t_xbc, &sh->full[st], col_c, row);
+        tma_load_2d(base + 16384, &t_xbc, &sh->full[st], col_c + 64, row);
+        tma_load_2d(base + kTileBytes, &t_xbc, &sh->full[st], col_b, row);
+        tma_load_2d(base + kTileBytes + 16384, &t_xbc, &sh->full[st], col_b + 64, row);
+        tma_load_2d(base + 2 * kTileBytes, &t_xbc, &sh->full[st], col_x, row);
       }
       if (!ok || *abort_flag) {   // leave no bulk copy in flight (bounded)
         const uint64_t tw = globaltimer_ns();
-        for (int s = 0; s < C::kStages; ++s) {
-          const int uses = (issued + C::kStages - 1 - s) / C::kStages;
+        for (int s = 0; s < kStages; ++s) {
+          const int uses = (issued + 1 - s) / 2;
           if (uses > 0)
-            while (!mbar_try_wait(&bars->full[s], (uses - 1) & 1) && globaltimer_ns() - tw < 2000000ull) {
+            while (!mbar_try_wait(&sh->full[s], (uses - 1) & 1) && globaltimer_ns() - tw < 2000000ull) {
             }
         }
       }
     }
   } else if (warp == 1) {
-    constexpr uint32_t i_g = make_idesc(128, 128, 0, 0, 1);   // C (K-major) x B (K-major)
-    constexpr uint32_t i_kn = make_idesc(128, P, 0, 1, 1);    // A K-major or in TMEM, B MN-major
-    constexpr uint32_t i_nn = make_idesc(128, P, 1, 1, 1);    // both MN-major
-    const uint32_t a_s = smem_u32(smem + C::kOffS), a_xp = smem_u32(smem + C::kOffXp);
-    for (int n = 0; n < n_chunks; ++n) {
-      const int st = n % C::kStages;
-      const uint32_t tc = smem_u32(smem + st * C::kStageBytes), tb = tc + kTileBytes, tx = tb + kTileBytes;
-      if (!mbar_wait(&bars->s_ready, n & 1, abort_flag) || !mbar_wait(&bars->full[st], (n / C::kStages) & 1, abort_flag)) {
+    constexpr uint32_t i_kk = make_idesc(128, 128, 0, 0, 1);    // G: C (K-major) x B (K-major)
+    constexpr uint32_t i_yo = make_idesc(128, 128, 0, 1, 1);    // Yo: C (K-major) x [S high | S low] (MN-major)
+    constexpr uint32_t i_y = make_idesc(128, kP, 0, 1, 1);      // Y: M (TMEM) x X (MN-major)
+    constexpr uint32_t i_t = make_idesc(128, kP, 1, 1, 1);      // T: B (MN-major) x X' (MN-major)
+    const uint32_t a_s = smem_u32(smem + kOffS), a_xp = smem_u32(smem + kOffXp);
+    auto tile = [&](int n) { return smem_u32(smem + (n & 1) * kStageBytes); };
+    auto issue_g = [&](int n) -> bool {
+      if (!mbar_wait(&sh->full[n & 1], (n >> 1) & 1, abort_flag)) {
         if (lane == 0) report_status(a.status, kWaitFullTimeout, 311, h, n);
-        break;
+        return false;
       }
       tc_fence_after();
       if (lane == 0) {
+        const uint32_t tc = tile(n), tb = tc + kTileBytes;
 #pragma unroll
         for (int k = 0; k < 8; ++k)   // K = state size
-          umma_bf16(tmem + kColG, make_smem_desc(tc + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024),
-                    make_smem_desc(tb + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024), i_g, k > 0 ? 1u : 0u);
-#pragma unroll
-        for (int k = 0; k < 16; ++k)   // state high, then low
-          umma_bf16(tmem + kColYo, make_smem_desc(tc + ((k & 7) >> 2) * 16384 + (k & 3) * 32, 16, 1024),
-                    make_smem_desc(a_s + (k >> 3) * C::kXBytes + (k & 7) * 2048, 16384, 1024), i_kn, k > 0 ? 1u : 0u);
-        tc_commit(&bars->g_full);
+          umma_bf16(tmem + kColG + (n & 1) * 128, make_smem_desc(tc + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024),
+                    make_smem_desc(tb + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024), i_kk, k > 0 ? 1u : 0u);
+        tc_commit(&sh->g_full[n & 1]);
       }
       __syncwarp();
-      if (!mbar_wait(&bars->m_ready, n & 1, abort_flag)) {
+      return true;
+    };
+    const bool ok = issue_g(0);
+    for (int n = 0; ok && n < n_chunks; ++n) {
+      // G(n + 1) goes into the buffer of M(n - 1), whose product Y(n - 1) was issued before and runs first
+      if (n + 1 < n_chunks && !issue_g(n + 1)) break;
+      const uint32_t tc = tile(n), tb = tc + kTileBytes, tx = tb + kTileBytes;
+      if (!mbar_wait(&sh->s_ready, n & 1, abort_flag)) {
         if (lane == 0) report_status(a.status, kWaitFullTimeout, 312, h, n);
         break;
       }
       tc_fence_after();
       if (lane == 0) {
 #pragma unroll
-        for (int k = 0; k < 16; ++k)   // K = tokens
-          umma_bf16_ts(tmem + kColY, tmem + kColG + (k >> 3) * 64 + (k & 7) * 8,
-                       make_smem_desc(tx + (k & 7) * 2048, 16384, 1024), i_kn, k > 0 ? 1u : 0u);
+        for (int k = 0; k < 8; ++k)   // K = state size; the second 64 columns are the low parts
+          umma_bf16(tmem + kColYo, make_smem_desc(tc + (k >> 2) * 16384 + (k & 3) * 32, 16, 1024),
+                    make_smem_desc(a_s + k * 2048, 16384, 1024), i_yo, k > 0 ? 1u : 0u);
+      }
+      __syncwarp();
+      if (!mbar_wait(&sh->m_ready[n & 1], (n >> 1) & 1, abort_flag)) {
+        if (lane == 0) report_status(a.status, kWaitFullTimeout, 313, h, n);
+        break;
+      }
+      tc_fence_after();
+      if (lane == 0) {
 #pragma unroll
-        for (int k = 0; k < 16; ++k)
+        for (int k = 0; k < 16; ++k)   // K = tokens; step k of M: high words at 16 k, low words at 16 k + 8
+          umma_bf16_ts(tmem + kColY, tmem + kColG + (n & 1) * 128 + (k >> 1) * 16 + (k & 1) * 8,
+                       make_smem_desc(tx + (k >> 1) * 2048, 16384, 1024), i_y, k > 0 ? 1u : 0u);
+      }
+      __syncwarp();
+      if (!mbar_wait(&sh->xp_ready, n & 1, abort_flag)) {
+        if (lane == 0) report_status(a.status, kWaitFullTimeout, 314, h, n);
+        break;
+      }
+      tc_fence_after();
+      if (lane == 0) {
+#pragma unroll
+        for (int k = 0; k < 16; ++k)   // K = tokens, X' high then low
           umma_bf16(tmem + kColT, make_smem_desc(tb + (k & 7) * 2048, 16384, 1024),
-                    make_smem_desc(a_xp + (k >> 3) * C::kXBytes + (k & 7) * 2048, 16384, 1024), i_nn, k > 0 ? 1u : 0u);
-        tc_commit(&bars->empty[st]);
-        tc_commit(&bars->y_full);
+                    make_smem_desc(a_xp + (k >> 3) * kXBytes + (k & 7) * 2048, 16384, 1024), i_t, k > 0 ? 1u : 0u);
+        tc_commit(&sh->empty[n & 1]);
+        tc_commit(&sh->y_full);
       }
       __syncwarp();
     }
-  } else {
+  } else if (warp < 2 + kGroup / 32) {
+    // ---- chunk warps: step sizes, M, X' ----
     const int q = warp & 3, half = (warp - 2) >> 2;
-    const int r = q * 32 + lane;   // row of every TMEM tile owned by this thread: a token of the chunk, or a state row
+    const int r = q * 32 + lane;   // token of the chunk
     const uint32_t lane_off = static_cast<uint32_t>(q * 32) << 16;
-    float2* cd = reinterpret_cast<float2*>(smem + C::kOffCd);
-    uint8_t* s_hi = smem + C::kOffS;
-    uint8_t* s_lo = s_hi + C::kXBytes;
-    uint8_t* xp_hi = smem + C::kOffXp;
-    uint8_t* xp_lo = xp_hi + C::kXBytes;
-    float* gs = a.state + ((static_cast<int64_t>(a.sb.ids[b]) * a.s.H + h) * kN + r) * P + half * kHalf;
+    uint8_t* xp_hi = smem + kOffXp;
+    uint8_t* xp_lo = xp_hi + kXBytes;
+    const float bias = a.dt_bias[h], decay = -expf(a.a_log[h]) * 1.4426950408889634f, dsk = a.d_skip[h];
+    auto load_dt = [&](int n) -> float {
+      const int t = n * kL + r;
+      return t < len ? __bfloat162float(a.dt_raw[static_cast<int64_t>(first + t) * a.ld_dt + h]) : 0.f;
+    };
+    float raw = load_dt(0);
+    bool ok = true;
+    // `ok` may differ between warps after a timeout, but every warp runs every iteration with all its barriers
+    for (int n = 0; n < n_chunks; ++n) {
+      const float dt = n * kL + r < len ? softplus_f(raw + bias) : 0.f;
+      float cum = dt * decay;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float t = __shfl_up_sync(0xffffffffu, cum, o);
+        if (lane >= o) cum += t;
+      }
+      if (half == 0 && lane == 31) sh->part[q] = cum;
+      if (n + 1 < n_chunks) raw = load_dt(n + 1);
+      chunk_sync();   // every warp is done with e of chunk n - 1
+      float c_end = 0.f;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float t = sh->part[k];
+        if (k < q) cum += t;
+        c_end += t;
+      }
+      if (half == 0) {
+        sh->c[n & (kCd - 1)][r] = cum;
+        sh->e[r] = cum - log2f(dt);
+        mbar_arrive(&sh->c_full[n & (kCd - 1)]);
+      }
+      chunk_sync();
+      // ---- M over G, sixteen columns at a time (the two warps of a row take alternate groups) ----
+      if (ok && !mbar_wait(&sh->g_full[n & 1], (n >> 1) & 1, abort_flag)) {
+        if (lane == 0) report_status(a.status, kWaitTmemFullTimeout, 316, h, n);
+        ok = false;
+      }
+      ok = __all_sync(0xffffffffu, ok);
+      if (ok) {
+        tc_fence_after();
+        const uint32_t tg = tmem + kColG + (n & 1) * 128 + lane_off;
+#pragma unroll 1
+        for (int gi = half; gi < 8; gi += 2) {
+          const int j0 = gi * 16;
+          uint32_t v[16], m[16];
+          if (j0 <= q * 32 + 31) {   // warp-uniform: part of the group is at or below the diagonal
+            tmem_ld_x16(tg + j0, v);
+            tmem_ld_wait();
+#pragma unroll
+            for (int j = 0; j < 16; j += 4) {
+              const float4 e = *reinterpret_cast<const float4*>(&sh->e[j0 + j]);
+              float f[4] = {__uint_as_float(v[j]) * ex2(cum - e.x), __uint_as_float(v[j + 1]) * ex2(cum - e.y),
+                            __uint_as_float(v[j + 2]) * ex2(cum - e.z), __uint_as_float(v[j + 3]) * ex2(cum - e.w)};
+#pragma unroll
+              for (int k = 0; k < 4; ++k) {
+                const int d = r - (j0 + j + k);
+                f[k] = d > 0 ? f[k] : (d == 0 ? f[k] + dsk : 0.f);
+              }
+#pragma unroll
+              for (int k = 0; k < 4; k += 2) {
+                const uint32_t hw = pack_bf16x2(f[k], f[k + 1]);
+                const float2 u = unpack_bf16x2(hw);
+                m[(j + k) / 2] = hw;
+                m[8 + (j + k) / 2] = pack_bf16x2(f[k] - u.x, f[k + 1] - u.y);
+              }
+            }
+          } else {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) m[j] = 0u;
+          }
+          tmem_st_32x16(tg + j0, m);
+        }
+        tmem_st_wait();
+        tc_fence_before();
+      }
+      mbar_arrive(&sh->m_ready[n & 1]);
+      // ---- X' (its buffer is free once the products of chunk n - 1 are done) ----
+      if (ok && n > 0 && !mbar_wait(&sh->y_full, (n - 1) & 1, abort_flag)) {
+        if (lane == 0) report_status(a.status, kWaitTmemFullTimeout, 317, h, n);
+        ok = false;
+      }
+      if (ok && !mbar_wait(&sh->full[n & 1], (n >> 1) & 1, abort_flag)) ok = false;
+      ok = __all_sync(0xffffffffu, ok);
+      if (ok) {
+        const uint8_t* tx = smem + (n & 1) * kStageBytes + 2 * kTileBytes;
+        const float w = ex2(c_end - cum) * dt;
+#pragma unroll
+        for (int j = 0; j < kP / 2; j += 8) {
+          const uint32_t o = swz(r, half * (kP / 2) + j);
+          const uint4 v = *reinterpret_cast<const uint4*>(tx + o);
+          const float2 f0 = unpack_bf16x2(v.x), f1 = unpack_bf16x2(v.y), f2 = unpack_bf16x2(v.z), f3 = unpack_bf16x2(v.w);
+          const float f[8] = {f0.x * w, f0.y * w, f1.x * w, f1.y * w, f2.x * w, f2.y * w, f3.x * w, f3.y * w};
+          uint4 hi, lo;
+          split8(f, hi, lo);
+          *reinterpret_cast<uint4*>(xp_hi + o) = hi;
+          *reinterpret_cast<uint4*>(xp_lo + o) = lo;
+        }
+        fence_proxy_async_smem();
+      }
+      mbar_arrive(&sh->xp_ready);
+    }
+  } else {
+    // ---- state warps: S operand, outputs, state update ----
+    constexpr int kHalf = kP / 2;
+    const int q = warp & 3, half = (warp - 2 - kGroup / 32) >> 2;
+    const int r = q * 32 + lane;   // row of the state, and token of the outputs
+    const uint32_t lane_off = static_cast<uint32_t>(q * 32) << 16;
+    uint8_t* s_hi = smem + kOffS;
+    uint8_t* s_lo = s_hi + kXBytes;
+    float* gs = a.state + ((static_cast<int64_t>(a.sb.ids[b]) * a.s.H + h) * kN + r) * a.s.P + p0 + half * kHalf;
     float S[kHalf];
     if (a.sb.start[b] > 0) {
 #pragma unroll
@@ -219,17 +362,8 @@ ssd_scan_sm100_kernel(const __grid_constant__ CUtensorMap t_xbc, const __grid_co
 #pragma unroll
       for (int j = 0; j < kHalf; ++j) S[j] = 0.f;
     }
-    const float bias = a.dt_bias[h], decay = -expf(a.a_log[h]) * 1.4426950408889634f, dsk = a.d_skip[h];
-    auto load_dt = [&](int n) -> float {
-      const int t = n * kL + r;
-      return (half == 0 && t < len) ? __bfloat162float(a.dt_raw[static_cast<int64_t>(first + t) * a.ld_dt + h]) : 0.f;
-    };
-    float raw = load_dt(0);
     bool ok = true;
-    // ok may differ between warps after a timeout, but every compute warp runs every iteration with all its barriers
     for (int n = 0; n < n_chunks; ++n) {
-      const int st = n % C::kStages;
-      // ---- publish the state the chunk starts from ----
 #pragma unroll
       for (int j = 0; j < kHalf; j += 8) {
         uint4 hi, lo;
@@ -239,133 +373,42 @@ ssd_scan_sm100_kernel(const __grid_constant__ CUtensorMap t_xbc, const __grid_co
         *reinterpret_cast<uint4*>(s_lo + o) = lo;
       }
       fence_proxy_async_smem();
-      mbar_arrive(&bars->s_ready);
-      // ---- step sizes and running log-decays of the chunk ----
-      float cum = 0.f, dt = 0.f;
-      if (half == 0) {
-        dt = n * kL + r < len ? softplus_f(raw + bias) : 0.f;
-        cum = dt * decay;
-#pragma unroll
-        for (int o = 1; o < 32; o <<= 1) {
-          const float t = __shfl_up_sync(0xffffffffu, cum, o);
-          if (lane >= o) cum += t;
-        }
-        if (lane == 31) bars->part[q] = cum;
-      }
-      compute_sync();
-      if (half == 0) {
-        for (int k = 0; k < q; ++k) cum += bars->part[k];
-        cd[r] = make_float2(cum, dt);
-      }
-      if (n + 1 < n_chunks) raw = load_dt(n + 1);
-      compute_sync();
-      const float2 mine = cd[r];
-      const float c_end = cd[kL - 1].x;
-      // ---- X' and the skip term's x ----
-      if (ok && !mbar_wait(&bars->full[st], (n / C::kStages) & 1, abort_flag)) ok = false;
-      ok = __all_sync(0xffffffffu, ok);
-      uint32_t xs[kHalf / 2];
-      if (ok) {
-        const uint8_t* tx = smem + st * C::kStageBytes + 2 * kTileBytes;
-        const float w = ex2(c_end - mine.x) * mine.y;
-#pragma unroll
-        for (int j = 0; j < kHalf; j += 8) {
-          const uint32_t o = swz(r, half * kHalf + j);
-          const uint4 v = *reinterpret_cast<const uint4*>(tx + o);
-          xs[j / 2] = v.x; xs[j / 2 + 1] = v.y; xs[j / 2 + 2] = v.z; xs[j / 2 + 3] = v.w;
-          float f[8];
-#pragma unroll
-          for (int k = 0; k < 4; ++k) {
-            const float2 u = unpack_bf16x2(xs[j / 2 + k]);
-            f[2 * k] = u.x * w;
-            f[2 * k + 1] = u.y * w;
-          }
-          uint4 hi, lo;
-          split8(f, hi, lo);
-          *reinterpret_cast<uint4*>(xp_hi + o) = hi;
-          *reinterpret_cast<uint4*>(xp_lo + o) = lo;
-        }
-        fence_proxy_async_smem();
-      }
-      // ---- G -> G * L ----
-      if (ok && !mbar_wait(&bars->g_full, n & 1, abort_flag)) {
-        if (lane == 0) report_status(a.status, kWaitTmemFullTimeout, 313, h, n);
+      mbar_arrive(&sh->s_ready);
+      if (ok && (!mbar_wait(&sh->c_full[n & (kCd - 1)], (n / kCd) & 1, abort_flag) || !mbar_wait(&sh->y_full, n & 1, abort_flag))) {
+        if (lane == 0) report_status(a.status, kWaitTmemFullTimeout, 318, h, n);
         ok = false;
       }
       ok = __all_sync(0xffffffffu, ok);
-      uint32_t gh[32], gl[32];
-      if (ok) {
-        tc_fence_after();
+      if (!ok) continue;
+      tc_fence_after();
+      const float* c = sh->c[n & (kCd - 1)];
+      const float ei = ex2(c[r]), ee = ex2(c[kL - 1]);
+      const int t = n * kL + r;
+      __nv_bfloat16* yo = a.y + static_cast<int64_t>(first + t) * inner + h * a.s.P + p0 + half * kHalf;
+      const uint32_t tc = tmem + half * kHalf + lane_off;
 #pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          const int j0 = half * 64 + c * 32;
-          if (j0 <= q * 32 + 31) {   // warp-uniform: some column of the block is at or below the diagonal
-            uint32_t v[32];
-            tmem_ld_32x32(tmem + kColG + j0 + lane_off, v);
-            tmem_ld_wait();
+      for (int g = 0; g < kHalf; g += 16) {
+        uint32_t v[16], hi[16], lo[16];
+        tmem_ld_x16(tc + kColT + g, v);
+        tmem_ld_wait();
 #pragma unroll
-            for (int j = 0; j < 32; j += 2) {
-              const float2 c0 = cd[j0 + j], c1 = cd[j0 + j + 1];
-              const float m0 = j0 + j <= r ? __uint_as_float(v[j]) * ex2(mine.x - c0.x) * c0.y : 0.f;
-              const float m1 = j0 + j + 1 <= r ? __uint_as_float(v[j + 1]) * ex2(mine.x - c1.x) * c1.y : 0.f;
-              const uint32_t hw = pack_bf16x2(m0, m1);
-              const float2 f = unpack_bf16x2(hw);
-              gh[c * 16 + j / 2] = hw;
-              gl[c * 16 + j / 2] = pack_bf16x2(m0 - f.x, m1 - f.y);
-            }
-          } else {
+        for (int j = 0; j < 16; ++j) S[g + j] = fmaf(S[g + j], ee, __uint_as_float(v[j]));
+        tmem_ld_x16(tc + kColY + g, v);
+        tmem_ld_x16(tc + kColYo + g, hi);
+        tmem_ld_x16(tc + kColYo + kP + g, lo);
+        tmem_ld_wait();
+        if (t < len) {
+          uint32_t o[8];
 #pragma unroll
-            for (int j = 0; j < 16; ++j) gh[c * 16 + j] = gl[c * 16 + j] = 0u;
-          }
+          for (int j = 0; j < 8; ++j)
+            o[j] = pack_bf16x2(
+                fmaf(ei, __uint_as_float(hi[2 * j]) + __uint_as_float(lo[2 * j]), __uint_as_float(v[2 * j])),
+                fmaf(ei, __uint_as_float(hi[2 * j + 1]) + __uint_as_float(lo[2 * j + 1]), __uint_as_float(v[2 * j + 1])));
+          *reinterpret_cast<uint4*>(yo + g) = make_uint4(o[0], o[1], o[2], o[3]);
+          *reinterpret_cast<uint4*>(yo + g + 8) = make_uint4(o[4], o[5], o[6], o[7]);
         }
-        tc_fence_before();
       }
-      compute_sync();   // every warp has read its part of G: the region may be overwritten
-      if (ok) {
-        tc_fence_after();
-        tmem_st_32x32(tmem + kColG + half * 32 + lane_off, gh);
-        tmem_st_32x32(tmem + kColG + 64 + half * 32 + lane_off, gl);
-        tmem_st_wait();
-        tc_fence_before();
-      }
-      mbar_arrive(&bars->m_ready);
-      if (ok && !mbar_wait(&bars->y_full, n & 1, abort_flag)) {
-        if (lane == 0) report_status(a.status, kWaitTmemFullTimeout, 314, h, n);
-        ok = false;
-      }
-      ok = __all_sync(0xffffffffu, ok);
-      if (ok) {
-        tc_fence_after();
-        const float ei = ex2(mine.x), ee = ex2(c_end);
-        const int t = n * kL + r;
-        __nv_bfloat16* yo = a.y + static_cast<int64_t>(first + t) * inner + h * P + half * kHalf;
-#pragma unroll
-        for (int c = 0; c < kHalf; c += 32) {
-          uint32_t v[32], u[32];
-          tmem_ld_32x32(tmem + kColY + half * kHalf + c + lane_off, v);
-          tmem_ld_32x32(tmem + kColYo + half * kHalf + c + lane_off, u);
-          tmem_ld_wait();
-          if (t < len) {
-#pragma unroll
-            for (int j = 0; j < 32; j += 8) {
-              uint32_t o[4];
-#pragma unroll
-              for (int k = 0; k < 4; ++k) {
-                const float2 x = unpack_bf16x2(xs[(c + j) / 2 + k]);
-                const int i = j + 2 * k;
-                o[k] = pack_bf16x2(fmaf(dsk, x.x, fmaf(ei, __uint_as_float(u[i]), __uint_as_float(v[i]))),
-                                   fmaf(dsk, x.y, fmaf(ei, __uint_as_float(u[i + 1]), __uint_as_float(v[i + 1]))));
-              }
-              *reinterpret_cast<uint4*>(yo + c + j) = make_uint4(o[0], o[1], o[2], o[3]);
-            }
-          }
-          tmem_ld_32x32(tmem + kColT + half * kHalf + c + lane_off, v);
-          tmem_ld_wait();
-#pragma unroll
-          for (int j = 0; j < 32; ++j) S[c + j] = fmaf(S[c + j], ee, __uint_as_float(v[j]));
-        }
-        tc_fence_before();
-      }
+      tc_fence_before();
     }
     if (ok) {
 #pragma unroll
@@ -380,24 +423,10 @@ ssd_scan_sm100_kernel(const __grid_constant__ CUtensorMap t_xbc, const __grid_co
   }
 }
 
-template <int P>
-cudaError_t ssd_launch(const CUtensorMap& m, const SsdArgs& a, cudaStream_t st) {
-  static bool configured = false;
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(ssd_scan_sm100_kernel<P>, cudaFuncAttributeMaxDynamicSharedMemorySize, SsdCfg<P>::kSmem);
-    if (e != cudaSuccess) return e;
-    configured = true;
-  }
-  static_assert(SsdCfg<P>::kSmem <= 227 * 1024, "shared memory");
-  static_assert(sizeof(SsdBars) <= 192, "barrier block");
-  ssd_scan_sm100_kernel<P><<<dim3(a.s.H, a.sb.n_seq), kThreads, SsdCfg<P>::kSmem, st>>>(m, a);
-  return cudaGetLastError();
-}
-
 }  // namespace
 
 bool ssd_scan_sm100_ok(const SsdShape& s) {
-  return s.N == kN && (s.P == 64 || s.P == 128) && s.G >= 1 && s.H % s.G == 0;
+  return s.N == kN && s.P >= kP && s.P % kP == 0 && s.G >= 1 && s.H % s.G == 0;
 }
 
 cudaError_t launch_ssd_scan_sm100(const SeqBatch& sb, const __nv_bfloat16* xbc, const __nv_bfloat16* dt_raw, int64_t ld_dt,
@@ -408,8 +437,15 @@ cudaError_t launch_ssd_scan_sm100(const SeqBatch& sb, const __nv_bfloat16* xbc, 
   CUtensorMap m;
   cudaError_t e = encode_tma_2d(&m, xbc, 2, cols, sb.n_tok, cols * 2, 64, kL);
   if (e != cudaSuccess) return e;
+  static bool configured = false;
+  if (!configured) {
+    e = cudaFuncSetAttribute(ssd_scan_sm100_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmem);
+    if (e != cudaSuccess) return e;
+    configured = true;
+  }
   const SsdArgs a{sb, dt_raw, ld_dt, dt_bias, a_log, d_skip, state, y, s, status};
-  return s.P == 64 ? ssd_launch<64>(m, a, st) : ssd_launch<128>(m, a, st);
+  ssd_scan_sm100_kernel<<<dim3(s.H * (s.P / kP), sb.n_seq), kThreads, kSmem, st>>>(m, a);
+  return cudaGetLastError();
 }
 
 }  // namespace b200

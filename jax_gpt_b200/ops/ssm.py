@@ -34,7 +34,7 @@ def ssm_conv(batch: PackedBatch, x, w, bias, ring) -> torch.Tensor:
 
 def chunked_ok(x, state) -> bool:
     """True when the tensor-core form of the recurrence takes these tensors."""
-    return x.is_cuda and x.dtype == torch.bfloat16 and state.shape[2] == 128 and state.shape[3] in (64, 128)
+    return x.is_cuda and x.dtype == torch.bfloat16 and state.shape[2] == 128 and state.shape[3] % 64 == 0
 
 
 def ssd_scan(batch: PackedBatch, xbc, dt_raw, dt_bias, a_log, d_skip, state, groups: int, chunked=None) -> torch.Tensor:

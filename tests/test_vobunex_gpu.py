@@ -120,15 +120,15 @@ def test_tensor_core_shapes_continued_prompt():
     assert float((got - want).pow(2).mean(-1).sqrt().max() / want.std(-1).mean()) < 0.12
 
 
-@pytest.mark.parametrize("P,H,G", [(64, 6, 3), (128, 2, 1)])
+@pytest.mark.parametrize("P,H,G", [(64, 6, 3), (128, 2, 1), (192, 2, 2)])
 def test_chunked_scan(P, H, G):
     """Chunk edges, tails, carried state; decays slow enough that an early token stays in the state across chunks."""
     from jax_gpt_b200.ops import ssm
     from jax_gpt_b200.ops.packed import PackedBatch, seq_begin
     N = 128
     g = torch.Generator().manual_seed(P)
-    lens = [127, 128, 129, 1, 260, 2]
-    b = PackedBatch.make([5, 0, 3, 1, 2, 4], lens, True, 300, DEV)
+    lens = [127, 128, 129, 1, 700, 2]
+    b = PackedBatch.make([5, 0, 3, 1, 2, 4], lens, True, 800, DEV)
     n, C = sum(lens), H * P + 2 * G * N
     xbc = torch.randn(n, C, generator=g).bfloat16()
     first = 0
