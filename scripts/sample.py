@@ -3,7 +3,7 @@ with the GPT-2 BPE, generate with the KV cache, decode and print.
 
     python scripts/sample.py --checkpoint_dir checkpoints/ --prompt "Hello" --new_tokens 50 --top_k 40
     python scripts/sample.py --preset gpt2-tiny --random-weights --prompt "abc"
-    python scripts/sample.py --model-dir DIR --prompt-ids 5,17,3        # any registered family that loads from a folder
+    python scripts/sample.py --model-dir DIR --prompt-ids 12,40,7        # any registered family that loads from a folder
 """
 from __future__ import annotations
 
