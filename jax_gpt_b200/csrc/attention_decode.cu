@@ -38,6 +38,7 @@ struct DecArgs {
   const int* seq_ids;
   const int* lens;
   int page_size, max_pages;
+  int window, keep_first;   // window > 0: of the valid keys only the last `window` and the first `keep_first` are seen
 };
 
 template <int D, int G>
@@ -55,13 +56,18 @@ attn_decode_split_kernel(const DecArgs a) {
   const int seq = a.table != nullptr ? a.seq_ids[b] : b;
   const int len = a.table != nullptr ? a.lens[seq] + a.len_add : (a.pos_ptr != nullptr ? a.pos_ptr[0] + a.len_add : a.len);
   const int* pages = a.table != nullptr ? a.table + static_cast<int64_t>(seq) * a.max_pages : nullptr;
-  // cache row of key t: the key index itself for a dense cache, page * page_size + offset for a paged one
+  // The seen keys are numbered through: the kept first ones, then the window (which may start among them).
+  const int n_keep = a.window > 0 ? min(a.keep_first, len) : 0;
+  const int w0 = a.window > 0 ? max(n_keep, len - a.window) : 0;
+  const int n_seen = n_keep + len - w0;
+  // cache row of seen key t: its position for a dense cache, page * page_size + offset for a paged one
   auto key_row = [&](int t) -> int64_t {
+    if (t >= n_keep) t += w0 - n_keep;
     if (pages == nullptr) return t;
     return static_cast<int64_t>(pages[t / a.page_size]) * a.page_size + t % a.page_size;
   };
-  const int per = ((len + n_splits - 1) / n_splits + KPS - 1) / KPS * KPS;
-  const int k0 = split * per, k1 = min(len, k0 + per);
+  const int per = ((n_seen + n_splits - 1) / n_splits + KPS - 1) / KPS * KPS;
+  const int k0 = split * per, k1 = min(n_seen, k0 + per);
 
   float qf[G][8];
 #pragma unroll
@@ -232,7 +238,7 @@ cudaError_t launch_attn_decode(const __nv_bfloat16* q, int64_t ldq, const __nv_b
       ldq % 8 != 0)
     return cudaErrorInvalidValue;
   DecArgs a{q, ldq, k, v, kv_stride_b, kv_stride_h, kv_stride_t, pos_ptr, len, len_add, H, Hkv,
-            scale * 1.4426950408889634f, part_o, part_ml, nullptr, nullptr, nullptr, 0, 0};
+            scale * 1.4426950408889634f, part_o, part_ml, nullptr, nullptr, nullptr, 0, 0, 0, 0};
   switch (D) {
     case 64: return decode_dispatch_g<64>(a, B, n_splits, out, ldo, stream);
     case 128: return decode_dispatch_g<128>(a, B, n_splits, out, ldo, stream);
@@ -244,12 +250,14 @@ cudaError_t launch_attn_decode(const __nv_bfloat16* q, int64_t ldq, const __nv_b
 cudaError_t launch_attn_decode_paged(const __nv_bfloat16* q, int64_t ldq, const __nv_bfloat16* pool, int width,
                                      const int* block_table, const int* seq_ids, const int* seq_lens, int len_add,
                                      int page_size, int max_pages, int B, int H, int Hkv, int D, float scale, int n_splits,
-                                     float* part_o, float* part_ml, __nv_bfloat16* out, int64_t ldo, cudaStream_t stream) {
-  if (H % Hkv != 0 || n_splits < 1 || width != 2 * Hkv * D || width % 8 != 0 || ldq % 8 != 0 || page_size < 1)
+                                     float* part_o, float* part_ml, __nv_bfloat16* out, int64_t ldo, cudaStream_t stream,
+                                     int window, int keep_first) {
+  if (H % Hkv != 0 || n_splits < 1 || width != 2 * Hkv * D || width % 8 != 0 || ldq % 8 != 0 || page_size < 1 || keep_first < 0)
     return cudaErrorInvalidValue;
   // a pool row holds K of every kv head, then V of every kv head
   DecArgs a{q, ldq, pool, pool + Hkv * D, 0, D, width, nullptr, 0, len_add, H, Hkv,
-            scale * 1.4426950408889634f, part_o, part_ml, block_table, seq_ids, seq_lens, page_size, max_pages};
+            scale * 1.4426950408889634f, part_o, part_ml, block_table, seq_ids, seq_lens, page_size, max_pages,
+            window, keep_first};
   switch (D) {
     case 64: return decode_dispatch_g<64>(a, B, n_splits, out, ldo, stream);
     case 128: return decode_dispatch_g<128>(a, B, n_splits, out, ldo, stream);

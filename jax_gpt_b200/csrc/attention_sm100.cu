@@ -19,6 +19,7 @@
 #include "attention_sm100.cuh"
 
 #include <algorithm>
+#include <climits>
 #include <cstdlib>
 
 #include "common.cuh"
@@ -43,6 +44,7 @@ struct FwdArgs {
   float* lse;
   int* status;
   const float* sink;        // [H] or nullptr: extra term exp(sink[h]) of the softmax denominator
+  int window, keep_first;   // keys j with i - j < window or j < keep_first are seen (window INT_MAX: all)
 };
 
 // D: width of q and k heads; DV: width of v heads (MLA prefill uses 192 / 128).
@@ -104,7 +106,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
   const int h = blockIdx.x, b = blockIdx.y;
   const int hkv = h / (a.H / a.Hkv);
   const int n_kv_all = (a.Tk + 127) / 128;
-  const int n_kv = a.causal ? min((a.q_pos0 + q_blk * 128 + 127) / 128 + 1, n_kv_all) : n_kv_all;
+  const int q0 = a.q_pos0 + q_blk * 128;     // position of the block's first query
+  const int n_seen = a.causal ? min((q0 + 127) / 128 + 1, n_kv_all) : n_kv_all;
+  // key tiles: those of the kept first keys, then those from the window of the first query on
+  const int n_keep = min((a.keep_first + 127) / 128, n_seen);
+  const int w_tile = max(n_keep, min(max(0, q0 - a.window + 1) / 128, n_seen));
+  const int n_kv = n_keep + n_seen - w_tile;
+  auto key_tile = [&](int j) { return j < n_keep ? j : w_tile + j - n_keep; };
   const int row0 = b * a.T + q_blk * 128;
   const int kv_row0 = b * a.kv_rows_b + hkv * a.kv_rows_h;
 
@@ -145,8 +153,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         }
         uint8_t* sK = smem + C::kOffK + s * C::kStageBytes;
         mbar_arrive_expect_tx(&bars->kv_full[s], C::kStageBytes);
-        load_tile<D>(sK, &tk, &bars->kv_full[s], hkv * a.k_col_h, kv_row0 + j * 128);
-        load_tile<DV>(sK + C::kQTile, &tv, &bars->kv_full[s], hkv * a.v_col_h, kv_row0 + j * 128);
+        const int kv_row = kv_row0 + key_tile(j) * 128;
+        load_tile<D>(sK, &tk, &bars->kv_full[s], hkv * a.k_col_h, kv_row);
+        load_tile<DV>(sK + C::kQTile, &tv, &bars->kv_full[s], hkv * a.v_col_h, kv_row);
       }
     }
   } else if (warp == 1) {
@@ -217,8 +226,13 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         break;
       }
       tc_fence_after();
-      const bool need_mask = (a.causal && j * 128 + 127 > a.q_pos0 + q_blk * 128) || ((j + 1) * 128 > a.Tk);
-      const int kv0 = j * 128 + half * 64;
+      const int kt0 = key_tile(j) * 128;
+      const bool need_mask = (a.causal && kt0 + 127 > q0) || kt0 + 128 > a.Tk ||
+                             (q0 + 127 - kt0 >= a.window && kt0 + 127 >= a.keep_first);
+      auto hidden = [&](int kv) {
+        return kv >= a.Tk || (a.causal && kv > qpos) || (qpos - kv >= a.window && kv >= a.keep_first);
+      };
+      const int kv0 = kt0 + half * 64;
       float mx = -INFINITY;
 #pragma unroll 1
       for (int c = 0; c < 2; ++c) {
@@ -228,10 +242,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           float s = __uint_as_float(v[i]);   // the (positive) softmax scale is applied to the maximum once, below
-          if (need_mask) {
-            const int kvpos = kv0 + c * 32 + i;
-            if (kvpos >= a.Tk || (a.causal && kvpos > qpos)) s = -INFINITY;
-          }
+          if (need_mask && hidden(kv0 + c * 32 + i)) s = -INFINITY;
           mx = fmaxf(mx, s);
         }
       }
@@ -260,8 +271,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
           float s0 = fmaf(__uint_as_float(v[i]), a.scale_log2, -mref), s1 = fmaf(__uint_as_float(v[i + 1]), a.scale_log2, -mref);
           if (need_mask) {
             const int kvpos = kv0 + c * 32 + i;
-            if (kvpos >= a.Tk || (a.causal && kvpos > qpos)) s0 = -INFINITY;
-            if (kvpos + 1 >= a.Tk || (a.causal && kvpos + 1 > qpos)) s1 = -INFINITY;
+            if (hidden(kvpos)) s0 = -INFINITY;
+            if (hidden(kvpos + 1)) s1 = -INFINITY;
           }
           const float p0 = exp2f(s0), p1 = exp2f(s1);
           rs += p0 + p1;
@@ -751,7 +762,8 @@ cudaError_t fwd_launch(const AttnTensors& t, const AttnShape& s, const AttnKvLay
     configured = true;
   }
   FwdArgs a{s.B, s.T, kv.Tk, s.H, s.Hkv, kv.q_pos0, kv.rows_b, kv.rows_h, kv.k_col_h, kv.v_col_h,
-            s.scale * kLog2e, s.causal, out, ldo, lse, status, s.sink};
+            s.scale * kLog2e, s.causal, out, ldo, lse, status, s.sink, s.window > 0 ? s.window : INT_MAX,
+            s.window > 0 ? std::min(s.keep_first, 1 << 30) : 0};
   dim3 grid(s.H, s.B, (s.T + 127) / 128);
   kernel<<<grid, kThreads, C::kSmem, stream>>>(tq, tk, tv, a);
   return cudaGetLastError();
@@ -802,7 +814,7 @@ cudaError_t bwd_launch(const AttnTensors& t, const AttnShape& s, const __nv_bflo
 
 cudaError_t launch_attn_fwd_kv(const AttnTensors& t, const AttnShape& s, const AttnKvLayout& kv, __nv_bfloat16* out,
                                int64_t ldo, float* lse, int* status, cudaStream_t stream) {
-  if (s.H % s.Hkv != 0) return cudaErrorInvalidValue;
+  if (s.H % s.Hkv != 0 || (s.window > 0 && (!s.causal || s.keep_first < 0))) return cudaErrorInvalidValue;
   const int dv = s.Dv > 0 ? s.Dv : s.D;
   if (s.D == 64 && dv == 64) {
     // two-tile kernel unless the single-tile one is asked for (B200_ATTN_FWD=1tile: comparisons, fallback)
@@ -810,7 +822,7 @@ cudaError_t launch_attn_fwd_kv(const AttnTensors& t, const AttnShape& s, const A
       const char* e = getenv("B200_ATTN_FWD");
       return e != nullptr && e[0] == '1';
     }();
-    if (!one_tile && s.sink == nullptr) return launch_attn_fwd2_d64(t, s, kv, out, ldo, lse, status, stream);
+    if (!one_tile && s.sink == nullptr && s.window <= 0) return launch_attn_fwd2_d64(t, s, kv, out, ldo, lse, status, stream);
     return fwd_launch<64, 64>(t, s, kv, out, ldo, lse, status, stream);
   }
   if (s.D == 128 && dv == 128) return fwd_launch<128, 128>(t, s, kv, out, ldo, lse, status, stream);

@@ -5,6 +5,7 @@
 #include <torch/library.h>
 #include <torch/torch.h>
 
+#include <algorithm>
 #include <cstring>
 #include <tuple>
 #include <vector>
@@ -316,7 +317,8 @@ void adamw_bf16_state(Tensor p, Tensor g, Tensor m, Tensor v, const Tensor& hp, 
 
 // q/k/v: 2-D bf16 views [B*T, H*D] (possibly column slices of one fused buffer).
 void attn_fwd(const Tensor& q, const Tensor& k, const Tensor& v, Tensor out, Tensor lse, int64_t B, int64_t T,
-              int64_t H, int64_t Hkv, int64_t D, double scale, bool causal, int64_t Dv, const c10::optional<Tensor>& sink) {
+              int64_t H, int64_t Hkv, int64_t D, double scale, bool causal, int64_t Dv, const c10::optional<Tensor>& sink,
+              int64_t window, int64_t keep_first) {
   c10::cuda::CUDAGuard guard(q.device());
   check_bf16_2d(q, "q");
   check_bf16_2d(k, "k");
@@ -329,6 +331,8 @@ void attn_fwd(const Tensor& q, const Tensor& k, const Tensor& v, Tensor out, Ten
     TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == at::kFloat && sink->numel() == H, "attn_fwd: sink is [H] fp32");
     s.sink = sink->data_ptr<float>();
   }
+  s.window = static_cast<int>(std::min<int64_t>(window, 1 << 30));
+  s.keep_first = static_cast<int>(std::min<int64_t>(keep_first, 1 << 30));
   B200_CHECK_CUDA(b200::launch_attn_fwd(t, s, bf16_mut(out), out.stride(0), lse.data_ptr<float>(), status_ptr(q),
                                         cur_stream()));
 }
@@ -450,7 +454,7 @@ void attn_decode(const Tensor& q, const Tensor& kcache, const Tensor& vcache, co
 // then V), block_table [max_seqs, max_pages] / seq_ids [B] / seq_lens [max_seqs] int32 on the device.
 void attn_decode_paged(const Tensor& q, const Tensor& pool, const Tensor& block_table, const Tensor& seq_ids,
                        const Tensor& seq_lens, int64_t len_add, int64_t H, int64_t Hkv, double scale, Tensor part_o,
-                       Tensor part_ml, Tensor out) {
+                       Tensor part_ml, Tensor out, int64_t window, int64_t keep_first) {
   c10::cuda::CUDAGuard guard(q.device());
   check_bf16_2d(q, "q");
   check_bf16_2d(out, "out");
@@ -472,7 +476,8 @@ void attn_decode_paged(const Tensor& q, const Tensor& pool, const Tensor& block_
       seq_ids.data_ptr<int>(), seq_lens.data_ptr<int>(), static_cast<int>(len_add), static_cast<int>(pool.size(1)),
       static_cast<int>(block_table.size(1)), static_cast<int>(B), static_cast<int>(H), static_cast<int>(Hkv),
       static_cast<int>(D), static_cast<float>(scale), static_cast<int>(part_o.size(2)), part_o.data_ptr<float>(),
-      part_ml.data_ptr<float>(), bf16_mut(out), out.stride(0), cur_stream()));
+      part_ml.data_ptr<float>(), bf16_mut(out), out.stride(0), cur_stream(),
+      static_cast<int>(std::min<int64_t>(window, 1 << 30)), static_cast<int>(std::min<int64_t>(keep_first, 1 << 30))));
 }
 
 void attn_bwd_probs(Tensor s, Tensor dp, const Tensor& lse, const Tensor& delta, int64_t c, int64_t q0, double scale,
@@ -544,7 +549,7 @@ TORCH_LIBRARY(b200, m) {
       &adamw);
   m.def(
       "attn_fwd(Tensor q, Tensor k, Tensor v, Tensor(a!) out, Tensor(b!) lse, int B, int T, int H, int Hkv, int D, "
-      "float scale, bool causal, int Dv, Tensor? sink=None) -> ()",
+      "float scale, bool causal, int Dv, Tensor? sink=None, int window=0, int keep_first=0) -> ()",
       &attn_fwd);
   m.def(
       "attn_bwd(Tensor q, Tensor k, Tensor v, Tensor out, Tensor dout, Tensor lse, Tensor(a!) delta, Tensor(b!) "
@@ -570,7 +575,7 @@ TORCH_LIBRARY(b200, m) {
       &attn_decode);
   m.def(
       "attn_decode_paged(Tensor q, Tensor pool, Tensor block_table, Tensor seq_ids, Tensor seq_lens, int len_add, int H, "
-      "int Hkv, float scale, Tensor(a!) part_o, Tensor(b!) part_ml, Tensor(c!) out) -> ()",
+      "int Hkv, float scale, Tensor(a!) part_o, Tensor(b!) part_ml, Tensor(c!) out, int window=0, int keep_first=0) -> ()",
       &attn_decode_paged);
   m.def("attn_bwd_probs(Tensor(a!) s, Tensor(b!) dp, Tensor lse, Tensor delta, int c, int q0, float scale, bool causal) -> ()", &attn_bwd_probs);
   m.def("norm_bwd_scratch_floats(int D) -> int", [](int64_t D) { return b200::norm_bwd_scratch_floats(static_cast<int>(D)); });

@@ -102,6 +102,10 @@ _Pragma("unroll") for (int j = 0; j < 32; ++j)
       f[j] = r * r;
     }
   }
+  if (args.epilogue == kEpiSilu) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) f[j] = __fdividef(f[j], 1.f + __expf(-f[j]));
+  }
   if (args.residual != nullptr && ks == 0) {
     const __nv_bfloat16* res = args.residual + static_cast<int64_t>(row) * args.ldr + col0;
     if (full && (args.ldr & 7) == 0) {
@@ -265,6 +269,10 @@ __device__ __forceinline__ void gemm_epilogue_group64(const GemmArgs& args, uint
         const float r = fmaxf(f[j], 0.f);
         f[j] = r * r;
       }
+    }
+    if (args.epilogue == kEpiSilu) {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) f[j] = __fdividef(f[j], 1.f + __expf(-f[j]));
     }
 #pragma unroll
     for (int j = 0; j < 32; j += 8) {

@@ -13,6 +13,7 @@ enum GemmEpilogue : int {
   kEpiGeluGrad = 2,  // out = acc * gelu_tanh'(aux_in)
   kEpiSiluMul = 3,   // reserved for SwiGLU-style epilogues
   kEpiRelu2 = 4,     // out = max(acc + bias, 0)^2
+  kEpiSilu = 5,      // out = silu(acc + bias)
 };
 enum GemmOut : int {
   kOutBf16 = 0,       // store bf16

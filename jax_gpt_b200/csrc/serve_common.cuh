@@ -1,6 +1,7 @@
-// Small device helpers of the serving kernels: typed loads and stores, block reductions.
+// Small helpers of the serving kernels: typed loads and stores, block reductions, page lookup.
 #pragma once
 #include "common.cuh"
+#include "serve_kernels.cuh"
 
 namespace b200 {
 
@@ -74,5 +75,24 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+
+// Row of position `pos` of cache slot `slot` in a page pool, or -1.
+__device__ __forceinline__ int64_t page_row(const PagedRows& pg, int slot, int pos) {
+  const int pi = pos / pg.page_size;
+  if (pi >= pg.max_pages) return -1;
+  const int page = pg.block_table[static_cast<int64_t>(slot) * pg.max_pages + pi];
+  if (page < 0 || page >= pg.n_pages) return -1;
+  return static_cast<int64_t>(page) * pg.page_size + pos % pg.page_size;
+}
+
+// Opts a kernel into `bytes` of dynamic shared memory once per new maximum.
+template <typename K>
+inline cudaError_t want_smem(K kernel, int bytes, int& have) {
+  if (bytes <= 48 * 1024 || bytes <= have) return cudaSuccess;
+  if (bytes > 227 * 1024) return cudaErrorInvalidValue;
+  cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+  if (e == cudaSuccess) have = bytes;
+  return e;
+}
 
 }  // namespace b200

@@ -1,7 +1,7 @@
 // Serving kernels of models whose layers run on packed (ragged) batches with a 32-bit residual: sequence
-// bookkeeping, embedding plus bigram table, norms, few-row linear layers (decode), multi-head latent attention over
-// paged latent rows (RMS-normed latents, interleaved rotary part, absorbed weights, softmax with a sink), and experts
-// chosen by a token table with a clamped gated activation.
+// bookkeeping, embedding plus bigram table, norms (also post-norm + residual + next pre-norm in one pass), few-row linear
+// layers (decode), multi-head latent attention over paged latent rows (RMS-normed latents, interleaved rotary part,
+// absorbed weights, softmax with a sink), and experts chosen by a token table or by a sigmoid router.
 //
 // Every kernel exists for fp32 and bf16 activations; accumulation, norms, angles, scores and softmax are fp32 in both.
 // This file is built without fast-math: the fp32 instances are meant to be exact to rounding.
@@ -143,6 +143,102 @@ void norm_rows_go(int mode, const float* x, const float* gamma, const float* bet
   else norm_rows_kernel<TO><<<rows, D >= 1024 ? 256 : (D >= 256 ? 128 : 64), 0, st>>>(mode, x, gamma, beta, out, D, eps);
 }
 
+// ---- post-norm into the residual, then the next pre-norm --------------------------------------------------------------
+// x = (add ? x : 0) + rms(y) gpost, out = rms(x) gnext in one pass over the row (out null: the first half only).
+template <typename TY, typename TO>
+__global__ void residual_norm_kernel(const TY* __restrict__ y, const float* __restrict__ gpost, float* __restrict__ x, int add,
+                                     const float* __restrict__ gnext, TO* __restrict__ out, int D, float eps) {
+  __shared__ float red[33];
+  const int64_t r0 = static_cast<int64_t>(blockIdx.x) * D;
+  float s = 0.f;
+  for (int i = threadIdx.x; i < D; i += blockDim.x) { const float v = ldf(y + r0 + i); s += v * v; }
+  const float iy = 1.f / sqrtf(block_sum(s, red) / D + eps);
+  s = 0.f;
+  for (int i = threadIdx.x; i < D; i += blockDim.x) {
+    const float v = (add ? x[r0 + i] : 0.f) + ldf(y + r0 + i) * iy * gpost[i];
+    x[r0 + i] = v;
+    s += v * v;
+  }
+  if (out == nullptr) return;
+  const float ix = 1.f / sqrtf(block_sum(s, red) / D + eps);
+  for (int i = threadIdx.x; i < D; i += blockDim.x) stf(out + r0 + i, x[r0 + i] * ix * gnext[i]);
+}
+
+template <typename T>
+__device__ __forceinline__ float4 ld4(const T* p) {
+  if constexpr (sizeof(T) == 2) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_bf16x2(v.x), b = unpack_bf16x2(v.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+  } else {
+    return *reinterpret_cast<const float4*>(p);
+  }
+}
+
+template <typename TY, typename TO, int kIt, int kThr>
+__global__ void __launch_bounds__(256)
+residual_norm_vec_kernel(const TY* __restrict__ y, const float* __restrict__ gpost, float* __restrict__ x, int add,
+                         const float* __restrict__ gnext, TO* __restrict__ out, int rows, int D, float eps) {
+  __shared__ float red[33];
+  constexpr int kPer = 256 / kThr;   // rows per block
+  const int row = blockIdx.x * kPer + threadIdx.x / kThr, t = threadIdx.x % kThr;
+  if (kThr == 32 && row >= rows) return;
+  auto total = [&](float v) { return kThr == 32 ? warp_sum(v) : block_sum(v, red); };
+  const int64_t r0 = static_cast<int64_t>(row) * D;
+  float4 v[kIt], a[kIt];
+  float s = 0.f;
+#pragma unroll
+  for (int k = 0; k < kIt; ++k) {
+    const int i = (k * kThr + t) * 4;
+    v[k] = a[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < D) {
+      v[k] = ld4(y + r0 + i);
+      if (add) a[k] = *reinterpret_cast<const float4*>(x + r0 + i);
+    }
+    s += (v[k].x * v[k].x + v[k].y * v[k].y) + (v[k].z * v[k].z + v[k].w * v[k].w);
+  }
+  const float iy = 1.f / sqrtf(total(s) / D + eps);
+  s = 0.f;
+#pragma unroll
+  for (int k = 0; k < kIt; ++k) {
+    const int i = (k * kThr + t) * 4;
+    if (i < D) {
+      const float4 g = *reinterpret_cast<const float4*>(gpost + i);
+      a[k].x += v[k].x * iy * g.x; a[k].y += v[k].y * iy * g.y; a[k].z += v[k].z * iy * g.z; a[k].w += v[k].w * iy * g.w;
+      *reinterpret_cast<float4*>(x + r0 + i) = a[k];
+      s += (a[k].x * a[k].x + a[k].y * a[k].y) + (a[k].z * a[k].z + a[k].w * a[k].w);
+    }
+  }
+  if (out == nullptr) return;
+  const float ix = 1.f / sqrtf(total(s) / D + eps);
+#pragma unroll
+  for (int k = 0; k < kIt; ++k) {
+    const int i = (k * kThr + t) * 4;
+    if (i < D) {
+      const float4 g = *reinterpret_cast<const float4*>(gnext + i);
+      const float4 r = make_float4(a[k].x * ix * g.x, a[k].y * ix * g.y, a[k].z * ix * g.z, a[k].w * ix * g.w);
+      if constexpr (sizeof(TO) == 2) *reinterpret_cast<uint2*>(out + r0 + i) = make_uint2(pack_bf16x2(r.x, r.y), pack_bf16x2(r.z, r.w));
+      else *reinterpret_cast<float4*>(out + r0 + i) = r;
+    }
+  }
+}
+
+template <typename TY, typename TO>
+void residual_norm_go(const TY* y, const float* gpost, float* x, int add, const float* gnext, TO* out, int rows, int D, float eps,
+                      cudaStream_t st) {
+  const bool vec = D % 4 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gpost) |
+                                   reinterpret_cast<uintptr_t>(gnext) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+#define B200_RN(IT, THR) \
+  residual_norm_vec_kernel<TY, TO, IT, THR><<<THR == 32 ? (rows + 7) / 8 : rows, 256, 0, st>>>(y, gpost, x, add, gnext, out, rows, D, eps)
+  if (vec && D <= 512 && rows >= 64) B200_RN(4, 32);
+  else if (vec && D <= 1024) B200_RN(1, 256);
+  else if (vec && D <= 2048) B200_RN(2, 256);
+  else if (vec && D <= 4096) B200_RN(4, 256);
+  else if (vec && D <= 8192) B200_RN(8, 256);
+  else residual_norm_kernel<TY, TO><<<rows, D >= 1024 ? 256 : (D >= 256 ? 128 : 64), 0, st>>>(y, gpost, x, add, gnext, out, D, eps);
+#undef B200_RN
+}
+
 // ---- few-row linear ------------------------------------------------------------------------------------------------
 constexpr int kLinWarps = 8;
 
@@ -151,16 +247,32 @@ __device__ __forceinline__ float row_act(float v, int act) {
     const float r = fmaxf(v, 0.f);
     return r * r;
   }
+  if (act == kActSilu) return silu_f(v);
   return v;
 }
 
-// A warp computes NR output features for up to MR rows; lanes stride the contraction in 16-byte vectors.
-template <typename T, int MR, int NR, bool kVec>
+template <typename T>
+__device__ __forceinline__ void rows_store(const RowsOut& o, int m, int n, float v) {
+  if (n >= o.n1) {
+    o.y2[static_cast<int64_t>(m) * o.ldy2 + n - o.n1] = v;
+    return;
+  }
+  v = row_act(v, o.act);
+  const int64_t i = static_cast<int64_t>(m) * o.ldy + n;
+  if (o.out_mode == 0) stf(static_cast<T*>(o.y) + i, v);
+  else if (o.out_mode == 1) static_cast<float*>(o.y)[i] = v;
+  else static_cast<float*>(o.y)[i] += v;
+}
+
+// A warp computes NR output features for up to MR rows; lanes stride the contraction in 16-byte vectors. kGlu (NR = 2):
+// one feature silu(gate) * up, rows n and N + n of w.
+template <typename T, int MR, int NR, bool kVec, bool kGlu>
 __global__ void __launch_bounds__(kLinWarps * 32)
-rows_linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, int64_t ldw, void* __restrict__ y,
-                   int64_t ldy, int M, int N, int K, int act, int out_mode) {
+rows_linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w, int64_t ldw, int M, int N, int K,
+                   const RowsOut out) {
+  static_assert(!kGlu || NR == 2, "gate and up");
   const int lane = threadIdx.x & 31;
-  const int n0 = (blockIdx.x * kLinWarps + (threadIdx.x >> 5)) * NR;
+  const int n0 = (blockIdx.x * kLinWarps + (threadIdx.x >> 5)) * (kGlu ? 1 : NR);
   const int m0 = blockIdx.y * MR;
   if (n0 >= N) return;
   float acc[MR][NR];
@@ -170,7 +282,7 @@ rows_linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w
     for (int r = 0; r < NR; ++r) acc[m][r] = 0.f;
   const T* wr[NR];
 #pragma unroll
-  for (int r = 0; r < NR; ++r) wr[r] = w + static_cast<int64_t>(n0 + r < N ? n0 + r : n0) * ldw;
+  for (int r = 0; r < NR; ++r) wr[r] = w + static_cast<int64_t>(kGlu ? n0 + r * N : (n0 + r < N ? n0 + r : n0)) * ldw;
   const T* xr[MR];
 #pragma unroll
   for (int m = 0; m < MR; ++m) xr[m] = x + static_cast<int64_t>(m0 + m < M ? m0 + m : m0) * ldx;
@@ -206,26 +318,24 @@ rows_linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w
 #pragma unroll
     for (int r = 0; r < NR; ++r) acc[m][r] = warp_sum(acc[m][r]);
 #pragma unroll
-  for (int m = 0; m < MR; ++m)
+  for (int m = 0; m < MR; ++m) {
+    if constexpr (kGlu) {
+      if (lane == m && m0 + m < M) rows_store<T>(out, m0 + m, n0, silu_f(acc[m][0]) * acc[m][1]);
+    } else {
 #pragma unroll
-    for (int r = 0; r < NR; ++r)
-      if (lane == ((m * NR + r) & 31) && m0 + m < M && n0 + r < N) {
-        const float v = row_act(acc[m][r], act);
-        const int64_t o = static_cast<int64_t>(m0 + m) * ldy + n0 + r;
-        if (out_mode == 0) stf(static_cast<T*>(y) + o, v);
-        else if (out_mode == 1) static_cast<float*>(y)[o] = v;
-        else static_cast<float*>(y)[o] += v;
-      }
+      for (int r = 0; r < NR; ++r)
+        if (lane == ((m * NR + r) & 31) && m0 + m < M && n0 + r < N) rows_store<T>(out, m0 + m, n0 + r, acc[m][r]);
+    }
+  }
 }
 
-template <typename T, int MR, int NR>
-void rows_linear_go(bool vec, const T* x, int64_t ldx, const T* w, int64_t ldw, void* y, int64_t ldy, int M, int N, int K,
-                    int act, int out_mode, cudaStream_t st) {
-  const dim3 grid((N + kLinWarps * NR - 1) / (kLinWarps * NR), (M + MR - 1) / MR);
-  if (vec)
-    rows_linear_kernel<T, MR, NR, true><<<grid, kLinWarps * 32, 0, st>>>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode);
-  else
-    rows_linear_kernel<T, MR, NR, false><<<grid, kLinWarps * 32, 0, st>>>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode);
+template <typename T, int MR, int NR, bool kGlu>
+void rows_linear_go(bool vec, const T* x, int64_t ldx, const T* w, int64_t ldw, int M, int N, int K, const RowsOut& out,
+                    cudaStream_t st) {
+  constexpr int kPer = kLinWarps * (kGlu ? 1 : NR);
+  const dim3 grid((N + kPer - 1) / kPer, (M + MR - 1) / MR);
+  if (vec) rows_linear_kernel<T, MR, NR, true, kGlu><<<grid, kLinWarps * 32, 0, st>>>(x, ldx, w, ldw, M, N, K, out);
+  else rows_linear_kernel<T, MR, NR, false, kGlu><<<grid, kLinWarps * 32, 0, st>>>(x, ldx, w, ldw, M, N, K, out);
 }
 
 // bf16, up to 8 * MT rows: weights are the A operand of mma.sync m16n8k16 (16 output features), activation rows the B
@@ -239,113 +349,115 @@ __device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a
                : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-template <int MT, int kW>   // kW warps per block
+template <int MT, int kW, bool kGlu>   // kW warps per block
 __global__ void __launch_bounds__(kW * 32)
 rows_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx, const __nv_bfloat16* __restrict__ w, int64_t ldw,
-                       void* __restrict__ y, int64_t ldy, int M, int N, int K, int act, int out_mode) {
-  __shared__ float red[kW][MT][32][4];
+                       int M, int N, int K, const RowsOut out) {
+  constexpr int kMat = kGlu ? 2 : 1;   // gate (and up) weights
+  __shared__ float red[kMat][kW][MT][32][4];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int n0 = blockIdx.x * 16;
   const __nv_bfloat16* w0 = w + static_cast<int64_t>(min(n0 + g, N - 1)) * ldw;
   const __nv_bfloat16* w1 = w + static_cast<int64_t>(min(n0 + g + 8, N - 1)) * ldw;
+  const int64_t up = static_cast<int64_t>(N) * ldw;
   const __nv_bfloat16* xr[MT];
 #pragma unroll
   for (int m = 0; m < MT; ++m) xr[m] = x + static_cast<int64_t>(min(m * 8 + g, M - 1)) * ldx;
-  float acc[MT][4];
+  float acc[kMat][MT][4];
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int q = 0; q < kMat; ++q)
 #pragma unroll
-    for (int j = 0; j < 4; ++j) acc[m][j] = 0.f;
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[q][m][j] = 0.f;
   const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
   constexpr int kU = MT == 1 ? 4 : 2;
   for (int kb = warp * 32; kb < K; kb += kW * 32 * kU) {
-    uint4 a[kU], c[kU], b[kU][MT];
+    uint4 a[kMat][kU], c[kMat][kU], b[kU][MT];
 #pragma unroll
     for (int u = 0; u < kU; ++u) {
       const int k = kb + u * kW * 32 + t * 8;
       const bool in = k < K;   // K is a multiple of 8
-      a[u] = in ? __ldg(reinterpret_cast<const uint4*>(w0 + k)) : zero;
-      c[u] = in ? __ldg(reinterpret_cast<const uint4*>(w1 + k)) : zero;
+#pragma unroll
+      for (int q = 0; q < kMat; ++q) {
+        a[q][u] = in ? __ldg(reinterpret_cast<const uint4*>(w0 + q * up + k)) : zero;
+        c[q][u] = in ? __ldg(reinterpret_cast<const uint4*>(w1 + q * up + k)) : zero;
+      }
 #pragma unroll
       for (int m = 0; m < MT; ++m) b[u][m] = in ? __ldg(reinterpret_cast<const uint4*>(xr[m] + k)) : zero;
     }
 #pragma unroll
     for (int u = 0; u < kU; ++u)
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        mma_16816(acc[m], a[u].x, c[u].x, a[u].y, c[u].y, b[u][m].x, b[u][m].y);
-        mma_16816(acc[m], a[u].z, c[u].z, a[u].w, c[u].w, b[u][m].z, b[u][m].w);
-      }
+      for (int q = 0; q < kMat; ++q)
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_16816(acc[q][m], a[q][u].x, c[q][u].x, a[q][u].y, c[q][u].y, b[u][m].x, b[u][m].y);
+          mma_16816(acc[q][m], a[q][u].z, c[q][u].z, a[q][u].w, c[q][u].w, b[u][m].z, b[u][m].w);
+        }
   }
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int q = 0; q < kMat; ++q)
 #pragma unroll
-    for (int j = 0; j < 4; ++j) red[warp][m][lane][j] = acc[m][j];
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) red[q][warp][m][lane][j] = acc[q][m][j];
   __syncthreads();
   // accumulator j of lane (g, t): feature g + 8 * (j / 2), row 2 t + j % 2
   for (int i = threadIdx.x; i < MT * 128; i += kW * 32) {
     const int m = i / 128, f = i % 16, r = (i / 16) % 8;
     const int src = (f % 8) * 4 + r / 2, j = (f / 8) * 2 + r % 2;
-    float v = 0.f;
+    float v[kMat];
 #pragma unroll
-    for (int q = 0; q < kW; ++q) v += red[q][m][src][j];
-    if (m * 8 + r < M && n0 + f < N) {
-      v = row_act(v, act);
-      const int64_t o = static_cast<int64_t>(m * 8 + r) * ldy + n0 + f;
-      if (out_mode == 0) static_cast<__nv_bfloat16*>(y)[o] = __float2bfloat16(v);
-      else if (out_mode == 1) static_cast<float*>(y)[o] = v;
-      else static_cast<float*>(y)[o] += v;
+    for (int p = 0; p < kMat; ++p) {
+      v[p] = 0.f;
+#pragma unroll
+      for (int q = 0; q < kW; ++q) v[p] += red[p][q][m][src][j];
     }
+    if (m * 8 + r < M && n0 + f < N) rows_store<__nv_bfloat16>(out, m * 8 + r, n0 + f, kGlu ? silu_f(v[0]) * v[kMat - 1] : v[0]);
   }
 }
 
-template <int MT>
-void rows_linear_mma_go(const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16* w, int64_t ldw, void* y, int64_t ldy, int M,
-                        int N, int K, int act, int out_mode, cudaStream_t st) {
+template <int MT, bool kGlu>
+void rows_linear_mma_go(const __nv_bfloat16* x, int64_t ldx, const __nv_bfloat16* w, int64_t ldw, int M, int N, int K,
+                        const RowsOut& out, cudaStream_t st) {
   const int grid = (N + 15) / 16;   // wide outputs: small blocks, so that all of them are resident at once
-  if (grid >= 296) rows_linear_mma_kernel<MT, 4><<<grid, 128, 0, st>>>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode);
-  else rows_linear_mma_kernel<MT, 8><<<grid, 256, 0, st>>>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode);
+  if (grid >= 296) rows_linear_mma_kernel<MT, 4, kGlu><<<grid, 128, 0, st>>>(x, ldx, w, ldw, M, N, K, out);
+  else rows_linear_mma_kernel<MT, 8, kGlu><<<grid, 256, 0, st>>>(x, ldx, w, ldw, M, N, K, out);
 }
 
-template <typename T>
-cudaError_t rows_linear_t(const void* x, int64_t ldx, const void* w, int64_t ldw, void* y, int64_t ldy, int M, int N, int K,
-                          int act, int out_mode, cudaStream_t st) {
+template <typename T, bool kGlu>
+cudaError_t rows_linear_t(const void* x, int64_t ldx, const void* w, int64_t ldw, int M, int N, int K, const RowsOut& out,
+                          cudaStream_t st) {
   const bool vec = K % Vec16<T>::n == 0 && ldx % Vec16<T>::n == 0 && ldw % Vec16<T>::n == 0 &&
                    (reinterpret_cast<uintptr_t>(x) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
   const T* xt = static_cast<const T*>(x);
   const T* wt = static_cast<const T*>(w);
-  // narrow outputs take fewer features per warp so that the grid still covers the SMs
   if constexpr (sizeof(T) == 2) {
     if (vec && M > 1 && M <= 32) {
-      if (M <= 8) rows_linear_mma_go<1>(xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st);
-      else if (M <= 16) rows_linear_mma_go<2>(xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st);
-      else rows_linear_mma_go<4>(xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st);
+      if (M <= 8) rows_linear_mma_go<1, kGlu>(xt, ldx, wt, ldw, M, N, K, out, st);
+      else if (M <= 16) rows_linear_mma_go<2, kGlu>(xt, ldx, wt, ldw, M, N, K, out, st);
+      else rows_linear_mma_go<4, kGlu>(xt, ldx, wt, ldw, M, N, K, out, st);
       return cudaGetLastError();
     }
   }
-  const bool wide = N >= 148 * kLinWarps * 4;
+  // narrow outputs take fewer features per warp so that the grid still covers the SMs
 #define B200_GO(MR)                                                                                       \
-  (wide ? rows_linear_go<T, MR, 4>(vec, xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st)             \
-        : (N >= 148 * kLinWarps * 2 ? rows_linear_go<T, MR, 2>(vec, xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st) \
-                                    : rows_linear_go<T, MR, 1>(vec, xt, ldx, wt, ldw, y, ldy, M, N, K, act, out_mode, st)))
-  if (M == 1) B200_GO(1);
-  else if (M == 2) B200_GO(2);
-  else if (M <= 4) B200_GO(4);
-  else B200_GO(8);
+  {                                                                                                       \
+    if constexpr (kGlu) rows_linear_go<T, MR, 2, true>(vec, xt, ldx, wt, ldw, M, N, K, out, st);          \
+    else if (N >= 148 * kLinWarps * 4) rows_linear_go<T, MR, 4, false>(vec, xt, ldx, wt, ldw, M, N, K, out, st); \
+    else if (N >= 148 * kLinWarps * 2) rows_linear_go<T, MR, 2, false>(vec, xt, ldx, wt, ldw, M, N, K, out, st); \
+    else rows_linear_go<T, MR, 1, false>(vec, xt, ldx, wt, ldw, M, N, K, out, st);                        \
+  }
+  if (M == 1) B200_GO(1)
+  else if (M == 2) B200_GO(2)
+  else if (M <= 4) B200_GO(4)
+  else B200_GO(8)
 #undef B200_GO
   return cudaGetLastError();
 }
 
 // ---- multi-head latent attention ------------------------------------------------------------------------------------
-// Row of position `pos` of cache slot `slot` in a page pool, or -1.
-__device__ __forceinline__ int64_t page_row(const PagedRows& pg, int slot, int pos) {
-  const int pi = pos / pg.page_size;
-  if (pi >= pg.max_pages) return -1;
-  const int page = pg.block_table[static_cast<int64_t>(slot) * pg.max_pages + pi];
-  if (page < 0 || page >= pg.n_pages) return -1;
-  return static_cast<int64_t>(page) * pg.page_size + pos % pg.page_size;
-}
-
 // Feature i of a rotary part read through `at(i)`, turned to position `pos`.
 template <typename F>
 __device__ __forceinline__ float rotated(const RopeTable& r, int pos, int i, F at) {
@@ -709,24 +821,79 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_o, const floa
   }
 }
 
-// ---- table-routed experts ---------------------------------------------------------------------------------------------
+// ---- experts -----------------------------------------------------------------------------------------------------
 __device__ __forceinline__ float clamped_glu(float g, float u, const GluArgs& a) {
   g = fminf(g, a.limit);
   u = fminf(fmaxf(u, -a.limit), a.limit);
-  return g * sigmoid_f(a.alpha * g) * (u + 1.f);
+  return g * sigmoid_f(a.alpha * g) * (u + a.shift);
+}
+
+// The next expert in order of falling logits (equal ones by index) after expert `pi` with logit `pv`; -1: none left.
+// Called by a whole warp with uniform arguments; every lane gets the result.
+__device__ __forceinline__ int next_best(const float* z, int E, float pv, int pi, float& value) {
+  float bv = -INFINITY;
+  int bi = -1;
+  for (int i = threadIdx.x & 31; i < E; i += 32) {
+    const float v = z[i];
+    if ((v < pv || (v == pv && i > pi)) && (bi < 0 || v > bv)) { bv = v; bi = i; }
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    if (oi >= 0 && (bi < 0 || ov > bv || (ov == bv && oi < bi))) { bv = ov; bi = oi; }
+  }
+  value = bv;
+  return bi;
+}
+
+// Expert number j of token m and the factor of the expert's input (a whole warp calls it). -1: bad token or table entry.
+__device__ __forceinline__ int choose_expert(const ExpertChoice& c, int m, int j, float& w) {
+  w = 1.f;
+  if (c.logits == nullptr) {
+    const int tok = c.tokens[m];
+    return tok >= 0 && tok < c.vocab ? c.table[static_cast<int64_t>(tok) * c.top + j] : -1;
+  }
+  const float* z = c.logits + static_cast<int64_t>(m) * c.E;
+  float v = INFINITY;
+  int e = -1;
+  for (int i = 0; i <= j; ++i) {
+    e = next_best(z, c.E, v, e, v);
+    if (e < 0) return -1;
+  }
+  w = sigmoid_f(v);
+  return e;
+}
+
+// One warp per token: ids and sigmoid scores of the `top` largest logits.
+__global__ void sigmoid_topk_kernel(const ExpertChoice c, int M, int* __restrict__ ids, float* __restrict__ weights, int* status) {
+  const int m = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (m >= M) return;
+  const float* z = c.logits + static_cast<int64_t>(m) * c.E;
+  float v = INFINITY;
+  int e = -1;
+  for (int j = 0; j < c.top; ++j) {
+    if (j == 0 || e >= 0) e = next_best(z, c.E, v, e, v);
+    if ((threadIdx.x & 31) == 0) {
+      if (e < 0) report_status(status, kBadArgument, 304, m, j);
+      ids[static_cast<int64_t>(m) * c.top + j] = e < 0 ? 0 : e;          // never past the expert table
+      weights[static_cast<int64_t>(m) * c.top + j] = e < 0 ? 0.f : sigmoid_f(v);
+    }
+  }
 }
 
 constexpr int kExpWarps = 8;
 
-// h[m * top + j, i] = glu(gate_e[i] . x[m], up_e[i] . x[m]) with e = table[token m, j]; w_gate_up [E, 2 I, D].
+// h[m * top + j, i] = glu(w gate_e[i] . x[m], w up_e[i] . x[m]) with the token's j-th expert e and its input factor w;
+// w_gate_up [E, 2 I, D].
 template <typename T, bool kVec>
 __global__ void __launch_bounds__(kExpWarps * 32)
-table_experts_up_kernel(const T* __restrict__ x, const int* __restrict__ tokens, const int* __restrict__ table, int vocab,
-                        int top, int E, const T* __restrict__ w, GluArgs glu, T* __restrict__ h, int D, int I, int* status) {
-  const int pair = blockIdx.x, m = pair / top;
-  const int tok = tokens[m];
-  const int e = tok >= 0 && tok < vocab ? table[static_cast<int64_t>(tok) * top + pair % top] : -1;
-  if (e < 0 || e >= E) {
+experts_up_kernel(const T* __restrict__ x, const ExpertChoice c, const T* __restrict__ w, GluArgs glu, T* __restrict__ h, int D,
+                  int I, int* status) {
+  const int pair = blockIdx.x, m = pair / c.top;
+  float wt;
+  const int e = choose_expert(c, m, pair % c.top, wt);
+  if (e < 0 || e >= c.E) {
     if (threadIdx.x == 0) report_status(status, kBadArgument, 303, m, e);
     return;
   }
@@ -759,26 +926,35 @@ table_experts_up_kernel(const T* __restrict__ x, const int* __restrict__ tokens,
     }
     g = warp_sum(g);
     u = warp_sum(u);
-    if (lane == 0) stf(h + static_cast<int64_t>(pair) * I + i, clamped_glu(g, u, glu));
+    if (lane == 0) stf(h + static_cast<int64_t>(pair) * I + i, clamped_glu(wt * g, wt * u, glu));
   }
 }
 
-// x[m, d] += 1 / top * sum_j down_e(j)[d] . h[m * top + j]; w_down [E, D, I].
+// x[m, d] += out_scale * sum_j down_e(j)[d] . h[m * top + j]; w_down [E, D, I]. Dynamic shared memory: top ints.
 template <typename T, bool kVec>
 __global__ void __launch_bounds__(kExpWarps * 32)
-table_experts_down_kernel(const T* __restrict__ h, const int* __restrict__ tokens, const int* __restrict__ table, int vocab,
-                          int top, int E, const T* __restrict__ w, float* __restrict__ x, int D, int I) {
+experts_down_kernel(const T* __restrict__ h, const ExpertChoice c, const T* __restrict__ w, float out_scale, float* __restrict__ x,
+                    int D, int I) {
+  extern __shared__ int chosen[];
   const int m = blockIdx.x;
-  const int tok = tokens[m];
-  if (tok < 0 || tok >= vocab) return;
   const int lane = threadIdx.x & 31;
+  if (threadIdx.x < 32) {
+    float v = INFINITY;
+    int e = -1;
+    for (int j = 0; j < c.top; ++j) {
+      if (c.logits == nullptr) e = choose_expert(c, m, j, v);
+      else if (j == 0 || e >= 0) e = next_best(c.logits + static_cast<int64_t>(m) * c.E, c.E, v, e, v);
+      if (lane == 0) chosen[j] = e;
+    }
+  }
+  __syncthreads();
   for (int d = blockIdx.y * kExpWarps + (threadIdx.x >> 5); d < D; d += gridDim.y * kExpWarps) {
     float acc = 0.f;
-    for (int j = 0; j < top; ++j) {
-      const int e = table[static_cast<int64_t>(tok) * top + j];
-      if (e < 0 || e >= E) continue;
+    for (int j = 0; j < c.top; ++j) {
+      const int e = chosen[j];
+      if (e < 0 || e >= c.E) continue;
       const T* wr = w + (static_cast<int64_t>(e) * D + d) * I;
-      const T* hr = h + (static_cast<int64_t>(m) * top + j) * I;
+      const T* hr = h + (static_cast<int64_t>(m) * c.top + j) * I;
       if constexpr (kVec) {
         constexpr int V = Vec16<T>::n;
 #pragma unroll 2
@@ -794,34 +970,38 @@ table_experts_down_kernel(const T* __restrict__ h, const int* __restrict__ token
       }
     }
     acc = warp_sum(acc);
-    if (lane == 0) x[static_cast<int64_t>(m) * D + d] += acc / top;
+    if (lane == 0) x[static_cast<int64_t>(m) * D + d] += acc * out_scale;
   }
 }
 
 __global__ void moe_gather_rows_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ idx,
                                        const int* __restrict__ pos, const int* __restrict__ offs_end,
-                                       const int* __restrict__ counts, int top, __nv_bfloat16* __restrict__ xs,
-                                       int* __restrict__ row_of, int D) {
+                                       const int* __restrict__ counts, const float* __restrict__ w_pair, int top,
+                                       __nv_bfloat16* __restrict__ xs, int* __restrict__ row_of, float* __restrict__ w_row, int D) {
   const int p = blockIdx.x, e = idx[p];
   const int row = offs_end[e] - counts[e] + pos[p];
-  if (threadIdx.x == 0) row_of[p] = row;
+  if (threadIdx.x == 0) {
+    row_of[p] = row;
+    if (w_pair != nullptr) w_row[row] = w_pair[p];
+  }
   const uint4* src = reinterpret_cast<const uint4*>(x + static_cast<int64_t>(p / top) * D);
   uint4* dst = reinterpret_cast<uint4*>(xs + static_cast<int64_t>(row) * D);
   for (int i = threadIdx.x; i < D / 8; i += blockDim.x) dst[i] = src[i];
 }
 
-__global__ void clamped_glu_kernel(const __nv_bfloat16* __restrict__ gu, GluArgs glu, __nv_bfloat16* __restrict__ h,
-                                   int64_t n8, int I8) {
+__global__ void clamped_glu_kernel(const __nv_bfloat16* __restrict__ gu, const float* __restrict__ w_row, GluArgs glu,
+                                   __nv_bfloat16* __restrict__ h, int64_t n8, int I8) {
   for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < n8;
        i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int64_t r = i / I8, c = i % I8;
+    const float w = w_row != nullptr ? w_row[r] : 1.f;
     float g[8], u[8];
     Vec16<__nv_bfloat16>::load(gu + (r * 2 * I8 + c) * 8, g);
     Vec16<__nv_bfloat16>::load(gu + (r * 2 * I8 + I8 + c) * 8, u);
     uint32_t o[4];
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      o[j] = pack_bf16x2(clamped_glu(g[2 * j], u[2 * j], glu), clamped_glu(g[2 * j + 1], u[2 * j + 1], glu));
+      o[j] = pack_bf16x2(clamped_glu(w * g[2 * j], w * u[2 * j], glu), clamped_glu(w * g[2 * j + 1], w * u[2 * j + 1], glu));
     *reinterpret_cast<uint4*>(h + i * 8) = make_uint4(o[0], o[1], o[2], o[3]);
   }
 }
@@ -850,16 +1030,6 @@ __global__ void moe_combine_rows_kernel(const __nv_bfloat16* __restrict__ ys, co
 }
 
 int threads_for(int n) { return n >= 1024 ? 256 : (n >= 256 ? 128 : 64); }
-
-// Opts a kernel into `bytes` of dynamic shared memory once per new maximum.
-template <typename K>
-cudaError_t want_smem(K kernel, int bytes, int& have) {
-  if (bytes <= 48 * 1024 || bytes <= have) return cudaSuccess;
-  if (bytes > 227 * 1024) return cudaErrorInvalidValue;
-  cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
-  if (e == cudaSuccess) have = bytes;
-  return e;
-}
 
 template <typename T>
 cudaError_t latent_attention_t(const SeqBatch& sb, const T* qf, const PagedRows& pages, int R, const float* sink, float scale,
@@ -932,11 +1102,29 @@ cudaError_t launch_norm_rows(bool f32_out, int mode, const float* x, const float
   return cudaGetLastError();
 }
 
-cudaError_t launch_rows_linear(bool f32, const void* x, int64_t ldx, const void* w, int64_t ldw, void* y, int64_t ldy,
-                               int M, int N, int K, int act, int out_mode, cudaStream_t st) {
-  if (M < 1 || N < 1 || K < 1) return cudaErrorInvalidValue;
-  return f32 ? rows_linear_t<float>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode, st)
-             : rows_linear_t<__nv_bfloat16>(x, ldx, w, ldw, y, ldy, M, N, K, act, out_mode, st);
+cudaError_t launch_residual_norm(bool y_f32, bool f32_out, const void* y, const float* gpost, float* x, bool add,
+                                 const float* gnext, void* out, int rows, int D, float eps, cudaStream_t st) {
+  const float* yf = static_cast<const float*>(y);
+  const __nv_bfloat16* yb = static_cast<const __nv_bfloat16*>(y);
+  if (f32_out) {
+    if (!y_f32) return cudaErrorInvalidValue;
+    residual_norm_go(yf, gpost, x, add, gnext, static_cast<float*>(out), rows, D, eps, st);
+  } else if (y_f32) {
+    residual_norm_go(yf, gpost, x, add, gnext, static_cast<__nv_bfloat16*>(out), rows, D, eps, st);
+  } else {
+    residual_norm_go(yb, gpost, x, add, gnext, static_cast<__nv_bfloat16*>(out), rows, D, eps, st);
+  }
+  return cudaGetLastError();
+}
+
+cudaError_t launch_rows_linear(bool f32, const void* x, int64_t ldx, const void* w, int64_t ldw, int M, int N, int K,
+                               const RowsOut& out, cudaStream_t st) {
+  if (M < 1 || N < 1 || K < 1 || (out.n1 < N && out.y2 == nullptr)) return cudaErrorInvalidValue;
+  if (out.act == kActSiluGlu)
+    return f32 ? rows_linear_t<float, true>(x, ldx, w, ldw, M, N, K, out, st)
+               : rows_linear_t<__nv_bfloat16, true>(x, ldx, w, ldw, M, N, K, out, st);
+  return f32 ? rows_linear_t<float, false>(x, ldx, w, ldw, M, N, K, out, st)
+             : rows_linear_t<__nv_bfloat16, false>(x, ldx, w, ldw, M, N, K, out, st);
 }
 
 cudaError_t launch_mla_prepare(bool f32, const SeqBatch& sb, const void* y, int64_t ldy, int q_rank, int R, int dr,
@@ -991,45 +1179,52 @@ cudaError_t launch_latent_attention(bool f32, const SeqBatch& sb, const void* qf
                                                  part_o, part_ml, static_cast<__nv_bfloat16*>(o_lat), st);
 }
 
-cudaError_t launch_table_experts_up(bool f32, const void* x, const int* tokens, const int* table, int vocab, int top, int E,
-                                    const void* w, GluArgs glu, void* h, int M, int D, int I, int* status, cudaStream_t st) {
+cudaError_t launch_experts_up(bool f32, const void* x, const ExpertChoice& c, const void* w, GluArgs glu, void* h, int M, int D,
+                              int I, int* status, cudaStream_t st) {
   const int per = (I + kExpWarps - 1) / kExpWarps;
-  const dim3 grid(M * top, per < 64 ? per : 64);
+  const dim3 grid(M * c.top, per < 64 ? per : 64);
   const bool vec = D % (f32 ? 4 : 8) == 0;
-#define B200_UP(T, V)                                                                                                      \
-  table_experts_up_kernel<T, V><<<grid, kExpWarps * 32, 0, st>>>(static_cast<const T*>(x), tokens, table, vocab, top, E,    \
-                                                                 static_cast<const T*>(w), glu, static_cast<T*>(h), D, I, status)
+#define B200_UP(T, V) \
+  experts_up_kernel<T, V><<<grid, kExpWarps * 32, 0, st>>>(static_cast<const T*>(x), c, static_cast<const T*>(w), glu, static_cast<T*>(h), D, I, status)
   if (f32) { if (vec) B200_UP(float, true); else B200_UP(float, false); }
   else { if (vec) B200_UP(__nv_bfloat16, true); else B200_UP(__nv_bfloat16, false); }
 #undef B200_UP
   return cudaGetLastError();
 }
 
-cudaError_t launch_table_experts_down(bool f32, const void* h, const int* tokens, const int* table, int vocab, int top,
-                                      int E, const void* w, float* x, int M, int D, int I, cudaStream_t st) {
+cudaError_t launch_experts_down(bool f32, const void* h, const ExpertChoice& c, const void* w, float out_scale, float* x, int M,
+                                int D, int I, cudaStream_t st) {
+  if (c.top * 4 > 48 * 1024) return cudaErrorInvalidValue;
   const int per = (D + kExpWarps - 1) / kExpWarps;
   const dim3 grid(M, per < 256 ? per : 256);
   const bool vec = I % (f32 ? 4 : 8) == 0;
-#define B200_DN(T, V)                                                                                                      \
-  table_experts_down_kernel<T, V><<<grid, kExpWarps * 32, 0, st>>>(static_cast<const T*>(h), tokens, table, vocab, top, E,  \
-                                                                   static_cast<const T*>(w), x, D, I)
+#define B200_DN(T, V) \
+  experts_down_kernel<T, V><<<grid, kExpWarps * 32, c.top * 4, st>>>(static_cast<const T*>(h), c, static_cast<const T*>(w), out_scale, x, D, I)
   if (f32) { if (vec) B200_DN(float, true); else B200_DN(float, false); }
   else { if (vec) B200_DN(__nv_bfloat16, true); else B200_DN(__nv_bfloat16, false); }
 #undef B200_DN
   return cudaGetLastError();
 }
 
-cudaError_t launch_moe_gather_rows(const __nv_bfloat16* x, const int* idx, const int* pos, const int* offs_end,
-                                   const int* counts, int top, __nv_bfloat16* xs, int* row_of, int M, int D, cudaStream_t st) {
-  if (D % 8 != 0) return cudaErrorInvalidValue;
-  moe_gather_rows_kernel<<<M * top, 128, 0, st>>>(x, idx, pos, offs_end, counts, top, xs, row_of, D);
+cudaError_t launch_sigmoid_topk(const ExpertChoice& c, int M, int* ids, float* weights, int* status, cudaStream_t st) {
+  if (c.top < 1 || c.top > c.E) return cudaErrorInvalidValue;
+  sigmoid_topk_kernel<<<(M + 7) / 8, 256, 0, st>>>(c, M, ids, weights, status);
   return cudaGetLastError();
 }
-cudaError_t launch_clamped_glu(const __nv_bfloat16* gu, GluArgs glu, __nv_bfloat16* h, int rows, int I, cudaStream_t st) {
+
+cudaError_t launch_moe_gather_rows(const __nv_bfloat16* x, const int* idx, const int* pos, const int* offs_end,
+                                   const int* counts, const float* w_pair, int top, __nv_bfloat16* xs, int* row_of, float* w_row,
+                                   int M, int D, cudaStream_t st) {
+  if (D % 8 != 0) return cudaErrorInvalidValue;
+  moe_gather_rows_kernel<<<M * top, 128, 0, st>>>(x, idx, pos, offs_end, counts, w_pair, top, xs, row_of, w_row, D);
+  return cudaGetLastError();
+}
+cudaError_t launch_clamped_glu(const __nv_bfloat16* gu, const float* w_row, GluArgs glu, __nv_bfloat16* h, int rows, int I,
+                               cudaStream_t st) {
   if (I % 8 != 0) return cudaErrorInvalidValue;
   const int64_t n8 = static_cast<int64_t>(rows) * (I / 8);
   const int grid = static_cast<int>((n8 + 255) / 256 < 148 * 16 ? (n8 + 255) / 256 : 148 * 16);
-  clamped_glu_kernel<<<grid > 0 ? grid : 1, 256, 0, st>>>(gu, glu, h, n8, I / 8);
+  clamped_glu_kernel<<<grid > 0 ? grid : 1, 256, 0, st>>>(gu, w_row, glu, h, n8, I / 8);
   return cudaGetLastError();
 }
 cudaError_t launch_moe_combine_rows(const __nv_bfloat16* ys, const int* row_of, int top, float w, float* x, int M, int D,

@@ -32,10 +32,24 @@ cudaError_t launch_embed_bigram(bool f32, const SeqBatch& sb, const int* tokens,
 cudaError_t launch_norm_rows(bool f32_out, int mode, const float* x, const float* gamma, const float* beta, void* out,
                              int rows, int D, float eps, cudaStream_t st);
 
-enum RowAct : int { kActNone = 0, kActRelu2 = 1 };
-// y[m, n] = act(sum_k x[m, k] w[n, k]); out_mode 0: activation dtype, 1: fp32, 2: added to fp32 y. Few rows.
-cudaError_t launch_rows_linear(bool f32, const void* x, int64_t ldx, const void* w, int64_t ldw, void* y, int64_t ldy,
-                               int M, int N, int K, int act, int out_mode, cudaStream_t st);
+// x[r, :] = (add ? x[r, :] : 0) + rms(y[r, :]) gpost; out[r, :] = rms(x[r, :]) gnext unless out is null. x fp32, y fp32
+// (y_f32) or bf16.
+cudaError_t launch_residual_norm(bool y_f32, bool f32_out, const void* y, const float* gpost, float* x, bool add,
+                                 const float* gnext, void* out, int rows, int D, float eps, cudaStream_t st);
+
+enum RowAct : int { kActNone = 0, kActRelu2 = 1, kActSilu = 2, kActSiluGlu = 3 };
+struct RowsOut {
+  void* y;             // [M, ldy]
+  int64_t ldy;
+  int act;             // kActSiluGlu: w holds 2 N rows, y = silu(gate) * up
+  int out_mode;        // 0: activation dtype, 1: fp32, 2: added to fp32 y
+  float* y2;           // features n >= n1 go to y2[m, n - n1] in fp32, without the activation (n1 = N: none do)
+  int64_t ldy2;
+  int n1;
+};
+// y[m, n] = act(sum_k x[m, k] w[n, k]). Few rows.
+cudaError_t launch_rows_linear(bool f32, const void* x, int64_t ldx, const void* w, int64_t ldw, int M, int N, int K,
+                               const RowsOut& out, cudaStream_t st);
 
 struct RopeTable {
   const float* cos;    // [max_pos, dims / 2], amplitude folded in
@@ -74,21 +88,87 @@ cudaError_t launch_latent_attention(bool f32, const SeqBatch& sb, const void* qf
                                     const float* sink, float scale, int H, int n_splits, float* part_o, float* part_ml,
                                     void* o_lat, cudaStream_t st);
 
-// Experts chosen by a table over token ids (experts of token t: table[t, :top], each with weight 1 / top).
-struct GluArgs {
-  float limit, alpha;  // g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(alpha * g) * (u + 1)
+// Experts of a token: table[token, :top] (each with weight 1 / top), or with `logits` [M, E] fp32 the `top` largest, whose
+// sigmoid scores multiply the expert's input.
+struct ExpertChoice {
+  const int* tokens;
+  const int* table;
+  int vocab;
+  const float* logits;
+  int top, E;
 };
-cudaError_t launch_table_experts_up(bool f32, const void* x, const int* tokens, const int* table, int vocab, int top, int E,
-                                    const void* w_gate_up, GluArgs glu, void* h, int M, int D, int I, int* status,
-                                    cudaStream_t st);
-cudaError_t launch_table_experts_down(bool f32, const void* h, const int* tokens, const int* table, int vocab, int top,
-                                      int E, const void* w_down, float* x, int M, int D, int I, cudaStream_t st);
-// Grouped path: rows of expert e start at offs[e]; pair p = (token, choice) sits in row offs[idx[p]] + pos[p].
+struct GluArgs {
+  float limit, alpha, shift;  // g = min(gate, limit), u = clamp(up, -limit, limit): g * sigmoid(alpha * g) * (u + shift)
+};
+// h[m * top + j] = glu of the token's j-th expert; x[m] += out_scale * sum of the experts' outputs.
+cudaError_t launch_experts_up(bool f32, const void* x, const ExpertChoice& c, const void* w_gate_up, GluArgs glu, void* h, int M,
+                              int D, int I, int* status, cudaStream_t st);
+cudaError_t launch_experts_down(bool f32, const void* h, const ExpertChoice& c, const void* w_down, float out_scale, float* x,
+                                int M, int D, int I, cudaStream_t st);
+cudaError_t launch_sigmoid_topk(const ExpertChoice& c, int M, int* ids, float* weights, int* status, cudaStream_t st);
+// Grouped path: rows of expert e start at offs[e]; pair p = (token, choice) sits in row offs[idx[p]] + pos[p]. w_pair
+// (optional) travels to w_row by the same permutation and scales gate and up before the activation.
 cudaError_t launch_moe_gather_rows(const __nv_bfloat16* x, const int* idx, const int* pos, const int* offs_end,
-                                   const int* counts, int top, __nv_bfloat16* xs, int* row_of, int M, int D, cudaStream_t st);
-cudaError_t launch_clamped_glu(const __nv_bfloat16* gu, GluArgs glu, __nv_bfloat16* h, int rows, int I, cudaStream_t st);
+                                   const int* counts, const float* w_pair, int top, __nv_bfloat16* xs, int* row_of, float* w_row,
+                                   int M, int D, cudaStream_t st);
+cudaError_t launch_clamped_glu(const __nv_bfloat16* gu, const float* w_row, GluArgs glu, __nv_bfloat16* h, int rows, int I,
+                               cudaStream_t st);
 cudaError_t launch_moe_combine_rows(const __nv_bfloat16* ys, const int* row_of, int top, float w, float* x, int M, int D,
                                     cudaStream_t st);
+
+// ---- windowed attention (window_attention.cu) ------------------------------------------------------------------------
+struct WindowMask {
+  int size, keep_first;   // i sees j when j <= i and (i - j < size or j < keep_first); no window: size 1 << 30
+};
+// y [n_tok, ldy] = [q of H heads | k of G heads], D wide. q [n_tok, H, D] = unit RMS norm of the rotated (y + bias); the
+// cache row becomes [k likewise | k as projected, the values]; both also go to k, v [n_tok, G, D] unless null. `rope` holds
+// half-split pairs (i, i + dims / 2) here.
+cudaError_t launch_qk_prepare(bool f32, const SeqBatch& sb, const void* y, int64_t ldy, const float* bias, int H, int G, int D,
+                              bool unit_norm, float eps, const RopeTable& rope, const PagedRows& pages, void* q, void* k, void* v,
+                              int* status, cudaStream_t st);
+// Softmax attention of q [n_tok, H, D] over the pages' rows [K | V] of G kv heads, any sizes. n_splits > 1 cuts the visible
+// keys into ranges merged by a second kernel (part_o [n_tok, H, S, D], part_ml [n_tok, H, S, 2] fp32).
+cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, int H, int G, int D,
+                                    WindowMask mask, float scale, int n_splits, float* part_o, float* part_ml, void* out,
+                                    cudaStream_t st);
+
+// ---- linear attention with a matrix state (linear_attention.cu, ssd_scan_sm100.cu) ---------------------------------------
+struct LinShape {
+  int H, N, P;            // heads, key width, value width; a row of qkv is [q (H N) | k (H N) | v (H P)]
+  float q_scale;
+  int silu;               // 1: q, k, v still need their SiLU
+};
+struct LinGates {
+  const float* decay;     // [H] fixed decay per head, or with `raw` set exponential gates:
+  const float* raw;       // [n_tok, ld] = [i (H) | f (H)] before bias and cap
+  int64_t ld;
+  const float* bias;      // [2 H]
+  float cap;
+  const float* vec;       // [slots, H, N + 1] = [n | m] at the start of the step
+  float* vec_new;         // [n_seq, H, N + 1] after it
+  float* den;             // [n_tok, H, 4] = {n . q, second part of n . q, exp(-m), -}
+};
+// state [slots, H, N, P] fp32 (ignored where start == 0, always written); y [n_tok, H P] fp32: the numerators.
+cudaError_t launch_linear_scan(bool f32, const SeqBatch& sb, const void* qkv, int64_t ld, const LinGates& g, float* state, float* y,
+                               const LinShape& s, cudaStream_t st);
+// One token per sequence.
+cudaError_t launch_linear_step(bool f32, const SeqBatch& sb, const void* qkv, int64_t ld, const LinGates& g, float* state, float* y,
+                               const LinShape& s, cudaStream_t st);
+// Chunked on tensor cores: bf16, N = 128, P a multiple of 64, q_scale > 0, activations applied. y bf16.
+bool linear_scan_sm100_ok(const LinShape& s);
+cudaError_t launch_linear_scan_sm100(const SeqBatch& sb, const __nv_bfloat16* qkv, int64_t ld, const LinGates& g, float* state,
+                                     __nv_bfloat16* y, const LinShape& s, int* status, cudaStream_t st);
+struct HeadNorm {
+  int parts;
+  float eps, den_eps;
+  const float* den;       // optional, with pieces = heads: y is divided by max(|n . q|, exp(-m)) + den_eps first
+  const float* vec_new;   // optional: copied to vec at the slot of the sequence, by the last row of every sequence
+  float* vec;
+  int vec_len;
+};
+// out = RMS norm over `parts` equal pieces of y, times gamma and sigmoid(z). y fp32 (y_f32) or activation dtype.
+cudaError_t launch_head_norm_gate(bool f32, bool y_f32, const SeqBatch& sb, const void* y, const void* z, int64_t ldz,
+                                  const float* gamma, void* out, int D, const HeadNorm& a, cudaStream_t st);
 
 // ---- state-space layers ------------------------------------------------------------------------------------------
 // Causal depthwise convolution of packed rows with bias and SiLU. ring [slots, taps, C] fp32 holds the raw input of

@@ -21,7 +21,7 @@ class Family:
     module: str                        # package with the configuration class, init_params, forward, generate
     config: str                        # name of the configuration class in it
     aliases: Tuple[str, ...] = ()      # values of architecture / architectures / model_type
-    from_dir: Optional[str] = None     # "module:function" (path, dtype, device) -> (config, params)
+    from_dir: Optional[str] = None     # "module:function" (path, dtype, device, family) -> (config, params)
     engine: Optional[str] = None       # step engine class in ``module``
 
     def mod(self):
@@ -32,12 +32,13 @@ class Family:
 
 
 _BASE = "jax_gpt_b200.models."
+_FOLDER = _BASE + "registry:_folder_with_config"
 FAMILIES: Dict[str, Family] = {f.name: f for f in (
     Family("gpt2", _BASE + "gpt2", "GPTConfig", ("GPT2LMHeadModel", "gpt2")),
     Family("qwen35", _BASE + "qwen35", "Qwen35Config", ("qwen3_5_moe",)),
     Family("deepseek_v3", _BASE + "deepseek_v3", "DeepSeekV3Config", ("DeepseekV3ForCausalLM", "deepseek_v3")),
-    Family("vobunex", _BASE + "vobunex", "VobunexConfig", ("Vobunex",), from_dir=_BASE + "registry:_vobunex_from_dir",
-           engine="VobunexEngine"),
+    Family("vobunex", _BASE + "vobunex", "VobunexConfig", ("Vobunex",), from_dir=_FOLDER, engine="VobunexEngine"),
+    Family("fovudra", _BASE + "fovudra", "FovudraConfig", ("Fovudra",), from_dir=_FOLDER, engine="FovudraEngine"),
 )}
 
 
@@ -60,7 +61,7 @@ def load_model(path: str, dtype=torch.bfloat16, device="cuda") -> Tuple[Family, 
     if f.from_dir is None:
         raise NotImplementedError(f"family {f.name!r} loads through its own scripts, not from a config.json folder")
     mod, fn = f.from_dir.split(":")
-    config, params = getattr(importlib.import_module(mod), fn)(path, dtype, device)
+    config, params = getattr(importlib.import_module(mod), fn)(path, dtype, device, f)
     return f, config, params
 
 
@@ -72,8 +73,8 @@ def load_engine(path: str, dtype=torch.bfloat16, device="cuda", **kw):
     return getattr(f.mod(), f.engine)(params, config, **kw)
 
 
-def _vobunex_from_dir(path, dtype, device):
+def _folder_with_config(path, dtype, device, family):
+    """Folders whose configuration class reads config.json (``from_dir``) and whose module loads tensors by name."""
     from ..utils.safetensors_dir import SafetensorsDir
-    from .vobunex import VobunexConfig, load_from_state_dict
-    config = VobunexConfig.from_dir(path)
-    return config, load_from_state_dict(SafetensorsDir(path), config, dtype, device)
+    config = family.config_class().from_dir(path)
+    return config, family.mod().load_from_state_dict(SafetensorsDir(path), config, dtype, device)

@@ -26,6 +26,7 @@ from ...ops.packed import PackedBatch, embed_bigram, norm_rows, seq_begin
 from ...ops.rope import rope_tables
 from ...ops.table_moe import table_moe
 from ...utils.profiling import scope
+from ..step_engine import forward_tokens, generate_tokens
 from .config import GLU_ALPHA, DenseMlp, LatentAttention, VobunexConfig
 
 
@@ -159,41 +160,16 @@ def init_params(config: VobunexConfig, key: int = 0, dtype=torch.float32, device
     return load_from_state_dict(random_state_dict(config, int(key), device=device if on_device else "cpu"), config, dtype, device)
 
 
-@torch.no_grad()
 def forward(params, tokens, config: VobunexConfig, cache: Optional[HybridPagedCache] = None, seq_ids: Optional[List] = None,
             is_decode: bool = False):
-    """tokens (B, T) -> logits (B, T, V). Sequences named by ``seq_ids`` continue from the cache when it holds them and
-    start at position 0 otherwise; ``is_decode`` is accepted for signature parity with the other families."""
+    """tokens (B, T) -> logits (B, T, V), see ``step_engine.forward_tokens``; ``is_decode`` is accepted for signature parity
+    with the other families."""
     from .engine import VobunexEngine
-    B, T = tokens.shape
-    seq_ids = list(range(B)) if seq_ids is None else list(seq_ids)
-    if cache is None:
-        per = (T + config.page_size - 1) // config.page_size
-        cache = make_cache(config, B * per, B, per, params["embed"].dtype, tokens.device)
-    eng = VobunexEngine(params, config, cache, use_cuda_graph=False)
-    return eng.step(seq_ids, tokens.tolist(), want=[list(range(T))] * B).reshape(B, T, -1)
+    return forward_tokens(VobunexEngine, params, tokens, config, cache, seq_ids)
 
 
-@torch.no_grad()
 def generate(params, prompt_tokens, config: VobunexConfig, max_new_tokens: int, temperature: float = 0.0,
              top_k: Optional[int] = None, key=None, cache: Optional[HybridPagedCache] = None, use_cuda_graph: bool = True):
-    """Continuation (B, max_new_tokens), greedy or sampled. ``prompt_tokens``: (B, T) tensor, or a list of token lists of
-    different lengths."""
-    from ..gpt2.model import sample_logits
+    """Continuation (B, max_new_tokens), see ``step_engine.generate_tokens``."""
     from .engine import VobunexEngine
-    prompts = prompt_tokens.tolist() if torch.is_tensor(prompt_tokens) else [list(p) for p in prompt_tokens]
-    device = params["embed"].device
-    gen = key if isinstance(key, torch.Generator) else torch.Generator().manual_seed(int(key) if key is not None else 0)
-    B = len(prompts)
-    if cache is None:
-        per = [(len(p) + max_new_tokens + config.page_size - 1) // config.page_size for p in prompts]
-        cache = make_cache(config, sum(per), B, max(per), params["embed"].dtype, device)
-    eng = VobunexEngine(params, config, cache, use_cuda_graph=use_cuda_graph)
-    ids = [("gen", b) for b in range(B)]
-    logits = eng.step(ids, prompts, want=[[len(p) - 1] for p in prompts])
-    out = [sample_logits(logits, temperature, top_k, gen)]
-    for _ in range(max_new_tokens - 1):
-        out.append(sample_logits(eng.decode(ids, out[-1]), temperature, top_k, gen))
-    for i in ids:
-        eng.release(i)
-    return torch.stack(out, dim=1)
+    return generate_tokens(VobunexEngine, params, prompt_tokens, config, max_new_tokens, temperature, top_k, key, cache, use_cuda_graph)

@@ -44,9 +44,10 @@ def _as2d(t):
     return t.as_strided((B * T, H * D), (t.stride(1), 1))
 
 
-def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None, sink=None):
+def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None, sink=None, window: int = 0, keep_first: int = 0):
     """Raw CUDA forward. Returns (out [B,T,H,D] bf16, lse [B,H,T] fp32 in log2 units). ``sink`` (H,) fp32 adds
-    exp(sink) to every softmax denominator of its head (and to lse)."""
+    exp(sink) to every softmax denominator of its head (and to lse). ``window`` > 0: query i sees keys j <= i with
+    i - j < window or j < keep_first; key tiles nobody sees are skipped."""
     B, T, H, D = q.shape
     Hkv, Dv = k.shape[2], v.shape[3]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -54,7 +55,8 @@ def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None, sink=None):
         out = torch.empty(B, T, H, Dv, device=q.device, dtype=torch.bfloat16)
     if lse is None:
         lse = torch.empty(B, H, T, device=q.device, dtype=torch.float32)
-    _ext.ops().attn_fwd(_as2d(q), _as2d(k), _as2d(v), _as2d(out), lse, B, T, H, Hkv, D, scale, causal, Dv, sink)
+    _ext.ops().attn_fwd(_as2d(q), _as2d(k), _as2d(v), _as2d(out), lse, B, T, H, Hkv, D, scale, causal, Dv, sink, window,
+                          keep_first)
     return out, lse
 
 
@@ -138,12 +140,13 @@ def attention_decode(q, cache_k, cache_v, kv_len=None, pos: Optional[torch.Tenso
 
 
 def attention_decode_paged(q, pool, block_table, seq_ids, seq_lens, n_kv_heads: int, len_add: int = 1, scale=None,
-                           scratch=None, out=None, max_len: Optional[int] = None):
+                           scratch=None, out=None, max_len: Optional[int] = None, window: int = 0, keep_first: int = 0):
     """One query token per sequence over a PAGED cache (cache/paged.py): ``pool`` (n_pages, page_size, 2 * Hkv * D)
     holds K of every kv head then V per cached token, ``block_table`` (max_seqs, max_pages) the page ids,
     ``seq_ids`` (B,) the sequence of every query row, ``seq_lens`` (max_seqs,) the committed lengths, all on the
     device; ``len_add`` keys beyond the committed length are attended (1: the new token's row is written, the length
-    not yet advanced). q (B, H, D). Returns (B, H, D)."""
+    not yet advanced). ``window`` > 0: only the last ``window`` keys and the first ``keep_first`` are seen.
+    q (B, H, D). Returns (B, H, D)."""
     B, H, D = q.shape
     Hkv = n_kv_heads
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -159,19 +162,23 @@ def attention_decode_paged(q, pool, block_table, seq_ids, seq_lens, n_kv_heads: 
             rows = pool[block_table[sid, (pos // ps).long()].long(), (pos % ps).long()]          # (n, 2 Hkv D)
             kk = rows[:, :Hkv * D].reshape(1, n, Hkv, D).to(q.dtype)
             vv = rows[:, Hkv * D:].reshape(1, n, Hkv, D).to(q.dtype)
+            if window > 0:
+                seen = (pos >= n - window) | (pos < keep_first)
+                kk, vv = kk[:, seen], vv[:, seen]
             outs.append(attention_ref(q[b:b + 1, None], kk, vv, causal=False, scale=scale)[:, 0])
         return torch.cat(outs)
     q2 = q.reshape(B, H * D)
     if q2.stride(1) != 1 or q2.stride(0) % 8 != 0 or q2.data_ptr() % 16 != 0:
         q2 = q2.contiguous()
     if scratch is None:
-        S = decode_splits(B, Hkv, max_len or block_table.shape[1] * pool.shape[1])
+        n_keys = max_len or block_table.shape[1] * pool.shape[1]
+        S = decode_splits(B, Hkv, min(n_keys, window + keep_first) if window > 0 else n_keys)
         scratch = (torch.empty(B, H, S, D, device=q.device, dtype=torch.float32),
                    torch.empty(B, H, S, 2, device=q.device, dtype=torch.float32))
     if out is None:
         out = torch.empty(B, H * D, device=q.device, dtype=torch.bfloat16)
     _ext.ops().attn_decode_paged(q2, pool, block_table, seq_ids, seq_lens, int(len_add), H, Hkv, scale, scratch[0],
-                                 scratch[1], out)
+                                 scratch[1], out, window, keep_first)
     return out.view(B, H, D)
 
 

@@ -14,7 +14,7 @@ import torch
 
 from .. import _ext
 
-EPI_NONE, EPI_GELU, EPI_GELU_GRAD, EPI_RELU2 = 0, 1, 2, 4
+EPI_NONE, EPI_GELU, EPI_GELU_GRAD, EPI_RELU2, EPI_SILU = 0, 1, 2, 4, 5
 OUT_BF16, OUT_F32, OUT_F32_ATOMIC = 0, 1, 2
 
 
@@ -46,6 +46,8 @@ def gemm_ref(a, b, *, a_mn_major=False, b_mn_major=False, out=None, bias=None, r
         acc = acc * gelu_tanh_grad(aux.float())
     elif epilogue == EPI_RELU2:
         acc = acc.clamp_min(0).square()
+    elif epilogue == EPI_SILU:
+        acc = torch.nn.functional.silu(acc)
     if residual is not None:
         acc = acc + residual.float()
     if out is None:
@@ -119,12 +121,18 @@ def linear_f32out(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 
 
 ROWS_KERNEL_MAX = {torch.bfloat16: 32, torch.float32: 8}   # rows up to which linear layers run on the few-row kernel
+_ROW_ACTS = {None: (0, EPI_NONE), "relu2": (1, EPI_RELU2), "silu": (2, EPI_SILU)}   # few-row kernel, GEMM epilogue
+_ROW_SILU_GLU = 3
+
+
+def _few_rows(x) -> bool:
+    return x.is_cuda and x.shape[0] <= ROWS_KERNEL_MAX.get(x.dtype, 0)
 
 
 def linear_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *, act: Optional[str] = None,
                 accumulate: bool = False, f32_out: bool = False) -> torch.Tensor:
-    """Inference linear layer with ``w`` stored (out, in) as checkpoints have it: ``act(x @ w.T)``; ``act`` is None or
-    "relu2" (the square of relu). ``accumulate`` adds into ``out`` (fp32: a 32-bit residual), ``f32_out`` returns fp32.
+    """Inference linear layer with ``w`` stored (out, in) as checkpoints have it: ``act(x @ w.T)``; ``act`` is None,
+    "relu2" (the square of relu) or "silu". ``accumulate`` adds into ``out`` (fp32: a 32-bit residual), ``f32_out`` returns fp32.
     x (M, in), bf16 or fp32, unit inner stride. On CUDA up to ``ROWS_KERNEL_MAX`` rows run on the few-row kernel
     (weights streamed once where the rows are 16-byte aligned), more rows on the tcgen05 GEMM in bf16 and on the library's fp32 GEMM in fp32."""
     M, N = x.shape[0], w.shape[0]
@@ -132,19 +140,49 @@ def linear_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = 
         assert not accumulate
         out = torch.empty(M, N, device=x.device, dtype=torch.float32 if f32_out else x.dtype)
     mode = 2 if accumulate else (1 if out.dtype == torch.float32 and x.dtype != torch.float32 else 0)
-    if x.is_cuda and M <= ROWS_KERNEL_MAX.get(x.dtype, 0):
-        _ext.ops().rows_linear(x, w, out, 1 if act == "relu2" else 0, mode)
+    if _few_rows(x):
+        _ext.ops().rows_linear(x, w, out, _ROW_ACTS[act][0], mode)
         return out
     if x.is_cuda and x.dtype == torch.bfloat16 and w.shape[1] % 8 == 0 and w.stride(0) % 8 == 0 and w.data_ptr() % 16 == 0:
         if x.stride(0) % 8 != 0 or x.data_ptr() % 16 != 0:
             x = x.contiguous()
         if act is None or mode == 0:
-            return gemm(x, w, out=out, epilogue=EPI_RELU2 if act == "relu2" else EPI_NONE,
+            return gemm(x, w, out=out, epilogue=_ROW_ACTS[act][1],
                         out_mode=(OUT_BF16, OUT_F32, OUT_F32_ATOMIC)[mode])
     y = x @ w.t() if mode == 0 else x.float() @ w.float().t()
     if act == "relu2":
         y = y.clamp_min(0).square()
+    elif act == "silu":
+        y = torch.nn.functional.silu(y)
     return out.add_(y) if accumulate else out.copy_(y)
+
+
+def linear_rows_f32_tail(x: torch.Tensor, w: torch.Tensor, n_tail: int):
+    """``x @ w.T`` in x's dtype and its last ``n_tail`` features as an fp32 tensor of their own (gates of a recurrence),
+    one launch where the few-row kernel runs."""
+    n = w.shape[0] - n_tail
+    if _few_rows(x):
+        y = torch.empty(x.shape[0], n, device=x.device, dtype=x.dtype)
+        tail = torch.empty(x.shape[0], n_tail, device=x.device, dtype=torch.float32)
+        _ext.ops().rows_linear(x, w, y, 0, 0, tail)
+        return y, tail
+    return linear_rows(x, w[:n]), linear_rows(x, w[n:], f32_out=True)
+
+
+def silu_glu_rows(x: torch.Tensor, w_gate_up: torch.Tensor) -> torch.Tensor:
+    """``silu(x @ gate.T) * (x @ up.T)`` with w_gate_up (2 I, in) = [gate | up]; the few-row kernel does it in one launch."""
+    M, I = x.shape[0], w_gate_up.shape[0] // 2
+    if _few_rows(x):
+        out = torch.empty(M, I, device=x.device, dtype=x.dtype)
+        _ext.ops().rows_linear(x, w_gate_up, out, _ROW_SILU_GLU, 0)
+        return out
+    gu = linear_rows(x, w_gate_up)
+    if x.is_cuda and x.dtype == torch.bfloat16 and I % 8 == 0:
+        out = torch.empty(M, I, device=x.device, dtype=x.dtype)
+        _ext.ops().clamped_glu(gu, float("inf"), 1.0, 0.0, None, out)
+        return out
+    g, u = gu.float().chunk(2, -1)
+    return (torch.nn.functional.silu(g) * u).to(x.dtype)
 
 
 class _LinearFn(torch.autograd.Function):

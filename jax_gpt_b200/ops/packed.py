@@ -13,7 +13,7 @@ from typing import List, Optional
 import torch
 
 from .. import _ext
-from .norm import LAYERNORM, norm_ref
+from .norm import LAYERNORM, RMSNORM, norm_ref
 
 
 @dataclass
@@ -111,3 +111,17 @@ def norm_rows(mode: int, x: torch.Tensor, gamma: torch.Tensor, beta: Optional[to
         _ext.ops().norm_rows(0 if mode == LAYERNORM else 1, x, gamma, beta, out, eps)
         return out
     return norm_ref(mode, x, gamma, beta, eps).to(dtype)
+
+
+def residual_norm_rows(y: torch.Tensor, gamma_post: torch.Tensor, x: torch.Tensor, gamma_next: Optional[torch.Tensor], eps: float,
+                       dtype, add: bool = True) -> Optional[torch.Tensor]:
+    """A sublayer's output ``y`` through its post-norm into the fp32 residual, and the next sublayer's normed input, in one
+    pass: ``x (+)= rms(y) gamma_post`` in place (``add`` False: assigned), returns ``rms(x) gamma_next`` in ``dtype`` (None
+    without ``gamma_next``)."""
+    out = torch.empty(x.shape, device=x.device, dtype=dtype) if gamma_next is not None else None
+    if x.is_cuda:
+        _ext.ops().residual_norm(y, gamma_post, x, add, gamma_next, out, eps)
+        return out
+    r = norm_ref(RMSNORM, y.float(), gamma_post, None, eps)
+    x.copy_(x + r if add else r)
+    return norm_ref(RMSNORM, x, gamma_next, None, eps).to(dtype) if out is not None else None

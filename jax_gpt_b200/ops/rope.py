@@ -83,9 +83,30 @@ def yarn_frequencies(dims: int, base: float, scaling=None):
     return [f / factor * r + f * (1.0 - r) for f, r in zip(freqs, ramp)], 0.1 * math.log(factor) + 1.0
 
 
+def banded_frequencies(dims: int, base: float, scaling=None):
+    """Frequencies [dims / 2] as Python floats. ``scaling`` is None or a mapping with ``factor``, ``low``, ``high``,
+    ``original``: waves shorter than original / high keep their frequency, waves longer than original / low are slowed by
+    ``factor``, those between are blended linearly in original / wavelength (the Llama 3.1 rule)."""
+    import math
+    out = []
+    for i in range(dims // 2):
+        f = base ** (-2.0 * i / dims)
+        if scaling:
+            turns = scaling["original"] * f / (2.0 * math.pi)       # original / wavelength
+            low, high = scaling["low"], scaling["high"]
+            keep = 1.0 if turns > high else 0.0 if turns < low else (turns - low) / (high - low) if high > low else 1.0
+            f = keep * f + (1.0 - keep) * f / scaling["factor"]
+        out.append(f)
+    return out
+
+
 def rope_tables(dims: int, base: float, n_pos: int, scaling=None, device="cpu"):
-    """(cos, sin) [n_pos, dims / 2] fp32 with the YaRN amplitude folded in; angles are taken in fp64 before rounding."""
-    freqs, amp = yarn_frequencies(dims, base, scaling)
+    """(cos, sin) [n_pos, dims / 2] fp32; angles are taken in fp64 before rounding. The scaling's keys tell its kind: YaRN
+    (``fast``, ``slow``; the amplitude is folded in) or wavelength bands (``low``, ``high``)."""
+    if scaling and "low" in scaling:
+        freqs, amp = banded_frequencies(dims, base, scaling), 1.0
+    else:
+        freqs, amp = yarn_frequencies(dims, base, scaling)
     ang = torch.arange(n_pos, dtype=torch.float64)[:, None] * torch.tensor(freqs, dtype=torch.float64)[None, :]
     return (ang.cos() * amp).float().to(device).contiguous(), (ang.sin() * amp).float().to(device).contiguous()
 
@@ -101,3 +122,15 @@ def rotate_interleaved(x: torch.Tensor, pos: torch.Tensor, tables) -> torch.Tens
     u, v = x[..., 0:dims:2], x[..., 1:dims:2]
     turned = torch.stack([u * c - v * s, v * c + u * s], dim=-1).flatten(-2)
     return torch.cat([turned, x[..., dims:]], dim=-1)
+
+
+def rotate_half_split(x: torch.Tensor, pos: torch.Tensor, tables) -> torch.Tensor:
+    """x (N, ..., d): of the first ``dims`` features, i and i + dims / 2 turn together by the angles of position ``pos[n]``."""
+    cos, sin = tables
+    half = cos.shape[1]
+    if half == 0:
+        return x
+    shape = [x.shape[0]] + [1] * (x.dim() - 2) + [half]
+    c, s = cos[pos.long()].reshape(shape), sin[pos.long()].reshape(shape)
+    u, v = x[..., :half], x[..., half:2 * half]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., 2 * half:]], dim=-1)
