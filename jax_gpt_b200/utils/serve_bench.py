@@ -1,12 +1,12 @@
-"""Serving benchmark of Vobunex beside the closest existing families at equal widths (random weights, one GPU).
+"""Serving benchmark of Vobunex and Fovudra beside the closest other families at equal widths (random weights, one GPU).
 
-    python bench.py --serve [--serve-part kernels|models|all]
+    python bench.py --serve [--serve-part kernels|models|all] [--serve-family vobunex|fovudra|all]
 
 ``models``: prefill and decode tokens/s of whole models. The hybrid (Mamba-2 + latent attention) stands beside the
 Qwen3.5-style hybrid (Gated DeltaNet + gated attention), latent-attention-only layers beside the DeepSeek-V3 layers; same
 width, depth, expert count and expert width, each family on its own serving path (decode: CUDA-graph engines, the
 others' experts on the fused expert kernel). ``kernels``: device time and roofline fraction of every kernel of a layer
-beside the like kernel of the other family.
+beside the like kernel of the other family. Fovudra's tables are made in utils/serve_bench_fovudra.py.
 
 Timing: CUDA events. Kernels are timed inside a captured graph that writes a 256 MB buffer (larger than L2) before every
 launch; the time of the same graph without the launches is subtracted. The roofline of a kernel is the slower of its
@@ -300,11 +300,13 @@ def _time_calls(fn, warmup, n):
     return statistics.median(ts)
 
 
-def _vobunex_run(cfg, B, T, steps, dev):
-    from ..models.vobunex import VobunexEngine, init_params, make_cache
-    params = init_params(cfg, 0, BF, dev, on_device=True)
+def step_engine_run(family, cfg, B, T, steps, dev):
+    """Prefill (last logits), decode and prefill (all logits) times of a family on the shared step engine."""
+    from ..models.registry import FAMILIES
+    f = FAMILIES[family]
+    params = f.mod().init_params(cfg, 0, BF, dev, on_device=True)
     per = (T + steps + 16 + cfg.page_size - 1) // cfg.page_size
-    eng = VobunexEngine(params, cfg, make_cache(cfg, B * per, B, per, BF, dev))
+    eng = getattr(f.mod(), f.engine)(params, cfg, f.mod().make_cache(cfg, B * per, B, per, BF, dev))
     tok = torch.randint(0, cfg.vocab_size, (B, T)).tolist()
     ids = list(range(B))
 
@@ -324,6 +326,19 @@ def _vobunex_run(cfg, B, T, steps, dev):
         state["t"] = eng.decode(ids, state["t"]).argmax(-1)
     dec = _time_calls(decode, 4, steps)
     return pre, dec, pre_all
+
+
+def _vobunex_run(cfg, B, T, steps, dev):
+    return step_engine_run("vobunex", cfg, B, T, steps, dev)
+
+
+def qwen_like(width, heads, experts, top, ff, vocab, shared_ff=128):
+    """The Qwen3.5-style hybrid of eight layers at the given widths."""
+    from ..models.qwen35 import Qwen35Config
+    return Qwen35Config(d_model=width, vocab_size=vocab, n_layers=8, max_position_embeddings=8192, gqa_n_q_heads=heads,
+                        gqa_n_kv_heads=heads // 8, gqa_head_dim=256, delta_n_qk_heads=16, delta_n_v_heads=2 * width // 128,
+                        delta_qk_head_dim=128, delta_v_head_dim=128, delta_chunk_size=64, n_routed_experts=experts,
+                        n_experts_per_token=top, moe_intermediate_size=ff, shared_expert_intermediate_size=shared_ff)
 
 
 def _qwen_run(cfg, B, T, steps, dev):
@@ -375,46 +390,54 @@ def _deepseek_run(cfg, B, T, steps, dev):
 def model_table(dev, sizes=((2048, 16), (4096, 32)), shapes=((1, 4096), (8, 1024)), steps: int = 24) -> list:
     """Prefill and decode tokens/s. ``sizes``: (width, attention heads); ``shapes``: (sequences, prompt length)."""
     from ..models.deepseek_v3 import DeepSeekV3Config
-    from ..models.qwen35 import Qwen35Config
     from ..models.vobunex import VobunexConfig
     E, top, ff, V = 64, 6, 1024, 65536
     rows = []
     for width, heads in sizes:
         hybrid = VobunexConfig.serving(width=width, n_mamba=6, n_attention=2, experts=E, top=top, ff=ff, heads=heads, vocab=V)
-        qwen = Qwen35Config(d_model=width, vocab_size=V, n_layers=8, max_position_embeddings=8192, gqa_n_q_heads=heads, gqa_n_kv_heads=heads // 8,
-                            gqa_head_dim=256, delta_n_qk_heads=16, delta_n_v_heads=2 * width // 128, delta_qk_head_dim=128,
-                            delta_v_head_dim=128, delta_chunk_size=64, n_routed_experts=E, n_experts_per_token=top,
-                            moe_intermediate_size=ff, shared_expert_intermediate_size=128)
+        qwen = qwen_like(width, heads, E, top, ff, V)
         latent = VobunexConfig.serving(width=width, n_mamba=0, n_attention=4, experts=E, top=top, ff=ff, heads=heads, vocab=V)
         ds = DeepSeekV3Config(d_model=width, vocab_size=V, n_layers=4, first_k_dense=0, max_position_embeddings=8192, n_heads=heads,
                               q_lora_rank=768, n_routed_experts=E, n_experts_per_token=top, n_group=1, topk_group=1,
                               moe_intermediate_size=ff)
-        for B, T in shapes:
-            row = {"width": width, "batch": B, "prompt": T}
-            for name, fn, cfg in (("vobunex_hybrid_8_layers", _vobunex_run, hybrid), ("qwen35_8_layers", _qwen_run, qwen),
-                                  ("vobunex_latent_4_layers", _vobunex_run, latent), ("deepseek_v3_4_layers", _deepseek_run, ds)):
-                try:
-                    pre, dec, *pre_all = fn(cfg, B, T, steps, dev)
-                    row[name] = {"prefill_ms": round(pre, 3), "prefill_tok_s": round(B * T / pre * 1e3), "decode_ms": round(dec, 4),
-                                 "decode_tok_s": round(B / dec * 1e3, 1)}
-                    if pre_all:      # the other families' prefill returns the logits of every position
-                        row[name]["prefill_all_logits_ms"] = round(pre_all[0], 3)
-                except Exception as e:  # noqa: BLE001 - a family that does not fit leaves the others' numbers
-                    row[name] = {"error": f"{type(e).__name__}: {str(e)[:200]}"}
-                _sync_free()
-            rows.append(row)
+        rows += model_rows(dev, width, shapes, steps, (("vobunex_hybrid_8_layers", _vobunex_run, hybrid), ("qwen35_8_layers", _qwen_run, qwen),
+                                                       ("vobunex_latent_4_layers", _vobunex_run, latent), ("deepseek_v3_4_layers", _deepseek_run, ds)))
     return rows
 
 
-def run(part: str = "all") -> dict:
+def model_rows(dev, width, shapes, steps, models) -> list:
+    """One row per shape; ``models``: (name, run function, configuration)."""
+    rows = []
+    for B, T in shapes:
+        row = {"width": width, "batch": B, "prompt": T}
+        for name, fn, cfg in models:
+            try:
+                pre, dec, *pre_all = fn(cfg, B, T, steps, dev)
+                row[name] = {"prefill_ms": round(pre, 3), "prefill_tok_s": round(B * T / pre * 1e3), "decode_ms": round(dec, 4),
+                             "decode_tok_s": round(B / dec * 1e3, 1)}
+                if pre_all:      # the other families' prefill returns the logits of every position
+                    row[name]["prefill_all_logits_ms"] = round(pre_all[0], 3)
+            except Exception as e:  # noqa: BLE001 - a family that does not fit leaves the others' numbers
+                row[name] = {"error": f"{type(e).__name__}: {str(e)[:200]}"}
+            _sync_free()
+        rows.append(row)
+    return rows
+
+
+def run(part: str = "all", family: str = "all") -> dict:
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
     out = {"data": "synthetic token ids, random weights", "dtype": "bf16 (fp32 residual, norms, states)"}
-    if part in ("kernels", "all"):
-        out["kernels"] = kernel_table(dev)
-        _sync_free()
-    if part in ("models", "all"):
-        out["models"] = model_table(dev)
+    from . import serve_bench_fovudra as fov
+    for name, kernels, models in (("vobunex", kernel_table, model_table), ("fovudra", fov.kernel_table, fov.model_table)):
+        if family not in (name, "all"):
+            continue
+        out[name] = {}
+        if part in ("kernels", "all"):
+            out[name]["kernels"] = kernels(dev)
+            _sync_free()
+        if part in ("models", "all"):
+            out[name]["models"] = models(dev)
     from .. import _ext
     _ext.check_status(dev)
     _sync_free()

@@ -9,7 +9,8 @@ that fits (doubling then bisection on out-of-memory, ``--max-batch`` caps it), t
 
 Timing is on the device with CUDA events, maximum over ranks (the reference uses host
 perf_counter and means only, scripts/bench_prefill_decode.py:246-264). ``--model`` selects the
-Qwen3.5 hybrid (``--config`` preset), the DeepSeek-V3 shape with its paged latent cache or Vobunex on its step engine.
+Qwen3.5 hybrid (``--config`` preset), the DeepSeek-V3 shape with its paged latent cache or Vobunex /
+Fovudra on the shared step engine.
 Results are printed and written as JSON to ``--out``.
 """
 from __future__ import annotations
@@ -19,7 +20,7 @@ import json
 import statistics
 import time
 
-from utils import fake_quant_w8a8, init_distributed, load_hf_dir, make_tp_dp_groups, qwen_config, vobunex_config
+from utils import fake_quant_w8a8, init_distributed, load_hf_dir, make_tp_dp_groups, qwen_config, step_engine_config
 
 import torch
 
@@ -118,23 +119,23 @@ def make_runner(args, device):
             logits, cache = forward(params, nxt[:, None], cfg, cache=cache, is_decode=True, ep_group=ep, tp_group=tp_group)
             return logits[:, -1].argmax(-1), cache
         return prefill, decode, cfg
-    if args.model == "vobunex":
+    if args.model in ("vobunex", "fovudra"):
         if args.tp > 1 or args.dp > 1 or args.w8a8 or args.fp8:
-            raise SystemExit("--tp / --dp / --w8a8 / --fp8 do not apply to --model vobunex")
-        from jax_gpt_b200.models.registry import load_model
-        from jax_gpt_b200.models.vobunex import VobunexEngine, init_params, make_cache
+            raise SystemExit(f"--tp / --dp / --w8a8 / --fp8 do not apply to --model {args.model}")
+        from jax_gpt_b200.models.registry import FAMILIES, load_model
+        family = FAMILIES[args.model]
         if args.model_dir and not args.random_weights:
-            _, cfg, params = load_model(args.model_dir, dtype, device)
+            family, cfg, params = load_model(args.model_dir, dtype, device)
         else:
-            cfg = vobunex_config(args.config if args.config != "mini" else "serving")
-            params = init_params(cfg, 0, dtype=dtype, device=device, on_device=device.type == "cuda")
+            cfg = step_engine_config(args.model, args.config if args.config != "mini" else "serving")
+            params = family.mod().init_params(cfg, 0, dtype=dtype, device=device, on_device=device.type == "cuda")
         plen, dlen = SCENARIOS[args.scenario]
         live = {}
 
         def prefill(B):
             live.clear()
             per = (plen + dlen + cfg.page_size - 1) // cfg.page_size
-            eng = VobunexEngine(params, cfg, make_cache(cfg, B * per, B, per, dtype, device), use_cuda_graph=not args.no_graph)
+            eng = getattr(family.mod(), family.engine)(params, cfg, family.mod().make_cache(cfg, B * per, B, per, dtype, device), use_cuda_graph=not args.no_graph)
             gen = torch.Generator().manual_seed(1234)
             tok = torch.randint(0, cfg.vocab_size, (B, plen), generator=gen)
             live["eng"] = eng
@@ -221,7 +222,7 @@ def find_max_batch(prefill, decode, cap):
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--model", default="qwen35", choices=["qwen35", "deepseek_v3", "vobunex"])
+    ap.add_argument("--model", default="qwen35", choices=["qwen35", "deepseek_v3", "vobunex", "fovudra"])
     ap.add_argument("--model-dir", default="", help="HF safetensors directory (random weights when empty)")
     ap.add_argument("--scenario", default="1k1k", choices=sorted(SCENARIOS))
     ap.add_argument("--tp", type=int, default=1)

@@ -85,10 +85,12 @@ def qwen_config(name: str):
             "full": Qwen35Config.full, "ns": Qwen35Config.ns, "tiny": Qwen35Config.tiny}[name]()
 
 
-def vobunex_config(name: str):
-    from jax_gpt_b200.models.vobunex import VobunexConfig
-    return {"tiny": VobunexConfig.tiny, "serving": VobunexConfig.serving,
-            "serving_wide": lambda: VobunexConfig.serving(width=4096, heads=32, ff=1536)}[name]()
+def step_engine_config(family: str, name: str):
+    """Preset of a family on the shared step engine (``--model vobunex`` / ``fovudra``)."""
+    from jax_gpt_b200.models.registry import FAMILIES
+    cls = FAMILIES[family].config_class()
+    wide = dict(width=4096, heads=32, ff=1536, **({"kv_heads": 4} if family == "fovudra" else {}))
+    return {"tiny": cls.tiny, "serving": cls.serving, "serving_wide": lambda: cls.serving(**wide)}[name]()
 
 
 class ByteTokenizer:
