@@ -187,32 +187,56 @@ attn_decode_split_kernel(const DecArgs a) {
   }
 }
 
-// out[b, h, :] = sum_s part_o[s] 2^(m_s - M) / sum_s l_s 2^(m_s - M); one CTA per (head, sequence), D threads.
+// out[b, h, :] = sum_s part_o[s] 2^(m_s - M) / sum_s l_s 2^(m_s - M); one CTA per (head, sequence). The ranges' weights go
+// through shared memory; kGroups groups of D threads each sum every kGroups-th range.
+constexpr int kMaxSplits = 256;
+
 template <int D>
-__global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                         int n_splits, __nv_bfloat16* __restrict__ out, int64_t ldo, int H) {
-  const int h = blockIdx.x, b = blockIdx.y, c = threadIdx.x;
+__global__ void __launch_bounds__(512)
+attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int n_splits,
+                         __nv_bfloat16* __restrict__ out, int64_t ldo, int H) {
+  constexpr int kGroups = 512 / D;
+  __shared__ float wt[kMaxSplits], acc_s[kGroups][D], red[1];
+  const int h = blockIdx.x, b = blockIdx.y, c = threadIdx.x % D, grp = threadIdx.x / D;
   const int64_t row0 = (static_cast<int64_t>(b) * H + h) * n_splits;
-  float mn = -INFINITY;
-  for (int s = 0; s < n_splits; ++s) mn = fmaxf(mn, part_ml[(row0 + s) * 2]);
-  float acc = 0.f, ls = 0.f;
-  for (int s = 0; s < n_splits; ++s) {
-    const float ms = part_ml[(row0 + s) * 2];
-    const float wt = (ms == -INFINITY) ? 0.f : exp2f(ms - mn);
-    acc = fmaf(part_o[(row0 + s) * D + c], wt, acc);
-    ls = fmaf(part_ml[(row0 + s) * 2 + 1], wt, ls);
+  if (threadIdx.x < 32) {
+    float mn = -INFINITY, ls = 0.f;
+    for (int s = threadIdx.x; s < n_splits; s += 32) mn = fmaxf(mn, part_ml[(row0 + s) * 2]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, o));
+    for (int s = threadIdx.x; s < n_splits; s += 32) {
+      const float ms = part_ml[(row0 + s) * 2];
+      const float w = (ms == -INFINITY) ? 0.f : exp2f(ms - mn);
+      wt[s] = w;
+      ls = fmaf(part_ml[(row0 + s) * 2 + 1], w, ls);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ls += __shfl_xor_sync(0xffffffffu, ls, o);
+    if (threadIdx.x == 0) red[0] = ls;
   }
-  out[static_cast<int64_t>(b) * ldo + h * D + c] = __float2bfloat16(ls > 0.f ? acc / ls : 0.f);
+  __syncthreads();
+  float acc = 0.f;
+#pragma unroll 8
+  for (int s = grp; s < n_splits; s += kGroups) acc = fmaf(part_o[(row0 + s) * D + c], wt[s], acc);
+  acc_s[grp][c] = acc;
+  __syncthreads();
+  if (grp == 0) {
+#pragma unroll
+    for (int g = 1; g < kGroups; ++g) acc += acc_s[g][c];
+    const float ls = red[0];
+    out[static_cast<int64_t>(b) * ldo + h * D + c] = __float2bfloat16(ls > 0.f ? acc / ls : 0.f);
+  }
 }
 
 template <int D, int G>
 cudaError_t decode_launch(const DecArgs& a, int B, int n_splits, __nv_bfloat16* out, int64_t ldo,
                           cudaStream_t stream) {
+  if (n_splits > kMaxSplits) return cudaErrorInvalidValue;
   dim3 grid(n_splits, a.Hkv, B);
   attn_decode_split_kernel<D, G><<<grid, kDecWarps * 32, 0, stream>>>(a);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return e;
-  attn_decode_merge_kernel<D><<<dim3(a.H, B), D, 0, stream>>>(a.part_o, a.part_ml, n_splits, out, ldo, a.H);
+  attn_decode_merge_kernel<D><<<dim3(a.H, B), 512, 0, stream>>>(a.part_o, a.part_ml, n_splits, out, ldo, a.H);
   return cudaGetLastError();
 }
 

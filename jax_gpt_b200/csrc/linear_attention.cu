@@ -182,8 +182,29 @@ linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
   const int64_t row = sb.cu[b];
   const T* x = qkv + row * ld;
   constexpr int kLanes = kStepCols / V, kRows = kStepThreads / kLanes;
+  constexpr int kAhead = V == 4 ? 8 : 16;   // state rows of a thread in flight; the first ones load before the gates are known
   const int r = threadIdx.x / kLanes, c = (threadIdx.x % kLanes) * V;
+  const bool live = c < cols;
   float* st = state + (static_cast<int64_t>(slot) * s.H + h) * N * P + p0 + c;
+  float S[kAhead][V];
+  auto load = [&](int n0) {
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i) {
+      const int n = n0 + i * kRows;
+#pragma unroll
+      for (int j = 0; j < V; ++j) S[i][j] = 0.f;
+      if (live && !fresh && n < N) {
+        const float* sp = st + static_cast<int64_t>(n) * P;
+        if constexpr (V == 4) {
+          const float4 f = *reinterpret_cast<const float4*>(sp);
+          S[i][0] = f.x; S[i][1] = f.y; S[i][2] = f.z; S[i][3] = f.w;
+        } else {
+          S[i][0] = sp[0];
+        }
+      }
+    }
+  };
+  load(r);
   for (int i = threadIdx.x; i < N; i += blockDim.x) {
     sq[i] = qkv_at(x + h * N + i, s.silu);
     sk[i] = qkv_at(x + (s.H + h) * N + i, s.silu);
@@ -203,32 +224,26 @@ linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
     a = gates.decay[h];
   }
   __syncthreads();
-  if (c < cols) {
+  if (live) {
     float acc[V], dx[V];
 #pragma unroll
     for (int j = 0; j < V; ++j) { acc[j] = 0.f; dx[j] = w * sv[c + j]; }
-#pragma unroll 8
-    for (int n = r; n < N; n += kRows) {
-      float S[V];
-      float* sp = st + static_cast<int64_t>(n) * P;
+    for (int n0 = r; n0 < N; n0 += kAhead * kRows) {
+      if (n0 != r) load(n0);
 #pragma unroll
-      for (int j = 0; j < V; ++j) S[j] = 0.f;
-      if (!fresh) {
-        if constexpr (V == 4) {
-          const float4 f = *reinterpret_cast<const float4*>(sp);
-          S[0] = f.x; S[1] = f.y; S[2] = f.z; S[3] = f.w;
-        } else {
-          S[0] = sp[0];
+      for (int i = 0; i < kAhead; ++i) {
+        const int n = n0 + i * kRows;
+        if (n >= N) break;
+        float* sp = st + static_cast<int64_t>(n) * P;
+        const float kn = sk[n], qn = sq[n];
+#pragma unroll
+        for (int j = 0; j < V; ++j) {
+          S[i][j] = fmaf(S[i][j], a, dx[j] * kn);
+          acc[j] = fmaf(S[i][j], qn, acc[j]);
         }
+        if constexpr (V == 4) *reinterpret_cast<float4*>(sp) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
+        else sp[0] = S[i][0];
       }
-      const float kn = sk[n], qn = sq[n];
-#pragma unroll
-      for (int j = 0; j < V; ++j) {
-        S[j] = fmaf(S[j], a, dx[j] * kn);
-        acc[j] = fmaf(S[j], qn, acc[j]);
-      }
-      if constexpr (V == 4) *reinterpret_cast<float4*>(sp) = make_float4(S[0], S[1], S[2], S[3]);
-      else sp[0] = S[0];
     }
 #pragma unroll
     for (int j = 0; j < V; ++j) part[r * kStepCols + c + j] = acc[j];
@@ -293,6 +308,7 @@ __device__ __forceinline__ void commit_vec(const HeadNorm& a, const SeqBatch& sb
   if (n != sb.cu[b + 1] - 1) return;
   const float* src = a.vec_new + (static_cast<int64_t>(b) * a.parts + h) * a.vec_len;
   float* dst = a.vec + (static_cast<int64_t>(sb.ids[b]) * a.parts + h) * a.vec_len;
+#pragma unroll 8
   for (int i = tid; i < a.vec_len; i += threads) dst[i] = src[i];
 }
 

@@ -288,7 +288,7 @@ rows_linear_kernel(const T* __restrict__ x, int64_t ldx, const T* __restrict__ w
   for (int m = 0; m < MR; ++m) xr[m] = x + static_cast<int64_t>(m0 + m < M ? m0 + m : m0) * ldx;
   if constexpr (kVec) {
     constexpr int V = Vec16<T>::n;
-#pragma unroll 2
+#pragma unroll (MR == 1 ? 4 : 2)
     for (int k = lane * V; k < K; k += 32 * V) {
       float wv[NR][V];
 #pragma unroll
@@ -445,7 +445,7 @@ cudaError_t rows_linear_t(const void* x, int64_t ldx, const void* w, int64_t ldw
 #define B200_GO(MR)                                                                                       \
   {                                                                                                       \
     if constexpr (kGlu) rows_linear_go<T, MR, 2, true>(vec, xt, ldx, wt, ldw, M, N, K, out, st);          \
-    else if (N >= 148 * kLinWarps * 4) rows_linear_go<T, MR, 4, false>(vec, xt, ldx, wt, ldw, M, N, K, out, st); \
+    else if (MR > 1 && N >= 148 * kLinWarps * 4) rows_linear_go<T, MR, 4, false>(vec, xt, ldx, wt, ldw, M, N, K, out, st); \
     else if (N >= 148 * kLinWarps * 2) rows_linear_go<T, MR, 2, false>(vec, xt, ldx, wt, ldw, M, N, K, out, st); \
     else rows_linear_go<T, MR, 1, false>(vec, xt, ldx, wt, ldw, M, N, K, out, st);                        \
   }
@@ -847,22 +847,38 @@ __device__ __forceinline__ int next_best(const float* z, int E, float pv, int pi
   return bi;
 }
 
-// Expert number j of token m and the factor of the expert's input (a whole warp calls it). -1: bad token or table entry.
-__device__ __forceinline__ int choose_expert(const ExpertChoice& c, int m, int j, float& w) {
-  w = 1.f;
-  if (c.logits == nullptr) {
-    const int tok = c.tokens[m];
-    return tok >= 0 && tok < c.vocab ? c.table[static_cast<int64_t>(tok) * c.top + j] : -1;
+// Experts of token m into `chosen` (shared memory, c.top entries, -1: bad token or table entry), scores' logits into
+// `score` when that is not null; `z` holds c.E floats of shared memory for the router. The whole block calls it. Ranks are
+// counted, one logit per thread: no chain of reductions.
+__device__ __forceinline__ void choose_experts(const ExpertChoice& c, int m, float* z, int* chosen, float* score) {
+  for (int j = threadIdx.x; j < c.top; j += blockDim.x) {
+    const int tok = c.logits == nullptr ? c.tokens[m] : -1;
+    chosen[j] = tok >= 0 && tok < c.vocab ? c.table[static_cast<int64_t>(tok) * c.top + j] : -1;
   }
-  const float* z = c.logits + static_cast<int64_t>(m) * c.E;
-  float v = INFINITY;
-  int e = -1;
-  for (int i = 0; i <= j; ++i) {
-    e = next_best(z, c.E, v, e, v);
-    if (e < 0) return -1;
+  if (c.logits != nullptr) {
+    const int pad = (c.E + 3) & ~3;
+    for (int i = threadIdx.x; i < pad; i += blockDim.x) z[i] = i < c.E ? c.logits[static_cast<int64_t>(m) * c.E + i] : -INFINITY;
+    __syncthreads();
+    for (int i = threadIdx.x; i < c.E; i += blockDim.x) {
+      const float v = z[i];
+      int rank = 0;
+#pragma unroll 4
+      for (int k = 0; k < pad; k += 4) {
+        const float4 o = *reinterpret_cast<const float4*>(z + k);
+        rank += (o.x > v || (o.x == v && k < i)) + (o.y > v || (o.y == v && k + 1 < i)) + (o.z > v || (o.z == v && k + 2 < i)) +
+                (o.w > v || (o.w == v && k + 3 < i));
+      }
+      if (rank < c.top && v == v) {
+        chosen[rank] = i;
+        if (score != nullptr) score[rank] = v;
+      }
+    }
   }
-  w = sigmoid_f(v);
-  return e;
+  __syncthreads();
+}
+// shared memory of choose_experts: logits, then experts, then scores
+__host__ __device__ __forceinline__ int choice_smem(const ExpertChoice& c) {
+  return 4 * ((c.logits != nullptr ? (c.E + 3) & ~3 : 0) + 2 * c.top);
 }
 
 // One warp per token: ids and sigmoid scores of the `top` largest logits.
@@ -890,9 +906,13 @@ template <typename T, bool kVec>
 __global__ void __launch_bounds__(kExpWarps * 32)
 experts_up_kernel(const T* __restrict__ x, const ExpertChoice c, const T* __restrict__ w, GluArgs glu, T* __restrict__ h, int D,
                   int I, int* status) {
+  extern __shared__ __align__(16) float zs[];
   const int pair = blockIdx.x, m = pair / c.top;
-  float wt;
-  const int e = choose_expert(c, m, pair % c.top, wt);
+  int* chosen = reinterpret_cast<int*>(zs + (choice_smem(c) / 4 - 2 * c.top));
+  float* score = reinterpret_cast<float*>(chosen + c.top);
+  choose_experts(c, m, zs, chosen, score);
+  const int e = chosen[pair % c.top];
+  const float wt = c.logits != nullptr ? sigmoid_f(score[pair % c.top]) : 1.f;
   if (e < 0 || e >= c.E) {
     if (threadIdx.x == 0) report_status(status, kBadArgument, 303, m, e);
     return;
@@ -905,7 +925,7 @@ experts_up_kernel(const T* __restrict__ x, const ExpertChoice c, const T* __rest
     float g = 0.f, u = 0.f;
     if constexpr (kVec) {
       constexpr int V = Vec16<T>::n;
-#pragma unroll 2
+#pragma unroll 4
       for (int k = lane * V; k < D; k += 32 * V) {
         float xv[V], gv[V], uv[V];
         Vec16<T>::load(xr + k, xv);
@@ -930,47 +950,56 @@ experts_up_kernel(const T* __restrict__ x, const ExpertChoice c, const T* __rest
   }
 }
 
-// x[m, d] += out_scale * sum_j down_e(j)[d] . h[m * top + j]; w_down [E, D, I]. Dynamic shared memory: top ints.
-template <typename T, bool kVec>
+// x[m, d] += out_scale * sum_j down_e(j)[d] . h[m * top + j]; w_down [E, D, I]. A warp owns an output feature and walks its
+// experts' rows kJ at a time (few rows: two, for more loads in flight; more rows: one, for more blocks).
+template <typename T, bool kVec, int kJ>
 __global__ void __launch_bounds__(kExpWarps * 32)
 experts_down_kernel(const T* __restrict__ h, const ExpertChoice c, const T* __restrict__ w, float out_scale, float* __restrict__ x,
                     int D, int I) {
-  extern __shared__ int chosen[];
-  const int m = blockIdx.x;
-  const int lane = threadIdx.x & 31;
-  if (threadIdx.x < 32) {
-    float v = INFINITY;
-    int e = -1;
-    for (int j = 0; j < c.top; ++j) {
-      if (c.logits == nullptr) e = choose_expert(c, m, j, v);
-      else if (j == 0 || e >= 0) e = next_best(c.logits + static_cast<int64_t>(m) * c.E, c.E, v, e, v);
-      if (lane == 0) chosen[j] = e;
-    }
-  }
-  __syncthreads();
+  extern __shared__ __align__(16) float zs[];
+  const int m = blockIdx.x, lane = threadIdx.x & 31;
+  int* chosen = reinterpret_cast<int*>(zs + (choice_smem(c) / 4 - 2 * c.top));
+  choose_experts(c, m, zs, chosen, nullptr);
+  const T* hm = h + static_cast<int64_t>(m) * c.top * I;
   for (int d = blockIdx.y * kExpWarps + (threadIdx.x >> 5); d < D; d += gridDim.y * kExpWarps) {
+    float* xo = x + static_cast<int64_t>(m) * D + d;
+    const float before = *xo;
     float acc = 0.f;
-    for (int j = 0; j < c.top; ++j) {
-      const int e = chosen[j];
-      if (e < 0 || e >= c.E) continue;
-      const T* wr = w + (static_cast<int64_t>(e) * D + d) * I;
-      const T* hr = h + (static_cast<int64_t>(m) * c.top + j) * I;
+    for (int j = 0; j < c.top; j += kJ) {
+      const T *wr[kJ], *hr[kJ];
+      bool ok[kJ];
+      float part[kJ];
+#pragma unroll
+      for (int q = 0; q < kJ; ++q) {   // a missing expert reads its neighbour's rows (or expert 0's) and counts nothing
+        const int e = j + q < c.top ? chosen[j + q] : -1;
+        ok[q] = e >= 0 && e < c.E;
+        wr[q] = w + (static_cast<int64_t>(ok[q] ? e : 0) * D + d) * I;
+        hr[q] = hm + static_cast<int64_t>(ok[q] ? j + q : 0) * I;
+        part[q] = 0.f;
+      }
       if constexpr (kVec) {
         constexpr int V = Vec16<T>::n;
-#pragma unroll 2
+#pragma unroll 4
         for (int k = lane * V; k < I; k += 32 * V) {
-          float hv[V], wv[V];
-          Vec16<T>::load(hr + k, hv);
-          Vec16<T>::load(wr + k, wv);
 #pragma unroll
-          for (int q = 0; q < V; ++q) acc = fmaf(hv[q], wv[q], acc);
+          for (int q = 0; q < kJ; ++q) {
+            float hv[V], wv[V];
+            Vec16<T>::load(hr[q] + k, hv);
+            Vec16<T>::load(wr[q] + k, wv);
+#pragma unroll
+            for (int t = 0; t < V; ++t) part[q] = fmaf(hv[t], wv[t], part[q]);
+          }
         }
       } else {
-        for (int k = lane; k < I; k += 32) acc = fmaf(ldf(hr + k), ldf(wr + k), acc);
+        for (int k = lane; k < I; k += 32)
+#pragma unroll
+          for (int q = 0; q < kJ; ++q) part[q] = fmaf(ldf(hr[q] + k), ldf(wr[q] + k), part[q]);
       }
+#pragma unroll
+      for (int q = 0; q < kJ; ++q) acc += ok[q] ? part[q] : 0.f;
     }
     acc = warp_sum(acc);
-    if (lane == 0) x[static_cast<int64_t>(m) * D + d] += acc * out_scale;
+    if (lane == 0) *xo = before + acc * out_scale;
   }
 }
 
@@ -1181,11 +1210,13 @@ cudaError_t launch_latent_attention(bool f32, const SeqBatch& sb, const void* qf
 
 cudaError_t launch_experts_up(bool f32, const void* x, const ExpertChoice& c, const void* w, GluArgs glu, void* h, int M, int D,
                               int I, int* status, cudaStream_t st) {
-  const int per = (I + kExpWarps - 1) / kExpWarps;
-  const dim3 grid(M * c.top, per < 64 ? per : 64);
+  // enough blocks for the loads in flight, few enough that the choice of the experts is not repeated too often
+  const int per = (I + kExpWarps - 1) / kExpWarps, want = 148 * (M <= 2 ? 16 : 8) / (M * c.top), smem = choice_smem(c);
+  const dim3 grid(M * c.top, want < 1 ? 1 : (want < per ? want : per));
+  if (smem > 48 * 1024) return cudaErrorInvalidValue;
   const bool vec = D % (f32 ? 4 : 8) == 0;
 #define B200_UP(T, V) \
-  experts_up_kernel<T, V><<<grid, kExpWarps * 32, 0, st>>>(static_cast<const T*>(x), c, static_cast<const T*>(w), glu, static_cast<T*>(h), D, I, status)
+  experts_up_kernel<T, V><<<grid, kExpWarps * 32, smem, st>>>(static_cast<const T*>(x), c, static_cast<const T*>(w), glu, static_cast<T*>(h), D, I, status)
   if (f32) { if (vec) B200_UP(float, true); else B200_UP(float, false); }
   else { if (vec) B200_UP(__nv_bfloat16, true); else B200_UP(__nv_bfloat16, false); }
 #undef B200_UP
@@ -1194,14 +1225,17 @@ cudaError_t launch_experts_up(bool f32, const void* x, const ExpertChoice& c, co
 
 cudaError_t launch_experts_down(bool f32, const void* h, const ExpertChoice& c, const void* w, float out_scale, float* x, int M,
                                 int D, int I, cudaStream_t st) {
-  if (c.top * 4 > 48 * 1024) return cudaErrorInvalidValue;
-  const int per = (D + kExpWarps - 1) / kExpWarps;
-  const dim3 grid(M, per < 256 ? per : 256);
+  const int per = (D + kExpWarps - 1) / kExpWarps, want = 148 * 16 / M, smem = choice_smem(c);
+  const dim3 grid(M, want < 1 ? 1 : (want < per ? want : per));
+  if (smem > 48 * 1024) return cudaErrorInvalidValue;
   const bool vec = I % (f32 ? 4 : 8) == 0;
 #define B200_DN(T, V) \
-  experts_down_kernel<T, V><<<grid, kExpWarps * 32, c.top * 4, st>>>(static_cast<const T*>(h), c, static_cast<const T*>(w), out_scale, x, D, I)
-  if (f32) { if (vec) B200_DN(float, true); else B200_DN(float, false); }
-  else { if (vec) B200_DN(__nv_bfloat16, true); else B200_DN(__nv_bfloat16, false); }
+  {                                                                                                                                         \
+    if (M <= 2) experts_down_kernel<T, V, 2><<<grid, kExpWarps * 32, smem, st>>>(static_cast<const T*>(h), c, static_cast<const T*>(w), out_scale, x, D, I); \
+    else experts_down_kernel<T, V, 1><<<grid, kExpWarps * 32, smem, st>>>(static_cast<const T*>(h), c, static_cast<const T*>(w), out_scale, x, D, I);        \
+  }
+  if (f32) { if (vec) B200_DN(float, true) else B200_DN(float, false) }
+  else { if (vec) B200_DN(__nv_bfloat16, true) else B200_DN(__nv_bfloat16, false) }
 #undef B200_DN
   return cudaGetLastError();
 }

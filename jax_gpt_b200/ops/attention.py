@@ -104,9 +104,9 @@ def attn_fwd_cached(q, cache_k, cache_v, kv_len: int, q_pos0: int, causal=True, 
 
 def decode_splits(batch: int, n_kv_heads: int, max_len: int) -> int:
     """Key ranges per (sequence, kv head) for ``attention_decode``: enough CTAs to cover the SMs about twice,
-    at least 64 keys per range."""
+    at least 16 keys per range (one step of its warps)."""
     want = max(1, 296 // max(1, batch * n_kv_heads))
-    return int(max(1, min(want, (max_len + 63) // 64, 64)))
+    return int(max(1, min(want, (max_len + 15) // 16, 128)))
 
 
 def attention_decode(q, cache_k, cache_v, kv_len=None, pos: Optional[torch.Tensor] = None, scale=None,

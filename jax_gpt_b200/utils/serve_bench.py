@@ -64,7 +64,7 @@ class _KernelTimer:
     def __call__(self, fn, bytes_: float = 0.0, flops: float = 0.0) -> dict:
         ms = max(self._run(fn) - self._run(None), 1e-4)
         roof = max(bytes_ / (self.peaks["hbm_gbs"] * 1e6), flops / (self.peaks["bf16_tflops"] * 1e9))
-        return {"us": round(ms * 1e3, 2), "roofline_us": round(roof * 1e3, 2), "frac": round(roof / ms, 3)}
+        return {"us": round(ms * 1e3, 2), "roofline_us": round(roof * 1e3, 2), "frac": float(f"{roof / ms:.3g}")}
 
 
 def _start_batch(seq_ids, lens, start, dev, max_len):
@@ -116,7 +116,7 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
         if other is not None:
             e["other"] = other
             e["other_kernel"] = other_name
-            e["distance_ratio"] = round(other["frac"] / max(mine["frac"], 1e-6), 2)   # > 1: further from the roofline than the other
+            e["distance_ratio"] = round(other["frac"] / max(mine["frac"], 1e-9), 2)   # > 1: further from the roofline than the other
         out[part][name] = e
 
     # ---- prefill: state-space layer beside the DeltaNet layer ----

@@ -35,7 +35,7 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
 
     def put(part, name, mine, other, other_name):
         part[name] = {"fovudra": mine, "other": other, "other_kernel": other_name,
-                      "distance_ratio": round(other["frac"] / max(mine["frac"], 1e-6), 2)}   # > 1: further from the roofline
+                      "distance_ratio": round(other["frac"] / max(mine["frac"], 1e-9), 2)}   # > 1: further from the roofline
     pre = out["prefill"]
     batch = _start_batch(list(range(seqs)), [seq_len] * seqs, 0, dev, seq_len)
 
@@ -150,8 +150,10 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
         qd = rn(B, Q, Dh)
         kb = lambda n: 2.0 * B * n * 2 * Gk * Dh
         dec = lambda w, kp: A.attention_decode_paged(qd, cache.pool[0], cache.block_table, idt, cache.seq_lens, Gk, 0, 0.09, max_len=ctx, window=w, keep_first=kp)
-        put(d, "paged attention, window + kept tokens", tm(lambda: dec(window, keep_first), kb(window + keep_first)), tm(lambda: dec(0, 0), kb(ctx)),
-            f"the same kernel, all {ctx} keys")
+        windowed = tm(lambda: dec(window, keep_first), kb(window + keep_first))
+        cache.seq_lens.fill_(window + keep_first)
+        put(d, "paged attention, window + kept tokens", windowed, tm(lambda: dec(0, 0), kb(window + keep_first)),
+            f"the same kernel, {window + keep_first} cached keys, all seen")
         y1 = rn(B, (Q + Gk) * Dh)
         xq1, n1w = rn(B, 1, Q, 256), rn(256)
         put(d, "bias, rotation, unit norm, cache write", tm(lambda: WA.qk_prepare(bd, y1, bqk, Q, Gk, Dh, True, 1e-5, rope, cache, 0, dense=False), 2.0 * B * Dh * (2 * Q + 3 * Gk)),
