@@ -5,6 +5,7 @@
     python -m jax_gpt_b200.utils.kernel_bench --op attn_bwd | norm_fwd | norm_bwd | adamw | ce
     python -m jax_gpt_b200.utils.kernel_bench --op mla_decode --B 32 --T 2304 --H 16
     python -m jax_gpt_b200.utils.kernel_bench --op ssd_scan --B 2 --T 4096 --H 64
+    python -m jax_gpt_b200.utils.kernel_bench --op gated_scan | decay_scan --B 2 --T 4096 --H 16
     python -m jax_gpt_b200.utils.kernel_bench --op gdn_prep_fwd | gdn_prep_bwd | gdn_prefill --B 1 --T 4096
 
 Each run does ``--warmup`` untimed launches, then times ``--iters`` launches with CUDA events on
@@ -214,6 +215,20 @@ def main(argv=None):
         fn = lambda: ssm.ssd_scan(batch, xbc, dt, db, al, dk, state, G)
         bytes_ = 2.0 * B * T * (C + H * 64 + H) + 4.0 * state.numel()
         flops = B * T / 128 * H * 2.0 * 128 * (128 * 128 + 3 * 128 * 64)
+    elif args.op in ("gated_scan", "decay_scan"):
+        # --B sequences of --T tokens, --H heads of 128 with keys of 128: exponential gates (mLSTM) or a fixed decay per head
+        from ..ops import linear_attention as LIN
+        from .serve_bench import _start_batch
+        B, T, H = args.B, args.T, args.H
+        batch = _start_batch(list(range(B)), [T] * B, 0, dev, T)
+        qkv = (torch.randn(B * T, 3 * H * 128, device=dev) * 0.3).to(torch.bfloat16)
+        state, vec = torch.zeros(B, H, 128, 128, device=dev), torch.zeros(B, H, 129, device=dev)
+        raw, bias = torch.randn(B * T, 2 * H, device=dev), torch.cat([torch.zeros(H), torch.full((H,), 4.0)]).to(dev)
+        gates = LIN.Gates(raw, bias, 15.0, vec) if args.op == "gated_scan" else None
+        decay = None if gates is not None else torch.full((H,), 0.99, device=dev)
+        fn = lambda: LIN.linear_scan(batch, qkv, state, gates=gates, decay=decay, q_scale=128 ** -0.5)
+        bytes_ = 8.0 * B * T * H * 128 + (24.0 * B * T * H if gates is not None else 0.0) + 4.0 * state.numel()
+        flops = B * T / 128 * H * 2.0 * 128 * (128 * 128 + 3 * 128 * 128)
     elif args.op == "mla_decode":
         # --B sequences of --T cached tokens each, --H heads (16 = DeepSeek-V3 with 8-way head sharding)
         from ..cache.paged import PagedCache
