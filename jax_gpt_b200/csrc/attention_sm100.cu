@@ -19,7 +19,6 @@
 #include "attention_sm100.cuh"
 
 #include <algorithm>
-#include <climits>
 #include <cstdlib>
 
 #include "common.cuh"
@@ -44,7 +43,7 @@ struct FwdArgs {
   float* lse;
   int* status;
   const float* sink;        // [H] or nullptr: extra term exp(sink[h]) of the softmax denominator
-  int window, keep_first;   // keys j with i - j < window or j < keep_first are seen (window INT_MAX: all)
+  int window, keep_first;   // kWindow instances: keys j with i - j < window or j < keep_first are seen
 };
 
 // D: width of q and k heads; DV: width of v heads (MLA prefill uses 192 / 128).
@@ -87,7 +86,10 @@ __device__ __forceinline__ void load_tile(uint8_t* dst, const CUtensorMap* m, ui
   for (int h = 0; h < D / 64; ++h) tma_load_2d(dst + h * 16384, m, bar, col0 + h * 64, row0);
 }
 
-template <int D, int DV>
+// bits 0 .. n - 1
+__device__ __forceinline__ uint32_t bits_below(int n) { return n <= 0 ? 0u : (n >= 32 ? 0xffffffffu : (1u << n) - 1u); }
+
+template <int D, int DV, bool kWindow>
 __global__ void __launch_bounds__(kThreads, (D == 64) ? 2 : 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                 const __grid_constant__ CUtensorMap tv, const __grid_constant__ FwdArgs a) {
@@ -109,10 +111,10 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
   const int q0 = a.q_pos0 + q_blk * 128;     // position of the block's first query
   const int n_seen = a.causal ? min((q0 + 127) / 128 + 1, n_kv_all) : n_kv_all;
   // key tiles: those of the kept first keys, then those from the window of the first query on
-  const int n_keep = min((a.keep_first + 127) / 128, n_seen);
-  const int w_tile = max(n_keep, min(max(0, q0 - a.window + 1) / 128, n_seen));
+  const int n_keep = kWindow ? min((a.keep_first + 127) / 128, n_seen) : 0;
+  const int w_tile = kWindow ? max(n_keep, min(max(0, q0 - a.window + 1) / 128, n_seen)) : 0;
   const int n_kv = n_keep + n_seen - w_tile;
-  auto key_tile = [&](int j) { return j < n_keep ? j : w_tile + j - n_keep; };
+  auto key_tile = [&](int j) { return kWindow && j >= n_keep ? w_tile + j - n_keep : j; };
   const int row0 = b * a.T + q_blk * 128;
   const int kv_row0 = b * a.kv_rows_b + hkv * a.kv_rows_h;
 
@@ -228,9 +230,14 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       tc_fence_after();
       const int kt0 = key_tile(j) * 128;
       const bool need_mask = (a.causal && kt0 + 127 > q0) || kt0 + 128 > a.Tk ||
-                             (q0 + 127 - kt0 >= a.window && kt0 + 127 >= a.keep_first);
-      auto hidden = [&](int kv) {
-        return kv >= a.Tk || (a.causal && kv > qpos) || (qpos - kv >= a.window && kv >= a.keep_first);
+                             (kWindow && q0 + 127 - kt0 >= a.window && kt0 + 127 >= a.keep_first);
+      // scores of 32 keys from position k0 on: those this row does not see become -inf
+      auto hide = [&](uint32_t (&v)[32], int k0) {
+        uint32_t seen = bits_below((a.causal ? min(qpos + 1, a.Tk) : a.Tk) - k0);
+        if (kWindow) seen &= ~bits_below(qpos - a.window + 1 - k0) | bits_below(a.keep_first - k0);
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+          if (!(seen >> i & 1u)) v[i] = 0xff800000u;
       };
       const int kv0 = kt0 + half * 64;
       float mx = -INFINITY;
@@ -239,12 +246,9 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         uint32_t v[32];
         tmem_ld_32x32(tmem + half * 64 + c * 32 + lane_off, v);
         tmem_ld_wait();
+        if (need_mask) hide(v, kv0 + c * 32);
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-          float s = __uint_as_float(v[i]);   // the (positive) softmax scale is applied to the maximum once, below
-          if (need_mask && hidden(kv0 + c * 32 + i)) s = -INFINITY;
-          mx = fmaxf(mx, s);
-        }
+        for (int i = 0; i < 32; ++i) mx = fmaxf(mx, __uint_as_float(v[i]));   // the (positive) scale is applied once, below
       }
       mx *= a.scale_log2;
       const __nv_bfloat16 mine = __float2bfloat16(mx);
@@ -265,16 +269,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         uint32_t v[32];
         tmem_ld_32x32(tmem + half * 64 + c * 32 + lane_off, v);
         tmem_ld_wait();
+        if (need_mask) hide(v, kv0 + c * 32);
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          float s0 = fmaf(__uint_as_float(v[i]), a.scale_log2, -mref), s1 = fmaf(__uint_as_float(v[i + 1]), a.scale_log2, -mref);
-          if (need_mask) {
-            const int kvpos = kv0 + c * 32 + i;
-            if (hidden(kvpos)) s0 = -INFINITY;
-            if (hidden(kvpos + 1)) s1 = -INFINITY;
-          }
-          const float p0 = exp2f(s0), p1 = exp2f(s1);
+          const float p0 = exp2f(fmaf(__uint_as_float(v[i]), a.scale_log2, -mref));
+          const float p1 = exp2f(fmaf(__uint_as_float(v[i + 1]), a.scale_log2, -mref));
           rs += p0 + p1;
           pk[i >> 1] = pack_bf16x2(p0, p1);
         }
@@ -744,7 +744,7 @@ cudaError_t make_map(CUtensorMap* m, const __nv_bfloat16* p, int64_t ld, int row
   return encode_tma_2d(m, p, 2, cols, rows, ld * 2, 64, 128);
 }
 
-template <int D, int DV>
+template <int D, int DV, bool kWindow = false>
 cudaError_t fwd_launch(const AttnTensors& t, const AttnShape& s, const AttnKvLayout& kv, __nv_bfloat16* out,
                        int64_t ldo, float* lse, int* status, cudaStream_t stream) {
   using C = FwdCfg<D, DV>;
@@ -754,7 +754,7 @@ cudaError_t fwd_launch(const AttnTensors& t, const AttnShape& s, const AttnKvLay
   if ((e = make_map(&tq, t.q, t.ldq, rows, s.H * D)) != cudaSuccess) return e;
   if ((e = encode_tma_2d(&tk, t.k, 2, kv.k_cols, kv.rows, t.ldk * 2, 64, 128)) != cudaSuccess) return e;
   if ((e = encode_tma_2d(&tv, t.v, 2, kv.v_cols, kv.rows, t.ldv * 2, 64, 128)) != cudaSuccess) return e;
-  auto kernel = attn_fwd_kernel<D, DV>;
+  auto kernel = attn_fwd_kernel<D, DV, kWindow>;
   static bool configured = false;
   if (!configured) {
     if ((e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmem)) != cudaSuccess)
@@ -762,8 +762,7 @@ cudaError_t fwd_launch(const AttnTensors& t, const AttnShape& s, const AttnKvLay
     configured = true;
   }
   FwdArgs a{s.B, s.T, kv.Tk, s.H, s.Hkv, kv.q_pos0, kv.rows_b, kv.rows_h, kv.k_col_h, kv.v_col_h,
-            s.scale * kLog2e, s.causal, out, ldo, lse, status, s.sink, s.window > 0 ? s.window : INT_MAX,
-            s.window > 0 ? std::min(s.keep_first, 1 << 30) : 0};
+            s.scale * kLog2e, s.causal, out, ldo, lse, status, s.sink, s.window, std::min(s.keep_first, 1 << 30)};
   dim3 grid(s.H, s.B, (s.T + 127) / 128);
   kernel<<<grid, kThreads, C::kSmem, stream>>>(tq, tk, tv, a);
   return cudaGetLastError();
@@ -816,13 +815,19 @@ cudaError_t launch_attn_fwd_kv(const AttnTensors& t, const AttnShape& s, const A
                                int64_t ldo, float* lse, int* status, cudaStream_t stream) {
   if (s.H % s.Hkv != 0 || (s.window > 0 && (!s.causal || s.keep_first < 0))) return cudaErrorInvalidValue;
   const int dv = s.Dv > 0 ? s.Dv : s.D;
+  if (s.window > 0) {
+    if (s.D == 64 && dv == 64) return fwd_launch<64, 64, true>(t, s, kv, out, ldo, lse, status, stream);
+    if (s.D == 128 && dv == 128) return fwd_launch<128, 128, true>(t, s, kv, out, ldo, lse, status, stream);
+    if (s.D == 256 && dv == 256) return fwd_launch<256, 256, true>(t, s, kv, out, ldo, lse, status, stream);
+    return cudaErrorInvalidValue;
+  }
   if (s.D == 64 && dv == 64) {
     // two-tile kernel unless the single-tile one is asked for (B200_ATTN_FWD=1tile: comparisons, fallback)
     static const bool one_tile = [] {
       const char* e = getenv("B200_ATTN_FWD");
       return e != nullptr && e[0] == '1';
     }();
-    if (!one_tile && s.sink == nullptr && s.window <= 0) return launch_attn_fwd2_d64(t, s, kv, out, ldo, lse, status, stream);
+    if (!one_tile && s.sink == nullptr) return launch_attn_fwd2_d64(t, s, kv, out, ldo, lse, status, stream);
     return fwd_launch<64, 64>(t, s, kv, out, ldo, lse, status, stream);
   }
   if (s.D == 128 && dv == 128) return fwd_launch<128, 128>(t, s, kv, out, ldo, lse, status, stream);
