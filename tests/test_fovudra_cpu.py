@@ -203,3 +203,35 @@ def test_presets_run():
     s = FovudraConfig.serving()
     assert len(s.layers) == 8 and len(s.attention_layers) == 2
     assert len({type(s.layers[i].mixer) for i in s.recurrent_layers}) == 2
+
+
+def test_engine_refuses_bad_steps_and_stays_usable():
+    cfg = K.CONFIGS["recurrent_only"]
+    w = K.weights(cfg, 24)
+    eng = K.engine(cfg, w, max_tokens=32, max_seqs=1)
+    with pytest.raises(ValueError):
+        eng.step(["a"], [[cfg["vocab"]]])
+    toks = K.tokens(cfg, 6, 7)
+    eng.step(["a"], [toks[:3]])
+    with pytest.raises(MemoryError):
+        eng.step(["b"], [[1]])
+    assert K.error(eng.step(["a"], [toks[3:]]), O.forward(toks, cfg, w)[-1:]) < TOL
+
+
+def test_sample_script_continues_token_ids(tmp_path):
+    import subprocess
+    from safetensors.torch import save_file
+    cfg = K.CONFIGS["aligned"]
+    w = K.weights(cfg, 50)
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    save_file({k: v.contiguous() for k, v in w.items()}, str(tmp_path / "model.safetensors"))
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    prompt = K.tokens(cfg, 7, 1)
+    r = subprocess.run([sys.executable, "scripts/sample.py", "--model-dir", str(tmp_path), "--dtype", "float32", "--temperature", "0", "--new_tokens",
+                        "5", "--prompt-ids", ",".join(map(str, prompt))], cwd=root, capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr
+    got = [list(map(int, l.split(","))) for l in r.stdout.splitlines() if l and not l.startswith("---")][0]
+    assert len(got) == 5
+    for n, t in enumerate(got):
+        lg = O.forward(prompt + got[:n], cfg, w)[-1]
+        assert float(lg.max() - lg[t]) < 1e-3
