@@ -2,7 +2,7 @@
 //   position i sees j when j <= i and (i - j < size or j < keep_first).
 //
 // qk_prepare turns a projection row [q heads | k heads] into attention operands (bias, half-split rotation, unit RMS norm
-// per head) and writes the cache row [K of every kv head | V of every kv head]; the values are the keys as projected.
+// per head) and writes the cache row [K of every kv head | V of every kv head]; the projected keys double as values.
 // window_attention is the attention for any sizes, fp32 or bf16, prompts that continue a cache and decode steps with split
 // keys; it walks only the key tiles that some query of the block can see. The tensor-core forms are in attention_sm100.cu
 // (whole prompts) and attention_decode.cu (one token).

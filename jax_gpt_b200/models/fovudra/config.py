@@ -23,7 +23,7 @@ class Rotary:
 
 @dataclass(frozen=True)
 class WindowAttention:
-    """Grouped-query attention over a sliding window and the first tokens; the values are the keys as projected."""
+    """Grouped-query attention over a sliding window and the first tokens; projected keys double as values."""
     heads: int
     kv_heads: int
     dim: int
@@ -150,7 +150,7 @@ def _layer(d: dict) -> Layer:
         if mixer.rot.dims > mixer.dim or mixer.rot.dims % 2:
             raise ValueError(f"rot.dims {mixer.rot.dims} does not fit dim {mixer.dim}")
         if mixer.heads % mixer.kv_heads or int(m.get("vdim", mixer.dim)) != mixer.dim:
-            raise ValueError("attention: heads must divide into kv_heads, and the values are the keys (vdim = dim)")
+            raise ValueError("attention: heads must divide into kv_heads, and keys double as values (vdim = dim)")
         if mixer.window < 1 or mixer.keep_first < 0:
             raise ValueError("attention: mask.size must be positive and mask.keep_first not negative")
     elif kind == "mlstm":

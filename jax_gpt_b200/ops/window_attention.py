@@ -2,7 +2,7 @@
 position i sees j when ``j <= i and (i - j < window or j < keep_first)``.
 
 ``qk_prepare`` makes attention operands of a projection row ``[q heads | k heads]`` (bias, half-split rotation, unit RMS norm
-per head) and writes the cache rows; the values are the keys as projected. ``window_attention`` then picks the form: whole
+per head) and writes the cache rows; the projected keys double as values. ``window_attention`` then picks the form: whole
 prompts of head width 64 / 128 / 256 on the tcgen05 flash kernel, decode steps of these widths on the paged decode kernel,
 every other case (other widths, fp32, prompts that continue a cache) on the any-size kernel of csrc/window_attention.cu.
 """
