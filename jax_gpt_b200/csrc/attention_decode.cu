@@ -39,15 +39,18 @@ struct DecArgs {
   const int* lens;
   int page_size, max_pages;
   int window, keep_first;   // window > 0: of the valid keys only the last `window` and the first `keep_first` are seen
+  int64_t v_stride_h;       // between the kv heads of V
 };
 
-template <int D, int G>
+// D: query and key width, DV: value width (D or 2 D).
+template <int D, int DV, int G>
 __global__ void __launch_bounds__(kDecWarps * 32)
 attn_decode_split_kernel(const DecArgs a) {
   constexpr int LPK = D / 8;          // lanes that share one key row
   constexpr int KPW = 32 / LPK;       // keys per warp step
   constexpr int KPS = KPW * kDecWarps;
-  __shared__ float sm_o[kDecWarps][G][D];
+  constexpr int EV = DV / LPK, NV = EV / 8;   // value features of a lane, in 16-byte pieces LPK * 8 features apart
+  __shared__ float sm_o[kDecWarps][G][DV];
   __shared__ float sm_m[kDecWarps][G], sm_l[kDecWarps][G];
   const int split = blockIdx.x, hkv = blockIdx.y, b = blockIdx.z;
   const int n_splits = gridDim.x;
@@ -81,16 +84,16 @@ attn_decode_split_kernel(const DecArgs a) {
       qf[g][2 * e + 1] = f.y * a.scale_log2;
     }
   }
-  float m[G], l[G], o[G][8];
+  float m[G], l[G], o[G][EV];
 #pragma unroll
   for (int g = 0; g < G; ++g) {
     m[g] = -INFINITY;
     l[g] = 0.f;
 #pragma unroll
-    for (int e = 0; e < 8; ++e) o[g][e] = 0.f;
+    for (int e = 0; e < EV; ++e) o[g][e] = 0.f;
   }
   const __nv_bfloat16* kb = a.k + b * a.kv_stride_b + hkv * a.kv_stride_h + sub * 8;
-  const __nv_bfloat16* vb = a.v + b * a.kv_stride_b + hkv * a.kv_stride_h + sub * 8;
+  const __nv_bfloat16* vb = a.v + b * a.kv_stride_b + hkv * a.v_stride_h + sub * 8;
   // Two keys per lane group in flight. The trip count is uniform over the warp (the shuffles below need every
   // lane); a lane group whose key is past the range loads nothing and skips the update.
   for (int base = k0 + warp * KPW; base < k1; base += 2 * KPS) {
@@ -99,23 +102,35 @@ attn_decode_split_kernel(const DecArgs a) {
     const uint4 zero = make_uint4(0, 0, 0, 0);
     const int64_t ra = has_a ? key_row(ka) * a.kv_stride_t : 0, rc = has_c ? key_row(kc) * a.kv_stride_t : 0;
     const uint4 kua = has_a ? *reinterpret_cast<const uint4*>(kb + ra) : zero;
-    const uint4 vua = has_a ? *reinterpret_cast<const uint4*>(vb + ra) : zero;
     const uint4 kuc = has_c ? *reinterpret_cast<const uint4*>(kb + rc) : zero;
-    const uint4 vuc = has_c ? *reinterpret_cast<const uint4*>(vb + rc) : zero;
+    uint4 vua[NV], vuc[NV];
+#pragma unroll
+    for (int p = 0; p < NV; ++p) {
+      vua[p] = has_a ? *reinterpret_cast<const uint4*>(vb + ra + p * D) : zero;
+      vuc[p] = has_c ? *reinterpret_cast<const uint4*>(vb + rc + p * D) : zero;
+    }
 #pragma unroll
     for (int which = 0; which < 2; ++which) {
       const uint4 ku = which == 0 ? kua : kuc;
-      const uint4 vu = which == 0 ? vua : vuc;
       const bool valid = which == 0 ? has_a : has_c;
-      const uint32_t kw[4] = {ku.x, ku.y, ku.z, ku.w}, vw[4] = {vu.x, vu.y, vu.z, vu.w};
-      float kf[8], vf[8];
+      const uint32_t kw[4] = {ku.x, ku.y, ku.z, ku.w};
+      float kf[8], vf[EV];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const float2 f = unpack_bf16x2(kw[e]), h = unpack_bf16x2(vw[e]);
+        const float2 f = unpack_bf16x2(kw[e]);
         kf[2 * e] = f.x;
         kf[2 * e + 1] = f.y;
-        vf[2 * e] = h.x;
-        vf[2 * e + 1] = h.y;
+      }
+#pragma unroll
+      for (int p = 0; p < NV; ++p) {
+        const uint4 vu = which == 0 ? vua[p] : vuc[p];
+        const uint32_t vw[4] = {vu.x, vu.y, vu.z, vu.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float2 f = unpack_bf16x2(vw[e]);
+          vf[8 * p + 2 * e] = f.x;
+          vf[8 * p + 2 * e + 1] = f.y;
+        }
       }
 #pragma unroll
       for (int g = 0; g < G; ++g) {
@@ -129,7 +144,7 @@ attn_decode_split_kernel(const DecArgs a) {
           const float alpha = exp2f(m[g] - mn), p = exp2f(s - mn);
           l[g] = fmaf(l[g], alpha, p);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) o[g][e] = fmaf(o[g][e], alpha, p * vf[e]);
+          for (int e = 0; e < EV; ++e) o[g][e] = fmaf(o[g][e], alpha, p * vf[e]);
           m[g] = mn;
         }
       }
@@ -147,7 +162,7 @@ attn_decode_split_kernel(const DecArgs a) {
       const float wb = (mo == -INFINITY) ? 0.f : exp2f(mo - mn);
       l[g] = l[g] * wa + lo * wb;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
+      for (int e = 0; e < EV; ++e) {
         const float oo = __shfl_xor_sync(0xffffffffu, o[g][e], off);
         o[g][e] = o[g][e] * wa + oo * wb;
       }
@@ -158,7 +173,7 @@ attn_decode_split_kernel(const DecArgs a) {
 #pragma unroll
     for (int g = 0; g < G; ++g) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) sm_o[warp][g][sub * 8 + e] = o[g][e];
+      for (int e = 0; e < EV; ++e) sm_o[warp][g][(e / 8) * D + sub * 8 + e % 8] = o[g][e];
       if (sub == 0) {
         sm_m[warp][g] = m[g];
         sm_l[warp][g] = l[g];
@@ -166,8 +181,8 @@ attn_decode_split_kernel(const DecArgs a) {
     }
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < G * D; i += kDecWarps * 32) {
-    const int g = i / D, c = i % D;
+  for (int i = threadIdx.x; i < G * DV; i += kDecWarps * 32) {
+    const int g = i / DV, c = i % DV;
     float mn = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kDecWarps; ++w) mn = fmaxf(mn, sm_m[w][g]);
@@ -179,7 +194,7 @@ attn_decode_split_kernel(const DecArgs a) {
       ls = fmaf(sm_l[w][g], wt, ls);
     }
     const int64_t row = (static_cast<int64_t>(b) * a.H + hkv * G + g) * n_splits + split;
-    a.part_o[row * D + c] = acc;
+    a.part_o[row * DV + c] = acc;
     if (c == 0) {
       a.part_ml[row * 2] = mn;
       a.part_ml[row * 2 + 1] = ls;
@@ -228,26 +243,26 @@ attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restri
   }
 }
 
-template <int D, int G>
+template <int D, int DV, int G>
 cudaError_t decode_launch(const DecArgs& a, int B, int n_splits, __nv_bfloat16* out, int64_t ldo,
                           cudaStream_t stream) {
   if (n_splits > kMaxSplits) return cudaErrorInvalidValue;
   dim3 grid(n_splits, a.Hkv, B);
-  attn_decode_split_kernel<D, G><<<grid, kDecWarps * 32, 0, stream>>>(a);
+  attn_decode_split_kernel<D, DV, G><<<grid, kDecWarps * 32, 0, stream>>>(a);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return e;
-  attn_decode_merge_kernel<D><<<dim3(a.H, B), 512, 0, stream>>>(a.part_o, a.part_ml, n_splits, out, ldo, a.H);
+  attn_decode_merge_kernel<DV><<<dim3(a.H, B), 512, 0, stream>>>(a.part_o, a.part_ml, n_splits, out, ldo, a.H);
   return cudaGetLastError();
 }
 
-template <int D>
+template <int D, int DV = D>
 cudaError_t decode_dispatch_g(const DecArgs& a, int B, int n_splits, __nv_bfloat16* out, int64_t ldo,
                               cudaStream_t stream) {
   switch (a.H / a.Hkv) {
-    case 1: return decode_launch<D, 1>(a, B, n_splits, out, ldo, stream);
-    case 2: return decode_launch<D, 2>(a, B, n_splits, out, ldo, stream);
-    case 4: return decode_launch<D, 4>(a, B, n_splits, out, ldo, stream);
-    case 8: return decode_launch<D, 8>(a, B, n_splits, out, ldo, stream);
+    case 1: return decode_launch<D, DV, 1>(a, B, n_splits, out, ldo, stream);
+    case 2: return decode_launch<D, DV, 2>(a, B, n_splits, out, ldo, stream);
+    case 4: return decode_launch<D, DV, 4>(a, B, n_splits, out, ldo, stream);
+    case 8: return decode_launch<D, DV, 8>(a, B, n_splits, out, ldo, stream);
     default: return cudaErrorInvalidValue;
   }
 }
@@ -262,7 +277,7 @@ cudaError_t launch_attn_decode(const __nv_bfloat16* q, int64_t ldq, const __nv_b
       ldq % 8 != 0)
     return cudaErrorInvalidValue;
   DecArgs a{q, ldq, k, v, kv_stride_b, kv_stride_h, kv_stride_t, pos_ptr, len, len_add, H, Hkv,
-            scale * 1.4426950408889634f, part_o, part_ml, nullptr, nullptr, nullptr, 0, 0, 0, 0};
+            scale * 1.4426950408889634f, part_o, part_ml, nullptr, nullptr, nullptr, 0, 0, 0, 0, kv_stride_h};
   switch (D) {
     case 64: return decode_dispatch_g<64>(a, B, n_splits, out, ldo, stream);
     case 128: return decode_dispatch_g<128>(a, B, n_splits, out, ldo, stream);
@@ -275,13 +290,18 @@ cudaError_t launch_attn_decode_paged(const __nv_bfloat16* q, int64_t ldq, const 
                                      const int* block_table, const int* seq_ids, const int* seq_lens, int len_add,
                                      int page_size, int max_pages, int B, int H, int Hkv, int D, float scale, int n_splits,
                                      float* part_o, float* part_ml, __nv_bfloat16* out, int64_t ldo, cudaStream_t stream,
-                                     int window, int keep_first) {
-  if (H % Hkv != 0 || n_splits < 1 || width != 2 * Hkv * D || width % 8 != 0 || ldq % 8 != 0 || page_size < 1 || keep_first < 0)
+                                     int window, int keep_first, int DV) {
+  if (DV == 0) DV = D;
+  if (H % Hkv != 0 || n_splits < 1 || width != Hkv * (D + DV) || width % 8 != 0 || ldq % 8 != 0 || page_size < 1 || keep_first < 0)
     return cudaErrorInvalidValue;
   // a pool row holds K of every kv head, then V of every kv head
   DecArgs a{q, ldq, pool, pool + Hkv * D, 0, D, width, nullptr, 0, len_add, H, Hkv,
             scale * 1.4426950408889634f, part_o, part_ml, block_table, seq_ids, seq_lens, page_size, max_pages,
             window, keep_first};
+  a.v_stride_h = DV;
+  if (DV == 2 * D && D == 64) return decode_dispatch_g<64, 128>(a, B, n_splits, out, ldo, stream);
+  if (DV == 2 * D && D == 128) return decode_dispatch_g<128, 256>(a, B, n_splits, out, ldo, stream);
+  if (DV != D) return cudaErrorInvalidValue;
   switch (D) {
     case 64: return decode_dispatch_g<64>(a, B, n_splits, out, ldo, stream);
     case 128: return decode_dispatch_g<128>(a, B, n_splits, out, ldo, stream);

@@ -2,14 +2,16 @@
 //
 //   S_t = a_t S_(t-1) + b_t k_t v_t^T        o_t = q_scale S_t^T q_t
 //
-// with a fixed decay per head (a_t = decay, b_t = 1), or with exponential gates from log values i, f and a running maximum
+// with a fixed decay per head (a_t = decay, b_t = 1), with a decay per key channel (a_t = diag(alpha_t), b_t = 1, log alpha =
+// log sigmoid(w2 low + bias2) / tau; Yang et al., "Gated Linear Attention Transformers with Hardware-Efficient Training"), or
+// with exponential gates from log values i, f and a running maximum
 // m (Beck et al., "xLSTM: Extended Long Short-Term Memory"):
 //   m_t = max(f_t + m_(t-1), i_t), a_t = exp(f_t + m_(t-1) - m_t), b_t = exp(i_t - m_t), n_t = a_t n_(t-1) + b_t k_t,
 //   o_t / (max(|q_scale n_t . q_t|, exp(-m_t)) + den_eps)
 // i = cap tanh(raw / cap), f = log sigmoid(cap tanh(raw / cap)).
 //
 // The gated scans leave the numerators in y and {n . q in two parts, exp(-m)} in `den`; head_norm_gate divides, applies the
-// RMS norm over equal pieces of the row, the gain and the sigmoid output gate. The chunked tensor-core form is in
+// RMS norm over equal pieces of the row, the gain and the output gate. The chunked tensor-core form is in
 // ssd_scan_sm100.cu. All gates, states and norms are fp32. This file is built without fast-math.
 #include "serve_common.cuh"
 #include "serve_kernels.cuh"
@@ -27,6 +29,17 @@ __device__ __forceinline__ void log_gates(const LinGates& g, int64_t row, int h,
   f = -softplus_f(-soft_cap(p[H + h] + g.bias[H + h], g.cap));
 }
 
+// decay of (row, head, key channel)
+template <typename T>
+__device__ __forceinline__ float channel_decay(const LinGates& g, int64_t row, int hn) {
+  const T *x = static_cast<const T*>(g.low) + row * g.ld_low, *w = static_cast<const T*>(g.w2) + static_cast<int64_t>(hn) * g.R;
+  float z = g.bias2[hn];
+  for (int r = 0; r < g.R; ++r) z = fmaf(ldf(x + r), ldf(w + r), z);
+  return expf(-softplus_f(-z) * g.inv_tau);
+}
+
+enum LinKind : int { kFixed = 0, kGatedExp = 1, kChannel = 2 };
+
 template <typename T>
 __device__ __forceinline__ float qkv_at(const T* p, int silu) {
   const float v = ldf(p);
@@ -38,10 +51,11 @@ __device__ __forceinline__ float qkv_at(const T* p, int silu) {
 // of the first columns also carry n and m (kGated).
 constexpr int kScanP = 16, kScanG = 8, kScanTok = 16;
 
-template <typename T, int NS, bool kGated>
+template <typename T, int NS, int kKind>
 __global__ void __launch_bounds__(kScanP * kScanG)
 linear_scan_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, const LinGates gates, float* __restrict__ state,
                    float* __restrict__ y, const LinShape s) {
+  constexpr bool kGated = kKind == kGatedExp;
   extern __shared__ float sm[];
   const int N = s.N, P = s.P;
   float* sK = sm;                       // [kScanTok][N]
@@ -50,6 +64,7 @@ linear_scan_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
   float* sA = sV + kScanTok * kScanP;   // [kScanTok] state factor
   float* sB = sA + kScanTok;            // [kScanTok] input factor
   float* sE = sB + kScanTok;            // [kScanTok] exp(-m)
+  float* sC = sE + kScanTok;            // [kScanTok][N] decays of the key channels (kChannel)
   const int h = blockIdx.x, p0 = blockIdx.y * kScanP, b = blockIdx.z;
   const int g = threadIdx.x % kScanG, p = threadIdx.x / kScanG;   // the eight row groups of a column are neighbours
   const int first = sb.cu[b], len = sb.cu[b + 1] - first;
@@ -65,7 +80,7 @@ linear_scan_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
     if constexpr (kGated) nn[i] = (!fresh && n < N) ? vec[n] : 0.f;
   }
   float m = kGated && !fresh ? vec[N] : 0.f;   // thread 0's copy advances
-  const float decay = kGated ? 0.f : gates.decay[h];
+  const float decay = kKind == kFixed ? gates.decay[h] : 0.f;
   for (int t0 = 0; t0 < len; t0 += kScanTok) {
     const int cnt = min(kScanTok, len - t0);
     __syncthreads();
@@ -73,6 +88,7 @@ linear_scan_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
       const T* row = qkv + static_cast<int64_t>(first + t0 + i / N) * ld + h * N + i % N;
       sQ[i] = qkv_at(row, s.silu);
       sK[i] = qkv_at(row + s.H * N, s.silu);
+      if constexpr (kKind == kChannel) sC[i] = channel_decay<T>(gates, first + t0 + i / N, h * N + i % N);
     }
     for (int i = threadIdx.x; i < cnt * kScanP; i += blockDim.x)
       sV[i] = p0 + i % kScanP < P ? qkv_at(qkv + static_cast<int64_t>(first + t0 + i / kScanP) * ld + 2 * s.H * N + h * P + p0 + i % kScanP, s.silu) : 0.f;
@@ -102,7 +118,7 @@ linear_scan_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
       for (int i = 0; i < NS; ++i) {
         const int n = g + i * kScanG;
         if (n < N) {
-          S[i] = fmaf(S[i], a, x * sK[t * N + n]);
+          S[i] = fmaf(S[i], kKind == kChannel ? sC[t * N + n] : a, x * sK[t * N + n]);
           acc = fmaf(S[i], sQ[t * N + n], acc);
           if constexpr (kGated) {
             nn[i] = fmaf(nn[i], a, w * sK[t * N + n]);
@@ -139,17 +155,17 @@ linear_scan_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
   }
 }
 
-template <typename T, bool kGated>
+template <typename T, int kKind>
 cudaError_t linear_scan_t(const SeqBatch& sb, const T* qkv, int64_t ld, const LinGates& g, float* state, float* y,
                           const LinShape& s, cudaStream_t st) {
   const dim3 grid(s.H, (s.P + kScanP - 1) / kScanP, sb.n_seq);
-  const int smem = 4 * (2 * kScanTok * s.N + kScanTok * kScanP + 3 * kScanTok);
+  const int smem = 4 * ((kKind == kChannel ? 3 : 2) * kScanTok * s.N + kScanTok * kScanP + 3 * kScanTok);
 #define B200_SCAN(NS)                                                                                                 \
   {                                                                                                                   \
     static int have = 0;                                                                                              \
-    const cudaError_t e = want_smem(linear_scan_kernel<T, NS, kGated>, smem, have);                                   \
+    const cudaError_t e = want_smem(linear_scan_kernel<T, NS, kKind>, smem, have);                                   \
     if (e != cudaSuccess) return e;                                                                                   \
-    linear_scan_kernel<T, NS, kGated><<<grid, kScanP * kScanG, smem, st>>>(sb, qkv, ld, g, state, y, s);              \
+    linear_scan_kernel<T, NS, kKind><<<grid, kScanP * kScanG, smem, st>>>(sb, qkv, ld, g, state, y, s);              \
   }
   if (s.N <= 64) B200_SCAN(8)
   else if (s.N <= 128) B200_SCAN(16)
@@ -165,10 +181,11 @@ cudaError_t linear_scan_t(const SeqBatch& sb, const T* qkv, int64_t ld, const Li
 // state row. The block of the first columns advances n and m.
 constexpr int kStepThreads = 256, kStepCols = 64;
 
-template <typename T, int V, bool kGated>
+template <typename T, int V, int kKind>
 __global__ void __launch_bounds__(kStepThreads)
 linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, const LinGates gates, float* __restrict__ state,
                    float* __restrict__ y, const LinShape s) {
+  constexpr bool kGated = kKind == kGatedExp;
   extern __shared__ float sm[];
   __shared__ float red[33];
   const int N = s.N, P = s.P;
@@ -176,7 +193,8 @@ linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
   float* sq = sm;                 // [N]
   float* sk = sq + N;             // [N]
   float* sv = sk + N;             // [kStepCols]
-  float* part = sv + kStepCols;   // [rows][cols]
+  float* sc = sv + kStepCols;     // [N] decays of the key channels (kChannel)
+  float* part = kKind == kChannel ? sc + N : sc;   // [rows][cols]
   const int slot = sb.ids[b];
   const bool fresh = sb.start[b] == 0;
   const int64_t row = sb.cu[b];
@@ -208,9 +226,10 @@ linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
   for (int i = threadIdx.x; i < N; i += blockDim.x) {
     sq[i] = qkv_at(x + h * N + i, s.silu);
     sk[i] = qkv_at(x + (s.H + h) * N + i, s.silu);
+    if constexpr (kKind == kChannel) sc[i] = channel_decay<T>(gates, row, h * N + i);
   }
   for (int i = threadIdx.x; i < cols; i += blockDim.x) sv[i] = qkv_at(x + 2 * s.H * N + h * P + p0 + i, s.silu);
-  float a, w = 1.f, m = 0.f;
+  float a = 0.f, w = 1.f, m = 0.f;
   const float* vec = nullptr;
   if constexpr (kGated) {
     vec = gates.vec + (static_cast<int64_t>(slot) * s.H + h) * (N + 1);
@@ -220,7 +239,7 @@ linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
     m = fmaxf(lf + m0, li);
     a = expf(lf + m0 - m);
     w = expf(li - m);
-  } else {
+  } else if constexpr (kKind == kFixed) {
     a = gates.decay[h];
   }
   __syncthreads();
@@ -235,10 +254,10 @@ linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
         const int n = n0 + i * kRows;
         if (n >= N) break;
         float* sp = st + static_cast<int64_t>(n) * P;
-        const float kn = sk[n], qn = sq[n];
+        const float kn = sk[n], qn = sq[n], an = kKind == kChannel ? sc[n] : a;
 #pragma unroll
         for (int j = 0; j < V; ++j) {
-          S[i][j] = fmaf(S[i][j], a, dx[j] * kn);
+          S[i][j] = fmaf(S[i][j], an, dx[j] * kn);
           acc[j] = fmaf(S[i][j], qn, acc[j]);
         }
         if constexpr (V == 4) *reinterpret_cast<float4*>(sp) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);
@@ -273,22 +292,22 @@ linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
   }
 }
 
-template <typename T, bool kGated>
+template <typename T, int kKind>
 cudaError_t linear_step_t(const SeqBatch& sb, const T* qkv, int64_t ld, const LinGates& g, float* state, float* y,
                           const LinShape& s, cudaStream_t st) {
   const dim3 grid(s.H, (s.P + kStepCols - 1) / kStepCols, sb.n_seq);
   if (s.P % 4 == 0) {
     static int have = 0;
-    const int smem = 4 * (2 * s.N + kStepCols + kStepThreads * 4);
-    const cudaError_t e = want_smem(linear_step_kernel<T, 4, kGated>, smem, have);
+    const int smem = 4 * ((kKind == kChannel ? 3 : 2) * s.N + kStepCols + kStepThreads * 4);
+    const cudaError_t e = want_smem(linear_step_kernel<T, 4, kKind>, smem, have);
     if (e != cudaSuccess) return e;
-    linear_step_kernel<T, 4, kGated><<<grid, kStepThreads, smem, st>>>(sb, qkv, ld, g, state, y, s);
+    linear_step_kernel<T, 4, kKind><<<grid, kStepThreads, smem, st>>>(sb, qkv, ld, g, state, y, s);
   } else {
     static int have = 0;
-    const int smem = 4 * (2 * s.N + kStepCols + kStepThreads);
-    const cudaError_t e = want_smem(linear_step_kernel<T, 1, kGated>, smem, have);
+    const int smem = 4 * ((kKind == kChannel ? 3 : 2) * s.N + kStepCols + kStepThreads);
+    const cudaError_t e = want_smem(linear_step_kernel<T, 1, kKind>, smem, have);
     if (e != cudaSuccess) return e;
-    linear_step_kernel<T, 1, kGated><<<grid, kStepThreads, smem, st>>>(sb, qkv, ld, g, state, y, s);
+    linear_step_kernel<T, 1, kKind><<<grid, kStepThreads, smem, st>>>(sb, qkv, ld, g, state, y, s);
   }
   return cudaGetLastError();
 }
@@ -326,9 +345,10 @@ __global__ void head_norm_gate_kernel(const SeqBatch sb, const TY* __restrict__ 
     ss += v * v;
   }
   const float inv = 1.f / sqrtf(block_sum(ss, red) / part + a.eps);
-  for (int i = threadIdx.x; i < part; i += blockDim.x)
-    stf(out + static_cast<int64_t>(n) * D + c0 + i,
-        buf[i] * inv * gamma[c0 + i] * sigmoid_f(ldf(z + static_cast<int64_t>(n) * ldz + c0 + i)));
+  for (int i = threadIdx.x; i < part; i += blockDim.x) {
+    const float zv = ldf(z + static_cast<int64_t>(n) * ldz + c0 + i);
+    stf(out + static_cast<int64_t>(n) * D + c0 + i, buf[i] * inv * gamma[c0 + i] * sigmoid_f(zv) * (a.gate == 1 ? zv : 1.f));
+  }
   commit_vec(a, sb, n, h, threadIdx.x, blockDim.x);
 }
 
@@ -382,7 +402,7 @@ head_norm_gate_vec_kernel(const SeqBatch sb, const TY* __restrict__ y, const __n
       float g[8];
       ld8(gamma + c0 + i, g);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) g[j] *= v[k][j] * inv * __fdividef(1.f, 1.f + __expf(-zv[k][j]));
+      for (int j = 0; j < 8; ++j) g[j] *= v[k][j] * inv * __fdividef(a.gate == 1 ? zv[k][j] : 1.f, 1.f + __expf(-zv[k][j]));
       *reinterpret_cast<uint4*>(out + static_cast<int64_t>(n) * D + c0 + i) =
           make_uint4(pack_bf16x2(g[0], g[1]), pack_bf16x2(g[2], g[3]), pack_bf16x2(g[4], g[5]), pack_bf16x2(g[6], g[7]));
     }
@@ -423,29 +443,28 @@ cudaError_t head_norm_gate_t(const SeqBatch& sb, const TY* y, const T* z, int64_
 
 }  // namespace
 
+#define B200_LIN(FN)                                                                                                    \
+  {                                                                                                                     \
+    if (f32) {                                                                                                          \
+      const float* x = static_cast<const float*>(qkv);                                                                  \
+      if (g.low != nullptr) return FN<float, kChannel>(sb, x, ld, g, state, y, s, st);                                  \
+      return g.raw != nullptr ? FN<float, kGatedExp>(sb, x, ld, g, state, y, s, st) : FN<float, kFixed>(sb, x, ld, g, state, y, s, st); \
+    }                                                                                                                   \
+    const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(qkv);                                                    \
+    if (g.low != nullptr) return FN<__nv_bfloat16, kChannel>(sb, x, ld, g, state, y, s, st);                            \
+    return g.raw != nullptr ? FN<__nv_bfloat16, kGatedExp>(sb, x, ld, g, state, y, s, st)                               \
+                            : FN<__nv_bfloat16, kFixed>(sb, x, ld, g, state, y, s, st);                                 \
+  }
 cudaError_t launch_linear_scan(bool f32, const SeqBatch& sb, const void* qkv, int64_t ld, const LinGates& g, float* state, float* y,
                                const LinShape& s, cudaStream_t st) {
-  const bool gated = g.raw != nullptr;
-  if (f32) {
-    const float* x = static_cast<const float*>(qkv);
-    return gated ? linear_scan_t<float, true>(sb, x, ld, g, state, y, s, st) : linear_scan_t<float, false>(sb, x, ld, g, state, y, s, st);
-  }
-  const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(qkv);
-  return gated ? linear_scan_t<__nv_bfloat16, true>(sb, x, ld, g, state, y, s, st)
-               : linear_scan_t<__nv_bfloat16, false>(sb, x, ld, g, state, y, s, st);
+  B200_LIN(linear_scan_t)
 }
 
 cudaError_t launch_linear_step(bool f32, const SeqBatch& sb, const void* qkv, int64_t ld, const LinGates& g, float* state, float* y,
                                const LinShape& s, cudaStream_t st) {
-  const bool gated = g.raw != nullptr;
-  if (f32) {
-    const float* x = static_cast<const float*>(qkv);
-    return gated ? linear_step_t<float, true>(sb, x, ld, g, state, y, s, st) : linear_step_t<float, false>(sb, x, ld, g, state, y, s, st);
-  }
-  const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(qkv);
-  return gated ? linear_step_t<__nv_bfloat16, true>(sb, x, ld, g, state, y, s, st)
-               : linear_step_t<__nv_bfloat16, false>(sb, x, ld, g, state, y, s, st);
+  B200_LIN(linear_step_t)
 }
+#undef B200_LIN
 
 cudaError_t launch_head_norm_gate(bool f32, bool y_f32, const SeqBatch& sb, const void* y, const void* z, int64_t ldz,
                                   const float* gamma, void* out, int D, const HeadNorm& a, cudaStream_t st) {

@@ -126,11 +126,67 @@ struct WindowMask {
 cudaError_t launch_qk_prepare(bool f32, const SeqBatch& sb, const void* y, int64_t ldy, const float* bias, int H, int G, int D,
                               bool unit_norm, float eps, const RopeTable& rope, const PagedRows& pages, void* q, void* k, void* v,
                               int* status, cudaStream_t st);
-// Softmax attention of q [n_tok, H, D] over the pages' rows [K | V] of G kv heads, any sizes. n_splits > 1 cuts the visible
-// keys into ranges merged by a second kernel (part_o [n_tok, H, S, D], part_ml [n_tok, H, S, 2] fp32).
-cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, int H, int G, int D,
+// Softmax attention of q [n_tok, H, D] over the pages' rows [K (G D) | V (G DV)] of G kv heads, any sizes. n_splits > 1 cuts the
+// visible keys into ranges merged by a second kernel (part_o [n_tok, H, S, DV], part_ml [n_tok, H, S, 2] fp32).
+cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, int H, int G, int D, int DV,
                                     WindowMask mask, float scale, int n_splits, float* part_o, float* part_ml, void* out,
                                     cudaStream_t st);
+
+// ---- interleaved rotation, rotated values (rotated_kv.cu) ----------------------------------------------------------------
+// Columns of a projection row and their biases ([heads * width] fp32 or null).
+struct QkvRows {
+  const void* y;
+  int64_t ld;
+  int q, k, v;
+  const float *bq, *bk, *bv;
+};
+// q, k turned by `rope`, v by `vrope` (interleaved pairs) into the cache row [K (G dk) | V (G dv)], q [n_tok, H, dkp] and, unless
+// null, k [n_tok, G, dkp], v [n_tok, G, dvp]; features past dk / dv are zero there.
+cudaError_t launch_qkv_rotate(bool f32, const SeqBatch& sb, const QkvRows& in, const RopeTable& rope, const RopeTable& vrope,
+                              const PagedRows& pages, int H, int G, int dk, int dv, int dkp, int dvp, void* q, void* k, void* v, int* status,
+                              cudaStream_t st);
+// out[n, h * dv + c] = scale sigmoid(g[n, h]) (o [n_tok, H, ldh] turned back by the row's position).
+cudaError_t launch_turn_back_gate(bool f32, const SeqBatch& sb, const void* o, int ldh, const void* g, int64_t ldg, const RopeTable& vrope,
+                                  float scale, int H, int dv, void* out, int64_t ldo, cudaStream_t st);
+
+// ---- residual streams and row activations (stream_kernels.cu) ------------------------------------------------------------
+constexpr int kMaxStreams = 16;
+struct StreamNorm {
+  float* xs;             // [rows, S, D] streams, updated in place
+  const float* bias;     // optional [D], added to y
+  const float* mix;      // [S, S] indexed [from, to]; null: the streams start with y
+  const float* w_out;    // [S] weight of y in every stream
+  const float* w_in;     // [S] weights of the streams in u
+  const float* gamma;    // [D]
+  float* u;              // optional [rows, D]: the combination before its norm
+  int rows, S, D, groups;
+  float eps;
+};
+// Streams of the sublayer output y [rows, D] and h = group norm of the next sublayer's input (null: none). y fp32 (y_f32) or bf16.
+cudaError_t launch_stream_norm(bool y_f32, bool f32_out, const void* y, const StreamNorm& a, void* h, cudaStream_t st);
+// out = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3 over rows of N features; coef [4].
+cudaError_t launch_poly_norm(bool f32, const void* z, int64_t ldz, const float* coef, void* out, int rows, int N, float eps, cudaStream_t st);
+
+// ---- gated linear recurrent unit (gated_lru.cu) ----------------------------------------------------------------------------
+struct LruArgs {
+  int W, blocks, taps;
+  const void* x;           // [n_tok, ldx] convolution input before its bias
+  int64_t ldx;
+  const float *x_bias, *conv, *conv_bias;   // [W], [W, taps] (current token last), [W]
+  float* ring;             // [slots, taps, W]: input of position p in row p % taps
+  const void* gates;       // [blocks, 2, W / blocks, W / blocks] = recurrence and input gate, (out, in)
+  const float* gates_bias; // [blocks, 2, W / blocks]
+  const float* decay;      // [W]: log a = -decay * gate
+  float* state;            // [slots, W], ignored where start == 0, always written
+  const void* y;           // [n_tok, ldy] output branch before bias and gelu
+  int64_t ldy;
+  const float* y_bias;     // [W]
+  float scale;
+  void* out;               // [n_tok, ldo]
+  int64_t ldo;
+};
+// log_a, inp: scratch [n_tok, W] fp32; log_a null: one token per sequence.
+cudaError_t launch_gated_lru(bool f32, const SeqBatch& sb, const LruArgs& a, float* log_a, float* inp, cudaStream_t st);
 
 // ---- linear attention with a matrix state (linear_attention.cu, ssd_scan_sm100.cu) ---------------------------------------
 struct LinShape {
@@ -147,6 +203,13 @@ struct LinGates {
   const float* vec;       // [slots, H, N + 1] = [n | m] at the start of the step
   float* vec_new;         // [n_seq, H, N + 1] after it
   float* den;             // [n_tok, H, 4] = {n . q, second part of n . q, exp(-m), -}
+  // or with `low` set a decay per key channel, alpha = sigmoid(w2 low + bias2)^(inv_tau):
+  const void* low;        // [n_tok, ld_low], R wide, activation dtype
+  int64_t ld_low;
+  const void* w2;         // [H N, R], activation dtype
+  const float* bias2;     // [H N]
+  int R;
+  float inv_tau;
 };
 // state [slots, H, N, P] fp32 (ignored where start == 0, always written); y [n_tok, H P] fp32: the numerators.
 cudaError_t launch_linear_scan(bool f32, const SeqBatch& sb, const void* qkv, int64_t ld, const LinGates& g, float* state, float* y,
@@ -165,8 +228,9 @@ struct HeadNorm {
   const float* vec_new;   // optional: copied to vec at the slot of the sequence, by the last row of every sequence
   float* vec;
   int vec_len;
+  int gate;               // 0: sigmoid(z), 1: silu(z)
 };
-// out = RMS norm over `parts` equal pieces of y, times gamma and sigmoid(z). y fp32 (y_f32) or activation dtype.
+// out = RMS norm over `parts` equal pieces of y, times gamma and the gate of z. y fp32 (y_f32) or activation dtype.
 cudaError_t launch_head_norm_gate(bool f32, bool y_f32, const SeqBatch& sb, const void* y, const void* z, int64_t ldz,
                                   const float* gamma, void* out, int D, const HeadNorm& a, cudaStream_t st);
 

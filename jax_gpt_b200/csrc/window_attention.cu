@@ -164,16 +164,30 @@ qk_prepare_vec_kernel(const PrepArgs a, const __nv_bfloat16* __restrict__ y, __n
 constexpr int kWaQ = 8, kWaK = 32, kWaWarps = 4, kWaMine = kWaQ / kWaWarps;
 
 template <typename T>
+__device__ __forceinline__ void stage_row(const T* __restrict__ src, bool live, int n, int lane, float* dst) {
+  if (live && n % Vec16<T>::n == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
+    for (int i = lane * Vec16<T>::n; i < n; i += 32 * Vec16<T>::n) {
+      float f[Vec16<T>::n];
+      Vec16<T>::load(src + i, f);
+#pragma unroll
+      for (int j = 0; j < Vec16<T>::n; ++j) dst[i + j] = f[j];
+    }
+  } else {
+    for (int i = lane; i < n; i += 32) dst[i] = live ? ldf(src + i) : 0.f;
+  }
+}
+
+template <typename T>
 __global__ void __launch_bounds__(kWaWarps * 32)
-window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows pages, int H, int G, int D, WindowMask mask,
-                   float scale, float* __restrict__ part_o, float* __restrict__ part_ml, T* __restrict__ out) {
+window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows pages, int H, int G, int D, int DV,
+                   WindowMask mask, float scale, float* __restrict__ part_o, float* __restrict__ part_ml, T* __restrict__ out) {
   extern __shared__ float sm[];
   const int DS = D | 1;                    // odd stride: lanes read a column of keys without bank conflicts
   float* sk = sm;                          // [kWaK][DS]
-  float* sv = sk + kWaK * DS;              // [kWaK][D]
-  float* sq = sv + kWaK * D;               // [kWaQ][D]
-  float* so = sq + kWaQ * D;               // [kWaQ][D]
-  float* sp = so + kWaQ * D;               // [kWaQ][kWaK]
+  float* sv = sk + kWaK * DS;              // [kWaK][DV]
+  float* sq = sv + kWaK * DV;              // [kWaQ][D]
+  float* so = sq + kWaQ * D;               // [kWaQ][DV]
+  float* sp = so + kWaQ * DV;              // [kWaQ][kWaK]
   const int split = blockIdx.y, S = gridDim.y, g = blockIdx.z, rep = H / G;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int tile = blockIdx.x, b = 0, r0 = -1, cnt = 0;      // tile -> (sequence, first pair)
@@ -195,10 +209,8 @@ window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows 
   const int n_tiles = n_keep + max(0, w1 - w0), per = (n_tiles + S - 1) / S;
   const int i0 = split * per, i1 = min(n_tiles, i0 + per);
   auto head = [&](int q) { return (static_cast<int64_t>(sb.cu[b] + (r0 + q) / rep) * H + g * rep + (r0 + q) % rep); };
-  for (int i = threadIdx.x; i < kWaQ * D; i += blockDim.x) {
-    sq[i] = i / D < cnt ? ldf(qx + head(i / D) * D + i % D) : 0.f;
-    so[i] = 0.f;
-  }
+  for (int i = threadIdx.x; i < kWaQ * D; i += blockDim.x) sq[i] = i / D < cnt ? ldf(qx + head(i / D) * D + i % D) : 0.f;
+  for (int i = threadIdx.x; i < kWaQ * DV; i += blockDim.x) so[i] = 0.f;
   float m[kWaMine], l[kWaMine];
   int pos[kWaMine];                        // position of the pair's token; -1: no pair
 #pragma unroll
@@ -213,25 +225,9 @@ window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows 
     __syncthreads();
     for (int k = warp; k < kWaK; k += kWaWarps) {
       const int64_t row = k0 + k <= p_hi ? page_row(pages, slot, k0 + k) : -1;
-      const T* src = static_cast<const T*>(pages.pool) + (row < 0 ? 0 : row) * pages.width + g * D;
-      const T* srv = src + G * D;
-      if (row >= 0 && D % Vec16<T>::n == 0) {
-        for (int i = lane * Vec16<T>::n; i < D; i += 32 * Vec16<T>::n) {
-          float f[Vec16<T>::n], e[Vec16<T>::n];
-          Vec16<T>::load(src + i, f);
-          Vec16<T>::load(srv + i, e);
-#pragma unroll
-          for (int j = 0; j < Vec16<T>::n; ++j) {
-            sk[k * DS + i + j] = f[j];
-            sv[k * D + i + j] = e[j];
-          }
-        }
-      } else {
-        for (int i = lane; i < D; i += 32) {
-          sk[k * DS + i] = row < 0 ? 0.f : ldf(src + i);
-          sv[k * D + i] = row < 0 ? 0.f : ldf(srv + i);
-        }
-      }
+      const T* base = static_cast<const T*>(pages.pool) + (row < 0 ? 0 : row) * pages.width;
+      stage_row(base + g * D, row >= 0, D, lane, sk + k * DS);
+      stage_row(base + G * D + g * DV, row >= 0, DV, lane, sv + k * DV);
     }
     __syncthreads();
     float s[kWaMine];
@@ -260,18 +256,18 @@ window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows 
       sp[(warp + j * kWaWarps) * kWaK + lane] = p;
     }
     __syncwarp();
-    for (int c = lane; c < D; c += 32) {
+    for (int c = lane; c < DV; c += 32) {
       float o[kWaMine];
 #pragma unroll
-      for (int j = 0; j < kWaMine; ++j) o[j] = so[(warp + j * kWaWarps) * D + c] * a[j];
+      for (int j = 0; j < kWaMine; ++j) o[j] = so[(warp + j * kWaWarps) * DV + c] * a[j];
 #pragma unroll 8
       for (int k = 0; k < kWaK; ++k) {
-        const float v = sv[k * D + c];
+        const float v = sv[k * DV + c];
 #pragma unroll
         for (int j = 0; j < kWaMine; ++j) o[j] = fmaf(sp[(warp + j * kWaWarps) * kWaK + k], v, o[j]);
       }
 #pragma unroll
-      for (int j = 0; j < kWaMine; ++j) so[(warp + j * kWaWarps) * D + c] = o[j];
+      for (int j = 0; j < kWaMine; ++j) so[(warp + j * kWaWarps) * DV + c] = o[j];
     }
   }
   if (i1 <= i0) __syncthreads();           // no tile in this range: the zeroed outputs below must be visible
@@ -282,9 +278,9 @@ window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows 
     const int64_t nh = head(q);
     if (S == 1) {
       const float w = 1.f / l[j];
-      for (int c = lane; c < D; c += 32) stf(out + nh * D + c, so[q * D + c] * w);
+      for (int c = lane; c < DV; c += 32) stf(out + nh * DV + c, so[q * DV + c] * w);
     } else {
-      for (int c = lane; c < D; c += 32) part_o[(nh * S + split) * D + c] = so[q * D + c];
+      for (int c = lane; c < DV; c += 32) part_o[(nh * S + split) * DV + c] = so[q * DV + c];
       if (lane == 0) {
         part_ml[(nh * S + split) * 2] = m[j];
         part_ml[(nh * S + split) * 2 + 1] = l[j];
@@ -311,15 +307,15 @@ __global__ void window_merge_kernel(const float* __restrict__ part_o, const floa
 }
 
 template <typename T>
-cudaError_t window_attention_t(const SeqBatch& sb, const T* q, const PagedRows& pages, int H, int G, int D, WindowMask mask,
-                               float scale, int n_splits, float* part_o, float* part_ml, T* out, cudaStream_t st) {
+cudaError_t window_attention_t(const SeqBatch& sb, const T* q, const PagedRows& pages, int H, int G, int D, int DV,
+                               WindowMask mask, float scale, int n_splits, float* part_o, float* part_ml, T* out, cudaStream_t st) {
   static int have = 0;
-  const int smem = 4 * (kWaK * ((D | 1) + D) + 2 * kWaQ * D + kWaQ * kWaK);
+  const int smem = 4 * (kWaK * ((D | 1) + DV) + kWaQ * (D + DV) + kWaQ * kWaK);
   cudaError_t e = want_smem(window_attn_kernel<T>, smem, have);
   if (e != cudaSuccess) return e;
   const dim3 grid(static_cast<unsigned>(static_cast<int64_t>(sb.n_tok) * (H / G) / kWaQ + sb.n_seq), n_splits, G);
-  window_attn_kernel<T><<<grid, kWaWarps * 32, smem, st>>>(sb, q, pages, H, G, D, mask, scale, part_o, part_ml, out);
-  if (n_splits > 1) window_merge_kernel<T><<<sb.n_tok * H, 128, 0, st>>>(part_o, part_ml, D, n_splits, out);
+  window_attn_kernel<T><<<grid, kWaWarps * 32, smem, st>>>(sb, q, pages, H, G, D, DV, mask, scale, part_o, part_ml, out);
+  if (n_splits > 1) window_merge_kernel<T><<<sb.n_tok * H, 128, 0, st>>>(part_o, part_ml, DV, n_splits, out);
   return cudaGetLastError();
 }
 
@@ -353,15 +349,15 @@ cudaError_t launch_qk_prepare(bool f32, const SeqBatch& sb, const void* y, int64
   return cudaGetLastError();
 }
 
-cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, int H, int G, int D,
+cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, int H, int G, int D, int DV,
                                     WindowMask mask, float scale, int n_splits, float* part_o, float* part_ml, void* out,
                                     cudaStream_t st) {
-  if (G < 1 || H % G != 0 || pages.width != 2 * G * D || mask.size < 1 || mask.keep_first < 0 || n_splits < 1 ||
+  if (G < 1 || H % G != 0 || pages.width != G * (D + DV) || mask.size < 1 || mask.keep_first < 0 || n_splits < 1 ||
       (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return cudaErrorInvalidValue;
-  return f32 ? window_attention_t<float>(sb, static_cast<const float*>(q), pages, H, G, D, mask, scale, n_splits, part_o, part_ml,
+  return f32 ? window_attention_t<float>(sb, static_cast<const float*>(q), pages, H, G, D, DV, mask, scale, n_splits, part_o, part_ml,
                                          static_cast<float*>(out), st)
-             : window_attention_t<__nv_bfloat16>(sb, static_cast<const __nv_bfloat16*>(q), pages, H, G, D, mask, scale, n_splits,
+             : window_attention_t<__nv_bfloat16>(sb, static_cast<const __nv_bfloat16*>(q), pages, H, G, D, DV, mask, scale, n_splits,
                                                  part_o, part_ml, static_cast<__nv_bfloat16*>(out), st);
 }
 

@@ -39,6 +39,7 @@ FAMILIES: Dict[str, Family] = {f.name: f for f in (
     Family("deepseek_v3", _BASE + "deepseek_v3", "DeepSeekV3Config", ("DeepseekV3ForCausalLM", "deepseek_v3")),
     Family("vobunex", _BASE + "vobunex", "VobunexConfig", ("Vobunex",), from_dir=_FOLDER, engine="VobunexEngine"),
     Family("fovudra", _BASE + "fovudra", "FovudraConfig", ("Fovudra",), from_dir=_FOLDER, engine="FovudraEngine"),
+    Family("munazen", _BASE + "munazen", "MunazenConfig", ("Munazen",), from_dir=_FOLDER, engine="MunazenEngine"),
 )}
 
 

@@ -139,19 +139,25 @@ def attention_decode(q, cache_k, cache_v, kv_len=None, pos: Optional[torch.Tenso
     return out.view(B, H, D)
 
 
+def decode_widths_ok(H: int, Hkv: int, D: int, Dv: int) -> bool:
+    """Head counts and widths that the paged decode kernel takes."""
+    return (D, Dv) in ((64, 64), (128, 128), (256, 256), (64, 128), (128, 256)) and H % Hkv == 0 and H // Hkv in (1, 2, 4, 8)
+
+
 def attention_decode_paged(q, pool, block_table, seq_ids, seq_lens, n_kv_heads: int, len_add: int = 1, scale=None,
-                           scratch=None, out=None, max_len: Optional[int] = None, window: int = 0, keep_first: int = 0):
+                           scratch=None, out=None, max_len: Optional[int] = None, window: int = 0, keep_first: int = 0,
+                           v_dim: int = 0):
     """One query token per sequence over a PAGED cache (cache/paged.py): ``pool`` (n_pages, page_size, 2 * Hkv * D)
     holds K of every kv head then V per cached token, ``block_table`` (max_seqs, max_pages) the page ids,
     ``seq_ids`` (B,) the sequence of every query row, ``seq_lens`` (max_seqs,) the committed lengths, all on the
     device; ``len_add`` keys beyond the committed length are attended (1: the new token's row is written, the length
     not yet advanced). ``window`` > 0: only the last ``window`` keys and the first ``keep_first`` are seen.
-    q (B, H, D). Returns (B, H, D)."""
+    q (B, H, D). Returns (B, H, D), or (B, H, v_dim) where the values have a width of their own."""
     B, H, D = q.shape
-    Hkv = n_kv_heads
+    Hkv, Dv = n_kv_heads, v_dim or q.shape[2]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
-    cuda_ok = (q.is_cuda and q.dtype == torch.bfloat16 and pool.dtype == torch.bfloat16 and D in (64, 128, 256)
-               and H % Hkv == 0 and (H // Hkv) in (1, 2, 4, 8) and pool.shape[-1] == 2 * Hkv * D)
+    cuda_ok = (q.is_cuda and q.dtype == torch.bfloat16 and pool.dtype == torch.bfloat16 and decode_widths_ok(H, Hkv, D, Dv)
+               and pool.shape[-1] == Hkv * (D + Dv))
     if not cuda_ok:
         outs = []
         ps = pool.shape[1]
@@ -159,9 +165,9 @@ def attention_decode_paged(q, pool, block_table, seq_ids, seq_lens, n_kv_heads: 
             sid = int(seq_ids[b])
             n = int(seq_lens[sid]) + len_add
             pos = torch.arange(n, device=pool.device)
-            rows = pool[block_table[sid, (pos // ps).long()].long(), (pos % ps).long()]          # (n, 2 Hkv D)
+            rows = pool[block_table[sid, (pos // ps).long()].long(), (pos % ps).long()]          # (n, Hkv (D + Dv))
             kk = rows[:, :Hkv * D].reshape(1, n, Hkv, D).to(q.dtype)
-            vv = rows[:, Hkv * D:].reshape(1, n, Hkv, D).to(q.dtype)
+            vv = rows[:, Hkv * D:].reshape(1, n, Hkv, Dv).to(q.dtype)
             if window > 0:
                 seen = (pos >= n - window) | (pos < keep_first)
                 kk, vv = kk[:, seen], vv[:, seen]
@@ -173,13 +179,13 @@ def attention_decode_paged(q, pool, block_table, seq_ids, seq_lens, n_kv_heads: 
     if scratch is None:
         n_keys = max_len or block_table.shape[1] * pool.shape[1]
         S = decode_splits(B, Hkv, min(n_keys, window + keep_first) if window > 0 else n_keys)
-        scratch = (torch.empty(B, H, S, D, device=q.device, dtype=torch.float32),
+        scratch = (torch.empty(B, H, S, Dv, device=q.device, dtype=torch.float32),
                    torch.empty(B, H, S, 2, device=q.device, dtype=torch.float32))
     if out is None:
-        out = torch.empty(B, H * D, device=q.device, dtype=torch.bfloat16)
+        out = torch.empty(B, H * Dv, device=q.device, dtype=torch.bfloat16)
     _ext.ops().attn_decode_paged(q2, pool, block_table, seq_ids, seq_lens, int(len_add), H, Hkv, scale, scratch[0],
                                  scratch[1], out, window, keep_first)
-    return out.view(B, H, D)
+    return out.view(B, H, Dv)
 
 
 class _AttnFn(torch.autograd.Function):

@@ -61,20 +61,21 @@ def key_splits(batch: PackedBatch, H: int, G: int, window: int, keep_first: int)
 
 
 def window_attention_any(batch: PackedBatch, q, cache, layer: int, G: int, window: int, keep_first: int, scale: float,
-                         n_splits: int = 0) -> torch.Tensor:
-    """q (N, H, D) over the cached rows of each token's own sequence. Returns (N, H, D)."""
+                         n_splits: int = 0, v_dim: int = 0) -> torch.Tensor:
+    """q (N, H, D) over the cached rows of each token's own sequence; values of width ``v_dim`` (0: D). Returns (N, H, v_dim)."""
     N, H, D = q.shape
+    DV = v_dim or D
     if q.is_cuda:
         S = n_splits or key_splits(batch, H, G, window, keep_first)
-        o = torch.empty_like(q)
-        po = torch.empty(N * H * S * D, device=q.device, dtype=torch.float32) if S > 1 else None
+        o = torch.empty(N, H, DV, device=q.device, dtype=q.dtype)
+        po = torch.empty(N * H * S * DV, device=q.device, dtype=torch.float32) if S > 1 else None
         pm = torch.empty(N * H * S * 2, device=q.device, dtype=torch.float32) if S > 1 else None
         _ext.ops().window_attention(*batch.desc, q, cache.pool[layer], cache.block_table, window, keep_first, scale, S, po, pm, o)
         return o
-    out = torch.empty_like(q)
+    out = torch.empty(N, H, DV, dtype=q.dtype)
     for c0, n, slot, start in batch.rows():
         rows = cache.gather(layer, slot, start + n).float()
-        k, v = (t.reshape(start + n, G, D).repeat_interleave(H // G, 1) for t in rows.split(G * D, -1))
+        k, v = (t.reshape(start + n, G, -1).repeat_interleave(H // G, 1) for t in rows.split([G * D, G * DV], -1))
         i, j = torch.arange(start, start + n)[:, None], torch.arange(start + n)[None, :]
         seen = (j <= i) & ((i - j < window) | (j < keep_first))
         s = torch.einsum("nhd,khd->hnk", q[c0:c0 + n].float(), k) * scale
@@ -83,19 +84,24 @@ def window_attention_any(batch: PackedBatch, q, cache, layer: int, G: int, windo
     return out
 
 
+def flash_prompts(batch: PackedBatch, q, k, v, scale: float, window: int = 0, keep_first: int = 0) -> torch.Tensor:
+    """Whole prompts on the flash kernel: dense q (N, H, D), k (N, G, D), v (N, G, DV). Returns (N, H, DV)."""
+    o = torch.empty(q.shape[0], q.shape[1], v.shape[2], device=q.device, dtype=q.dtype)
+    same = len(set(batch.lens)) == 1
+    parts = [(0, batch.n_tok, batch.n_seq)] if same else [(sum(batch.lens[:b]), n, 1) for b, n in enumerate(batch.lens)]
+    for c0, n, B in parts:
+        as4 = lambda t: t[c0:c0 + n].unflatten(0, (B, n // B))
+        A.attn_fwd(as4(q), as4(k), as4(v), True, scale, out=as4(o), window=window, keep_first=keep_first)
+    return o
+
+
 def window_attention(batch: PackedBatch, q, k, v, cache, layer: int, G: int, window: Optional[int], keep_first: int,
                      scale: float) -> torch.Tensor:
     """q (N, H, D) and, for whole prompts on the flash kernel, the dense k, v (N, G, D) of ``qk_prepare``. Returns (N, H D)."""
     N, H, D = q.shape
     window = window or NO_WINDOW
     if k is not None and flash_ok(batch, q, D):
-        o = torch.empty(N, H, D, device=q.device, dtype=q.dtype)
-        same = len(set(batch.lens)) == 1
-        parts = [(0, N, batch.n_seq)] if same else [(sum(batch.lens[:b]), n, 1) for b, n in enumerate(batch.lens)]
-        for c0, n, B in parts:
-            as4 = lambda t: t[c0:c0 + n].unflatten(0, (B, n // B))
-            A.attn_fwd(as4(q), as4(k), as4(v), True, scale, out=as4(o), window=window, keep_first=keep_first)
-        return o.view(N, H * D)
+        return flash_prompts(batch, q, k, v, scale, window, keep_first).view(N, H * D)
     if decode_ok(batch, q, H, G, D):
         # the step has advanced the lengths already: len_add 0
         return A.attention_decode_paged(q, cache.pool[layer], cache.block_table, batch.ids, cache.seq_lens, G, 0, scale,
