@@ -1,0 +1,417 @@
+// Linear attention with a decay per key channel on packed batches, chunked (Yang et al., "Gated Linear Attention Transformers with
+// Hardware-Efficient Training"): S_t = diag(alpha_t) S_(t-1) + k_t v_t^T, o_t = q_scale S_t^T q_t. With F the running sum of
+// log alpha in a chunk of 64 tokens and S the state before it,
+//   o_i   = (q_i exp(F_i))^T S + sum_(j <= i) A_ij v_j,      A_ij = sum_n q_in k_jn exp(F_in - F_jn)
+//   S_new = diag(exp(F_end)) S + sum_j (k_j exp(F_end - F_j)) v_j^T
+// Every exponent that is formed is at most 0, but for the 16 x 16 blocks on the diagonal of A: those are taken relative to the block's
+// middle token where its decays allow that, and pair by pair where they are too strong.
+//
+// Two launches. Nothing in the first depends on the state: a block per chunk and head makes the decays, the scaled queries and keys and
+// A, and leaves them as the shared-memory image (rows padded by 16 bytes) that the second one copies in. The second walks the chunks of
+// a sequence with the state of a head and 32 value columns in registers. Every fp32 operand (scaled queries and keys, A, the state as
+// an operand) enters its product as a high and a low bf16 part; values are bf16 already. mma.sync: the operands of a step are
+// 64 rows high and the state has to come back to registers every step.
+//
+// This file is built without fast-math and names its fast intrinsics.
+#include "serve_common.cuh"
+#include "serve_kernels.cuh"
+
+namespace b200 {
+
+namespace {
+
+using Bf = __nv_bfloat16;
+constexpr int kC = 64, kSub = 16, kLdA = kC + 8, kPrepThreads = 320, kScanThreads = 256, kPs = 32, kLdP = kPs + 8;
+
+struct Image {   // one (chunk, head); offsets in bytes
+  int N, ld;     // key width, row stride of the scaled queries and keys
+  __host__ __device__ explicit Image(int n) : N(n), ld(n + 8) {}
+  __host__ __device__ int rows() const { return kC * ld * 2; }                     // one of qh, ql, kh, kl
+  __host__ __device__ int a() const { return 4 * rows(); }                         // high, then low part of A
+  __host__ __device__ int tiles() const { return a() + 2 * kC * kLdA * 2; }        // what the scan copies
+  __host__ __device__ int bytes() const { return tiles() + N * 4; }                // and exp(F_end), fp32
+};
+
+struct Chunk {
+  int b, t0, cnt;   // sequence, first token in it, tokens
+};
+__device__ __forceinline__ Chunk chunk_at(const SeqBatch& sb, int tile) {
+  for (int b = 0; b < sb.n_seq; ++b) {
+    const int len = sb.cu[b + 1] - sb.cu[b], n = (len + kC - 1) / kC;
+    if (tile < n) return {b, tile * kC, min(kC, len - tile * kC)};
+    tile -= n;
+  }
+  return {-1, 0, 0};
+}
+
+__device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)));
+}
+__device__ __forceinline__ void cp16(void* dst, const void* src, bool live) {   // 16 bytes, zeros where not live
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+// x = hi + lo with both in bf16
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(x, y);
+  const float2 h = unpack_bf16x2(hi);
+  lo = pack_bf16x2(x - h.x, y - h.y);
+}
+// log sigmoid(z)
+__device__ __forceinline__ float log_sigmoid_fast(float z) {
+  const float e = __expf(-fabsf(z));
+  const float l = e < 0.03f ? e * (1.f - e * (0.5f - e * (1.f / 3 - e * 0.25f))) : __logf(1.f + e);
+  return fminf(z, 0.f) - l;
+}
+
+// ---- decays, scaled operands, A ------------------------------------------------------------------------------------------
+__host__ __device__ __forceinline__ int low_ld(int R) { return (R + 3) / 4 * 4; }
+__host__ __device__ __forceinline__ int prep_smem(int N, int R) {
+  return kC * (N + 8) * 4 + 2 * kC * (N + 8) * 2 + low_ld(R) * (kC + N) * 4;
+}
+
+// two elements of an operand scaled by exp(dir (F - ref)), split
+__device__ __forceinline__ void scaled2(const Bf* x, const float* F, const float* ref, float dir, uint32_t& hi, uint32_t& lo) {
+  const float2 v = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x)), f = *reinterpret_cast<const float2*>(F), r = *reinterpret_cast<const float2*>(ref);
+  split2(v.x * __expf(dir * (f.x - r.x)), v.y * __expf(dir * (f.y - r.y)), hi, lo);
+}
+
+__global__ void __launch_bounds__(kPrepThreads)
+gla_prep_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const LinGates gt, const LinShape s, unsigned char* __restrict__ images) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  const Chunk ch = chunk_at(sb, blockIdx.x);
+  if (ch.b < 0) return;
+  const int N = s.N, h = blockIdx.y, R = gt.R, ldl = low_ld(R), ldn = N + 8;
+  const Image im(N);
+  unsigned char* img = images + (static_cast<int64_t>(blockIdx.x) * s.H + h) * im.bytes();
+  float* sF = reinterpret_cast<float*>(smem);              // [kC][ldn]
+  Bf* sQ = reinterpret_cast<Bf*>(sF + kC * ldn);           // [kC][ldn]
+  Bf* sK = sQ + kC * ldn;                                  // [kC][ldn]
+  float* sL = reinterpret_cast<float*>(sK + kC * ldn);     // [kC][ldl] low-rank rows
+  float* sW = sL + kC * ldl;                               // [ldl][N]
+  const int64_t row0 = sb.cu[ch.b] + ch.t0;
+  const int tid = threadIdx.x, chunks = N / 8;
+  for (int i = tid; i < kC * chunks; i += kPrepThreads) {
+    const int t = i / chunks, c = i % chunks * 8;
+    uint4 q = make_uint4(0u, 0u, 0u, 0u), k = q;
+    if (t < ch.cnt) {
+      const Bf* row = qkv + (row0 + t) * ld + h * N + c;
+      q = *reinterpret_cast<const uint4*>(row);
+      k = *reinterpret_cast<const uint4*>(row + s.H * N);
+    }
+    *reinterpret_cast<uint4*>(sQ + t * ldn + c) = q;
+    *reinterpret_cast<uint4*>(sK + t * ldn + c) = k;
+  }
+  for (int i = tid; i < kC * ldl; i += kPrepThreads) {
+    const int t = i / ldl, r = i % ldl;
+    sL[i] = t < ch.cnt && r < R ? ldf(static_cast<const Bf*>(gt.low) + (row0 + t) * gt.ld_low + r) : 0.f;
+  }
+  for (int i = tid; i < ldl * N; i += kPrepThreads) {
+    const int n = i / ldl, r = i % ldl;
+    sW[r * N + n] = r < R ? ldf(static_cast<const Bf*>(gt.w2) + (static_cast<int64_t>(h) * N + n) * R + r) : 0.f;
+  }
+  __syncthreads();
+  // ---- running sums of log alpha: a thread per channel and run of tokens ----
+  int groups = 8;
+  while (groups > 1 && groups * N > kPrepThreads) groups >>= 1;
+  const int run = kC / groups, n = tid % N, tg = tid / N;
+  if (tg < groups) {
+    const float b2 = gt.bias2[h * N + n];
+    float F = 0.f;
+    for (int t0 = tg * run; t0 < (tg + 1) * run; t0 += 8) {
+      float z[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) z[j] = b2;
+      for (int r = 0; r < ldl; r += 4) {
+        const float w0 = sW[r * N + n], w1 = sW[(r + 1) * N + n], w2 = sW[(r + 2) * N + n], w3 = sW[(r + 3) * N + n];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const float4 x = *reinterpret_cast<const float4*>(sL + (t0 + j) * ldl + r);
+          z[j] = fmaf(x.x, w0, fmaf(x.y, w1, fmaf(x.z, w2, fmaf(x.w, w3, z[j]))));
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        if (t0 + j < ch.cnt) F = fmaf(log_sigmoid_fast(z[j]), gt.inv_tau, F);
+        sF[(t0 + j) * ldn + n] = F;
+      }
+    }
+  }
+  __syncthreads();
+  if (groups > 1) {
+    float off = 0.f;
+    if (tg < groups)
+      for (int i = 0; i < tg; ++i) off += sF[((i + 1) * run - 1) * ldn + n];
+    __syncthreads();
+    if (tg < groups && tg > 0)
+      for (int t = tg * run; t < (tg + 1) * run; ++t) sF[t * ldn + n] += off;
+    __syncthreads();
+  }
+  // ---- scaled queries and keys ----
+  const float* end = sF + (kC - 1) * ldn;
+  for (int i = tid; i < kC * chunks; i += kPrepThreads) {
+    const int t = i / chunks, c = i % chunks * 8;
+    float q[8], k[8];
+    Vec16<Bf>::load(sQ + t * ldn + c, q);
+    Vec16<Bf>::load(sK + t * ldn + c, k);
+    uint32_t qh[4], ql[4], kh[4], kl[4];
+#pragma unroll
+    for (int j = 0; j < 8; j += 2) {
+      const float f0 = sF[t * ldn + c + j], f1 = sF[t * ldn + c + j + 1];
+      split2(q[j] * s.q_scale * __expf(f0), q[j + 1] * s.q_scale * __expf(f1), qh[j / 2], ql[j / 2]);
+      split2(k[j] * __expf(end[c + j] - f0), k[j + 1] * __expf(end[c + j + 1] - f1), kh[j / 2], kl[j / 2]);
+    }
+    unsigned char* d = img + (t * ldn + c) * 2;
+    *reinterpret_cast<uint4*>(d) = make_uint4(qh[0], qh[1], qh[2], qh[3]);
+    *reinterpret_cast<uint4*>(d + im.rows()) = make_uint4(ql[0], ql[1], ql[2], ql[3]);
+    *reinterpret_cast<uint4*>(d + 2 * im.rows()) = make_uint4(kh[0], kh[1], kh[2], kh[3]);
+    *reinterpret_cast<uint4*>(d + 3 * im.rows()) = make_uint4(kl[0], kl[1], kl[2], kl[3]);
+  }
+  for (int i = tid; i < N; i += kPrepThreads) reinterpret_cast<float*>(img + im.tiles())[i] = expf(end[i]);
+  // ---- A: a warp per 16 x 16 block, six below the diagonal and four on it ----
+  const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  int I, J;
+  if (warp < 6) {
+    I = warp < 1 ? 1 : warp < 3 ? 2 : 3;
+    J = warp - (I == 1 ? 0 : I == 2 ? 1 : 3);
+  } else {
+    I = J = warp - 6;
+  }
+  const bool diag = I == J;
+  Bf *ah = reinterpret_cast<Bf*>(img + im.a()) + I * kSub * kLdA + J * kSub, *al = ah + kC * kLdA;
+  const float* ref = sF + (J * kSub + (diag ? kSub / 2 - 1 : kSub - 1)) * ldn;
+  if (diag) {
+    float spread = 0.f;
+    for (int c = lane; c < N; c += 32) spread = fmaxf(spread, fmaxf(sF[I * kSub * ldn + c] - ref[c], ref[c] - sF[(I * kSub + kSub - 1) * ldn + c]));
+    if (warp_max(spread) > 60.f) {   // the factors would leave fp32's range: pair by pair
+      for (int i = 0; i < kSub; ++i)
+        for (int j = 0; j < kSub; ++j) {
+          float v = 0.f;
+          if (j <= i)
+            for (int c = lane; c < N; c += 32) {
+              const int qi = (I * kSub + i) * ldn + c, kj = (I * kSub + j) * ldn + c;
+              v = fmaf(ldf(sQ + qi) * ldf(sK + kj), __expf(sF[qi] - sF[kj]), v);
+            }
+          v = warp_sum(v) * s.q_scale;
+          if (lane == 0) {
+            const Bf hi = __float2bfloat16(v);
+            ah[i * kLdA + j] = hi;
+            al[i * kLdA + j] = __float2bfloat16(v - __bfloat162float(hi));
+          }
+        }
+      return;
+    }
+  }
+  float acc[2][4] = {};
+  const int i0 = (I * kSub + g) * ldn, j0 = (J * kSub + g) * ldn;
+  for (int kb = 0; kb < N; kb += 16) {
+    uint32_t xh[4], xl[4], yh[4], yl[4];   // queries; keys of the two column tiles
+#pragma unroll
+    for (int p = 0; p < 2; ++p) {
+      const int c = kb + 2 * t + 8 * p;
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        scaled2(sQ + i0 + r * 8 * ldn + c, sF + i0 + r * 8 * ldn + c, ref + c, 1.f, xh[2 * p + r], xl[2 * p + r]);
+        scaled2(sK + j0 + r * 8 * ldn + c, sF + j0 + r * 8 * ldn + c, ref + c, -1.f, yh[2 * r + p], yl[2 * r + p]);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      mma_16816(acc[m], xh, yh[2 * m], yh[2 * m + 1]);
+      mma_16816(acc[m], xh, yl[2 * m], yl[2 * m + 1]);
+      mma_16816(acc[m], xl, yh[2 * m], yh[2 * m + 1]);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int i = g + 8 * r, j = m * 8 + 2 * t;
+      const float v0 = !diag || j <= i ? acc[m][2 * r] * s.q_scale : 0.f, v1 = !diag || j + 1 <= i ? acc[m][2 * r + 1] * s.q_scale : 0.f;
+      uint32_t hi, lo;
+      split2(v0, v1, hi, lo);
+      *reinterpret_cast<uint32_t*>(ah + i * kLdA + j) = hi;
+      *reinterpret_cast<uint32_t*>(al + i * kLdA + j) = lo;
+    }
+}
+
+// ---- scan over the chunks --------------------------------------------------------------------------------------------------
+__host__ __device__ __forceinline__ int stage_bytes(int N) { return Image(N).tiles() + kC * kLdP * 2; }
+__host__ __device__ __forceinline__ int scan_smem(int N) { return 2 * stage_bytes(N) + 2 * 2 * N * kLdP * 2; }
+
+__global__ void __launch_bounds__(kScanThreads)
+gla_scan_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const unsigned char* __restrict__ images, float* __restrict__ state,
+                Bf* __restrict__ y, const LinShape s) {
+  extern __shared__ __align__(16) unsigned char smem[];
+  const int N = s.N, P = s.P, h = blockIdx.x, p0 = blockIdx.y * kPs, b = blockIdx.z;
+  const Image im(N);
+  const int ldn = im.ld, stage = stage_bytes(N);
+  Bf* sS = reinterpret_cast<Bf*>(smem + 2 * stage);        // [2 buffers][high, low][N][kLdP]
+  const int first = sb.cu[b], len = sb.cu[b + 1] - first, chunks = (len + kC - 1) / kC;
+  int tile0 = 0;
+  for (int i = 0; i < b; ++i) tile0 += (sb.cu[i + 1] - sb.cu[i] + kC - 1) / kC;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  auto image = [&](int c) { return images + (static_cast<int64_t>(tile0 + c) * s.H + h) * im.bytes(); };
+  auto load = [&](int c) {
+    unsigned char* d = smem + (c & 1) * stage;
+    const unsigned char* src = image(c);
+    for (int i = tid * 16; i < im.tiles(); i += kScanThreads * 16) cp16(d + i, src + i, true);
+    Bf* sv = reinterpret_cast<Bf*>(d + im.tiles());
+    const Bf* v = qkv + 2 * s.H * N + h * P + p0;
+    for (int i = tid; i < kC * (kPs / 8); i += kScanThreads) {
+      const int r = i / (kPs / 8), cc = i % (kPs / 8) * 8;
+      const bool live = c * kC + r < len && p0 + cc < P;
+      cp16(sv + r * kLdP + cc, live ? v + static_cast<int64_t>(first + c * kC + r) * ld + cc : v, live);
+    }
+    cp_commit();
+  };
+  load(0);
+  // state rows of this warp: keys 16 warp + g, + 8; columns 8 m + 2 t, + 1
+  const bool owner = warp * 16 < N;
+  float* st = state + (static_cast<int64_t>(sb.ids[b]) * s.H + h) * N * P;
+  const bool fresh = sb.start[b] == 0;
+  float S[4][4];
+  auto each_state = [&](auto&& f) {
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int key = warp * 16 + g + 8 * (e / 2), p = p0 + m * 8 + 2 * t + e % 2;
+        f(S[m][e], key, p, owner && p < P);
+      }
+  };
+  each_state([&](float& v, int key, int p, bool live) { v = live && !fresh ? st[static_cast<int64_t>(key) * P + p] : 0.f; });
+  auto publish = [&](int buf) {
+    if (!owner) return;
+    Bf *hi = sS + buf * 2 * N * kLdP, *lo = hi + N * kLdP;
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        uint32_t a, c;
+        split2(S[m][2 * r], S[m][2 * r + 1], a, c);
+        const int at = (warp * 16 + g + 8 * r) * kLdP + m * 8 + 2 * t;
+        *reinterpret_cast<uint32_t*>(hi + at) = a;
+        *reinterpret_cast<uint32_t*>(lo + at) = c;
+      }
+  };
+  publish(0);
+  const int mt = warp >> 1, nh = (warp & 1) * 16;          // output rows 16 mt .., columns nh ..
+  const int r16 = lane & 15, c8 = (lane >> 4) * 8;
+  for (int c = 0; c < chunks; ++c) {
+    float fe[2] = {0.f, 0.f};
+    if (owner) {
+      const float* e = reinterpret_cast<const float*>(image(c) + im.tiles());
+      fe[0] = e[warp * 16 + g];
+      fe[1] = e[warp * 16 + g + 8];
+    }
+    cp_wait_all();
+    __syncthreads();                                       // this chunk's operands and state are visible, the other buffers are free
+    if (c + 1 < chunks) load(c + 1);
+    const unsigned char* d = smem + (c & 1) * stage;
+    const Bf *qh = reinterpret_cast<const Bf*>(d), *ql = qh + kC * ldn, *kh = ql + kC * ldn, *kl = kh + kC * ldn;
+    const Bf *ah = reinterpret_cast<const Bf*>(d + im.a()), *al = ah + kC * kLdA, *sv = reinterpret_cast<const Bf*>(d + im.tiles());
+    const Bf *sh = sS + (c & 1) * 2 * N * kLdP, *sl = sh + N * kLdP;
+    const int cnt = min(kC, len - c * kC);
+    // ---- outputs ----
+    if (mt * 16 < cnt) {
+      float o[2][4] = {};
+      for (int k = 0; k < N; k += 16) {
+        uint32_t xh[4], xl[4], zh[4], zl[4];
+        ldsm4(xh, qh + (mt * 16 + r16) * ldn + k + c8);
+        ldsm4(xl, ql + (mt * 16 + r16) * ldn + k + c8);
+        ldsm4_t(zh, sh + (k + r16) * kLdP + nh + c8);
+        ldsm4_t(zl, sl + (k + r16) * kLdP + nh + c8);
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          mma_16816(o[m], xh, zh[2 * m], zh[2 * m + 1]);
+          mma_16816(o[m], xh, zl[2 * m], zl[2 * m + 1]);
+          mma_16816(o[m], xl, zh[2 * m], zh[2 * m + 1]);
+        }
+      }
+      for (int k = 0; k <= mt; ++k) {
+        uint32_t xh[4], xl[4], z[4];
+        ldsm4(xh, ah + (mt * 16 + r16) * kLdA + k * 16 + c8);
+        ldsm4(xl, al + (mt * 16 + r16) * kLdA + k * 16 + c8);
+        ldsm4_t(z, sv + (k * 16 + r16) * kLdP + nh + c8);
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          mma_16816(o[m], xh, z[2 * m], z[2 * m + 1]);
+          mma_16816(o[m], xl, z[2 * m], z[2 * m + 1]);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int row = mt * 16 + g + 8 * r, p = p0 + nh + m * 8 + 2 * t;
+          if (row < cnt && p < P)
+            *reinterpret_cast<uint32_t*>(y + (static_cast<int64_t>(first + c * kC + row) * s.H + h) * P + p) = pack_bf16x2(o[m][2 * r], o[m][2 * r + 1]);
+        }
+    }
+    // ---- state ----
+    if (owner) {
+#pragma unroll
+      for (int m = 0; m < 4; ++m)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) S[m][e] *= fe[e / 2];
+      const int tok = (lane & 7) + (lane >> 4) * 8, key = warp * 16 + ((lane >> 3) & 1) * 8;
+#pragma unroll
+      for (int k = 0; k < kC; k += 16) {
+        uint32_t xh[4], xl[4], z0[4], z1[4];
+        ldsm4_t(xh, kh + (k + tok) * ldn + key);
+        ldsm4_t(xl, kl + (k + tok) * ldn + key);
+        ldsm4_t(z0, sv + (k + r16) * kLdP + c8);
+        ldsm4_t(z1, sv + (k + r16) * kLdP + 16 + c8);
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          mma_16816(S[m], xh, z0[2 * m], z0[2 * m + 1]);
+          mma_16816(S[m], xl, z0[2 * m], z0[2 * m + 1]);
+          mma_16816(S[2 + m], xh, z1[2 * m], z1[2 * m + 1]);
+          mma_16816(S[2 + m], xl, z1[2 * m], z1[2 * m + 1]);
+        }
+      }
+      publish((c + 1) & 1);
+    }
+  }
+  each_state([&](float& v, int key, int p, bool live) { if (live) st[static_cast<int64_t>(key) * P + p] = v; });
+}
+
+}  // namespace
+
+bool gla_chunked_ok(const LinShape& s, int64_t ld, int R) {
+  return s.N % 16 == 0 && s.N <= 128 && s.P % 8 == 0 && ld % 8 == 0 && R <= 64 && s.silu == 0 && scan_smem(s.N) <= 227 * 1024;
+}
+
+int64_t gla_chunked_scratch(const SeqBatch& sb, const LinShape& s) {
+  return static_cast<int64_t>(sb.n_tok / kC + sb.n_seq) * s.H * Image(s.N).bytes();
+}
+
+cudaError_t launch_gla_chunked(const SeqBatch& sb, const Bf* qkv, int64_t ld, const LinGates& g, float* state, Bf* y, const LinShape& s,
+                               void* scratch, cudaStream_t st) {
+  if (!gla_chunked_ok(s, ld, g.R) || ((reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(scratch) | reinterpret_cast<uintptr_t>(y)) & 15) != 0)
+    return cudaErrorInvalidValue;
+  static int have_prep = 0, have_scan = 0;
+  const int ps = prep_smem(s.N, g.R), ss = scan_smem(s.N);
+  cudaError_t e = want_smem(gla_prep_kernel, ps, have_prep);
+  if (e == cudaSuccess) e = want_smem(gla_scan_kernel, ss, have_scan);
+  if (e != cudaSuccess) return e;
+  unsigned char* img = static_cast<unsigned char*>(scratch);
+  gla_prep_kernel<<<dim3(sb.n_tok / kC + sb.n_seq, s.H), kPrepThreads, ps, st>>>(sb, qkv, ld, g, s, img);
+  gla_scan_kernel<<<dim3(s.H, (s.P + kPs - 1) / kPs, sb.n_seq), kScanThreads, ss, st>>>(sb, qkv, ld, img, state, y, s);
+  return cudaGetLastError();
+}
+
+}  // namespace b200

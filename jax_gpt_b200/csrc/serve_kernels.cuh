@@ -185,8 +185,9 @@ struct LruArgs {
   void* out;               // [n_tok, ldo]
   int64_t ldo;
 };
-// log_a, inp: scratch [n_tok, W] fp32; log_a null: one token per sequence.
-cudaError_t launch_gated_lru(bool f32, const SeqBatch& sb, const LruArgs& a, float* log_a, float* inp, cudaStream_t st);
+// scratch: gated_lru_scratch floats (8-byte aligned), or null for one token per sequence.
+int64_t gated_lru_scratch(bool f32, const SeqBatch& sb, const LruArgs& a);
+cudaError_t launch_gated_lru(bool f32, const SeqBatch& sb, const LruArgs& a, float* scratch, cudaStream_t st);
 
 // ---- linear attention with a matrix state (linear_attention.cu, ssd_scan_sm100.cu) ---------------------------------------
 struct LinShape {
@@ -221,6 +222,12 @@ cudaError_t launch_linear_step(bool f32, const SeqBatch& sb, const void* qkv, in
 bool linear_scan_sm100_ok(const LinShape& s);
 cudaError_t launch_linear_scan_sm100(const SeqBatch& sb, const __nv_bfloat16* qkv, int64_t ld, const LinGates& g, float* state,
                                      __nv_bfloat16* y, const LinShape& s, int* status, cudaStream_t st);
+// Decays per key channel, chunked on tensor cores (gla_chunk.cu): bf16, N a multiple of 16 up to 128, P and ld multiples of 8, R <= 64,
+// activations applied. scratch: gla_chunked_scratch bytes. y bf16.
+bool gla_chunked_ok(const LinShape& s, int64_t ld, int R);
+int64_t gla_chunked_scratch(const SeqBatch& sb, const LinShape& s);
+cudaError_t launch_gla_chunked(const SeqBatch& sb, const __nv_bfloat16* qkv, int64_t ld, const LinGates& g, float* state, __nv_bfloat16* y,
+                               const LinShape& s, void* scratch, cudaStream_t st);
 struct HeadNorm {
   int parts;
   float eps, den_eps;

@@ -34,9 +34,8 @@ def gated_lru(batch: PackedBatch, x, y, w: LruWeights, ring, state, scale: float
     ``ring`` and ``state`` are advanced. ``out`` (N, W) may be a column slice."""
     N, W = x.shape
     if x.is_cuda:
-        scratch = lambda: None if batch.single else torch.empty(N, W, device=x.device, dtype=torch.float32)
         _ext.ops().gated_lru(*batch.desc, x, w.x_bias, w.conv, w.conv_bias, ring, w.gates, w.gates_bias, w.decay, state, y, w.y_bias,
-                             scale, out, scratch(), scratch())
+                             scale, out)
         return
     taps = w.conv.shape[1]
     nb = w.gates.shape[0]

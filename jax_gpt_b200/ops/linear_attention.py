@@ -3,7 +3,7 @@ with a fixed decay per head, a decay per key channel (gated linear attention), o
 and a normaliser (mLSTM).
 
 Kernels: csrc/linear_attention.cu (token by token, one-token step, norm and output gate), csrc/ssd_scan_sm100.cu (chunked on
-tcgen05). State per cache slot: ``state`` [slots, H, N, P] fp32; gated layers also carry ``vec`` [slots, H, N + 1] fp32 = the
+tcgen05), csrc/gla_chunk.cu (chunked, decays per key channel). State per cache slot: ``state`` [slots, H, N, P] fp32; gated layers also carry ``vec`` [slots, H, N + 1] fp32 = the
 normaliser and the running maximum, both scaled by exp(-maximum). A sequence that starts at position 0 ignores them.
 """
 from __future__ import annotations
@@ -57,6 +57,12 @@ def chunked_ok(batch: PackedBatch, x: torch.Tensor, N: int, P: int) -> bool:
     return x.is_cuda and x.dtype == torch.bfloat16 and not batch.single and N == 128 and P % 64 == 0
 
 
+def channels_chunked_ok(batch: PackedBatch, x: torch.Tensor, N: int, P: int, rank: int) -> bool:
+    """The same for a decay per key channel (csrc/gla_chunk.cu)."""
+    return (x.is_cuda and x.dtype == torch.bfloat16 and not batch.single and N % 16 == 0 and N <= 128 and P % 8 == 0 and rank <= 64
+            and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0)
+
+
 def log_gates(raw, bias, cap: float):
     """(log input gate, log forget gate), each (N, H)."""
     i, f = (cap * torch.tanh((raw + bias) / cap)).chunk(2, -1)
@@ -72,7 +78,8 @@ def linear_scan(batch: PackedBatch, qkv, state, *, decay=None, gates: Optional[G
     N = batch.n_tok
     if qkv.is_cuda:
         if kind is None:
-            chunked = not silu and channels is None and chunked_ok(batch, qkv, Nk, P)
+            chunked = not silu and (chunked_ok(batch, qkv, Nk, P) if channels is None else
+                                    channels_chunked_ok(batch, qkv, Nk, P, channels.w.shape[1]))
             kind = STEP if batch.single else CHUNKED if chunked else TOKENS
         new = lambda *s: torch.empty(*s, device=qkv.device, dtype=torch.float32)
         y = torch.empty(N, H * P, device=qkv.device, dtype=torch.bfloat16) if kind == CHUNKED else new(N, H * P)
