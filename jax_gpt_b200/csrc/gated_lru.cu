@@ -6,8 +6,7 @@
 //
 // Any sizes: gates of eight rows at a time (a warp per channel), then a scan with a thread per channel; one token per sequence:
 // all of it in one launch. bf16 prompts: the gates are tensor-core products with channels as rows and tokens as columns, so that a
-// warp holds all tokens of a chunk for its 16 channels and scans them in registers; chunk totals first, then a scan over the
-// chunks, then the outputs.
+// warp holds all tokens of a chunk for its 16 channels and scans them in registers; then a scan over the chunks, then the outputs.
 //
 // Gates, decays and states are fp32. This file is built without fast-math; the tensor-core kernel names its fast intrinsics.
 #include "serve_common.cuh"
@@ -158,33 +157,35 @@ cudaError_t lru_gates_go(const SeqBatch& sb, const LruArgs& a, float* log_a, flo
 }
 
 // ---- bf16 prompts on tensor cores --------------------------------------------------------------------------------------
-// Block: a chunk of 64 tokens of one sequence and up to 128 channels of one gate block, a warp per 16 channels. The convolved
-// inputs of the whole gate block are staged as rows (token, channel) in a high and a low bf16 part; mma.sync m16n8k16 with gate weights as the 16-row
-// operand and tokens as columns (tcgen05 would need both products of 16 channels spread over TMEM lanes, one channel a lane, and
-// the scan back through tcgen05.ld; here the accumulators are where the scan wants them). Column g of tile n is token
-// 16 (g / 2) + 2 n + g % 2, so that a lane's 16 columns are 16 consecutive tokens of its two channels: the scan is a loop in the
-// lane and one composition over four lanes. Contraction indices are permuted alike on both sides, which leaves the sums unchanged.
-constexpr int kChunk = 64, kSlice = 128;
+// lru_chunk: a block per chunk of 64 tokens of one sequence and up to 128 channels of one gate block, a warp per 16 channels. The
+// convolved inputs of the whole gate block are staged as rows (token, channel) in a high and a low bf16 part; mma.sync m16n8k16 with
+// gate weights as the 16-row operand and tokens as columns (tcgen05 would leave a channel per TMEM lane, and the scan would take it
+// back through tcgen05.ld; here the accumulators are where the scan wants them). Column g of tile n is token 16 (g / 2) + 2 n + g % 2,
+// so that a lane's 16 columns are 16 consecutive tokens of its two channels: the scan is a loop in the lane and one composition over
+// four lanes. Contraction indices are permuted alike on both sides, which leaves the sums unchanged. Every token's composition
+// (factor, offset) from the chunk's start goes to memory, the start states follow from a scan over the chunks (lru_prefix), and
+// lru_output makes the outputs.
+constexpr int kChunk = 64, kSlice = 128, kStripTok = 4;
 
-__device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
 __device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
   f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
 }
-__device__ __forceinline__ float fast_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
-// 1 - exp(-x) for x >= 0, with e = exp(-x / 2)
-__device__ __forceinline__ float one_minus_exp(float x, float e) {
-  const float p = x * (1.f - x * (0.5f - x * (1.f / 6 - x * (1.f / 24 - x * (1.f / 120 - x * (1.f / 720))))));
-  return x < 0.25f ? p : 1.f - e * e;
+// a = exp(-x) and 1 - a^2 for x >= 0, both to fp32 rounding also where a is close to 1
+__device__ __forceinline__ void decay_pair(float x, float& a, float& om) {
+  const float p = x * (1.f - x * (0.5f - x * (1.f / 6 - x * (1.f / 24 - x * (1.f / 120)))));
+  const float e = ex2_approx(-kLog2e * x);
+  const float d = x < 0.125f ? p : 1.f - e;
+  a = x < 0.125f ? 1.f - p : e;
+  om = d * (2.f - d);
 }
 __host__ __device__ __forceinline__ int staged_ld(int wb) {   // row stride of the staged inputs: 64 bytes past a multiple of 128
   const int k = (wb + 31) / 32;
   return (k % 2 == 0 ? k + 1 : k) * 32;
 }
+// rows turn by 16 bytes every 16 tokens: lanes that read one channel of tokens 16 apart hit different banks
+__host__ __device__ __forceinline__ int staged_size(int wb) { return kChunk * staged_ld(wb) + kChunk / 16 * 8; }
+__device__ __forceinline__ int staged_row(int tok, int ldu) { return tok * ldu + (tok >> 4) * 8; }
 
 struct ChunkOf {
   int b, t0, cnt;   // sequence, first token in it, tokens
@@ -198,169 +199,205 @@ __device__ __forceinline__ ChunkOf chunk_of(const SeqBatch& sb, int tile) {
   return {-1, 0, 0};
 }
 
-// kFinal: outputs from the chunk's start state `starts`; otherwise the chunk's composition (factor, offset) to `totals`.
-template <bool kFinal>
 __global__ void __launch_bounds__(kSlice * 2, 2)
-lru_chunk_kernel(const SeqBatch sb, const LruArgs a, float2* __restrict__ totals, const float* __restrict__ starts) {
+lru_chunk_kernel(const SeqBatch sb, const LruArgs a, float2* __restrict__ steps, float2* __restrict__ totals) {
   using B = __nv_bfloat16;
   extern __shared__ __align__(16) unsigned char smem[];
   const ChunkOf ch = chunk_of(sb, blockIdx.x);
   if (ch.b < 0) return;
   const int wb = a.W / a.blocks, ldu = staged_ld(wb), blk = blockIdx.y, c0 = blockIdx.z * kSlice, cc = min(kSlice, wb - c0);
-  B* su = reinterpret_cast<B*>(smem);                                    // [kChunk][ldu] high parts
-  B* sl = su + kChunk * ldu;                                             // [kChunk][ldu] low parts
-  float* sw = reinterpret_cast<float*>(sl + kChunk * ldu);               // [2 + taps][wb], later
-  float* sS = sw;                                                        // [kChunk][cc] (kFinal)
+  B* su = reinterpret_cast<B*>(smem);                          // high parts
+  B* sl = su + staged_size(wb);                                // low parts
+  float* sw = reinterpret_cast<float*>(sl + staged_size(wb));  // [3 + taps][wb]: x_bias, conv_bias, conv_bias + sum(conv) x_bias, taps
   const int first = sb.cu[ch.b], start = sb.start[ch.b], slot = sb.ids[ch.b];
   const B* x = static_cast<const B*>(a.x);
-  // ---- convolution: eight channels of a token at a time; biases and taps are staged as rows ----
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3, cw = c0 + warp * 16;
+  const B* wr = static_cast<const B*>(a.gates) + (static_cast<int64_t>(blk) * 2 * wb + min(cw, wb - 16) + g) * wb;
+  const B* wi = wr + static_cast<int64_t>(wb) * wb;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  struct Weights {
+    uint4 r0, r1, i0, i1;
+  };
+  auto weights = [&](int kb) {
+    const int k = kb + t * 8;
+    if (k >= wb) return Weights{zero, zero, zero, zero};
+    return Weights{__ldg(reinterpret_cast<const uint4*>(wr + k)), __ldg(reinterpret_cast<const uint4*>(wr + 8 * wb + k)),
+                   __ldg(reinterpret_cast<const uint4*>(wi + k)), __ldg(reinterpret_cast<const uint4*>(wi + 8 * wb + k))};
+  };
   for (int i = threadIdx.x; i < wb; i += blockDim.x) {
     const int c = blk * wb + i;
-    sw[i] = a.x_bias[c];
-    sw[wb + i] = a.conv_bias[c];
-    for (int k = 0; k < a.taps; ++k) sw[(2 + k) * wb + i] = a.conv[static_cast<int64_t>(c) * a.taps + k];
+    const float xb = a.x_bias[c], cb = a.conv_bias[c];
+    float sum = 0.f;
+    for (int k = 0; k < a.taps; ++k) {
+      const float w = a.conv[static_cast<int64_t>(c) * a.taps + k];
+      sw[(3 + k) * wb + i] = w;
+      sum += w;
+    }
+    sw[i] = xb;
+    sw[wb + i] = cb;
+    sw[2 * wb + i] = fmaf(sum, xb, cb);
   }
-  __syncthreads();
+  // ---- convolution: four tokens of eight channels at a time ----
   const int groups = wb / 8;
-  for (int i = threadIdx.x; i < groups * kChunk; i += blockDim.x) {
-    const int k8 = i % groups * 8, tok = i / groups, c = blk * wb + k8;
-    uint32_t hi[4] = {0u, 0u, 0u, 0u}, lo[4] = {0u, 0u, 0u, 0u};
-    if (tok < ch.cnt) {
-      float xb[8], acc[8];
-      load8(sw + k8, xb);
-      load8(sw + wb + k8, acc);
-      for (int k = 0; k < a.taps; ++k) {
-        const int p = start + ch.t0 + tok - (a.taps - 1) + k;
-        if (p < 0) continue;
-        float v[8], w[8];
-        load8(sw + (2 + k) * wb + k8, w);
-        if (p >= start) {
-          Vec16<B>::load(x + static_cast<int64_t>(first + p - start) * a.ldx + c, v);
+  auto put = [&](int tok, int k8, const float (&v)[8]) {
+    uint32_t hi[4], lo[4];
 #pragma unroll
-          for (int j = 0; j < 8; ++j) v[j] += xb[j];
+    for (int j = 0; j < 4; ++j) {
+      hi[j] = pack_bf16x2(v[2 * j], v[2 * j + 1]);
+      const float2 h = unpack_bf16x2(hi[j]);
+      lo[j] = pack_bf16x2(v[2 * j] - h.x, v[2 * j + 1] - h.y);
+    }
+    const int at = staged_row(tok, ldu) + k8;
+    *reinterpret_cast<uint4*>(su + at) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    *reinterpret_cast<uint4*>(sl + at) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+  };
+  const int items = groups * (kChunk / kStripTok);
+  uint4 raw[7];   // inputs of tokens -3 .. 3 of this thread's first strip, loaded ahead of the barrier
+  auto fetch = [&](int i) {
+    const int k8 = i % groups * 8, t0 = i / groups * kStripTok;
+    const B* xr = x + static_cast<int64_t>(first + ch.t0) * a.ldx + blk * wb + k8;
+#pragma unroll
+    for (int k = 0; k < 7; ++k) {
+      const int r = t0 - 3 + k;
+      raw[k] = r > t0 - a.taps && r < ch.cnt && ch.t0 + r >= 0 ? *reinterpret_cast<const uint4*>(xr + static_cast<int64_t>(r) * a.ldx) : zero;
+    }
+  };
+  if (threadIdx.x < items) fetch(threadIdx.x);
+  __syncthreads();
+  for (int i = threadIdx.x; i < items; i += blockDim.x) {
+    if (i != threadIdx.x) fetch(i);
+    const int k8 = i % groups * 8, t0 = i / groups * kStripTok, c = blk * wb + k8;
+    if (a.taps <= 4 && ch.t0 + t0 >= a.taps - 1) {     // every input lies in this portion
+      float w[4][8], cb[8];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const int kk = k - (4 - a.taps);
+        if (kk >= 0) {
+          load8(sw + (3 + kk) * wb + k8, w[k]);
         } else {
-          load8(a.ring + (static_cast<int64_t>(slot) * a.taps + p % a.taps) * a.W + c, v);
-        }
 #pragma unroll
-        for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[j], v[j], acc[j]);
+          for (int j = 0; j < 8; ++j) w[k][j] = 0.f;
+        }
+      }
+      load8(sw + 2 * wb + k8, cb);
+      float v[kStripTok][8];
+#pragma unroll
+      for (int q = 0; q < kStripTok; ++q)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[q][j] = cb[j];
+#pragma unroll
+      for (int k = 0; k < 7; ++k) {
+        const uint32_t u[4] = {raw[k].x, raw[k].y, raw[k].z, raw[k].w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float2 f = unpack_bf16x2(u[j]);
+#pragma unroll
+          for (int q = 0; q < kStripTok; ++q)
+            if (k - q >= 0 && k - q < 4) {
+              v[q][2 * j] = fmaf(w[k - q][2 * j], f.x, v[q][2 * j]);
+              v[q][2 * j + 1] = fmaf(w[k - q][2 * j + 1], f.y, v[q][2 * j + 1]);
+            }
+        }
       }
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        hi[j] = pack_bf16x2(acc[2 * j], acc[2 * j + 1]);
-        const float2 h = unpack_bf16x2(hi[j]);
-        lo[j] = pack_bf16x2(acc[2 * j] - h.x, acc[2 * j + 1] - h.y);
+      for (int q = 0; q < kStripTok; ++q) put(t0 + q, k8, v[q]);
+    } else {
+      for (int q = 0; q < kStripTok; ++q) {
+        float acc[8], xb[8];
+        load8(sw + wb + k8, acc);
+        load8(sw + k8, xb);
+        for (int k = 0; k < a.taps; ++k) {
+          const int p = start + ch.t0 + min(t0 + q, ch.cnt - 1) - (a.taps - 1) + k;
+          if (p < 0) continue;
+          float v[8], w[8];
+          load8(sw + (3 + k) * wb + k8, w);
+          if (p >= start) {
+            Vec16<B>::load(x + static_cast<int64_t>(first + p - start) * a.ldx + c, v);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] += xb[j];
+          } else {
+            load8(a.ring + (static_cast<int64_t>(slot) * a.taps + p % a.taps) * a.W + c, v);
+          }
+#pragma unroll
+          for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[j], v[j], acc[j]);
+        }
+        put(t0 + q, k8, acc);
       }
     }
-    *reinterpret_cast<uint4*>(su + tok * ldu + k8) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-    *reinterpret_cast<uint4*>(sl + tok * ldu + k8) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
   }
-  for (int i = threadIdx.x; i < kChunk * ((ldu - wb) / 8); i += blockDim.x) {   // the contraction's tail
-    const int per = (ldu - wb) / 8;
-    *reinterpret_cast<uint4*>(su + (i / per) * ldu + wb + (i % per) * 8) = make_uint4(0u, 0u, 0u, 0u);
-    *reinterpret_cast<uint4*>(sl + (i / per) * ldu + wb + (i % per) * 8) = make_uint4(0u, 0u, 0u, 0u);
+  const int tail = (ldu - wb) / 8;   // the contraction's tail
+  for (int i = threadIdx.x; i < kChunk * tail; i += blockDim.x) {
+    const int at = staged_row(i / tail, ldu) + wb + (i % tail) * 8;
+    *reinterpret_cast<uint4*>(su + at) = zero;
+    *reinterpret_cast<uint4*>(sl + at) = zero;
   }
+  Weights next = weights(0);
   __syncthreads();
+  if (warp * 16 >= cc) return;
   // ---- gates ----
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3, cw = c0 + warp * 16;
-  if (warp * 16 < cc) {
-    float r[8][4], v[8][4];
+  float r[8][4], v[8][4];
+#pragma unroll
+  for (int n = 0; n < 8; ++n)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) r[n][j] = v[n][j] = 0.f;
+  const int ub = staged_row((g >> 1) * 16 + (g & 1), ldu);
+  for (int kb = 0; kb < wb; kb += 32) {
+    const Weights w = next;
+    if (kb + 32 < wb) next = weights(kb + 32);
+#pragma unroll
+    for (int part = 0; part < 2; ++part) {
+      const B* u0 = (part == 0 ? su : sl) + ub + kb + t * 8;
+#pragma unroll
+      for (int n = 0; n < 8; ++n) {
+        const uint4 u = *reinterpret_cast<const uint4*>(u0 + 2 * n * ldu);
+        mma_bf16_16816(r[n], w.r0.x, w.r1.x, w.r0.y, w.r1.y, u.x, u.y);
+        mma_bf16_16816(v[n], w.i0.x, w.i1.x, w.i0.y, w.i1.y, u.x, u.y);
+        mma_bf16_16816(r[n], w.r0.z, w.r1.z, w.r0.w, w.r1.w, u.z, u.w);
+        mma_bf16_16816(v[n], w.i0.z, w.i1.z, w.i0.w, w.i1.w, u.z, u.w);
+      }
+    }
+  }
+  // ---- decays and inputs, scan: element j of tile n is channel g + 8 (j / 2), token 16 t + 2 n + j % 2 ----
+  const int live = ch.cnt - 16 * t;   // tokens of this lane
+  float2* sp = steps + static_cast<int64_t>(first + ch.t0 + 16 * t) * a.W;
+  const int ut = staged_row(16 * t, ldu);
+#pragma unroll
+  for (int h = 0; h < 2; ++h) {
+    const int cb = cw + g + 8 * h, c = blk * wb + cb;
+    const float br = a.gates_bias[(blk * 2) * wb + cb], bi = a.gates_bias[(blk * 2 + 1) * wb + cb], dec = a.decay[c];
+    float P = 1.f, Q = 0.f;
 #pragma unroll
     for (int n = 0; n < 8; ++n)
 #pragma unroll
-      for (int j = 0; j < 4; ++j) r[n][j] = v[n][j] = 0.f;
-    const B* wr = static_cast<const B*>(a.gates) + (static_cast<int64_t>(blk) * 2 * wb + cw + g) * wb;
-    const B* wi = wr + static_cast<int64_t>(wb) * wb;
-    const B* ub = su + ((g >> 1) * 16 + (g & 1)) * ldu;
-    const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
-    for (int kb = 0; kb < wb; kb += 32) {
-      const int k = kb + t * 8;
-      const bool in = k < wb;
-      const uint4 r0 = in ? __ldg(reinterpret_cast<const uint4*>(wr + k)) : zero, r1 = in ? __ldg(reinterpret_cast<const uint4*>(wr + 8 * wb + k)) : zero;
-      const uint4 i0 = in ? __ldg(reinterpret_cast<const uint4*>(wi + k)) : zero, i1 = in ? __ldg(reinterpret_cast<const uint4*>(wi + 8 * wb + k)) : zero;
+      for (int e = 0; e < 2; ++e) {
+        const int j = 2 * n + e;
+        float al, om;
+        decay_pair(dec * sigmoid_approx(r[n][2 * h + e] + br), al, om);
+        const float u = __bfloat162float(su[ut + j * ldu + cb]) + __bfloat162float(sl[ut + j * ldu + cb]);
+        float in = sqrt_approx(om) * sigmoid_approx(v[n][2 * h + e] + bi) * u;
+        if (j >= live) { al = 1.f; in = 0.f; }
+        P *= al;
+        Q = fmaf(al, Q, in);
+        r[n][2 * h + e] = P;       // compositions from the lane's first token on
+        v[n][2 * h + e] = Q;
+      }
 #pragma unroll
-      for (int n = 0; n < 8; ++n) {
-#pragma unroll
-        for (int part = 0; part < 2; ++part) {
-          const uint4 u = *reinterpret_cast<const uint4*>(ub + (part * kChunk + 2 * n) * ldu + k);
-          mma_16816(r[n], r0.x, r1.x, r0.y, r1.y, u.x, u.y);
-          mma_16816(v[n], i0.x, i1.x, i0.y, i1.y, u.x, u.y);
-          mma_16816(r[n], r0.z, r1.z, r0.w, r1.w, u.z, u.w);
-          mma_16816(v[n], i0.z, i1.z, i0.w, i1.w, u.z, u.w);
-        }
+    for (int o = 1; o < 4; o <<= 1) {
+      const float Po = __shfl_up_sync(0xffffffffu, P, o, 4), Qo = __shfl_up_sync(0xffffffffu, Q, o, 4);
+      if (t >= o) {
+        Q = fmaf(P, Qo, Q);
+        P *= Po;
       }
     }
-    // ---- decays and inputs, scan: element j of tile n is channel g + 8 (j / 2), token 16 t + 2 n + j % 2 ----
+    float Pe = __shfl_up_sync(0xffffffffu, P, 1, 4), Qe = __shfl_up_sync(0xffffffffu, Q, 1, 4);
+    if (t == 0) { Pe = 1.f; Qe = 0.f; }
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int cb = cw + g + 8 * h, c = blk * wb + cb;
-      const float br = a.gates_bias[(blk * 2) * wb + cb], bi = a.gates_bias[(blk * 2 + 1) * wb + cb], dec = a.decay[c];
-      float P = 1.f, Q = 0.f;
+    for (int n = 0; n < 8; ++n)
 #pragma unroll
-      for (int n = 0; n < 8; ++n)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int tok = 16 * t + 2 * n + e;
-          const float la = -dec * fast_sigmoid(r[n][2 * h + e] + br);
-          float al = expf(la);
-          const float om = one_minus_exp(-2.f * la, al);
-          float in = sqrtf(om) * fast_sigmoid(v[n][2 * h + e] + bi) * (__bfloat162float(su[tok * ldu + cb]) + __bfloat162float(sl[tok * ldu + cb]));
-          if (tok >= ch.cnt) { al = 1.f; in = 0.f; }
-          r[n][2 * h + e] = al;
-          v[n][2 * h + e] = in;
-          P *= al;
-          Q = fmaf(al, Q, in);
-        }
-#pragma unroll
-      for (int o = 1; o < 4; o <<= 1) {
-        const float Po = __shfl_up_sync(0xffffffffu, P, o, 4), Qo = __shfl_up_sync(0xffffffffu, Q, o, 4);
-        if (t >= o) {
-          Q = fmaf(P, Qo, Q);
-          P *= Po;
-        }
-      }
-      const int64_t at = static_cast<int64_t>(blockIdx.x) * a.W + c;
-      if constexpr (!kFinal) {
-        if (t == 3) totals[at] = make_float2(P, Q);
-      } else {
-        const float Pe = __shfl_up_sync(0xffffffffu, P, 1, 4), Qe = __shfl_up_sync(0xffffffffu, Q, 1, 4), S0 = starts[at];
-        float S = t > 0 ? fmaf(Pe, S0, Qe) : S0;
-        int col = warp * 16 + g + 8 * h + 8 * t;   // columns of a row turn by 8 every 16 tokens: the lanes hit different banks
-        if (col >= cc) col -= cc;
-        if (col >= cc) col -= cc;
-#pragma unroll
-        for (int n = 0; n < 8; ++n)
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            S = fmaf(r[n][2 * h + e], S, v[n][2 * h + e]);
-            sS[(16 * t + 2 * n + e) * cc + col] = S;
-          }
-      }
-    }
-  }
-  if constexpr (kFinal) {
-    __syncthreads();
-    // ---- output gate ----
-    const int per = cc / 8;
-    for (int i = threadIdx.x; i < ch.cnt * per; i += blockDim.x) {
-      const int tok = i / per, c8 = i % per * 8, c = blk * wb + c0 + c8;
-      const int64_t n = first + ch.t0 + tok;
-      int col = c8 + 8 * (tok >> 4);
-      if (col >= cc) col -= cc;
-      if (col >= cc) col -= cc;
-      const float4 s0 = *reinterpret_cast<const float4*>(sS + tok * cc + col), s1 = *reinterpret_cast<const float4*>(sS + tok * cc + col + 4);
-      const float S[8] = {s0.x, s0.y, s0.z, s0.w, s1.x, s1.y, s1.z, s1.w};
-      float y[8];
-      Vec16<B>::load(static_cast<const B*>(a.y) + n * a.ldy + c, y);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        const float z = y[j] + a.y_bias[c + j];
-        // z (1 + tanh(w)) / 2 = z / (1 + exp(-2 w))
-        const float w2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
-        y[j] = a.scale * S[j] * z * fast_sigmoid(w2);
-      }
-      *reinterpret_cast<uint4*>(static_cast<B*>(a.out) + n * a.ldo + c) =
-          make_uint4(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]), pack_bf16x2(y[4], y[5]), pack_bf16x2(y[6], y[7]));
-    }
+      for (int e = 0; e < 2; ++e)
+        if (2 * n + e < live)
+          sp[static_cast<int64_t>(2 * n + e) * a.W + c] = make_float2(r[n][2 * h + e] * Pe, fmaf(r[n][2 * h + e], Qe, v[n][2 * h + e]));
+    if (t == 3) totals[static_cast<int64_t>(blockIdx.x) * a.W + c] = make_float2(P, Q);
   }
 }
 
@@ -374,42 +411,83 @@ lru_prefix_kernel(const SeqBatch sb, const LruArgs a, const float2* __restrict__
   const int n = (sb.cu[b + 1] - sb.cu[b] + kChunk - 1) / kChunk;
   float* sp = a.state + static_cast<int64_t>(sb.ids[b]) * a.W + c;
   float S = sb.start[b] > 0 ? *sp : 0.f;
-  constexpr int kAhead = 16;
-  for (int i0 = 0; i0 < n; i0 += kAhead) {
+  const float2* src = totals + tile * a.W + c;
+  float* dst = starts + tile * a.W + c;
+  constexpr int kAhead = 32;
+  int i = 0;
+  for (; i + kAhead <= n; i += kAhead) {
     float2 v[kAhead];
 #pragma unroll
-    for (int j = 0; j < kAhead; ++j) v[j] = totals[(tile + min(i0 + j, n - 1)) * a.W + c];
+    for (int j = 0; j < kAhead; ++j) v[j] = __ldcg(src + static_cast<int64_t>(i + j) * a.W);
 #pragma unroll
     for (int j = 0; j < kAhead; ++j) {
-      if (i0 + j >= n) break;
-      starts[(tile + i0 + j) * a.W + c] = S;
+      dst[static_cast<int64_t>(i + j) * a.W] = S;
       S = fmaf(v[j].x, S, v[j].y);
     }
   }
+  for (; i < n; ++i) {
+    const float2 v = __ldcg(src + static_cast<int64_t>(i) * a.W);
+    dst[static_cast<int64_t>(i) * a.W] = S;
+    S = fmaf(v.x, S, v.y);
+  }
   *sp = S;
+}
+
+// Outputs: S = factor * start + offset per token and channel, eight channels per thread; a block per 16 tokens of a chunk.
+__global__ void __launch_bounds__(256)
+lru_output_kernel(const SeqBatch sb, const LruArgs a, const float2* __restrict__ steps, const float* __restrict__ starts) {
+  using B = __nv_bfloat16;
+  const ChunkOf ch = chunk_of(sb, blockIdx.x);
+  if (ch.b < 0) return;
+  const int c = (blockIdx.z * 32 + (threadIdx.x & 31)) * 8;
+  if (c >= a.W) return;
+  float S0[8], yb[8];
+  load8(starts + static_cast<int64_t>(blockIdx.x) * a.W + c, S0);
+  load8(a.y_bias + c, yb);
+#pragma unroll
+  for (int q = 0; q < 2; ++q) {
+    const int tok = blockIdx.y * 16 + q * 8 + (threadIdx.x >> 5);
+    if (tok >= ch.cnt) return;
+    const int64_t n = sb.cu[ch.b] + ch.t0 + tok;
+    const float4* p = reinterpret_cast<const float4*>(steps + n * a.W + c);
+    float y[8];
+    Vec16<B>::load(static_cast<const B*>(a.y) + n * a.ldy + c, y);
+#pragma unroll
+    for (int j = 0; j < 8; j += 2) {
+      const float4 f = __ldcs(p + j / 2);
+      const float s[2] = {fmaf(f.x, S0[j], f.y), fmaf(f.z, S0[j + 1], f.w)};
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float z = y[j + e] + yb[j + e];
+        // z (1 + tanh(w)) / 2 = z / (1 + exp(-2 w))
+        y[j + e] = a.scale * s[e] * z * sigmoid_approx(1.5957691216057308f * fmaf(0.044715f * z * z, z, z));
+      }
+    }
+    *reinterpret_cast<uint4*>(static_cast<B*>(a.out) + n * a.ldo + c) =
+        make_uint4(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]), pack_bf16x2(y[4], y[5]), pack_bf16x2(y[6], y[7]));
+  }
 }
 
 bool lru_chunks_ok(const LruArgs& a) {
   const int wb = a.W / a.blocks;
   return wb % 16 == 0 && wb <= 512 && a.taps <= 8 && ((a.ldx | a.ldy | a.ldo) & 7) == 0 &&
-         ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.out) |
+         ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.out) | reinterpret_cast<uintptr_t>(a.y_bias) |
            reinterpret_cast<uintptr_t>(a.gates) | reinterpret_cast<uintptr_t>(a.ring)) & 15) == 0;
 }
 
-// scratch: totals [tiles, W] float2, then starts [tiles, W], with tiles = n_tok / 64 + n_seq
+// scratch: steps [n_tok, W] float2, totals [tiles, W] float2, starts [tiles, W], with tiles = n_tok / 64 + n_seq
 cudaError_t lru_chunks_go(const SeqBatch& sb, const LruArgs& a, float* scratch, cudaStream_t st) {
   const int wb = a.W / a.blocks, tiles = sb.n_tok / kChunk + sb.n_seq, threads = min(wb, kSlice) * 2;
-  const int rows = (2 + a.taps) * wb * 4, u = 2 * kChunk * staged_ld(wb) * 2, smem_u = u + rows, smem = u + max(rows, kChunk * min(wb, kSlice) * 4);
-  static int have0 = 0, have1 = 0;
-  cudaError_t e = want_smem(lru_chunk_kernel<false>, smem_u, have0);
-  if (e == cudaSuccess) e = want_smem(lru_chunk_kernel<true>, smem, have1);
+  const int smem = 2 * staged_size(wb) * 2 + (3 + a.taps) * wb * 4;
+  static int have = 0;
+  const cudaError_t e = want_smem(lru_chunk_kernel, smem, have);
   if (e != cudaSuccess) return e;
-  float2* totals = reinterpret_cast<float2*>(scratch);
-  float* starts = scratch + static_cast<int64_t>(tiles) * a.W * 2;
-  const dim3 grid(tiles, a.blocks, (wb + kSlice - 1) / kSlice);
-  lru_chunk_kernel<false><<<grid, threads, smem_u, st>>>(sb, a, totals, nullptr);
+  float2* steps = reinterpret_cast<float2*>(scratch);
+  float2* totals = steps + static_cast<int64_t>(sb.n_tok) * a.W;
+  float* starts = reinterpret_cast<float*>(totals + static_cast<int64_t>(tiles) * a.W);
+  lru_chunk_kernel<<<dim3(tiles, a.blocks, (wb + kSlice - 1) / kSlice), threads, smem, st>>>(sb, a, steps, totals);
   lru_prefix_kernel<<<dim3((a.W + 63) / 64, sb.n_seq), 64, 0, st>>>(sb, a, totals, starts);
-  lru_chunk_kernel<true><<<grid, threads, smem, st>>>(sb, a, nullptr, starts);
+  lru_output_kernel<<<dim3(tiles, kChunk / 16, (a.W + 255) / 256), 256, 0, st>>>(sb, a, steps, starts);
   return lru_ring_go<__nv_bfloat16>(sb, a, st);
 }
 
@@ -430,7 +508,7 @@ cudaError_t lru_t(const SeqBatch& sb, const LruArgs& a, float* scratch, cudaStre
 
 int64_t gated_lru_scratch(bool f32, const SeqBatch& sb, const LruArgs& a) {
   const int64_t tiles = sb.n_tok / kChunk + sb.n_seq;
-  return !f32 && lru_chunks_ok(a) ? 3 * tiles * a.W : 2 * static_cast<int64_t>(sb.n_tok) * a.W;
+  return (2 * static_cast<int64_t>(sb.n_tok) + (!f32 && lru_chunks_ok(a) ? 3 * tiles : 0)) * a.W;
 }
 
 cudaError_t launch_gated_lru(bool f32, const SeqBatch& sb, const LruArgs& a, float* scratch, cudaStream_t st) {

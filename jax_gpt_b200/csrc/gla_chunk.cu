@@ -45,9 +45,7 @@ __device__ __forceinline__ Chunk chunk_at(const SeqBatch& sb, int tile) {
 }
 
 __device__ __forceinline__ void mma_16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+  mma_bf16_16816(d, a[0], a[1], a[2], a[3], b0, b1);
 }
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -69,26 +67,28 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
   const float2 h = unpack_bf16x2(hi);
   lo = pack_bf16x2(x - h.x, y - h.y);
 }
-// log sigmoid(z)
-__device__ __forceinline__ float log_sigmoid_fast(float z) {
-  const float e = __expf(-fabsf(z));
-  const float l = e < 0.03f ? e * (1.f - e * (0.5f - e * (1.f / 3 - e * 0.25f))) : __logf(1.f + e);
-  return fminf(z, 0.f) - l;
+// log2 sigmoid(z), to fp32 rounding of the logarithm also where the sigmoid is close to 1
+__device__ __forceinline__ float log2_sigmoid(float z) {
+  const float e = ex2_approx(-kLog2e * fabsf(z));
+  const float l = e < 0.03f ? kLog2e * e * (1.f - e * (0.5f - e * (1.f / 3 - e * 0.25f))) : lg2_approx(1.f + e);
+  return fmaf(kLog2e, fminf(z, 0.f), -l);
 }
 
 // ---- decays, scaled operands, A ------------------------------------------------------------------------------------------
-__host__ __device__ __forceinline__ int low_ld(int R) { return (R + 3) / 4 * 4; }
+// Sums of log alpha are kept in units of log 2 and run within 16 tokens, so that neighbours' differences stay exact however far the
+// chunk has decayed; [kC][N + 8] with rows turned by 8 words every 16 tokens. T(m) below is the sum of all of block m.
+__host__ __device__ __forceinline__ int low_ld(int R) { return (R + 15) / 16 * 16 + 8; }
 __host__ __device__ __forceinline__ int prep_smem(int N, int R) {
-  return kC * (N + 8) * 4 + 2 * kC * (N + 8) * 2 + low_ld(R) * (kC + N) * 4;
+  return (kC * (N + 8) + kC / 16 * 8) * 4 + 2 * kC * (N + 8) * 2 + kC * low_ld(R) * 2;
 }
 
-// two elements of an operand scaled by exp(dir (F - ref)), split
-__device__ __forceinline__ void scaled2(const Bf* x, const float* F, const float* ref, float dir, uint32_t& hi, uint32_t& lo) {
-  const float2 v = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x)), f = *reinterpret_cast<const float2*>(F), r = *reinterpret_cast<const float2*>(ref);
-  split2(v.x * __expf(dir * (f.x - r.x)), v.y * __expf(dir * (f.y - r.y)), hi, lo);
+// two elements of an operand scaled by 2^(dir (F - ref)), split
+__device__ __forceinline__ void scaled2(const Bf* x, const float* F, const float2& r, float dir, uint32_t& hi, uint32_t& lo) {
+  const float2 v = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x)), f = *reinterpret_cast<const float2*>(F);
+  split2(v.x * ex2_approx(dir * (f.x - r.x)), v.y * ex2_approx(dir * (f.y - r.y)), hi, lo);
 }
 
-__global__ void __launch_bounds__(kPrepThreads)
+__global__ void __launch_bounds__(kPrepThreads, 2)
 gla_prep_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const LinGates gt, const LinShape s, unsigned char* __restrict__ images) {
   extern __shared__ __align__(16) unsigned char smem[];
   const Chunk ch = chunk_at(sb, blockIdx.x);
@@ -96,92 +96,99 @@ gla_prep_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const
   const int N = s.N, h = blockIdx.y, R = gt.R, ldl = low_ld(R), ldn = N + 8;
   const Image im(N);
   unsigned char* img = images + (static_cast<int64_t>(blockIdx.x) * s.H + h) * im.bytes();
-  float* sF = reinterpret_cast<float*>(smem);              // [kC][ldn]
-  Bf* sQ = reinterpret_cast<Bf*>(sF + kC * ldn);           // [kC][ldn]
-  Bf* sK = sQ + kC * ldn;                                  // [kC][ldn]
-  float* sL = reinterpret_cast<float*>(sK + kC * ldn);     // [kC][ldl] low-rank rows
-  float* sW = sL + kC * ldl;                               // [ldl][N]
+  float* sF = reinterpret_cast<float*>(smem);
+  Bf* sQ = reinterpret_cast<Bf*>(sF + kC * ldn + kC / 16 * 8);   // [kC][ldn]
+  Bf* sK = sQ + kC * ldn;                                        // [kC][ldn]
+  Bf* sL = sK + kC * ldn;                                        // [kC][ldl] low-rank rows
+  auto row_of = [&](int tok) { return tok * ldn + (tok >> 4) * 8; };
   const int64_t row0 = sb.cu[ch.b] + ch.t0;
-  const int tid = threadIdx.x, chunks = N / 8;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3, chunks = N / 8;
+  const int cpad = ldl - 8;
+  for (int i = tid; i < kC * cpad; i += kPrepThreads) {
+    const int k = i / cpad, r = i % cpad;
+    sL[k * ldl + r] = k < ch.cnt && r < R ? static_cast<const Bf*>(gt.low)[(row0 + k) * gt.ld_low + r] : __float2bfloat16(0.f);
+  }
   for (int i = tid; i < kC * chunks; i += kPrepThreads) {
-    const int t = i / chunks, c = i % chunks * 8;
-    uint4 q = make_uint4(0u, 0u, 0u, 0u), k = q;
-    if (t < ch.cnt) {
-      const Bf* row = qkv + (row0 + t) * ld + h * N + c;
-      q = *reinterpret_cast<const uint4*>(row);
-      k = *reinterpret_cast<const uint4*>(row + s.H * N);
-    }
-    *reinterpret_cast<uint4*>(sQ + t * ldn + c) = q;
-    *reinterpret_cast<uint4*>(sK + t * ldn + c) = k;
+    const int k = i / chunks, c = i % chunks * 8;
+    const Bf* row = qkv + (row0 + k) * ld + h * N + c;
+    cp16(sQ + k * ldn + c, k < ch.cnt ? row : qkv, k < ch.cnt);
+    cp16(sK + k * ldn + c, k < ch.cnt ? row + s.H * N : qkv, k < ch.cnt);
   }
-  for (int i = tid; i < kC * ldl; i += kPrepThreads) {
-    const int t = i / ldl, r = i % ldl;
-    sL[i] = t < ch.cnt && r < R ? ldf(static_cast<const Bf*>(gt.low) + (row0 + t) * gt.ld_low + r) : 0.f;
-  }
-  for (int i = tid; i < ldl * N; i += kPrepThreads) {
-    const int n = i / ldl, r = i % ldl;
-    sW[r * N + n] = r < R ? ldf(static_cast<const Bf*>(gt.w2) + (static_cast<int64_t>(h) * N + n) * R + r) : 0.f;
-  }
+  cp_commit();
   __syncthreads();
-  // ---- running sums of log alpha: a thread per channel and run of tokens ----
-  int groups = 8;
-  while (groups > 1 && groups * N > kPrepThreads) groups >>= 1;
-  const int run = kC / groups, n = tid % N, tg = tid / N;
-  if (tg < groups) {
-    const float b2 = gt.bias2[h * N + n];
-    float F = 0.f;
-    for (int t0 = tg * run; t0 < (tg + 1) * run; t0 += 8) {
-      float z[8];
+  // ---- running sums of log alpha: a warp per 16 channels (rows of the product w2 low^T) and all tokens; column g of tile m is token
+  // 16 (g / 2) + 2 m + g % 2, which gives a lane 16 consecutive tokens of its two channels ----
+  if (warp * 16 < N) {
+    float z[8][4];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) z[j] = b2;
-      for (int r = 0; r < ldl; r += 4) {
-        const float w0 = sW[r * N + n], w1 = sW[(r + 1) * N + n], w2 = sW[(r + 2) * N + n], w3 = sW[(r + 3) * N + n];
+    for (int m = 0; m < 8; ++m)
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          const float4 x = *reinterpret_cast<const float4*>(sL + (t0 + j) * ldl + r);
-          z[j] = fmaf(x.x, w0, fmaf(x.y, w1, fmaf(x.z, w2, fmaf(x.w, w3, z[j]))));
+      for (int e = 0; e < 4; ++e) z[m][e] = gt.bias2[h * N + warp * 16 + g + 8 * (e / 2)];
+    const Bf* w = static_cast<const Bf*>(gt.w2) + (static_cast<int64_t>(h) * N + warp * 16 + g) * R;
+    auto pair = [&](const Bf* p, int r) {
+      const unsigned short* u = reinterpret_cast<const unsigned short*>(p);
+      return (r < R ? static_cast<uint32_t>(u[r]) : 0u) | (r + 1 < R ? static_cast<uint32_t>(u[r + 1]) << 16 : 0u);
+    };
+    for (int k = 0; k < cpad; k += 16) {
+      const int r = k + 2 * t;
+      const uint32_t a0 = pair(w, r), a1 = pair(w + 8 * R, r), a2 = pair(w, r + 8), a3 = pair(w + 8 * R, r + 8);
+      const Bf* l = sL + ((g >> 1) * 16 + (g & 1)) * ldl + r;
+#pragma unroll
+      for (int m = 0; m < 8; ++m)
+        mma_bf16_16816(z[m], a0, a1, a2, a3, *reinterpret_cast<const uint32_t*>(l + 2 * m * ldl), *reinterpret_cast<const uint32_t*>(l + 2 * m * ldl + 8));
+    }
+    const int live = ch.cnt - 16 * t;
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      float F = 0.f;
+#pragma unroll
+      for (int m = 0; m < 8; ++m)
+#pragma unroll
+        for (int p = 0; p < 2; ++p) {
+          if (2 * m + p < live) F = fmaf(log2_sigmoid(z[m][2 * e + p]), gt.inv_tau, F);
+          z[m][2 * e + p] = F;
         }
-      }
+      float* f = sF + row_of(16 * t) + warp * 16 + g + 8 * e;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        if (t0 + j < ch.cnt) F = fmaf(log_sigmoid_fast(z[j]), gt.inv_tau, F);
-        sF[(t0 + j) * ldn + n] = F;
-      }
+      for (int m = 0; m < 8; ++m)
+#pragma unroll
+        for (int p = 0; p < 2; ++p) f[(2 * m + p) * ldn] = z[m][2 * e + p];
     }
   }
+  cp_wait_all();
   __syncthreads();
-  if (groups > 1) {
-    float off = 0.f;
-    if (tg < groups)
-      for (int i = 0; i < tg; ++i) off += sF[((i + 1) * run - 1) * ldn + n];
-    __syncthreads();
-    if (tg < groups && tg > 0)
-      for (int t = tg * run; t < (tg + 1) * run; ++t) sF[t * ldn + n] += off;
-    __syncthreads();
-  }
   // ---- scaled queries and keys ----
-  const float* end = sF + (kC - 1) * ldn;
+  auto total = [&](int m, int c) { return *reinterpret_cast<const float2*>(sF + row_of(m * kSub + kSub - 1) + c); };   // T(m)
   for (int i = tid; i < kC * chunks; i += kPrepThreads) {
-    const int t = i / chunks, c = i % chunks * 8;
-    float q[8], k[8];
-    Vec16<Bf>::load(sQ + t * ldn + c, q);
-    Vec16<Bf>::load(sK + t * ldn + c, k);
+    const int k = i / chunks, c = i % chunks * 8, own = k / kSub;
+    const uint4 q4 = *reinterpret_cast<const uint4*>(sQ + k * ldn + c), k4 = *reinterpret_cast<const uint4*>(sK + k * ldn + c);
+    const uint32_t qw[4] = {q4.x, q4.y, q4.z, q4.w}, kw[4] = {k4.x, k4.y, k4.z, k4.w};
+    const float* f = sF + row_of(k) + c;
     uint32_t qh[4], ql[4], kh[4], kl[4];
 #pragma unroll
-    for (int j = 0; j < 8; j += 2) {
-      const float f0 = sF[t * ldn + c + j], f1 = sF[t * ldn + c + j + 1];
-      split2(q[j] * s.q_scale * __expf(f0), q[j + 1] * s.q_scale * __expf(f1), qh[j / 2], ql[j / 2]);
-      split2(k[j] * __expf(end[c + j] - f0), k[j + 1] * __expf(end[c + j + 1] - f1), kh[j / 2], kl[j / 2]);
+    for (int j = 0; j < 4; ++j) {
+      const float2 F = *reinterpret_cast<const float2*>(f + 2 * j);
+      float2 from = F, to = make_float2(-F.x, -F.y);   // from the chunk's start, to its end
+#pragma unroll
+      for (int m = 0; m < kC / kSub; ++m) {
+        const float2 T = total(m, c + 2 * j);
+        if (m < own) { from.x += T.x; from.y += T.y; }
+        else { to.x += T.x; to.y += T.y; }
+      }
+      const float2 q = unpack_bf16x2(qw[j]), kk = unpack_bf16x2(kw[j]);
+      split2(q.x * s.q_scale * ex2_approx(from.x), q.y * s.q_scale * ex2_approx(from.y), qh[j], ql[j]);
+      split2(kk.x * ex2_approx(to.x), kk.y * ex2_approx(to.y), kh[j], kl[j]);
     }
-    unsigned char* d = img + (t * ldn + c) * 2;
+    unsigned char* d = img + (k * ldn + c) * 2;
     *reinterpret_cast<uint4*>(d) = make_uint4(qh[0], qh[1], qh[2], qh[3]);
     *reinterpret_cast<uint4*>(d + im.rows()) = make_uint4(ql[0], ql[1], ql[2], ql[3]);
     *reinterpret_cast<uint4*>(d + 2 * im.rows()) = make_uint4(kh[0], kh[1], kh[2], kh[3]);
     *reinterpret_cast<uint4*>(d + 3 * im.rows()) = make_uint4(kl[0], kl[1], kl[2], kl[3]);
   }
-  for (int i = tid; i < N; i += kPrepThreads) reinterpret_cast<float*>(img + im.tiles())[i] = expf(end[i]);
+  for (int i = tid; i < N; i += kPrepThreads)
+    reinterpret_cast<float*>(img + im.tiles())[i] =
+        exp2f((sF[row_of(15) + i] + sF[row_of(31) + i]) + (sF[row_of(47) + i] + sF[row_of(63) + i]));
   // ---- A: a warp per 16 x 16 block, six below the diagonal and four on it ----
-  const int warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   int I, J;
   if (warp < 6) {
     I = warp < 1 ? 1 : warp < 3 ? 2 : 3;
@@ -191,19 +198,17 @@ gla_prep_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const
   }
   const bool diag = I == J;
   Bf *ah = reinterpret_cast<Bf*>(img + im.a()) + I * kSub * kLdA + J * kSub, *al = ah + kC * kLdA;
-  const float* ref = sF + (J * kSub + (diag ? kSub / 2 - 1 : kSub - 1)) * ldn;
+  const float *ref = sF + row_of(J * kSub + (diag ? kSub / 2 - 1 : kSub - 1)), *FI = sF + row_of(I * kSub), *FJ = sF + row_of(J * kSub);
   if (diag) {
     float spread = 0.f;
-    for (int c = lane; c < N; c += 32) spread = fmaxf(spread, fmaxf(sF[I * kSub * ldn + c] - ref[c], ref[c] - sF[(I * kSub + kSub - 1) * ldn + c]));
-    if (warp_max(spread) > 60.f) {   // the factors would leave fp32's range: pair by pair
+    for (int c = lane; c < N; c += 32) spread = fmaxf(spread, fmaxf(FI[c] - ref[c], ref[c] - FI[(kSub - 1) * ldn + c]));
+    if (warp_max(spread) > 80.f) {   // the factors would leave fp32's range: pair by pair
       for (int i = 0; i < kSub; ++i)
         for (int j = 0; j < kSub; ++j) {
           float v = 0.f;
           if (j <= i)
-            for (int c = lane; c < N; c += 32) {
-              const int qi = (I * kSub + i) * ldn + c, kj = (I * kSub + j) * ldn + c;
-              v = fmaf(ldf(sQ + qi) * ldf(sK + kj), __expf(sF[qi] - sF[kj]), v);
-            }
+            for (int c = lane; c < N; c += 32)
+              v = fmaf(ldf(sQ + (I * kSub + i) * ldn + c) * ldf(sK + (I * kSub + j) * ldn + c), ex2_approx(FI[i * ldn + c] - FI[j * ldn + c]), v);
           v = warp_sum(v) * s.q_scale;
           if (lane == 0) {
             const Bf hi = __float2bfloat16(v);
@@ -215,16 +220,25 @@ gla_prep_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const
     }
   }
   float acc[2][4] = {};
-  const int i0 = (I * kSub + g) * ldn, j0 = (J * kSub + g) * ldn;
+  const Bf *q0 = sQ + (I * kSub + g) * ldn, *k0 = sK + (J * kSub + g) * ldn;
+  const float *fi = FI + g * ldn, *fj = FJ + g * ldn;
+#pragma unroll 2
   for (int kb = 0; kb < N; kb += 16) {
     uint32_t xh[4], xl[4], yh[4], yl[4];   // queries; keys of the two column tiles
 #pragma unroll
     for (int p = 0; p < 2; ++p) {
       const int c = kb + 2 * t + 8 * p;
+      const float2 rf = *reinterpret_cast<const float2*>(ref + c);
+      float2 rq = diag ? rf : make_float2(0.f, 0.f);   // the blocks between J and I, negative
+      for (int m = J + 1; m < I; ++m) {
+        const float2 T = total(m, c);
+        rq.x -= T.x;
+        rq.y -= T.y;
+      }
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        scaled2(sQ + i0 + r * 8 * ldn + c, sF + i0 + r * 8 * ldn + c, ref + c, 1.f, xh[2 * p + r], xl[2 * p + r]);
-        scaled2(sK + j0 + r * 8 * ldn + c, sF + j0 + r * 8 * ldn + c, ref + c, -1.f, yh[2 * r + p], yl[2 * r + p]);
+        scaled2(q0 + r * 8 * ldn + c, fi + r * 8 * ldn + c, rq, 1.f, xh[2 * p + r], xl[2 * p + r]);
+        scaled2(k0 + r * 8 * ldn + c, fj + r * 8 * ldn + c, rf, -1.f, yh[2 * r + p], yl[2 * r + p]);
       }
     }
 #pragma unroll
@@ -251,11 +265,12 @@ gla_prep_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const
 __host__ __device__ __forceinline__ int stage_bytes(int N) { return Image(N).tiles() + kC * kLdP * 2; }
 __host__ __device__ __forceinline__ int scan_smem(int N) { return 2 * stage_bytes(N) + 2 * 2 * N * kLdP * 2; }
 
+template <int kN>   // key width, 0: any
 __global__ void __launch_bounds__(kScanThreads)
 gla_scan_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const unsigned char* __restrict__ images, float* __restrict__ state,
                 Bf* __restrict__ y, const LinShape s) {
   extern __shared__ __align__(16) unsigned char smem[];
-  const int N = s.N, P = s.P, h = blockIdx.x, p0 = blockIdx.y * kPs, b = blockIdx.z;
+  const int N = kN > 0 ? kN : s.N, P = s.P, h = blockIdx.x, p0 = blockIdx.y * kPs, b = blockIdx.z;
   const Image im(N);
   const int ldn = im.ld, stage = stage_bytes(N);
   Bf* sS = reinterpret_cast<Bf*>(smem + 2 * stage);        // [2 buffers][high, low][N][kLdP]
@@ -327,31 +342,38 @@ gla_scan_kernel(const SeqBatch sb, const Bf* __restrict__ qkv, int64_t ld, const
     const int cnt = min(kC, len - c * kC);
     // ---- outputs ----
     if (mt * 16 < cnt) {
-      float o[2][4] = {};
+      float o[2][4] = {}, o1[2][4] = {}, o2[2][4] = {};   // separate sums: short chains of dependent products
+#pragma unroll
       for (int k = 0; k < N; k += 16) {
         uint32_t xh[4], xl[4], zh[4], zl[4];
         ldsm4(xh, qh + (mt * 16 + r16) * ldn + k + c8);
-        ldsm4(xl, ql + (mt * 16 + r16) * ldn + k + c8);
         ldsm4_t(zh, sh + (k + r16) * kLdP + nh + c8);
+        ldsm4(xl, ql + (mt * 16 + r16) * ldn + k + c8);
         ldsm4_t(zl, sl + (k + r16) * kLdP + nh + c8);
 #pragma unroll
         for (int m = 0; m < 2; ++m) {
           mma_16816(o[m], xh, zh[2 * m], zh[2 * m + 1]);
-          mma_16816(o[m], xh, zl[2 * m], zl[2 * m + 1]);
-          mma_16816(o[m], xl, zh[2 * m], zh[2 * m + 1]);
+          mma_16816(o1[m], xh, zl[2 * m], zl[2 * m + 1]);
+          mma_16816(o2[m], xl, zh[2 * m], zh[2 * m + 1]);
         }
       }
-      for (int k = 0; k <= mt; ++k) {
+#pragma unroll
+      for (int k = 0; k < kC / 16; ++k) {
+        if (k > mt) break;
         uint32_t xh[4], xl[4], z[4];
         ldsm4(xh, ah + (mt * 16 + r16) * kLdA + k * 16 + c8);
         ldsm4(xl, al + (mt * 16 + r16) * kLdA + k * 16 + c8);
         ldsm4_t(z, sv + (k * 16 + r16) * kLdP + nh + c8);
 #pragma unroll
         for (int m = 0; m < 2; ++m) {
-          mma_16816(o[m], xh, z[2 * m], z[2 * m + 1]);
-          mma_16816(o[m], xl, z[2 * m], z[2 * m + 1]);
+          mma_16816(o1[m], xh, z[2 * m], z[2 * m + 1]);
+          mma_16816(o2[m], xl, z[2 * m], z[2 * m + 1]);
         }
       }
+#pragma unroll
+      for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[m][e] += o1[m][e] + o2[m][e];
 #pragma unroll
       for (int m = 0; m < 2; ++m)
 #pragma unroll
@@ -403,14 +425,24 @@ cudaError_t launch_gla_chunked(const SeqBatch& sb, const Bf* qkv, int64_t ld, co
                                void* scratch, cudaStream_t st) {
   if (!gla_chunked_ok(s, ld, g.R) || ((reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(scratch) | reinterpret_cast<uintptr_t>(y)) & 15) != 0)
     return cudaErrorInvalidValue;
-  static int have_prep = 0, have_scan = 0;
+  static int have_prep = 0;
   const int ps = prep_smem(s.N, g.R), ss = scan_smem(s.N);
   cudaError_t e = want_smem(gla_prep_kernel, ps, have_prep);
-  if (e == cudaSuccess) e = want_smem(gla_scan_kernel, ss, have_scan);
   if (e != cudaSuccess) return e;
   unsigned char* img = static_cast<unsigned char*>(scratch);
   gla_prep_kernel<<<dim3(sb.n_tok / kC + sb.n_seq, s.H), kPrepThreads, ps, st>>>(sb, qkv, ld, g, s, img);
-  gla_scan_kernel<<<dim3(s.H, (s.P + kPs - 1) / kPs, sb.n_seq), kScanThreads, ss, st>>>(sb, qkv, ld, img, state, y, s);
+  const dim3 grid(s.H, (s.P + kPs - 1) / kPs, sb.n_seq);
+#define B200_SCAN(N)                                                                             \
+  {                                                                                              \
+    static int have = 0;                                                                         \
+    e = want_smem(gla_scan_kernel<N>, ss, have);                                                 \
+    if (e != cudaSuccess) return e;                                                              \
+    gla_scan_kernel<N><<<grid, kScanThreads, ss, st>>>(sb, qkv, ld, img, state, y, s);           \
+  }
+  if (s.N == 128) B200_SCAN(128)
+  else if (s.N == 64) B200_SCAN(64)
+  else B200_SCAN(0)
+#undef B200_SCAN
   return cudaGetLastError();
 }
 

@@ -342,13 +342,6 @@ void rows_linear_go(bool vec, const T* x, int64_t ldx, const T* w, int64_t ldw, 
 // operand. Every lane loads 16 contiguous bytes of a weight row and of an activation row; the products' k index is
 // permuted the same way on both sides, which leaves the sums unchanged. The warps of a block split the contraction.
 // Bound by the stream of weights: tcgen05 tiles would be 94 % padding here.
-__device__ __forceinline__ void mma_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
-                                          uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-
 template <int MT, int kW, bool kGlu>   // kW warps per block
 __global__ void __launch_bounds__(kW * 32)
 rows_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx, const __nv_bfloat16* __restrict__ w, int64_t ldw,
@@ -392,8 +385,8 @@ rows_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx, const _
       for (int q = 0; q < kMat; ++q)
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
-          mma_16816(acc[q][m], a[q][u].x, c[q][u].x, a[q][u].y, c[q][u].y, b[u][m].x, b[u][m].y);
-          mma_16816(acc[q][m], a[q][u].z, c[q][u].z, a[q][u].w, c[q][u].w, b[u][m].z, b[u][m].w);
+          mma_bf16_16816(acc[q][m], a[q][u].x, c[q][u].x, a[q][u].y, c[q][u].y, b[u][m].x, b[u][m].y);
+          mma_bf16_16816(acc[q][m], a[q][u].z, c[q][u].z, a[q][u].w, c[q][u].w, b[u][m].z, b[u][m].w);
         }
   }
 #pragma unroll
