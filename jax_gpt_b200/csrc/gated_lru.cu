@@ -468,10 +468,128 @@ lru_output_kernel(const SeqBatch sb, const LruArgs a, const float2* __restrict__
   }
 }
 
+// ---- bf16, one token per sequence ----------------------------------------------------------------------------------------
+// Block: 16 channels and up to eight sequences (the columns of the gates' products); its four warps split the contraction. Everything
+// that does not depend on the gates is loaded first.
+__global__ void __launch_bounds__(128)
+lru_step_kernel(const SeqBatch sb, const LruArgs a) {
+  using B = __nv_bfloat16;
+  extern __shared__ __align__(16) unsigned char smem[];
+  __shared__ float red[4][2][32][4];
+  const int wb = a.W / a.blocks, ldu = staged_ld(wb), ch0 = blockIdx.x * 16, blk = ch0 / wb, k0 = ch0 % wb, n0 = blockIdx.y * 8;
+  B* su = reinterpret_cast<B*>(smem);   // [8][ldu] high parts
+  B* sl = su + 8 * ldu;                 // [8][ldu] low parts
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const B* wr = static_cast<const B*>(a.gates) + (static_cast<int64_t>(blk) * 2 * wb + k0 + g) * wb;
+  const B* wi = wr + static_cast<int64_t>(wb) * wb;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  uint4 w[4];
+  auto weights = [&](int kb) {
+    const int k = kb + t * 8;
+    const bool in = k < wb;
+    w[0] = in ? __ldg(reinterpret_cast<const uint4*>(wr + k)) : zero;
+    w[1] = in ? __ldg(reinterpret_cast<const uint4*>(wr + 8 * wb + k)) : zero;
+    w[2] = in ? __ldg(reinterpret_cast<const uint4*>(wi + k)) : zero;
+    w[3] = in ? __ldg(reinterpret_cast<const uint4*>(wi + 8 * wb + k)) : zero;
+  };
+  weights(warp * 32);
+  // this thread's output: channel c of sequence n
+  const int n = n0 + threadIdx.x / 16, kc = k0 + threadIdx.x % 16, c = blk * wb + kc;
+  const bool live = n < sb.n_seq;
+  const int slot = live ? sb.ids[n] : 0, pos = live ? sb.start[n] : 0;
+  float* sp = a.state + static_cast<int64_t>(slot) * a.W + c;
+  const float S0 = live && pos > 0 ? *sp : 0.f;
+  const float yv = live ? ldf(static_cast<const B*>(a.y) + static_cast<int64_t>(n) * a.ldy + c) + a.y_bias[c] : 0.f;
+  const float xv = live ? ldf(static_cast<const B*>(a.x) + static_cast<int64_t>(n) * a.ldx + c) + a.x_bias[c] : 0.f;
+  const float br = a.gates_bias[blk * 2 * wb + kc], bi = a.gates_bias[(blk * 2 + 1) * wb + kc], dec = a.decay[c];
+  for (int i = threadIdx.x; i < 8 * (ldu / 8); i += 128) {
+    const int q = i / (ldu / 8), k8 = i % (ldu / 8) * 8, m = n0 + q, cc = blk * wb + k8;
+    uint32_t hi[4] = {0u, 0u, 0u, 0u}, lo[4] = {0u, 0u, 0u, 0u};
+    if (k8 < wb && m < sb.n_seq) {
+      const int sm = sb.ids[m], pm = sb.start[m];
+      float acc[8], xb[8], v[8];
+      load8(a.conv_bias + cc, acc);
+      load8(a.x_bias + cc, xb);
+      Vec16<B>::load(static_cast<const B*>(a.x) + static_cast<int64_t>(m) * a.ldx + cc, v);
+      const float* cw = a.conv + static_cast<int64_t>(cc) * a.taps;
+      if (a.taps == 4) {
+        float r[3][8];
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) r[k][j] = 0.f;
+          if (pm - 3 + k >= 0) load8(a.ring + (static_cast<int64_t>(sm) * 4 + (pm - 3 + k) % 4) * a.W + cc, r[k]);
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          const float4 f = *reinterpret_cast<const float4*>(cw + 4 * j);
+          acc[j] = fmaf(f.x, r[0][j], fmaf(f.y, r[1][j], fmaf(f.z, r[2][j], fmaf(f.w, v[j] + xb[j], acc[j]))));
+        }
+      } else {
+        for (int k = 0; k + 1 < a.taps; ++k) {
+          const int p = pm - (a.taps - 1) + k;
+          if (p < 0) continue;
+          float r[8];
+          load8(a.ring + (static_cast<int64_t>(sm) * a.taps + p % a.taps) * a.W + cc, r);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) acc[j] = fmaf(cw[j * a.taps + k], r[j], acc[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[j] = fmaf(cw[j * a.taps + a.taps - 1], v[j] + xb[j], acc[j]);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        hi[j] = pack_bf16x2(acc[2 * j], acc[2 * j + 1]);
+        const float2 h = unpack_bf16x2(hi[j]);
+        lo[j] = pack_bf16x2(acc[2 * j] - h.x, acc[2 * j + 1] - h.y);
+      }
+    }
+    *reinterpret_cast<uint4*>(su + q * ldu + k8) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+    *reinterpret_cast<uint4*>(sl + q * ldu + k8) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+  }
+  __syncthreads();
+  float r[4] = {0.f, 0.f, 0.f, 0.f}, v[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int kb = warp * 32; kb < wb; kb += 128) {
+    if (kb != warp * 32) weights(kb);
+#pragma unroll
+    for (int part = 0; part < 2; ++part) {
+      const uint4 u = *reinterpret_cast<const uint4*>((part == 0 ? su : sl) + g * ldu + kb + t * 8);
+      mma_bf16_16816(r, w[0].x, w[1].x, w[0].y, w[1].y, u.x, u.y);
+      mma_bf16_16816(v, w[2].x, w[3].x, w[2].y, w[3].y, u.x, u.y);
+      mma_bf16_16816(r, w[0].z, w[1].z, w[0].w, w[1].w, u.z, u.w);
+      mma_bf16_16816(v, w[2].z, w[3].z, w[2].w, w[3].w, u.z, u.w);
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    red[warp][0][lane][j] = r[j];
+    red[warp][1][lane][j] = v[j];
+  }
+  __syncthreads();
+  if (!live) return;
+  // accumulator j of lane (g, t): channel g + 8 (j / 2), sequence 2 t + j % 2
+  const int q = threadIdx.x / 16, ci = threadIdx.x % 16, src = (ci % 8) * 4 + q / 2, j = (ci / 8) * 2 + q % 2;
+  float zr = br, zi = bi;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    zr += red[k][0][src][j];
+    zi += red[k][1][src][j];
+  }
+  const float u = __bfloat162float(su[q * ldu + kc]) + __bfloat162float(sl[q * ldu + kc]);
+  float al, om;
+  decay_pair(dec * sigmoid_approx(zr), al, om);
+  const float S = fmaf(al, S0, sqrt_approx(om) * sigmoid_approx(zi) * u);
+  *sp = S;
+  a.ring[(static_cast<int64_t>(slot) * a.taps + pos % a.taps) * a.W + c] = xv;   // not a row that the other blocks read
+  const float gelu = yv * sigmoid_approx(1.5957691216057308f * fmaf(0.044715f * yv * yv, yv, yv));
+  stf(static_cast<B*>(a.out) + static_cast<int64_t>(n) * a.ldo + c, a.scale * S * gelu);
+}
+
 bool lru_chunks_ok(const LruArgs& a) {
   const int wb = a.W / a.blocks;
   return wb % 16 == 0 && wb <= 512 && a.taps <= 8 && ((a.ldx | a.ldy | a.ldo) & 7) == 0 &&
          ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.out) | reinterpret_cast<uintptr_t>(a.y_bias) |
+           reinterpret_cast<uintptr_t>(a.x_bias) | reinterpret_cast<uintptr_t>(a.conv) | reinterpret_cast<uintptr_t>(a.conv_bias) |
            reinterpret_cast<uintptr_t>(a.gates) | reinterpret_cast<uintptr_t>(a.ring)) & 15) == 0;
 }
 
@@ -493,10 +611,14 @@ cudaError_t lru_chunks_go(const SeqBatch& sb, const LruArgs& a, float* scratch, 
 
 template <typename T>
 cudaError_t lru_t(const SeqBatch& sb, const LruArgs& a, float* scratch, cudaStream_t st) {
-  if (scratch == nullptr) return lru_gates_go<T, true>(sb, a, nullptr, nullptr, st);
   if constexpr (sizeof(T) == 2) {
-    if (lru_chunks_ok(a)) return lru_chunks_go(sb, a, scratch, st);
+    if (lru_chunks_ok(a)) {
+      if (scratch != nullptr) return lru_chunks_go(sb, a, scratch, st);
+      lru_step_kernel<<<dim3(a.W / 16, (sb.n_seq + 7) / 8), 128, 2 * 8 * staged_ld(a.W / a.blocks) * 2, st>>>(sb, a);
+      return cudaGetLastError();
+    }
   }
+  if (scratch == nullptr) return lru_gates_go<T, true>(sb, a, nullptr, nullptr, st);
   float *log_a = scratch, *inp = scratch + static_cast<int64_t>(sb.n_tok) * a.W;
   const cudaError_t e = lru_gates_go<T, false>(sb, a, log_a, inp, st);
   if (e != cudaSuccess) return e;

@@ -10,7 +10,7 @@ that fits (doubling then bisection on out-of-memory, ``--max-batch`` caps it), t
 Timing is on the device with CUDA events, maximum over ranks (the reference uses host
 perf_counter and means only, scripts/bench_prefill_decode.py:246-264). ``--model`` selects the
 Qwen3.5 hybrid (``--config`` preset), the DeepSeek-V3 shape with its paged latent cache or Vobunex /
-Fovudra on the shared step engine.
+Fovudra / Munazen on the shared step engine.
 Results are printed and written as JSON to ``--out``.
 """
 from __future__ import annotations
@@ -119,7 +119,7 @@ def make_runner(args, device):
             logits, cache = forward(params, nxt[:, None], cfg, cache=cache, is_decode=True, ep_group=ep, tp_group=tp_group)
             return logits[:, -1].argmax(-1), cache
         return prefill, decode, cfg
-    if args.model in ("vobunex", "fovudra"):
+    if args.model in ("vobunex", "fovudra", "munazen"):
         if args.tp > 1 or args.dp > 1 or args.w8a8 or args.fp8:
             raise SystemExit(f"--tp / --dp / --w8a8 / --fp8 do not apply to --model {args.model}")
         from jax_gpt_b200.models.registry import FAMILIES, load_model
@@ -222,7 +222,7 @@ def find_max_batch(prefill, decode, cap):
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--model", default="qwen35", choices=["qwen35", "deepseek_v3", "vobunex", "fovudra"])
+    ap.add_argument("--model", default="qwen35", choices=["qwen35", "deepseek_v3", "vobunex", "fovudra", "munazen"])
     ap.add_argument("--model-dir", default="", help="HF safetensors directory (random weights when empty)")
     ap.add_argument("--scenario", default="1k1k", choices=sorted(SCENARIOS))
     ap.add_argument("--tp", type=int, default=1)

@@ -207,7 +207,7 @@ def test_gated_lru(W, blocks, taps, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
-@pytest.mark.parametrize("W,blocks,taps", [(256, 2, 4), (30, 3, 5), (1024, 8, 4), (24, 24, 1)])
+@pytest.mark.parametrize("W,blocks,taps", [(256, 2, 4), (30, 3, 5), (1024, 8, 4), (24, 24, 1), (96, 2, 3), (1024, 2, 1), (48, 3, 6)])
 @pytest.mark.parametrize("B", [1, 3, 8, 19])
 def test_gated_lru_one_token_steps(W, blocks, taps, B, dtype):
     """Steps from position 0 on against the recurrence over the whole sequence."""
@@ -233,7 +233,7 @@ def test_gated_lru_one_token_steps(W, blocks, taps, B, dtype):
         u = O.causal_conv(D(x[:, b].float() + xb), D(conv), D(cb))
         S, last = O.rglru_recurrence(u, O.sigmoid(O.block_linear(u, D(ra), D(rab))), O.sigmoid(O.block_linear(u, D(ri), D(rib))), D(lam))
         assert rel(torch.stack(got)[:, b], 1.5 * S * O.gelu_tanh(D(y[:, b].float() + yb))) < (4e-3 if dtype == torch.bfloat16 else 2e-6)
-        assert rel(state[slots[b]], last) < 2e-6
+        assert rel(state[slots[b]], last) < (1e-5 if dtype == torch.bfloat16 else 2e-6)
 
 
 # ---- linear attention with a decay per key channel -------------------------------------------------------------------------
