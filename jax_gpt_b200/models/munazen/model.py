@@ -7,7 +7,7 @@ operations pick the form that fits the batch).
 
 Everything between two sublayers (bias, streams, next combination, group norm) is one kernel. Parallel layers: one projection for both
 branches; attention operands and cache row in one kernel, attention on the tcgen05 flash kernel, the paged decode kernel or the any-size
-kernel; the recurrent unit from convolution to gated output; both branches write the row that one output projection reads. Gated linear
+kernel; the recurrent unit from convolution to gated output on a second stream; both branches write the row that one output projection reads. Gated linear
 attention: one projection, the scan, then norm and output gate in one kernel.
 """
 from __future__ import annotations
@@ -24,6 +24,7 @@ from ...ops.gemm import linear_rows
 from ...ops.packed import PackedBatch, embed_bigram, seq_begin
 from ...ops.rope import rope_tables
 from ...ops.streams import Connection, group_norm_rows, poly_norm, stream_norm
+from ...utils.overlap import beside
 from ...utils.profiling import scope
 from ..step_engine import forward_tokens, generate_tokens
 from .config import GatedLinear, MunazenConfig, Parallel
@@ -62,12 +63,14 @@ def parallel_mixer(h, mp, m: Parallel, batch: PackedBatch, cache: HybridPagedCac
     a, W = m.left, m.right.width
     (cq, ck, cv, cx, cy, cg), _ = m.segments()
     y = linear_rows(h, mp["in"])
+    both = torch.empty(h.shape[0], a.heads * a.vdim + W, device=h.device, dtype=h.dtype)
+    lru_done = beside(h.device, lambda: gated_lru(batch, y[:, cx:cx + W], y[:, cy:cy + W], mp["lru"], cache.rings[run], cache.states[run],
+                                                  m.right_scale, both[:, -W:]))
     wide = RKV.flash_widths(batch, h.dtype, h.is_cuda, a.dim, a.vdim)
     q, k, v = RKV.qkv_rotate(batch, y, (cq, ck, cv), mp["qkv_b"], a.heads, a.kv_heads, a.dim, a.vdim, rope[0], rope[1], cache.paged, layer, wide)
     o = RKV.causal_attention(batch, q, k, v, cache.paged, layer, a.kv_heads, a.vdim, a.scale)
-    both = torch.empty(h.shape[0], a.heads * a.vdim + W, device=h.device, dtype=h.dtype)
     RKV.turn_back_gate(batch, o, y[:, cg:cg + a.heads], rope[1], m.left_scale, both[:, :-W])
-    gated_lru(batch, y[:, cx:cx + W], y[:, cy:cy + W], mp["lru"], cache.rings[run], cache.states[run], m.right_scale, both[:, -W:])
+    lru_done()
     return linear_rows(both, mp["o"])
 
 
