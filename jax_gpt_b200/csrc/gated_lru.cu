@@ -35,6 +35,9 @@ __device__ __forceinline__ float conv_at(const LruArgs& a, int first, int start,
   return acc;
 }
 
+// exp(la) S + in as a change of S: decays close to 1 keep their distance from it, whose rounding would add up over a long memory
+__device__ __forceinline__ float decayed(float S, float la, float in) { return S + fmaf(expm1f(la), S, in); }
+
 // ---- gates, any sizes; kStep: the whole unit for one token per sequence ----------------------------------------------------
 constexpr int kLruTok = 8, kLruWarps = 8;
 
@@ -85,7 +88,7 @@ lru_gates_kernel(const SeqBatch sb, const LruArgs a, int per_block, float* __res
     if constexpr (kStep) {
       const int b = sb.tok_seq[n], slot = sb.ids[b];
       float* sp = a.state + static_cast<int64_t>(slot) * a.W + c;
-      const float S = fmaf(expf(la), sb.start[b] > 0 ? *sp : 0.f, in);
+      const float S = decayed(sb.start[b] > 0 ? *sp : 0.f, la, in);
       *sp = S;
       const float y = gelu_f(ldf(static_cast<const T*>(a.y) + static_cast<int64_t>(n) * a.ldy + c) + a.y_bias[c]);
       stf(static_cast<T*>(a.out) + static_cast<int64_t>(n) * a.ldo + c, a.scale * S * y);
@@ -119,7 +122,7 @@ lru_scan_kernel(const SeqBatch sb, const LruArgs a, const float* __restrict__ lo
 #pragma unroll
     for (int j = 0; j < kAhead; ++j) {
       if (n0 + j >= end) break;
-      S = fmaf(expf(la[j]), S, in[j]);
+      S = decayed(S, la[j], in[j]);
       stf(static_cast<T*>(a.out) + static_cast<int64_t>(n0 + j) * a.ldo + c, a.scale * S * gelu_f(y[j] + yb));
     }
   }
@@ -171,11 +174,11 @@ __device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
   const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
   f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
 }
-// a = exp(-x) and 1 - a^2 for x >= 0, both to fp32 rounding also where a is close to 1
-__device__ __forceinline__ void decay_pair(float x, float& a, float& om) {
+// a = exp(-x), d = 1 - a and 1 - a^2 for x >= 0, all to fp32 rounding also where a is close to 1
+__device__ __forceinline__ void decay_pair(float x, float& d, float& a, float& om) {
   const float p = x * (1.f - x * (0.5f - x * (1.f / 6 - x * (1.f / 24 - x * (1.f / 120)))));
   const float e = ex2_approx(-kLog2e * x);
-  const float d = x < 0.125f ? p : 1.f - e;
+  d = x < 0.125f ? p : 1.f - e;
   a = x < 0.125f ? 1.f - p : e;
   om = d * (2.f - d);
 }
@@ -371,8 +374,8 @@ lru_chunk_kernel(const SeqBatch sb, const LruArgs a, float2* __restrict__ steps,
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int j = 2 * n + e;
-        float al, om;
-        decay_pair(dec * sigmoid_approx(r[n][2 * h + e] + br), al, om);
+        float d, al, om;
+        decay_pair(dec * sigmoid_approx(r[n][2 * h + e] + br), d, al, om);
         const float u = __bfloat162float(su[ut + j * ldu + cb]) + __bfloat162float(sl[ut + j * ldu + cb]);
         float in = sqrt_approx(om) * sigmoid_approx(v[n][2 * h + e] + bi) * u;
         if (j >= live) { al = 1.f; in = 0.f; }
@@ -576,9 +579,9 @@ lru_step_kernel(const SeqBatch sb, const LruArgs a) {
     zi += red[k][1][src][j];
   }
   const float u = __bfloat162float(su[q * ldu + kc]) + __bfloat162float(sl[q * ldu + kc]);
-  float al, om;
-  decay_pair(dec * sigmoid_approx(zr), al, om);
-  const float S = fmaf(al, S0, sqrt_approx(om) * sigmoid_approx(zi) * u);
+  float d, al, om;
+  decay_pair(dec * sigmoid_approx(zr), d, al, om);
+  const float S = S0 + fmaf(-d, S0, sqrt_approx(om) * sigmoid_approx(zi) * u);
   *sp = S;
   a.ring[(static_cast<int64_t>(slot) * a.taps + pos % a.taps) * a.W + c] = xv;   // not a row that the other blocks read
   const float gelu = yv * sigmoid_approx(1.5957691216057308f * fmaf(0.044715f * yv * yv, yv, yv));

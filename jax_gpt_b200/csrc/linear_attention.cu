@@ -29,13 +29,13 @@ __device__ __forceinline__ void log_gates(const LinGates& g, int64_t row, int h,
   f = -softplus_f(-soft_cap(p[H + h] + g.bias[H + h], g.cap));
 }
 
-// decay of (row, head, key channel)
+// decay of (row, head, key channel), less 1: S + (decay - 1) S keeps the distance of slow decays from 1
 template <typename T>
 __device__ __forceinline__ float channel_decay(const LinGates& g, int64_t row, int hn) {
   const T *x = static_cast<const T*>(g.low) + row * g.ld_low, *w = static_cast<const T*>(g.w2) + static_cast<int64_t>(hn) * g.R;
   float z = g.bias2[hn];
   for (int r = 0; r < g.R; ++r) z = fmaf(ldf(x + r), ldf(w + r), z);
-  return expf(-softplus_f(-z) * g.inv_tau);
+  return expm1f(-softplus_f(-z) * g.inv_tau);
 }
 
 enum LinKind : int { kFixed = 0, kGatedExp = 1, kChannel = 2 };
@@ -118,7 +118,8 @@ linear_scan_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
       for (int i = 0; i < NS; ++i) {
         const int n = g + i * kScanG;
         if (n < N) {
-          S[i] = fmaf(S[i], kKind == kChannel ? sC[t * N + n] : a, x * sK[t * N + n]);
+          if constexpr (kKind == kChannel) S[i] += fmaf(S[i], sC[t * N + n], x * sK[t * N + n]);
+          else S[i] = fmaf(S[i], a, x * sK[t * N + n]);
           acc = fmaf(S[i], sQ[t * N + n], acc);
           if constexpr (kGated) {
             nn[i] = fmaf(nn[i], a, w * sK[t * N + n]);
@@ -257,7 +258,8 @@ linear_step_kernel(const SeqBatch sb, const T* __restrict__ qkv, int64_t ld, con
         const float kn = sk[n], qn = sq[n], an = kKind == kChannel ? sc[n] : a;
 #pragma unroll
         for (int j = 0; j < V; ++j) {
-          S[i][j] = fmaf(S[i][j], an, dx[j] * kn);
+          if constexpr (kKind == kChannel) S[i][j] += fmaf(S[i][j], an, dx[j] * kn);
+          else S[i][j] = fmaf(S[i][j], an, dx[j] * kn);
           acc[j] = fmaf(S[i][j], qn, acc[j]);
         }
         if constexpr (V == 4) *reinterpret_cast<float4*>(sp) = make_float4(S[i][0], S[i][1], S[i][2], S[i][3]);

@@ -304,6 +304,34 @@ def test_channel_decay_steps_of_any_size(H, N, P, R, dtype):
         assert rel(got[r], want) < (2e-2 if dtype == torch.bfloat16 else 2e-5), r
 
 
+@pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
+def test_slow_decays_do_not_drift(dtype):
+    """Thousands of tokens with decays close to 1: a systematic error of the decay would add up to far more than rounding."""
+    from jax_gpt_b200.ops import linear_attention as LIN
+    from jax_gpt_b200.ops.gated_lru import LruWeights, gated_lru, lru_decay
+    g = torch.Generator().manual_seed(9)
+    n, W = 3000, 64
+    r = lambda *s: torch.randn(*s, generator=g)
+    x, y = (0.1 * r(n, W) + 1).to(dtype), r(n, W).to(dtype)
+    ra, ri, rab, rib, lam = (r(1, W, W) * 0.02).to(dtype), (r(1, W, W) * 0.02).to(dtype), r(1, W), 3 + r(1, W), -9 + 0.3 * r(W)
+    conv, zero = torch.ones(W, 1), torch.zeros(W)
+    dv = lambda t: t.contiguous().to(DEV)
+    w = LruWeights(dv(zero), dv(zero), dv(conv), dv(zero), dv(torch.stack([ra, ri], 1)), dv(torch.stack([rab, rib], 1)), dv(lru_decay(lam)))
+    state, out = torch.zeros(1, W, device=DEV), torch.empty(n, W, dtype=dtype, device=DEV)
+    gated_lru(begin([0], [n], [0]), dv(x), dv(y), w, torch.zeros(1, 1, W, device=DEV), state, 1.0, out)
+    D = lambda t: t.double()
+    _, last = O.rglru_recurrence(D(x), O.sigmoid(O.block_linear(D(x), D(ra), D(rab))), O.sigmoid(O.block_linear(D(x), D(ri), D(rib))), D(lam))
+    assert rel(state[0], last) < 3e-6
+    H, N, P = 1, 16, 16
+    qkv = (0.1 * r(n, H * (2 * N + P)) + 1).to(dtype)
+    low, w2, b2 = r(n, 4).to(dtype), (0.1 * r(H * N, 4)).to(dtype), 4 + r(H * N)
+    S = torch.zeros(1, H, N, P, device=DEV)
+    LIN.linear_scan(begin([0], [n], [0]), dv(qkv), S, channels=LIN.ChannelDecay(dv(low), dv(w2), dv(b2), 20.0))
+    q, k, v = [t.reshape(n, H, -1) for t in D(qkv).split([H * N, H * N, H * P], -1)]
+    _, want = O.channel_decay_recurrence(q, k, v, _log_alpha(low, w2, b2, 20.0, H, N))
+    assert rel(S[0], want) < (2e-5 if dtype == torch.bfloat16 else 3e-6)
+
+
 # ---- attention operands -----------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", [torch.bfloat16, torch.float32])
 @pytest.mark.parametrize("H,G,dk,dv,dims,dense", [(8, 2, 128, 128, 128, (128, 128)), (3, 3, 40, 72, 24, (128, 128)), (4, 1, 12, 20, 6, None),
