@@ -5,7 +5,8 @@
     python -m jax_gpt_b200.utils.kernel_bench --op attn_bwd | norm_fwd | norm_bwd | adamw | ce
     python -m jax_gpt_b200.utils.kernel_bench --op mla_decode --B 32 --T 2304 --H 16
     python -m jax_gpt_b200.utils.kernel_bench --op ssd_scan --B 2 --T 4096 --H 64
-    python -m jax_gpt_b200.utils.kernel_bench --op gated_scan | decay_scan --B 2 --T 4096 --H 16
+    python -m jax_gpt_b200.utils.kernel_bench --op gated_scan | decay_scan | channel_scan --B 2 --T 4096 --H 16
+    python -m jax_gpt_b200.utils.kernel_bench --op gated_lru --B 2 --T 4096 --H 16
     python -m jax_gpt_b200.utils.kernel_bench --op gdn_prep_fwd | gdn_prep_bwd | gdn_prefill --B 1 --T 4096
 
 Each run does ``--warmup`` untimed launches, then times ``--iters`` launches with CUDA events on
@@ -215,8 +216,22 @@ def main(argv=None):
         fn = lambda: ssm.ssd_scan(batch, xbc, dt, db, al, dk, state, G)
         bytes_ = 2.0 * B * T * (C + H * 64 + H) + 4.0 * state.numel()
         flops = B * T / 128 * H * 2.0 * 128 * (128 * 128 + 3 * 128 * 64)
-    elif args.op in ("gated_scan", "decay_scan"):
-        # --B sequences of --T tokens, --H heads of 128 with keys of 128: exponential gates (mLSTM) or a fixed decay per head
+    elif args.op == "gated_lru":
+        # --B sequences of --T tokens, --H gate blocks of 128 channels, four taps
+        from ..ops.gated_lru import LruWeights, gated_lru
+        from .serve_bench import _start_batch
+        B, T, H, W = args.B, args.T, args.H, args.H * 128
+        batch = _start_batch(list(range(B)), [T] * B, 0, dev, T)
+        vec = lambda *s: torch.randn(*s, device=dev)
+        w = LruWeights(vec(W), vec(W), vec(W, 4), vec(W), (vec(H, 2, 128, 128) * 128 ** -0.5).to(torch.bfloat16), vec(H, 2, 128), torch.rand(W, device=dev) * 0.1)
+        xy, out = vec(B * T, 2 * W).to(torch.bfloat16), torch.empty(B * T, W, device=dev, dtype=torch.bfloat16)
+        ring, state = torch.zeros(B, 4, W, device=dev), torch.zeros(B, W, device=dev)
+        fn = lambda: gated_lru(batch, xy[:, :W], xy[:, W:], w, ring, state, 1.0, out)
+        bytes_ = 6.0 * B * T * W + 2.0 * w.gates.numel()
+        flops = 2.0 * B * T * W * 2 * 128
+    elif args.op in ("gated_scan", "decay_scan", "channel_scan"):
+        # --B sequences of --T tokens, --H heads of 128 with keys of 128: exponential gates (mLSTM), a fixed decay per head, or a
+        # decay per key channel from 16 low-rank columns
         from ..ops import linear_attention as LIN
         from .serve_bench import _start_batch
         B, T, H = args.B, args.T, args.H
@@ -225,8 +240,12 @@ def main(argv=None):
         state, vec = torch.zeros(B, H, 128, 128, device=dev), torch.zeros(B, H, 129, device=dev)
         raw, bias = torch.randn(B * T, 2 * H, device=dev), torch.cat([torch.zeros(H), torch.full((H,), 4.0)]).to(dev)
         gates = LIN.Gates(raw, bias, 15.0, vec) if args.op == "gated_scan" else None
-        decay = None if gates is not None else torch.full((H,), 0.99, device=dev)
-        fn = lambda: LIN.linear_scan(batch, qkv, state, gates=gates, decay=decay, q_scale=128 ** -0.5)
+        channels = None
+        if args.op == "channel_scan":
+            low, w2 = (torch.randn(n, 16, device=dev).to(torch.bfloat16) for n in (B * T, H * 128))
+            channels = LIN.ChannelDecay(low, w2 * 0.25, torch.randn(H * 128, device=dev) + 2, 16.0)
+        decay = torch.full((H,), 0.99, device=dev) if args.op == "decay_scan" else None
+        fn = lambda: LIN.linear_scan(batch, qkv, state, gates=gates, decay=decay, channels=channels, q_scale=128 ** -0.5)
         bytes_ = 8.0 * B * T * H * 128 + (24.0 * B * T * H if gates is not None else 0.0) + 4.0 * state.numel()
         flops = B * T / 128 * H * 2.0 * 128 * (128 * 128 + 3 * 128 * 128)
     elif args.op == "mla_decode":
