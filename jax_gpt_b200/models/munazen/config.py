@@ -141,14 +141,14 @@ class MunazenConfig:
                 loop: Optional[Tuple[int, int, int]] = None, vocab: int = 65536) -> "MunazenConfig":
         """Layers with the widths of a real model: attention heads of 128, recurrent units over the model width in blocks of 128,
         linear-attention heads of 128 over the model width, gated-linear layers spread evenly."""
-        rot = Rotary(500000.0, dim, (("factor", 8.0), ("fast", 32.0), ("original", 8192.0), ("slow", 1.0)))
+        rot = Rotary(1e6, dim, (("factor", 4.0), ("fast", 32.0), ("original", 8192.0), ("slow", 1.0)))
         p = Parallel(RotatedAttention(heads, kv_heads, dim, vdim, dim ** -0.5, rot), GatedLru(width, width // lru_block, 4), 1.0, 1.0)
         g = GatedLinear(width // gla_vdim, gla_dim, gla_vdim, 16.0)
         n = n_parallel + n_gla
         every = max(1, n // max(1, n_gla))
         mlp = PolyMlp(ff or 4 * width)
         mixers = [g if n_gla > 0 and i % every == every - 1 and i // every < n_gla else p for i in range(n)]
-        return MunazenConfig(vocab_size=vocab, width=width, norm_eps=1e-6, norm_groups=4, streams=streams, loop=loop,
+        return MunazenConfig(vocab_size=vocab, width=width, norm_eps=1e-5, norm_groups=8, streams=streams, loop=loop,
                              layers=tuple(Layer(m, mlp) for m in mixers))
 
 

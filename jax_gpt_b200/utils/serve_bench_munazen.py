@@ -55,8 +55,8 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
     put(pre, "channel-decay scan (beside the gated scan)", pre["channel-decay scan"]["munazen"], mlstm, "mLSTM scan")
     gam = rn(inner, dtype=f32)
     s1 = LIN.Numerators(LIN.linear_scan(batch, qkv, state, decay=decay).y)
-    put(pre, "head norm, SiLU gate", tm(lambda: LIN.head_norm_gate(batch, s1, z, gam, H, 1e-6, BF, silu=True), 6.0 * N * inner),
-        tm(lambda: LIN.head_norm_gate(batch, s1, z, gam, 1, 1e-6, BF), 6.0 * N * inner), "lightning norm, sigmoid gate")
+    put(pre, "head norm, SiLU gate", tm(lambda: LIN.head_norm_gate(batch, s1, z, gam, H, 1e-5, BF, silu=True), 6.0 * N * inner),
+        tm(lambda: LIN.head_norm_gate(batch, s1, z, gam, 1, 1e-5, BF), 6.0 * N * inner), "lightning norm, sigmoid gate")
     lw = LruWeights(rn(W, dtype=f32), rn(W, dtype=f32), rn(W, 4, dtype=f32), rn(W, dtype=f32), rn(nb, 2, K, K) * K ** -0.5, rn(nb, 2, K, dtype=f32),
                     torch.rand(W, device=dev) * 0.1)
     xy, both = rn(N, 2 * W), torch.empty(N, 2 * W, device=dev, dtype=BF)
@@ -70,12 +70,12 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
     x16, g1, g2 = rn(N, D), rn(D, dtype=f32), rn(D, dtype=f32)
     x32, xs = rn(N, D, dtype=f32), rn(N, streams, D, dtype=f32)
     conn = Connection(rn(streams, dtype=f32), torch.eye(streams, device=dev), rn(streams, dtype=f32))
-    res = tm(lambda: residual_norm_rows(x16, g1, x32, g2, 1e-6, BF), 12.0 * N * D)
-    put(pre, "streams, next combination, group norm", tm(lambda: stream_norm(x16, xs, conn, conn.w_in, g1, 4, 1e-6, BF, bias=g2), (4.0 + 8.0 * streams) * N * D),
+    res = tm(lambda: residual_norm_rows(x16, g1, x32, g2, 1e-5, BF), 12.0 * N * D)
+    put(pre, "streams, next combination, group norm", tm(lambda: stream_norm(x16, xs, conn, conn.w_in, g1, 8, 1e-5, BF, bias=g2), (4.0 + 8.0 * streams) * N * D),
         res, "post-norm, residual, next norm")
     zf, coef = rn(N, ff), torch.tensor([0.5, 0.3, 0.2, 0.0], device=dev)
     gu, gh = rn(N, 2 * ff), torch.empty(N, ff, device=dev, dtype=BF)
-    put(pre, "polynomial activation", tm(lambda: poly_norm(zf, coef, 1e-6), 4.0 * N * ff),
+    put(pre, "polynomial activation", tm(lambda: poly_norm(zf, coef, 1e-5), 4.0 * N * ff),
         tm(lambda: _ext.ops().clamped_glu(gu, float("inf"), 1.0, 0.0, None, gh), 6.0 * N * ff), "gate times up (clamped_glu)")
     del gu, gh
     n_in = (heads + 2 * kv_heads) * K + 2 * W + 16
@@ -89,7 +89,7 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
 
     # ---- prefill: attention ----
     Q, G = heads, kv_heads
-    rope, vrope = rope_tables(K, 5e5, ctx + seq_len, None, dev), rope_tables(K, 5e5, ctx + seq_len, None, dev)
+    rope, vrope = rope_tables(K, 1e6, ctx + seq_len, None, dev), rope_tables(K, 1e6, ctx + seq_len, None, dev)
     per = max(seq_len, ctx) // 64 + 2
     n_seq = max(max(decode_batches), seqs)
     cache = PagedCache(1, [2 * G * K], n_seq * per, 64, n_seq, per, BF, dev)
@@ -101,7 +101,7 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
     rotate = lambda yy, bt, dense: RKV.qkv_rotate(bt, yy, cols, bq, Q, G, K, K, rope, vrope, cache, 0, dense)
     y_qk, b_qk = rn(N, (Q + G) * K), rn((Q + G) * K, dtype=f32)
     put(pre, "bias, rotation of q k v, cache write", tm(lambda: rotate(yq, batch, (K, K)), 2.0 * N * K * ((Q + 2 * G) * 2 + 2 * G)),
-        tm(lambda: WA.qk_prepare(batch, y_qk, b_qk, Q, G, K, True, 1e-6, rope, cache, 0, dense=True), 2.0 * N * K * ((Q + G) * 2 + 3 * G)),
+        tm(lambda: WA.qk_prepare(batch, y_qk, b_qk, Q, G, K, True, 1e-5, rope, cache, 0, dense=True), 2.0 * N * K * ((Q + G) * 2 + 3 * G)),
         "bias, rotation, unit norm, cache write")
     q, k, v = rotate(yq, batch, (K, K))
     as4 = lambda t: t.unflatten(0, (seqs, seq_len))
@@ -111,7 +111,7 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
     put(pre, "flash attention, keys of 64 padded to 128", tm(lambda: WA.flash_prompts(batch, q, k, v, 0.09), 0, fa(64, K)), causal, "the same kernel, keys of 128")
     o = rn(N, Q, K)
     put(pre, "turn back, head gate", tm(lambda: RKV.turn_back_gate(batch, o, yq[:, -16:][:, :Q], vrope, 1.0, both[:, :Q * K]), 4.0 * N * Q * K),
-        tm(lambda: LIN.head_norm_gate(batch, s1, z, gam, 1, 1e-6, BF), 6.0 * N * inner), "lightning norm, sigmoid gate")
+        tm(lambda: LIN.head_norm_gate(batch, s1, z, gam, 1, 1e-5, BF), 6.0 * N * inner), "lightning norm, sigmoid gate")
     del yq, y_qk, q, k, v, o, both, s1, z, x16
     _ext.check_status(dev)
 
@@ -125,7 +125,7 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
         def step(kind):
             s = LIN.linear_scan(bd, qk1[:, :3 * inner], st1, channels=ch1, q_scale=K ** -0.5) if kind else \
                 LIN.linear_scan(bd, qk1[:, :3 * inner], st1, decay=decay, silu=True)
-            LIN.head_norm_gate(bd, s, z1, gam, H if kind else 1, 1e-6, BF, silu=bool(kind))
+            LIN.head_norm_gate(bd, s, z1, gam, H if kind else 1, 1e-5, BF, silu=bool(kind))
         b_step = 8.0 * st1.numel() + 2.0 * B * 5 * inner
         light = tm(lambda: step(0), b_step)
         put(d, "channel-decay step + norm", tm(lambda: step(1), b_step + 2.0 * w2.numel()), light, "lightning step + norm")
@@ -149,17 +149,17 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
             dec, "the same kernel, both 128")
         y1, yk1 = rn(B, n_in), rn(B, (Q + G) * K)
         put(d, "bias, rotation of q k v, cache write", tm(lambda: rotate(y1, bd, None), 2.0 * B * K * (2 * Q + 4 * G)),
-            tm(lambda: WA.qk_prepare(bd, yk1, b_qk, Q, G, K, True, 1e-6, rope, cache, 0, dense=False), 2.0 * B * K * (2 * Q + 3 * G)),
+            tm(lambda: WA.qk_prepare(bd, yk1, b_qk, Q, G, K, True, 1e-5, rope, cache, 0, dense=False), 2.0 * B * K * (2 * Q + 3 * G)),
             "bias, rotation, unit norm, cache write")
         od = rn(B, Q, K)
-        gate1 = tm(lambda: LIN.head_norm_gate(bd, LIN.Numerators(z1), z1, gam, 1, 1e-6, BF), 6.0 * B * inner)
+        gate1 = tm(lambda: LIN.head_norm_gate(bd, LIN.Numerators(z1), z1, gam, 1, 1e-5, BF), 6.0 * B * inner)
         put(d, "turn back, head gate", tm(lambda: RKV.turn_back_gate(bd, od, y1[:, -16:][:, :Q], vrope, 1.0, o1[:, :Q * K]), 4.0 * B * Q * K), gate1,
             "lightning norm, sigmoid gate")
         xb, yb, xr, xs1 = rn(B, D), rn(B, D), rn(B, D, dtype=f32), rn(B, streams, D, dtype=f32)
-        put(d, "streams, next combination, group norm", tm(lambda: stream_norm(yb, xs1, conn, conn.w_in, g1, 4, 1e-6, BF, bias=g2), (4.0 + 8.0 * streams) * B * D),
-            tm(lambda: residual_norm_rows(yb, g1, xr, g2, 1e-6, BF), 12.0 * B * D), "post-norm, residual, next norm")
+        put(d, "streams, next combination, group norm", tm(lambda: stream_norm(yb, xs1, conn, conn.w_in, g1, 8, 1e-5, BF, bias=g2), (4.0 + 8.0 * streams) * B * D),
+            tm(lambda: residual_norm_rows(yb, g1, xr, g2, 1e-5, BF), 12.0 * B * D), "post-norm, residual, next norm")
         z1f = rn(B, ff)
-        put(d, "polynomial activation", tm(lambda: poly_norm(z1f, coef, 1e-6), 4.0 * B * ff), gate1, "lightning norm, sigmoid gate")
+        put(d, "polynomial activation", tm(lambda: poly_norm(z1f, coef, 1e-5), 4.0 * B * ff), gate1, "lightning norm, sigmoid gate")
         yo = torch.empty(B, 3 * D, device=dev, dtype=BF)
         lin = tm(lambda: gemm(xb, w_in[:3 * D], out=yo), 6.0 * D * D)
         for name, fn, w in (("projection q k v x y g", lambda: linear_rows(xb, w_in), w_in), ("projection of both branches", lambda: linear_rows(o1, w_o), w_o),
