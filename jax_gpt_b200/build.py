@@ -29,7 +29,7 @@ NVCC_FLAGS = [
 # Sources whose fp32 instances are exact to rounding: no approximate division, square root, exponential or denormal
 # flush (kernels in them that want the fast intrinsics name them).
 PRECISE_SOURCES = {"serve_kernels.cu", "ssm_kernels.cu", "ssd_scan_sm100.cu", "window_attention.cu", "linear_attention.cu",
-                   "rotated_kv.cu", "stream_kernels.cu", "gated_lru.cu", "gla_chunk.cu"}
+                   "rotated_kv.cu", "mixed_kv.cu", "stream_kernels.cu", "gated_lru.cu", "gla_chunk.cu"}
 
 
 def _cuda_home() -> str:

@@ -12,6 +12,7 @@
 #include "attention_sm100.cuh"
 
 #include "common.cuh"
+#include "softcap.cuh"
 
 namespace b200 {
 
@@ -40,10 +41,15 @@ struct DecArgs {
   int page_size, max_pages;
   int window, keep_first;   // window > 0: of the valid keys only the last `window` and the first `keep_first` are seen
   int64_t v_stride_h;       // between the kv heads of V
+  // pool > 0 (paged, keep_first 0): the mean rows of the blocks of `pool` tokens that lie wholly before the window are seen too; they sit
+  // in pages of ceil(page_size / pool) rows, in the page of a block's last token
+  const __nv_bfloat16* pooled;
+  int pool;
+  SoftCap cap;              // kCap instances
 };
 
 // D: query and key width, DV: value width (D or 2 D).
-template <int D, int DV, int G>
+template <int D, int DV, int G, bool kCap, bool kPool>
 __global__ void __launch_bounds__(kDecWarps * 32)
 attn_decode_split_kernel(const DecArgs a) {
   constexpr int LPK = D / 8;          // lanes that share one key row
@@ -60,12 +66,18 @@ attn_decode_split_kernel(const DecArgs a) {
   const int len = a.table != nullptr ? a.lens[seq] + a.len_add : (a.pos_ptr != nullptr ? a.pos_ptr[0] + a.len_add : a.len);
   const int* pages = a.table != nullptr ? a.table + static_cast<int64_t>(seq) * a.max_pages : nullptr;
   // The seen keys are numbered through: the kept first ones, then the window (which may start among them).
-  const int n_keep = a.window > 0 ? min(a.keep_first, len) : 0;
-  const int w0 = a.window > 0 ? max(n_keep, len - a.window) : 0;
+  const int n_keep = kPool ? max(0, len - a.window) / a.pool : (a.window > 0 ? min(a.keep_first, len) : 0);
+  const int w0 = a.window > 0 ? max(kPool ? 0 : n_keep, len - a.window) : 0;
   const int n_seen = n_keep + len - w0;
   // cache row of seen key t: its position for a dense cache, page * page_size + offset for a paged one
+  const int block_rows = kPool ? (a.page_size + a.pool - 1) / a.pool : 0;
   auto key_row = [&](int t) -> int64_t {
-    if (t >= n_keep) t += w0 - n_keep;
+    if (t >= n_keep) {
+      t += w0 - n_keep;
+    } else if (kPool) {
+      const int pi = (t * a.pool + a.pool - 1) / a.page_size;
+      return static_cast<int64_t>(pages[pi]) * block_rows + t - pi * a.page_size / a.pool;
+    }
     if (pages == nullptr) return t;
     return static_cast<int64_t>(pages[t / a.page_size]) * a.page_size + t % a.page_size;
   };
@@ -80,8 +92,8 @@ attn_decode_split_kernel(const DecArgs a) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const float2 f = unpack_bf16x2(w[e]);
-      qf[g][2 * e] = f.x * a.scale_log2;
-      qf[g][2 * e + 1] = f.y * a.scale_log2;
+      qf[g][2 * e] = kCap ? f.x : f.x * a.scale_log2;
+      qf[g][2 * e + 1] = kCap ? f.y : f.y * a.scale_log2;
     }
   }
   float m[G], l[G], o[G][EV];
@@ -94,6 +106,8 @@ attn_decode_split_kernel(const DecArgs a) {
   }
   const __nv_bfloat16* kb = a.k + b * a.kv_stride_b + hkv * a.kv_stride_h + sub * 8;
   const __nv_bfloat16* vb = a.v + b * a.kv_stride_b + hkv * a.v_stride_h + sub * 8;
+  const __nv_bfloat16* kp = kPool ? a.pooled + hkv * a.kv_stride_h + sub * 8 : nullptr;   // the same in the rows of means
+  const __nv_bfloat16* vp = kPool ? a.pooled + (a.v - a.k) + hkv * a.v_stride_h + sub * 8 : nullptr;
   // Two keys per lane group in flight. The trip count is uniform over the warp (the shuffles below need every
   // lane); a lane group whose key is past the range loads nothing and skips the update.
   for (int base = k0 + warp * KPW; base < k1; base += 2 * KPS) {
@@ -101,13 +115,15 @@ attn_decode_split_kernel(const DecArgs a) {
     const bool has_a = ka < k1, has_c = kc < k1;
     const uint4 zero = make_uint4(0, 0, 0, 0);
     const int64_t ra = has_a ? key_row(ka) * a.kv_stride_t : 0, rc = has_c ? key_row(kc) * a.kv_stride_t : 0;
-    const uint4 kua = has_a ? *reinterpret_cast<const uint4*>(kb + ra) : zero;
-    const uint4 kuc = has_c ? *reinterpret_cast<const uint4*>(kb + rc) : zero;
+    const bool pa = kPool && ka < n_keep, pc = kPool && kc < n_keep;
+    const __nv_bfloat16 *va = pa ? vp : vb, *vc = pc ? vp : vb;
+    const uint4 kua = has_a ? *reinterpret_cast<const uint4*>((pa ? kp : kb) + ra) : zero;
+    const uint4 kuc = has_c ? *reinterpret_cast<const uint4*>((pc ? kp : kb) + rc) : zero;
     uint4 vua[NV], vuc[NV];
 #pragma unroll
     for (int p = 0; p < NV; ++p) {
-      vua[p] = has_a ? *reinterpret_cast<const uint4*>(vb + ra + p * D) : zero;
-      vuc[p] = has_c ? *reinterpret_cast<const uint4*>(vb + rc + p * D) : zero;
+      vua[p] = has_a ? *reinterpret_cast<const uint4*>(va + ra + p * D) : zero;
+      vuc[p] = has_c ? *reinterpret_cast<const uint4*>(vc + rc + p * D) : zero;
     }
 #pragma unroll
     for (int which = 0; which < 2; ++which) {
@@ -139,6 +155,7 @@ attn_decode_split_kernel(const DecArgs a) {
         for (int e = 0; e < 8; ++e) s = fmaf(qf[g][e], kf[e], s);
 #pragma unroll
         for (int off = LPK / 2; off > 0; off >>= 1) s += __shfl_xor_sync(0xffffffffu, s, off);
+        if (kCap) s = soft_cap(s, a.cap);
         if (valid) {
           const float mn = fmaxf(m[g], s);
           const float alpha = exp2f(m[g] - mn), p = exp2f(s - mn);
@@ -202,20 +219,21 @@ attn_decode_split_kernel(const DecArgs a) {
   }
 }
 
-// out[b, h, :] = sum_s part_o[s] 2^(m_s - M) / sum_s l_s 2^(m_s - M); one CTA per (head, sequence). The ranges' weights go
-// through shared memory; kGroups groups of D threads each sum every kGroups-th range.
+// out[b, h, :] = sum_s part_o[s] 2^(m_s - M) / (sum_s l_s 2^(m_s - M) + the sink's weight); one CTA per (head, sequence). The
+// ranges' weights go through shared memory; kGroups groups of D threads each sum every kGroups-th range.
 constexpr int kMaxSplits = 256;
 
 template <int D>
 __global__ void __launch_bounds__(512)
 attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int n_splits,
-                         __nv_bfloat16* __restrict__ out, int64_t ldo, int H) {
+                         __nv_bfloat16* __restrict__ out, int64_t ldo, int H, const float* __restrict__ sink) {
   constexpr int kGroups = 512 / D;
   __shared__ float wt[kMaxSplits], acc_s[kGroups][D], red[1];
   const int h = blockIdx.x, b = blockIdx.y, c = threadIdx.x % D, grp = threadIdx.x / D;
   const int64_t row0 = (static_cast<int64_t>(b) * H + h) * n_splits;
   if (threadIdx.x < 32) {
-    float mn = -INFINITY, ls = 0.f;
+    const float sk = sink != nullptr ? sink[h] * 1.4426950408889634f : -INFINITY;
+    float mn = sk, ls = 0.f;
     for (int s = threadIdx.x; s < n_splits; s += 32) mn = fmaxf(mn, part_ml[(row0 + s) * 2]);
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, o));
@@ -227,7 +245,7 @@ attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restri
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) ls += __shfl_xor_sync(0xffffffffu, ls, o);
-    if (threadIdx.x == 0) red[0] = ls;
+    if (threadIdx.x == 0) red[0] = ls + (sink != nullptr ? exp2f(sk - mn) : 0.f);
   }
   __syncthreads();
   float acc = 0.f;
@@ -245,24 +263,27 @@ attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restri
 
 template <int D, int DV, int G>
 cudaError_t decode_launch(const DecArgs& a, int B, int n_splits, __nv_bfloat16* out, int64_t ldo,
-                          cudaStream_t stream) {
-  if (n_splits > kMaxSplits) return cudaErrorInvalidValue;
+                          cudaStream_t stream, const float* sink) {
+  const bool cap = a.cap.out > 0.f;
+  if (n_splits > kMaxSplits || (a.pool > 0 && cap)) return cudaErrorInvalidValue;
   dim3 grid(n_splits, a.Hkv, B);
-  attn_decode_split_kernel<D, DV, G><<<grid, kDecWarps * 32, 0, stream>>>(a);
+  if (a.pool > 0) attn_decode_split_kernel<D, DV, G, false, true><<<grid, kDecWarps * 32, 0, stream>>>(a);
+  else if (cap) attn_decode_split_kernel<D, DV, G, true, false><<<grid, kDecWarps * 32, 0, stream>>>(a);
+  else attn_decode_split_kernel<D, DV, G, false, false><<<grid, kDecWarps * 32, 0, stream>>>(a);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return e;
-  attn_decode_merge_kernel<DV><<<dim3(a.H, B), 512, 0, stream>>>(a.part_o, a.part_ml, n_splits, out, ldo, a.H);
+  attn_decode_merge_kernel<DV><<<dim3(a.H, B), 512, 0, stream>>>(a.part_o, a.part_ml, n_splits, out, ldo, a.H, sink);
   return cudaGetLastError();
 }
 
 template <int D, int DV = D>
 cudaError_t decode_dispatch_g(const DecArgs& a, int B, int n_splits, __nv_bfloat16* out, int64_t ldo,
-                              cudaStream_t stream) {
+                              cudaStream_t stream, const float* sink = nullptr) {
   switch (a.H / a.Hkv) {
-    case 1: return decode_launch<D, DV, 1>(a, B, n_splits, out, ldo, stream);
-    case 2: return decode_launch<D, DV, 2>(a, B, n_splits, out, ldo, stream);
-    case 4: return decode_launch<D, DV, 4>(a, B, n_splits, out, ldo, stream);
-    case 8: return decode_launch<D, DV, 8>(a, B, n_splits, out, ldo, stream);
+    case 1: return decode_launch<D, DV, 1>(a, B, n_splits, out, ldo, stream, sink);
+    case 2: return decode_launch<D, DV, 2>(a, B, n_splits, out, ldo, stream, sink);
+    case 4: return decode_launch<D, DV, 4>(a, B, n_splits, out, ldo, stream, sink);
+    case 8: return decode_launch<D, DV, 8>(a, B, n_splits, out, ldo, stream, sink);
     default: return cudaErrorInvalidValue;
   }
 }
@@ -277,7 +298,7 @@ cudaError_t launch_attn_decode(const __nv_bfloat16* q, int64_t ldq, const __nv_b
       ldq % 8 != 0)
     return cudaErrorInvalidValue;
   DecArgs a{q, ldq, k, v, kv_stride_b, kv_stride_h, kv_stride_t, pos_ptr, len, len_add, H, Hkv,
-            scale * 1.4426950408889634f, part_o, part_ml, nullptr, nullptr, nullptr, 0, 0, 0, 0, kv_stride_h};
+            scale * 1.4426950408889634f, part_o, part_ml, nullptr, nullptr, nullptr, 0, 0, 0, 0, kv_stride_h, nullptr, 0, SoftCap{0.f, 0.f}};
   switch (D) {
     case 64: return decode_dispatch_g<64>(a, B, n_splits, out, ldo, stream);
     case 128: return decode_dispatch_g<128>(a, B, n_splits, out, ldo, stream);
@@ -290,8 +311,9 @@ cudaError_t launch_attn_decode_paged(const __nv_bfloat16* q, int64_t ldq, const 
                                      const int* block_table, const int* seq_ids, const int* seq_lens, int len_add,
                                      int page_size, int max_pages, int B, int H, int Hkv, int D, float scale, int n_splits,
                                      float* part_o, float* part_ml, __nv_bfloat16* out, int64_t ldo, cudaStream_t stream,
-                                     int window, int keep_first, int DV) {
+                                     int window, int keep_first, int DV, const DecodeScores& sc) {
   if (DV == 0) DV = D;
+  if (sc.pool > 0 && (sc.pooled == nullptr || window < 1 || keep_first > 0)) return cudaErrorInvalidValue;
   if (H % Hkv != 0 || n_splits < 1 || width != Hkv * (D + DV) || width % 8 != 0 || ldq % 8 != 0 || page_size < 1 || keep_first < 0)
     return cudaErrorInvalidValue;
   // a pool row holds K of every kv head, then V of every kv head
@@ -299,13 +321,16 @@ cudaError_t launch_attn_decode_paged(const __nv_bfloat16* q, int64_t ldq, const 
             scale * 1.4426950408889634f, part_o, part_ml, block_table, seq_ids, seq_lens, page_size, max_pages,
             window, keep_first};
   a.v_stride_h = DV;
-  if (DV == 2 * D && D == 64) return decode_dispatch_g<64, 128>(a, B, n_splits, out, ldo, stream);
-  if (DV == 2 * D && D == 128) return decode_dispatch_g<128, 256>(a, B, n_splits, out, ldo, stream);
+  a.pooled = sc.pooled;
+  a.pool = sc.pool;
+  if (sc.softcap > 0.f) a.cap = SoftCap{2.f * 1.4426950408889634f * scale / sc.softcap, sc.softcap * 1.4426950408889634f};
+  if (DV == 2 * D && D == 64) return decode_dispatch_g<64, 128>(a, B, n_splits, out, ldo, stream, sc.sink);
+  if (DV == 2 * D && D == 128) return decode_dispatch_g<128, 256>(a, B, n_splits, out, ldo, stream, sc.sink);
   if (DV != D) return cudaErrorInvalidValue;
   switch (D) {
-    case 64: return decode_dispatch_g<64>(a, B, n_splits, out, ldo, stream);
-    case 128: return decode_dispatch_g<128>(a, B, n_splits, out, ldo, stream);
-    case 256: return decode_dispatch_g<256>(a, B, n_splits, out, ldo, stream);
+    case 64: return decode_dispatch_g<64>(a, B, n_splits, out, ldo, stream, sc.sink);
+    case 128: return decode_dispatch_g<128>(a, B, n_splits, out, ldo, stream, sc.sink);
+    case 256: return decode_dispatch_g<256>(a, B, n_splits, out, ldo, stream, sc.sink);
     default: return cudaErrorInvalidValue;
   }
 }

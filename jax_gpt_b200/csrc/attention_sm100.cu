@@ -22,6 +22,7 @@
 #include <cstdlib>
 
 #include "common.cuh"
+#include "softcap.cuh"
 #include "tma_host.h"
 
 namespace b200 {
@@ -43,8 +44,13 @@ struct FwdArgs {
   float* lse;
   int* status;
   const float* sink;        // [H] or nullptr: extra term exp(sink[h]) of the softmax denominator
-  int window, keep_first;   // kWindow instances: keys j with i - j < window or j < keep_first are seen
+  int window, keep_first;   // windowed instances: keys j with i - j < window or j < keep_first are seen
+  int pool, pool_rows;      // kPooled: keys 0 .. pool_rows - 1 are block means, tokens follow (q_pos0 = pool_rows)
+  SoftCap cap;              // kCap instances
 };
+
+// What a query sees besides the causal rule: everything, a window and kept first keys, a window and block means before it.
+enum FwdMask : int { kAll = 0, kWindowed = 1, kPooled = 2 };
 
 // D: width of q and k heads; DV: width of v heads (MLA prefill uses 192 / 128).
 template <int D, int DV>
@@ -89,11 +95,12 @@ __device__ __forceinline__ void load_tile(uint8_t* dst, const CUtensorMap* m, ui
 // bits 0 .. n - 1
 __device__ __forceinline__ uint32_t bits_below(int n) { return n <= 0 ? 0u : (n >= 32 ? 0xffffffffu : (1u << n) - 1u); }
 
-template <int D, int DV, bool kWindow>
+template <int D, int DV, int kMask, bool kCap>
 __global__ void __launch_bounds__(kThreads, (D == 64) ? 2 : 1)
 attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk,
                 const __grid_constant__ CUtensorMap tv, const __grid_constant__ FwdArgs a) {
   using C = FwdCfg<D, DV>;
+  constexpr bool kWindow = kMask != kAll;
   extern __shared__ __align__(1024) uint8_t smem[];
   if ((smem_u32(smem) & 1023u) != 0) {
     if (threadIdx.x == 0) report_status(a.status, kBadArgument, 1, 0, 0);
@@ -110,9 +117,12 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
   const int n_kv_all = (a.Tk + 127) / 128;
   const int q0 = a.q_pos0 + q_blk * 128;     // position of the block's first query
   const int n_seen = a.causal ? min((q0 + 127) / 128 + 1, n_kv_all) : n_kv_all;
-  // key tiles: those of the kept first keys, then those from the window of the first query on
-  const int n_keep = kWindow ? min((a.keep_first + 127) / 128, n_seen) : 0;
-  const int w_tile = kWindow ? max(n_keep, min(max(0, q0 - a.window + 1) / 128, n_seen)) : 0;
+  // key tiles: those of the kept first keys or of the block means, then those from the window of the first query on
+  auto first_keys = [&](int pos) { return kMask == kPooled ? max(0, pos - a.pool_rows - a.window + 1) / a.pool : a.keep_first; };
+  const int n_keep = kMask == kPooled ? min((first_keys(q0 + 127) + 127) / 128, a.pool_rows / 128)
+                                      : (kWindow ? min((a.keep_first + 127) / 128, n_seen) : 0);
+  const int w_tile = kMask == kPooled ? max(a.pool_rows, q0 - a.window + 1) / 128
+                                      : (kWindow ? max(n_keep, min(max(0, q0 - a.window + 1) / 128, n_seen)) : 0);
   const int n_kv = n_keep + n_seen - w_tile;
   auto key_tile = [&](int j) { return kWindow && j >= n_keep ? w_tile + j - n_keep : j; };
   const int row0 = b * a.T + q_blk * 128;
@@ -214,6 +224,7 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
     const int qi = q_blk * 128 + r;      // query index inside the sequence
     const int qpos = a.q_pos0 + qi;
     const uint32_t lane_off = static_cast<uint32_t>(q * 32) << 16;
+    const int first = kWindow ? first_keys(qpos) : 0;
     __nv_bfloat16* xchg = reinterpret_cast<__nv_bfloat16*>(smem + C::kOffXchg);  // [2][128]
     constexpr int DH = DV / 2;
     float m = -INFINITY, l = 0.f;
@@ -229,12 +240,15 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
       }
       tc_fence_after();
       const int kt0 = key_tile(j) * 128;
-      const bool need_mask = (a.causal && kt0 + 127 > q0) || kt0 + 128 > a.Tk ||
-                             (kWindow && q0 + 127 - kt0 >= a.window && kt0 + 127 >= a.keep_first);
+      const bool means = kMask == kPooled && j < n_keep;
+      const bool need_mask = means ? kt0 + 128 > first_keys(q0)
+                                   : ((a.causal && kt0 + 127 > q0) || kt0 + 128 > a.Tk ||
+                                      (kWindow && q0 + 127 - kt0 >= a.window && (kMask == kPooled || kt0 + 127 >= a.keep_first)));
       // scores of 32 keys from position k0 on: those this row does not see become -inf
       auto hide = [&](uint32_t (&v)[32], int k0) {
         uint32_t seen = bits_below((a.causal ? min(qpos + 1, a.Tk) : a.Tk) - k0);
-        if (kWindow) seen &= ~bits_below(qpos - a.window + 1 - k0) | bits_below(a.keep_first - k0);
+        if (kMask == kWindowed) seen &= ~bits_below(qpos - a.window + 1 - k0) | bits_below(first - k0);
+        if (kMask == kPooled) seen = means ? bits_below(first - k0) : seen & ~bits_below(qpos - a.window + 1 - k0);
 #pragma unroll
         for (int i = 0; i < 32; ++i)
           if (!(seen >> i & 1u)) v[i] = 0xff800000u;
@@ -250,7 +264,8 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
 #pragma unroll
         for (int i = 0; i < 32; ++i) mx = fmaxf(mx, __uint_as_float(v[i]));   // the (positive) scale is applied once, below
       }
-      mx *= a.scale_log2;
+      if (kCap) mx = mx == -INFINITY ? mx : soft_cap(mx, a.cap);   // monotone: the capped maximum
+      else mx *= a.scale_log2;
       const __nv_bfloat16 mine = __float2bfloat16(mx);
       xchg[half * 128 + r] = mine;
       mbar_arrive(&bars->x_ready);
@@ -273,8 +288,18 @@ attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ 
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          const float p0 = exp2f(fmaf(__uint_as_float(v[i]), a.scale_log2, -mref));
-          const float p1 = exp2f(fmaf(__uint_as_float(v[i + 1]), a.scale_log2, -mref));
+          float p0, p1;
+          if constexpr (kCap) {
+            p0 = exp2f(soft_cap(__uint_as_float(v[i]), a.cap) - mref);
+            p1 = exp2f(soft_cap(__uint_as_float(v[i + 1]), a.cap) - mref);
+            if (need_mask) {   // the cap of -inf is finite
+              p0 = v[i] == 0xff800000u ? 0.f : p0;
+              p1 = v[i + 1] == 0xff800000u ? 0.f : p1;
+            }
+          } else {
+            p0 = exp2f(fmaf(__uint_as_float(v[i]), a.scale_log2, -mref));
+            p1 = exp2f(fmaf(__uint_as_float(v[i + 1]), a.scale_log2, -mref));
+          }
           rs += p0 + p1;
           pk[i >> 1] = pack_bf16x2(p0, p1);
         }
@@ -744,7 +769,7 @@ cudaError_t make_map(CUtensorMap* m, const __nv_bfloat16* p, int64_t ld, int row
   return encode_tma_2d(m, p, 2, cols, rows, ld * 2, 64, 128);
 }
 
-template <int D, int DV, bool kWindow = false>
+template <int D, int DV, int kMask = kAll, bool kCap = false>
 cudaError_t fwd_launch(const AttnTensors& t, const AttnShape& s, const AttnKvLayout& kv, __nv_bfloat16* out,
                        int64_t ldo, float* lse, int* status, cudaStream_t stream) {
   using C = FwdCfg<D, DV>;
@@ -754,7 +779,7 @@ cudaError_t fwd_launch(const AttnTensors& t, const AttnShape& s, const AttnKvLay
   if ((e = make_map(&tq, t.q, t.ldq, rows, s.H * D)) != cudaSuccess) return e;
   if ((e = encode_tma_2d(&tk, t.k, 2, kv.k_cols, kv.rows, t.ldk * 2, 64, 128)) != cudaSuccess) return e;
   if ((e = encode_tma_2d(&tv, t.v, 2, kv.v_cols, kv.rows, t.ldv * 2, 64, 128)) != cudaSuccess) return e;
-  auto kernel = attn_fwd_kernel<D, DV, kWindow>;
+  auto kernel = attn_fwd_kernel<D, DV, kMask, kCap>;
   static bool configured = false;
   if (!configured) {
     if ((e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kSmem)) != cudaSuccess)
@@ -762,7 +787,8 @@ cudaError_t fwd_launch(const AttnTensors& t, const AttnShape& s, const AttnKvLay
     configured = true;
   }
   FwdArgs a{s.B, s.T, kv.Tk, s.H, s.Hkv, kv.q_pos0, kv.rows_b, kv.rows_h, kv.k_col_h, kv.v_col_h,
-            s.scale * kLog2e, s.causal, out, ldo, lse, status, s.sink, s.window, std::min(s.keep_first, 1 << 30)};
+            s.scale * kLog2e, s.causal, out, ldo, lse, status, s.sink, s.window, std::min(s.keep_first, 1 << 30), s.pool, s.pool_rows, SoftCap{0.f, 0.f}};
+  if (kCap) a.cap = SoftCap{2.f * kLog2e * s.scale / s.softcap, s.softcap * kLog2e};
   dim3 grid(s.H, s.B, (s.T + 127) / 128);
   kernel<<<grid, kThreads, C::kSmem, stream>>>(tq, tk, tv, a);
   return cudaGetLastError();
@@ -815,12 +841,23 @@ cudaError_t launch_attn_fwd_kv(const AttnTensors& t, const AttnShape& s, const A
                                int64_t ldo, float* lse, int* status, cudaStream_t stream) {
   if (s.H % s.Hkv != 0 || (s.window > 0 && (!s.causal || s.keep_first < 0))) return cudaErrorInvalidValue;
   const int dv = s.Dv > 0 ? s.Dv : s.D;
-  if (s.window > 0) {
-    if (s.D == 64 && dv == 64) return fwd_launch<64, 64, true>(t, s, kv, out, ldo, lse, status, stream);
-    if (s.D == 128 && dv == 128) return fwd_launch<128, 128, true>(t, s, kv, out, ldo, lse, status, stream);
-    if (s.D == 256 && dv == 256) return fwd_launch<256, 256, true>(t, s, kv, out, ldo, lse, status, stream);
-    return cudaErrorInvalidValue;
+#define B200_FWD(MASK, CAP)                                                                                          \
+  {                                                                                                                  \
+    if (s.D == 64 && dv == 64) return fwd_launch<64, 64, MASK, CAP>(t, s, kv, out, ldo, lse, status, stream);        \
+    if (s.D == 128 && dv == 128) return fwd_launch<128, 128, MASK, CAP>(t, s, kv, out, ldo, lse, status, stream);    \
+    if (s.D == 256 && dv == 256) return fwd_launch<256, 256, MASK, CAP>(t, s, kv, out, ldo, lse, status, stream);    \
+    if (s.D == 192 && dv == 128) return fwd_launch<192, 128, MASK, CAP>(t, s, kv, out, ldo, lse, status, stream);    \
+    return cudaErrorInvalidValue;                                                                                    \
   }
+  if (s.softcap > 0.f) {
+    if (s.window > 0 || s.pool > 0) return cudaErrorInvalidValue;
+    B200_FWD(kAll, true)
+  }
+  if (s.pool > 0) {
+    if (s.window < 1 || s.keep_first > 0 || s.pool_rows % 128 != 0 || kv.q_pos0 != s.pool_rows) return cudaErrorInvalidValue;
+    B200_FWD(kPooled, false)
+  }
+  if (s.window > 0) B200_FWD(kWindowed, false)
   if (s.D == 64 && dv == 64) {
     // two-tile kernel unless the single-tile one is asked for (B200_ATTN_FWD=1tile: comparisons, fallback)
     static const bool one_tile = [] {
@@ -830,23 +867,21 @@ cudaError_t launch_attn_fwd_kv(const AttnTensors& t, const AttnShape& s, const A
     if (!one_tile && s.sink == nullptr) return launch_attn_fwd2_d64(t, s, kv, out, ldo, lse, status, stream);
     return fwd_launch<64, 64>(t, s, kv, out, ldo, lse, status, stream);
   }
-  if (s.D == 128 && dv == 128) return fwd_launch<128, 128>(t, s, kv, out, ldo, lse, status, stream);
-  if (s.D == 256 && dv == 256) return fwd_launch<256, 256>(t, s, kv, out, ldo, lse, status, stream);
-  if (s.D == 192 && dv == 128) return fwd_launch<192, 128>(t, s, kv, out, ldo, lse, status, stream);
-  return cudaErrorInvalidValue;
+  B200_FWD(kAll, false)
+#undef B200_FWD
 }
 
 cudaError_t launch_attn_fwd(const AttnTensors& t, const AttnShape& s, __nv_bfloat16* out, int64_t ldo, float* lse,
                             int* status, cudaStream_t stream) {
   const int dv = s.Dv > 0 ? s.Dv : s.D;
   AttnKvLayout kv;
-  kv.Tk = s.T;
-  kv.q_pos0 = 0;
-  kv.rows_b = s.T;
+  kv.Tk = s.pool_rows + s.T;
+  kv.q_pos0 = s.pool_rows;
+  kv.rows_b = kv.Tk;
   kv.rows_h = 0;
   kv.k_col_h = s.D;
   kv.v_col_h = dv;
-  kv.rows = static_cast<uint64_t>(s.B) * s.T;
+  kv.rows = static_cast<uint64_t>(s.B) * kv.Tk;
   kv.k_cols = static_cast<uint64_t>(s.Hkv) * s.D;
   kv.v_cols = static_cast<uint64_t>(s.Hkv) * dv;
   return launch_attn_fwd_kv(t, s, kv, out, ldo, lse, status, stream);

@@ -23,6 +23,10 @@ struct AttnShape {
   const float* sink = nullptr;  // forward: [H] fp32, exp(sink[h]) joins every denominator of head h (no key, no value, not scaled)
   // forward, causal: a query at position i sees keys j <= i with i - j < window or j < keep_first; 0: no window
   int window = 0, keep_first = 0;
+  float softcap = 0.f;      // forward, without a window: > 0: scores become softcap * tanh(scale * score / softcap)
+  // forward, with a window: K and V of a sequence start with `pool_rows` rows (a multiple of 128) of block means, then its T tokens;
+  // query i sees mean b when the block b pool .. b pool + pool - 1 lies wholly before its window
+  int pool = 0, pool_rows = 0;
 };
 
 // Where the keys and values of (batch b, kv head hkv) live. Token-major activations: K and V are [B*Tk, Hkv*D]
@@ -82,6 +86,15 @@ cudaError_t launch_attn_decode(const __nv_bfloat16* q, int64_t ldq, const __nv_b
                                int len, int len_add, int B, int H, int Hkv, int D, float scale, int n_splits,
                                float* part_o, float* part_ml, __nv_bfloat16* out, int64_t ldo, cudaStream_t stream);
 
+struct DecodeScores {
+  float softcap = 0.f;                      // > 0: scores become softcap * tanh(score / softcap)
+  const float* sink = nullptr;              // [H] fp32: exp(sink[h]) joins the denominator of head h
+  // pool > 0 (with a window, no kept first keys): besides the window one mean row per block of `pool` tokens wholly before it is seen;
+  // pooled [n_pages, ceil(page_size / pool), width], a block's row in the page of its last token, in order. Not with a soft cap.
+  const __nv_bfloat16* pooled = nullptr;
+  int pool = 0;
+};
+
 // The same decode attention over a PAGED cache: pool [n_pages, page_size, width] bf16 with width = 2 * Hkv * D (K of
 // every kv head, then V), block_table [max_seqs, max_pages] int32, seq_ids [B], seq_lens [max_seqs] (device); the
 // number of valid keys of a sequence is seq_lens[seq] + len_add (len_add = 1 when the new token's row has been written
@@ -91,7 +104,7 @@ cudaError_t launch_attn_decode_paged(const __nv_bfloat16* q, int64_t ldq, const 
                                      const int* block_table, const int* seq_ids, const int* seq_lens, int len_add,
                                      int page_size, int max_pages, int B, int H, int Hkv, int D, float scale, int n_splits,
                                      float* part_o, float* part_ml, __nv_bfloat16* out, int64_t ldo, cudaStream_t stream,
-                                     int window = 0, int keep_first = 0, int DV = 0);
+                                     int window = 0, int keep_first = 0, int DV = 0, const DecodeScores& sc = DecodeScores{});
 
 // dst[r, c] (bf16, row stride ldd) = src[r, c] (fp32, row stride lds), for an M x N block.
 // In-place elementwise step of the recomputed attention backward: s [rows, kv] bf16 scores -> probabilities,

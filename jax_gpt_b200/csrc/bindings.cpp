@@ -54,7 +54,7 @@ Tensor status(int64_t device) { return status_tensor(static_cast<int>(device)); 
 // out[M,N] = epilogue(alpha * A @ B^T ...). a: [M,K] (or [K,M] if a_mn_major); b: [N,K] (or [K,N]).
 void gemm(const Tensor& a, bool a_mn_major, const Tensor& b, bool b_mn_major, Tensor out,
           const c10::optional<Tensor>& bias, const c10::optional<Tensor>& residual, const c10::optional<Tensor>& aux,
-          int64_t epilogue, int64_t out_mode, double alpha, int64_t split_k) {
+          int64_t epilogue, int64_t out_mode, double alpha, int64_t split_k, double act_a, double act_b) {
   c10::cuda::CUDAGuard guard(a.device());
   check_bf16_2d(a, "a");
   check_bf16_2d(b, "b");
@@ -100,6 +100,8 @@ void gemm(const Tensor& a, bool a_mn_major, const Tensor& b, bool b_mn_major, Te
     g.ldaux = aux->stride(0);
   }
   g.alpha = static_cast<float>(alpha);
+  g.act_a = static_cast<float>(act_a);
+  g.act_b = static_cast<float>(act_b);
   g.split_k = static_cast<int>(split_k);
   g.status = status_ptr(a);
   B200_CHECK_CUDA(b200::launch_gemm_bf16(bf16_ptr(a), a.stride(0), a_mn_major ? 1 : 0, bf16_ptr(b), b.stride(0),
@@ -318,7 +320,7 @@ void adamw_bf16_state(Tensor p, Tensor g, Tensor m, Tensor v, const Tensor& hp, 
 // q/k/v: 2-D bf16 views [B*T, H*D] (possibly column slices of one fused buffer).
 void attn_fwd(const Tensor& q, const Tensor& k, const Tensor& v, Tensor out, Tensor lse, int64_t B, int64_t T,
               int64_t H, int64_t Hkv, int64_t D, double scale, bool causal, int64_t Dv, const c10::optional<Tensor>& sink,
-              int64_t window, int64_t keep_first) {
+              int64_t window, int64_t keep_first, double softcap, int64_t pool, int64_t pool_rows) {
   c10::cuda::CUDAGuard guard(q.device());
   check_bf16_2d(q, "q");
   check_bf16_2d(k, "k");
@@ -333,6 +335,11 @@ void attn_fwd(const Tensor& q, const Tensor& k, const Tensor& v, Tensor out, Ten
   }
   s.window = static_cast<int>(std::min<int64_t>(window, 1 << 30));
   s.keep_first = static_cast<int>(std::min<int64_t>(keep_first, 1 << 30));
+  s.softcap = static_cast<float>(softcap);
+  s.pool = static_cast<int>(pool);
+  s.pool_rows = static_cast<int>(pool_rows);
+  TORCH_CHECK(pool >= 0 && pool_rows >= 0 && (pool > 0 || pool_rows == 0) && k.size(0) >= B * (pool_rows + T) && v.size(0) >= B * (pool_rows + T) &&
+                  q.size(0) >= B * T, "attn_fwd: q [B T, H D], k and v [B (pool_rows + T), Hkv D]");
   B200_CHECK_CUDA(b200::launch_attn_fwd(t, s, bf16_mut(out), out.stride(0), lse.data_ptr<float>(), status_ptr(q),
                                         cur_stream()));
 }
@@ -454,7 +461,8 @@ void attn_decode(const Tensor& q, const Tensor& kcache, const Tensor& vcache, co
 // then V), block_table [max_seqs, max_pages] / seq_ids [B] / seq_lens [max_seqs] int32 on the device.
 void attn_decode_paged(const Tensor& q, const Tensor& pool, const Tensor& block_table, const Tensor& seq_ids,
                        const Tensor& seq_lens, int64_t len_add, int64_t H, int64_t Hkv, double scale, Tensor part_o,
-                       Tensor part_ml, Tensor out, int64_t window, int64_t keep_first) {
+                       Tensor part_ml, Tensor out, int64_t window, int64_t keep_first, double softcap,
+                       const c10::optional<Tensor>& sink, const c10::optional<Tensor>& pooled, int64_t pool_block) {
   c10::cuda::CUDAGuard guard(q.device());
   check_bf16_2d(q, "q");
   check_bf16_2d(out, "out");
@@ -470,6 +478,19 @@ void attn_decode_paged(const Tensor& q, const Tensor& pool, const Tensor& block_
                   part_ml.is_contiguous() && part_o.dim() == 4 && part_o.size(0) >= B && part_o.size(1) == H &&
                   part_o.size(3) == DV && part_ml.numel() * DV == part_o.numel() * 2,
               "attn_decode_paged: part_o [B, H, splits, DV], part_ml [B, H, splits, 2] fp32");
+  b200::DecodeScores sc;
+  sc.softcap = static_cast<float>(softcap);
+  if (sink.has_value()) {
+    TORCH_CHECK(sink->is_cuda() && sink->scalar_type() == at::kFloat && sink->numel() == H, "attn_decode_paged: sink is [H] fp32");
+    sc.sink = sink->data_ptr<float>();
+  }
+  if (pooled.has_value()) {
+    TORCH_CHECK(pool_block >= 1 && pooled->dim() == 3 && pooled->is_contiguous() && pooled->scalar_type() == at::kBFloat16 && pooled->size(0) == pool.size(0) &&
+                    pooled->size(1) == (pool.size(1) + pool_block - 1) / pool_block && pooled->size(2) == pool.size(2),
+                "attn_decode_paged: pooled [n_pages, ceil(page_size / pool), width]");
+    sc.pooled = bf16_ptr(*pooled);
+    sc.pool = static_cast<int>(pool_block);
+  }
   B200_CHECK_CUDA(b200::launch_attn_decode_paged(
       bf16_ptr(q), q.stride(0), bf16_ptr(pool), static_cast<int>(pool.size(2)), block_table.data_ptr<int>(),
       seq_ids.data_ptr<int>(), seq_lens.data_ptr<int>(), static_cast<int>(len_add), static_cast<int>(pool.size(1)),
@@ -477,7 +498,7 @@ void attn_decode_paged(const Tensor& q, const Tensor& pool, const Tensor& block_
       static_cast<int>(D), static_cast<float>(scale), static_cast<int>(part_o.size(2)), part_o.data_ptr<float>(),
       part_ml.data_ptr<float>(), bf16_mut(out), out.stride(0), cur_stream(),
       static_cast<int>(std::min<int64_t>(window, 1 << 30)), static_cast<int>(std::min<int64_t>(keep_first, 1 << 30)),
-      static_cast<int>(DV)));
+      static_cast<int>(DV), sc));
 }
 
 void attn_bwd_probs(Tensor s, Tensor dp, const Tensor& lse, const Tensor& delta, int64_t c, int64_t q0, double scale,
@@ -515,7 +536,7 @@ TORCH_LIBRARY(b200, m) {
   m.def("status(int device) -> Tensor", &status);
   m.def(
       "gemm(Tensor a, bool a_mn_major, Tensor b, bool b_mn_major, Tensor(a!) out, Tensor? bias, Tensor? residual, "
-      "Tensor? aux, int epilogue, int out_mode, float alpha, int split_k) -> ()",
+      "Tensor? aux, int epilogue, int out_mode, float alpha, int split_k, float act_a=0.0, float act_b=0.0) -> ()",
       &gemm);
   m.def(
       "gemm_gathered_a_staged(int[] gather_ptrs, int[] ready_ptrs, int rows_per_src, int K, int rank, Tensor b, "
@@ -549,7 +570,8 @@ TORCH_LIBRARY(b200, m) {
       &adamw);
   m.def(
       "attn_fwd(Tensor q, Tensor k, Tensor v, Tensor(a!) out, Tensor(b!) lse, int B, int T, int H, int Hkv, int D, "
-      "float scale, bool causal, int Dv, Tensor? sink=None, int window=0, int keep_first=0) -> ()",
+      "float scale, bool causal, int Dv, Tensor? sink=None, int window=0, int keep_first=0, float softcap=0.0, int pool=0, "
+      "int pool_rows=0) -> ()",
       &attn_fwd);
   m.def(
       "attn_bwd(Tensor q, Tensor k, Tensor v, Tensor out, Tensor dout, Tensor lse, Tensor(a!) delta, Tensor(b!) "
@@ -575,7 +597,8 @@ TORCH_LIBRARY(b200, m) {
       &attn_decode);
   m.def(
       "attn_decode_paged(Tensor q, Tensor pool, Tensor block_table, Tensor seq_ids, Tensor seq_lens, int len_add, int H, "
-      "int Hkv, float scale, Tensor(a!) part_o, Tensor(b!) part_ml, Tensor(c!) out, int window=0, int keep_first=0) -> ()",
+      "int Hkv, float scale, Tensor(a!) part_o, Tensor(b!) part_ml, Tensor(c!) out, int window=0, int keep_first=0, "
+      "float softcap=0.0, Tensor? sink=None, Tensor? pooled=None, int pool_block=0) -> ()",
       &attn_decode_paged);
   m.def("attn_bwd_probs(Tensor(a!) s, Tensor(b!) dp, Tensor lse, Tensor delta, int c, int q0, float scale, bool causal) -> ()", &attn_bwd_probs);
   m.def("norm_bwd_scratch_floats(int D) -> int", [](int64_t D) { return b200::norm_bwd_scratch_floats(static_cast<int>(D)); });

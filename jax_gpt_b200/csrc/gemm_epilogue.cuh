@@ -7,6 +7,11 @@
 
 namespace b200 {
 
+// exp(z) - 1 - z is off by a rounding of 1 at most, far below a bf16 step of z / 2 wherever that matters.
+__device__ __forceinline__ float xielu(float z, float a, float b) {
+  return fmaf(0.5f, z, z > 0.f ? a * z * z : b * (__expf(z) - 1.f - z));
+}
+
 // v: the 32 fp32 accumulator values of row `row`, columns [col0, col0 + 32); ks: the tile's K split
 // (bias and residual are added by split 0 only).
 __device__ __forceinline__ void gemm_epilogue_chunk(const GemmArgs& args, const uint32_t (&v)[32], int row, int col0,
@@ -105,6 +110,10 @@ _Pragma("unroll") for (int j = 0; j < 32; ++j)
   if (args.epilogue == kEpiSilu) {
 #pragma unroll
     for (int j = 0; j < 32; ++j) f[j] = __fdividef(f[j], 1.f + __expf(-f[j]));
+  }
+  if (args.epilogue == kEpiXielu) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) f[j] = xielu(f[j], args.act_a, args.act_b);
   }
   if (args.residual != nullptr && ks == 0) {
     const __nv_bfloat16* res = args.residual + static_cast<int64_t>(row) * args.ldr + col0;
@@ -273,6 +282,10 @@ __device__ __forceinline__ void gemm_epilogue_group64(const GemmArgs& args, uint
     if (args.epilogue == kEpiSilu) {
 #pragma unroll
       for (int j = 0; j < 32; ++j) f[j] = __fdividef(f[j], 1.f + __expf(-f[j]));
+    }
+    if (args.epilogue == kEpiXielu) {
+#pragma unroll
+      for (int j = 0; j < 32; ++j) f[j] = xielu(f[j], args.act_a, args.act_b);
     }
 #pragma unroll
     for (int j = 0; j < 32; j += 8) {

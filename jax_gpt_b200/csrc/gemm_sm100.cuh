@@ -14,6 +14,7 @@ enum GemmEpilogue : int {
   kEpiSiluMul = 3,   // reserved for SwiGLU-style epilogues
   kEpiRelu2 = 4,     // out = max(acc + bias, 0)^2
   kEpiSilu = 5,      // out = silu(acc + bias)
+  kEpiXielu = 6,     // z = acc + bias; out = act_a z^2 + z / 2 for z > 0, act_b (exp(z) - 1 - z) + z / 2 otherwise
 };
 enum GemmOut : int {
   kOutBf16 = 0,       // store bf16
@@ -39,6 +40,7 @@ struct GemmArgs {
   int epilogue;
   int out_mode;
   float alpha;
+  float act_a, act_b;             // kEpiXielu
   int split_k;
   int* status;
   // kOutBf16PeerRed: rows [r*rows_per_peer, (r+1)*rows_per_peer) of the logical output live

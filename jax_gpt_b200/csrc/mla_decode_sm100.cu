@@ -113,9 +113,10 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap t_pool, const __grid_const
   const int split = blockIdx.x, hb = blockIdx.y, b = blockIdx.z;
   const int sid = a.seq_ids[b];
   const int len = a.seq_lens[sid];
-  const int n_tiles = (len + kTile - 1) / kTile;
-  const int t0 = static_cast<int>(static_cast<int64_t>(n_tiles) * split / a.n_splits);
-  const int t1 = static_cast<int>(static_cast<int64_t>(n_tiles) * (split + 1) / a.n_splits);
+  const int first = a.window > 0 ? max(0, len - a.window) : 0;   // first token seen
+  const int tile0 = first / kTile, n_tiles = (len + kTile - 1) / kTile - tile0;
+  const int t0 = tile0 + static_cast<int>(static_cast<int64_t>(n_tiles) * split / a.n_splits);
+  const int t1 = tile0 + static_cast<int>(static_cast<int64_t>(n_tiles) * (split + 1) / a.n_splits);
   const int n_it = t1 - t0;
   const int h0 = hb * kHeads;
 
@@ -278,7 +279,8 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap t_pool, const __grid_const
         uint32_t v[kHeads];
         tmem_ld_cols<kHeads>(tmem + Cfg::kColS + g * kHeads + lane_off, v);
         tmem_ld_wait();
-        const bool valid = lane < 16 && (t0 + it) * kTile + row < len;
+        const int tok = (t0 + it) * kTile + row;
+        const bool valid = lane < 16 && tok < len && tok >= first;
 #pragma unroll
         for (int h = 0; h < kHeads; ++h) s[h] = valid ? __uint_as_float(v[h]) * a.scale_log2 : -INFINITY;
         float mine = -INFINITY;

@@ -25,6 +25,7 @@ struct MlaDecodeArgs {
   float* part_lse;                // [batch, 2 * n_splits, heads] log2-sum-exp of each partial (-inf when empty)
   int* status;
   const float* sink = nullptr;    // [heads] fp32 or nullptr: exp(sink[h]) joins the softmax denominator of head h
+  int window = 0;                 // > 0: only the last `window` tokens are seen
 };
 
 // q [batch * heads, 576] bf16 (absorbed nope part | rotated rope part); pool: one layer of the page pool,

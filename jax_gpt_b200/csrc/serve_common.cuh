@@ -2,6 +2,7 @@
 #pragma once
 #include "common.cuh"
 #include "serve_kernels.cuh"
+#include "softcap.cuh"
 
 namespace b200 {
 
@@ -76,20 +77,9 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
-// Single-instruction approximations (about 2^-22 relative, denormals flushed) for kernels that name them.
-__device__ __forceinline__ float ex2_approx(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 __device__ __forceinline__ float lg2_approx(float x) {
   float y;
   asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ float rcp_approx(float x) {
-  float y;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
 __device__ __forceinline__ float sqrt_approx(float x) {
@@ -115,6 +105,18 @@ __device__ __forceinline__ int64_t page_row(const PagedRows& pg, int slot, int p
   if (page < 0 || page >= pg.n_pages) return -1;
   return static_cast<int64_t>(page) * pg.page_size + pos % pg.page_size;
 }
+
+// Row of the mean of positions b P .. b P + P - 1 in a pool of such rows: it lies in the page of its last token, whose rows
+// [page, 0 .. ceil(page_size / P)) hold the blocks that end there in order. -1: no such page.
+__device__ __forceinline__ int64_t pooled_row(const PagedRows& pg, int P, int slot, int b) {
+  const int pi = (b * P + P - 1) / pg.page_size;
+  if (pi >= pg.max_pages) return -1;
+  const int page = pg.block_table[static_cast<int64_t>(slot) * pg.max_pages + pi];
+  if (page < 0 || page >= pg.n_pages) return -1;
+  return static_cast<int64_t>(page) * ((pg.page_size + P - 1) / P) + b - pi * pg.page_size / P;
+}
+// Blocks of P tokens that lie wholly before the window of a query at `pos`.
+__device__ __forceinline__ int blocks_seen(int pos, int window, int P) { return max(0, pos - window + 1) / P; }
 
 // Opts a kernel into `bytes` of dynamic shared memory once per new maximum.
 template <typename K>

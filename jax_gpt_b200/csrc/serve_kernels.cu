@@ -242,12 +242,13 @@ void residual_norm_go(const TY* y, const float* gpost, float* x, int add, const 
 // ---- few-row linear ------------------------------------------------------------------------------------------------
 constexpr int kLinWarps = 8;
 
-__device__ __forceinline__ float row_act(float v, int act) {
-  if (act == kActRelu2) {
+__device__ __forceinline__ float row_act(float v, const RowsOut& o) {
+  if (o.act == kActRelu2) {
     const float r = fmaxf(v, 0.f);
     return r * r;
   }
-  if (act == kActSilu) return silu_f(v);
+  if (o.act == kActSilu) return silu_f(v);
+  if (o.act == kActXielu) return (v > 0.f ? o.act_a * v * v : o.act_b * (expm1f(v) - v)) + 0.5f * v;
   return v;
 }
 
@@ -257,7 +258,7 @@ __device__ __forceinline__ void rows_store(const RowsOut& o, int m, int n, float
     o.y2[static_cast<int64_t>(m) * o.ldy2 + n - o.n1] = v;
     return;
   }
-  v = row_act(v, o.act);
+  v = row_act(v, o);
   const int64_t i = static_cast<int64_t>(m) * o.ldy + n;
   if (o.out_mode == 0) stf(static_cast<T*>(o.y) + i, v);
   else if (o.out_mode == 1) static_cast<float*>(o.y)[i] = v;
@@ -474,7 +475,7 @@ __global__ void mla_prepare_kernel(const SeqBatch sb, const T* __restrict__ y, i
   float sq = 0.f, sk = 0.f;
   for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = ldf(row + i); sq += v * v; }
   for (int i = threadIdx.x; i < R; i += blockDim.x) { const float v = ldf(kv + i); sk += v * v; }
-  const float iq = 1.f / sqrtf(block_sum(sq, red) / q_rank + eps);
+  const float iq = q_rank > 0 ? 1.f / sqrtf(block_sum(sq, red) / q_rank + eps) : 0.f;
   const float ik = 1.f / sqrtf(block_sum(sk, red) / R + eps);
   for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
     stf(cq + static_cast<int64_t>(n) * q_rank + i, ldf(row + i) * iq * q_gamma[i]);
@@ -496,14 +497,14 @@ __global__ void mla_prepare_kernel(const SeqBatch sb, const T* __restrict__ y, i
 
 // One block per token: query heads rotated in place, keys assembled.
 template <typename T>
-__global__ void mla_rope_qk_kernel(const SeqBatch sb, T* __restrict__ q, const T* __restrict__ kn, int64_t ldkn,
+__global__ void mla_rope_qk_kernel(const SeqBatch sb, T* __restrict__ q, int64_t ldq, const T* __restrict__ kn, int64_t ldkn,
                                    const T* __restrict__ lat, int64_t ldlat, int R, T* __restrict__ k, int H, int dn, int dr,
                                    const RopeTable rope) {
   const int n = blockIdx.x;
   const int b = sb.tok_seq[n];
   const int pos = sb.start[b] + n - sb.cu[b];
   const int half = rope.dims / 2, D = dn + dr;
-  T* qr = q + static_cast<int64_t>(n) * H * D;
+  T* qr = q + static_cast<int64_t>(n) * ldq;
   for (int i = threadIdx.x; i < H * half; i += blockDim.x) {
     const int h = i / half, j = i % half;
     const float c = rope.cos[static_cast<int64_t>(pos) * half + j], s = rope.sin[static_cast<int64_t>(pos) * half + j];
@@ -537,14 +538,14 @@ constexpr int kAbsCols = 64;  // latent columns per block of the query absorptio
 // the warps split the contraction over dn; partial sums meet in shuffles and in shared memory.
 template <typename T, bool kVec>
 __global__ void __launch_bounds__(256)
-mla_absorb_q_kernel(const SeqBatch sb, const T* __restrict__ q, const T* __restrict__ w_uk, T* __restrict__ qf, int H, int dn,
+mla_absorb_q_kernel(const SeqBatch sb, const T* __restrict__ q, int64_t ldq, const T* __restrict__ w_uk, T* __restrict__ qf, int H, int dn,
                     int dr, int R, const RopeTable rope) {
   extern __shared__ float sm[];   // [kAbsTok][dn + dr], then [8 warps][kAbsTok][kAbsCols]
   const int D = dn + dr, h = blockIdx.y, n0 = blockIdx.x * kAbsTok;
   float* red = sm + kAbsTok * D;
   const int cnt = min(kAbsTok, sb.n_tok - n0);
   for (int i = threadIdx.x; i < kAbsTok * D; i += blockDim.x)
-    sm[i] = i < cnt * D ? ldf(q + (static_cast<int64_t>(n0 + i / D) * H + h) * D + i % D) : 0.f;
+    sm[i] = i < cnt * D ? ldf(q + static_cast<int64_t>(n0 + i / D) * ldq + h * D + i % D) : 0.f;
   __syncthreads();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int c0 = blockIdx.z * kAbsCols + (lane & 7) * 8, dg = warp * 4 + (lane >> 3);   // 32 slices of dn
@@ -614,8 +615,8 @@ mla_absorb_q_kernel(const SeqBatch sb, const T* __restrict__ q, const T* __restr
 // A warp computes one value feature of a head for up to 8 tokens; lanes stride the latent.
 template <typename T, bool kVec>
 __global__ void __launch_bounds__(256)
-mla_absorb_out_kernel(const T* __restrict__ o_lat, const T* __restrict__ w_uv, T* __restrict__ o, int n_tok, int H, int dv,
-                      int R) {
+mla_absorb_out_kernel(const T* __restrict__ o_lat, const T* __restrict__ w_uv, const T* __restrict__ gate, int64_t ldg,
+                      T* __restrict__ o, int n_tok, int H, int dv, int R) {
   extern __shared__ float sm[];   // [kAbsTok][R]
   const int h = blockIdx.y, n0 = blockIdx.x * kAbsTok;
   const int cnt = min(kAbsTok, n_tok - n0);
@@ -662,8 +663,35 @@ mla_absorb_out_kernel(const T* __restrict__ o_lat, const T* __restrict__ w_uv, T
     }
 #pragma unroll
     for (int t = 0; t < kAbsTok; ++t) {
-      const float s = warp_sum(acc[t]);
-      if (lane == t && t < cnt) stf(o + (static_cast<int64_t>(n0 + t) * H + h) * dv + v, s);
+      float s = warp_sum(acc[t]);
+      if (lane == t && t < cnt) {
+        if (gate != nullptr) s *= sigmoid_f(ldf(gate + (n0 + t) * ldg + h * dv + v));
+        stf(o + (static_cast<int64_t>(n0 + t) * H + h) * dv + v, s);
+      }
+    }
+  }
+}
+
+// o *= sigmoid(gate), rows of N features; kVec: a 16-byte vector of features per thread and step.
+template <typename T, bool kVec>
+__global__ void __launch_bounds__(256)
+sigmoid_gate_kernel(T* __restrict__ o, const T* __restrict__ gate, int64_t ldg, int64_t total, int N) {
+  constexpr int V = kVec ? Vec16<T>::n : 1;
+  for (int64_t i = (static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x) * V; i < total;
+       i += static_cast<int64_t>(gridDim.x) * blockDim.x * V) {
+    const T* g = gate + i / N * ldg + i % N;
+    if constexpr (kVec) {
+      float a[V], b[V];
+      Vec16<T>::load(o + i, a);
+      Vec16<T>::load(g, b);
+#pragma unroll
+      for (int j = 0; j < V; ++j) a[j] *= sizeof(T) == 2 ? sigmoid_approx(b[j]) : sigmoid_f(b[j]);
+      if constexpr (sizeof(T) == 2)
+        *reinterpret_cast<uint4*>(o + i) = make_uint4(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]), pack_bf16x2(a[4], a[5]), pack_bf16x2(a[6], a[7]));
+      else
+        *reinterpret_cast<float4*>(o + i) = make_float4(a[0], a[1], a[2], a[3]);
+    } else {
+      stf(o + i, ldf(o + i) * sigmoid_f(ldf(g)));
     }
   }
 }
@@ -677,7 +705,7 @@ constexpr int kLaQ = 8, kLaK = 32, kLaWarps = 4, kLaMine = kLaQ / kLaWarps;
 template <typename T>
 __global__ void __launch_bounds__(kLaWarps * 32)
 latent_attn_kernel(const SeqBatch sb, const T* __restrict__ qf, const PagedRows pages, int R,
-                   const float* __restrict__ sink, float scale, int H, float* __restrict__ part_o,
+                   const float* __restrict__ sink, float scale, int window, int H, float* __restrict__ part_o,
                    float* __restrict__ part_ml, T* __restrict__ o_lat) {
   extern __shared__ float sm[];
   const int W = pages.width, WS = W | 1;   // odd stride: lanes read a column of keys without bank conflicts
@@ -702,8 +730,9 @@ latent_attn_kernel(const SeqBatch sb, const T* __restrict__ qf, const PagedRows 
   const int slot = sb.ids[b], start = sb.start[b];
   const int64_t g0 = static_cast<int64_t>(sb.cu[b]) * H + r0;   // first pair in the packed arrays
   const int n_keys = start + (r0 + cnt - 1) / H + 1;
-  const int tiles_k = (n_keys + kLaK - 1) / kLaK, per = (tiles_k + S - 1) / S;
-  const int kt0 = split * per, kt1 = min(tiles_k, kt0 + per);
+  const int tile0 = max(0, start + r0 / H - window + 1) / kLaK;   // from the window of the first query on
+  const int tiles_k = (n_keys + kLaK - 1) / kLaK, per = (tiles_k - tile0 + S - 1) / S;
+  const int kt0 = tile0 + split * per, kt1 = min(tiles_k, kt0 + per);
   for (int i = threadIdx.x; i < kLaQ * W; i += blockDim.x) sq[i] = i < cnt * W ? ldf(qf + g0 * W + i) : 0.f;
   for (int i = threadIdx.x; i < kLaQ * R; i += blockDim.x) so[i] = 0.f;
   float m[kLaMine], l[kLaMine];
@@ -747,7 +776,8 @@ latent_attn_kernel(const SeqBatch sb, const T* __restrict__ qf, const PagedRows 
     float a[kLaMine];
 #pragma unroll
     for (int j = 0; j < kLaMine; ++j) {
-      const float sc = kt * kLaK + lane <= pos[j] ? s[j] * scale : -INFINITY;
+      const int kp = kt * kLaK + lane;
+      const float sc = kp <= pos[j] && pos[j] - kp < window ? s[j] * scale : -INFINITY;
       const float mn = fmaxf(m[j], warp_max(sc));
       const float ref = mn == -INFINITY ? 0.f : mn;   // nothing seen yet: every weight below is 0
       const float p = expf(sc - ref);
@@ -1055,19 +1085,19 @@ int threads_for(int n) { return n >= 1024 ? 256 : (n >= 256 ? 128 : 64); }
 
 template <typename T>
 cudaError_t latent_attention_t(const SeqBatch& sb, const T* qf, const PagedRows& pages, int R, const float* sink, float scale,
-                               int H, int n_splits, float* part_o, float* part_ml, T* o_lat, cudaStream_t st) {
+                               int window, int H, int n_splits, float* part_o, float* part_ml, T* o_lat, cudaStream_t st) {
   static int have = 0;
   const int smem = 4 * (kLaK * (pages.width + 1) + kLaQ * pages.width + kLaQ * R + kLaQ * kLaK);
   cudaError_t e = want_smem(latent_attn_kernel<T>, smem, have);
   if (e != cudaSuccess) return e;
   const dim3 grid(static_cast<unsigned>(static_cast<int64_t>(sb.n_tok) * H / kLaQ + sb.n_seq), n_splits);
-  latent_attn_kernel<T><<<grid, kLaWarps * 32, smem, st>>>(sb, qf, pages, R, sink, scale, H, part_o, part_ml, o_lat);
+  latent_attn_kernel<T><<<grid, kLaWarps * 32, smem, st>>>(sb, qf, pages, R, sink, scale, window, H, part_o, part_ml, o_lat);
   if (n_splits > 1) latent_merge_kernel<T><<<sb.n_tok * H, 128, 0, st>>>(part_o, part_ml, sink, H, R, n_splits, o_lat);
   return cudaGetLastError();
 }
 
 template <typename T>
-cudaError_t absorb_q_t(const SeqBatch& sb, const T* q, const T* w_uk, T* qf, int H, int dn, int dr, int R,
+cudaError_t absorb_q_t(const SeqBatch& sb, const T* q, int64_t ldq, const T* w_uk, T* qf, int H, int dn, int dr, int R,
                        const RopeTable& rope, cudaStream_t st) {
   static int have_v = 0, have_s = 0;
   const int smem = 4 * (kAbsTok * (dn + dr) + 8 * kAbsTok * kAbsCols);
@@ -1075,13 +1105,13 @@ cudaError_t absorb_q_t(const SeqBatch& sb, const T* q, const T* w_uk, T* qf, int
   cudaError_t e = vec ? want_smem(mla_absorb_q_kernel<T, true>, smem, have_v) : want_smem(mla_absorb_q_kernel<T, false>, smem, have_s);
   if (e != cudaSuccess) return e;
   const dim3 grid((sb.n_tok + kAbsTok - 1) / kAbsTok, H, (R + kAbsCols - 1) / kAbsCols);
-  if (vec) mla_absorb_q_kernel<T, true><<<grid, 256, smem, st>>>(sb, q, w_uk, qf, H, dn, dr, R, rope);
-  else mla_absorb_q_kernel<T, false><<<grid, 256, smem, st>>>(sb, q, w_uk, qf, H, dn, dr, R, rope);
+  if (vec) mla_absorb_q_kernel<T, true><<<grid, 256, smem, st>>>(sb, q, ldq, w_uk, qf, H, dn, dr, R, rope);
+  else mla_absorb_q_kernel<T, false><<<grid, 256, smem, st>>>(sb, q, ldq, w_uk, qf, H, dn, dr, R, rope);
   return cudaGetLastError();
 }
 
 template <typename T>
-cudaError_t absorb_out_t(const T* o_lat, const T* w_uv, T* o, int n_tok, int H, int dv, int R, cudaStream_t st) {
+cudaError_t absorb_out_t(const T* o_lat, const T* w_uv, const T* gate, int64_t ldg, T* o, int n_tok, int H, int dv, int R, cudaStream_t st) {
   static int have_v = 0, have_s = 0;
   const int smem = 4 * kAbsTok * R;
   const bool vec = R % Vec16<T>::n == 0 && ((reinterpret_cast<uintptr_t>(w_uv) | reinterpret_cast<uintptr_t>(o_lat)) & 15) == 0;
@@ -1090,8 +1120,8 @@ cudaError_t absorb_out_t(const T* o_lat, const T* w_uv, T* o, int n_tok, int H, 
   const int tiles = (n_tok + kAbsTok - 1) / kAbsTok;
   const int per = (dv + 7) / 8, z = tiles * H < 148 ? (per < 16 ? per : 16) : 1;
   const dim3 grid(tiles, H, z);
-  if (vec) mla_absorb_out_kernel<T, true><<<grid, 256, smem, st>>>(o_lat, w_uv, o, n_tok, H, dv, R);
-  else mla_absorb_out_kernel<T, false><<<grid, 256, smem, st>>>(o_lat, w_uv, o, n_tok, H, dv, R);
+  if (vec) mla_absorb_out_kernel<T, true><<<grid, 256, smem, st>>>(o_lat, w_uv, gate, ldg, o, n_tok, H, dv, R);
+  else mla_absorb_out_kernel<T, false><<<grid, 256, smem, st>>>(o_lat, w_uv, gate, ldg, o, n_tok, H, dv, R);
   return cudaGetLastError();
 }
 
@@ -1163,41 +1193,53 @@ cudaError_t launch_mla_prepare(bool f32, const SeqBatch& sb, const void* y, int6
   return cudaGetLastError();
 }
 
-cudaError_t launch_mla_rope_qk(bool f32, const SeqBatch& sb, void* q, const void* kn, int64_t ldkn, const void* lat,
+cudaError_t launch_mla_rope_qk(bool f32, const SeqBatch& sb, void* q, int64_t ldq, const void* kn, int64_t ldkn, const void* lat,
                                int64_t ldlat, int R, void* k, int H, int dn, int dr, const RopeTable& rope, cudaStream_t st) {
   if (f32)
-    mla_rope_qk_kernel<float><<<sb.n_tok, 256, 0, st>>>(sb, static_cast<float*>(q), static_cast<const float*>(kn), ldkn,
+    mla_rope_qk_kernel<float><<<sb.n_tok, 256, 0, st>>>(sb, static_cast<float*>(q), ldq, static_cast<const float*>(kn), ldkn,
                                                         static_cast<const float*>(lat), ldlat, R, static_cast<float*>(k), H, dn, dr, rope);
   else
     mla_rope_qk_kernel<__nv_bfloat16><<<sb.n_tok, 256, 0, st>>>(
-        sb, static_cast<__nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(kn), ldkn, static_cast<const __nv_bfloat16*>(lat),
+        sb, static_cast<__nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(kn), ldkn, static_cast<const __nv_bfloat16*>(lat),
         ldlat, R, static_cast<__nv_bfloat16*>(k), H, dn, dr, rope);
   return cudaGetLastError();
 }
 
-cudaError_t launch_mla_absorb_q(bool f32, const SeqBatch& sb, const void* q, const void* w_uk, void* qf, int H, int dn,
+cudaError_t launch_mla_absorb_q(bool f32, const SeqBatch& sb, const void* q, int64_t ldq, const void* w_uk, void* qf, int H, int dn,
                                 int dr, int R, const RopeTable& rope, cudaStream_t st) {
-  return f32 ? absorb_q_t<float>(sb, static_cast<const float*>(q), static_cast<const float*>(w_uk), static_cast<float*>(qf), H, dn,
+  return f32 ? absorb_q_t<float>(sb, static_cast<const float*>(q), ldq, static_cast<const float*>(w_uk), static_cast<float*>(qf), H, dn,
                                  dr, R, rope, st)
-             : absorb_q_t<__nv_bfloat16>(sb, static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(w_uk),
+             : absorb_q_t<__nv_bfloat16>(sb, static_cast<const __nv_bfloat16*>(q), ldq, static_cast<const __nv_bfloat16*>(w_uk),
                                          static_cast<__nv_bfloat16*>(qf), H, dn, dr, R, rope, st);
 }
 
-cudaError_t launch_mla_absorb_out(bool f32, const void* o_lat, const void* w_uv, void* o, int n_tok, int H, int dv, int R,
-                                  cudaStream_t st) {
-  return f32 ? absorb_out_t<float>(static_cast<const float*>(o_lat), static_cast<const float*>(w_uv), static_cast<float*>(o), n_tok,
-                                   H, dv, R, st)
+cudaError_t launch_mla_absorb_out(bool f32, const void* o_lat, const void* w_uv, const void* gate, int64_t ldg, void* o, int n_tok, int H,
+                                  int dv, int R, cudaStream_t st) {
+  return f32 ? absorb_out_t<float>(static_cast<const float*>(o_lat), static_cast<const float*>(w_uv), static_cast<const float*>(gate), ldg,
+                                   static_cast<float*>(o), n_tok, H, dv, R, st)
              : absorb_out_t<__nv_bfloat16>(static_cast<const __nv_bfloat16*>(o_lat), static_cast<const __nv_bfloat16*>(w_uv),
-                                           static_cast<__nv_bfloat16*>(o), n_tok, H, dv, R, st);
+                                           static_cast<const __nv_bfloat16*>(gate), ldg, static_cast<__nv_bfloat16*>(o), n_tok, H, dv, R, st);
+}
+
+cudaError_t launch_sigmoid_gate(bool f32, void* o, const void* gate, int64_t ldg, int rows, int N, cudaStream_t st) {
+  const int V = f32 ? 4 : 8;
+  const bool vec = N % V == 0 && ldg % V == 0 && ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate)) & 15) == 0;
+  const int64_t total = static_cast<int64_t>(rows) * N, blocks = (total / (vec ? V : 1) + 255) / 256;
+  const int grid = static_cast<int>(blocks < 148 * 16 ? (blocks < 1 ? 1 : blocks) : 148 * 16);
+#define B200_GATE(T, K) sigmoid_gate_kernel<T, K><<<grid, 256, 0, st>>>(static_cast<T*>(o), static_cast<const T*>(gate), ldg, total, N)
+  if (f32) { if (vec) B200_GATE(float, true); else B200_GATE(float, false); }
+  else { if (vec) B200_GATE(__nv_bfloat16, true); else B200_GATE(__nv_bfloat16, false); }
+#undef B200_GATE
+  return cudaGetLastError();
 }
 
 cudaError_t launch_latent_attention(bool f32, const SeqBatch& sb, const void* qf, const PagedRows& pages, int R,
-                                    const float* sink, float scale, int H, int n_splits, float* part_o, float* part_ml,
+                                    const float* sink, float scale, int window, int H, int n_splits, float* part_o, float* part_ml,
                                     void* o_lat, cudaStream_t st) {
-  if (n_splits < 1 || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr))) return cudaErrorInvalidValue;
-  return f32 ? latent_attention_t<float>(sb, static_cast<const float*>(qf), pages, R, sink, scale, H, n_splits, part_o, part_ml,
+  if (window < 1 || n_splits < 1 || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr))) return cudaErrorInvalidValue;
+  return f32 ? latent_attention_t<float>(sb, static_cast<const float*>(qf), pages, R, sink, scale, window, H, n_splits, part_o, part_ml,
                                          static_cast<float*>(o_lat), st)
-             : latent_attention_t<__nv_bfloat16>(sb, static_cast<const __nv_bfloat16*>(qf), pages, R, sink, scale, H, n_splits,
+             : latent_attention_t<__nv_bfloat16>(sb, static_cast<const __nv_bfloat16*>(qf), pages, R, sink, scale, window, H, n_splits,
                                                  part_o, part_ml, static_cast<__nv_bfloat16*>(o_lat), st);
 }
 

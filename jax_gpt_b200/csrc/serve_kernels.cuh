@@ -37,7 +37,8 @@ cudaError_t launch_norm_rows(bool f32_out, int mode, const float* x, const float
 cudaError_t launch_residual_norm(bool y_f32, bool f32_out, const void* y, const float* gpost, float* x, bool add,
                                  const float* gnext, void* out, int rows, int D, float eps, cudaStream_t st);
 
-enum RowAct : int { kActNone = 0, kActRelu2 = 1, kActSilu = 2, kActSiluGlu = 3 };
+// kActXielu: a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 otherwise
+enum RowAct : int { kActNone = 0, kActRelu2 = 1, kActSilu = 2, kActSiluGlu = 3, kActXielu = 4 };
 struct RowsOut {
   void* y;             // [M, ldy]
   int64_t ldy;
@@ -46,6 +47,7 @@ struct RowsOut {
   float* y2;           // features n >= n1 go to y2[m, n - n1] in fp32, without the activation (n1 = N: none do)
   int64_t ldy2;
   int n1;
+  float act_a, act_b;  // kActXielu
 };
 // y[m, n] = act(sum_k x[m, k] w[n, k]). Few rows.
 cudaError_t launch_rows_linear(bool f32, const void* x, int64_t ldx, const void* w, int64_t ldw, int M, int N, int K,
@@ -62,7 +64,7 @@ struct PagedRows {
   int page_size, max_pages, n_pages, width;
 };
 
-// y [n_tok, ldy] = [down-projected query: q_rank | compressed kv: R | rotary key: dr]. cq = RMS norm of the first
+// y [n_tok, ldy] = [down-projected query: q_rank (may be 0) | compressed kv: R | rotary key: dr]. cq = RMS norm of the first
 // part; the token's cache row becomes [RMS norm of the second | rotated third], also written to lat [n_tok, R + dr]
 // when that is not null.
 cudaError_t launch_mla_prepare(bool f32, const SeqBatch& sb, const void* y, int64_t ldy, int q_rank, int R, int dr,
@@ -71,21 +73,23 @@ cudaError_t launch_mla_prepare(bool f32, const SeqBatch& sb, const void* y, int6
 
 // Decompressed prefill operands: rotates the last dr features of every query head in place (q [n_tok, H, dn + dr])
 // and writes k [n_tok, H, dn + dr] = [kn | lat[:, R:]].
-cudaError_t launch_mla_rope_qk(bool f32, const SeqBatch& sb, void* q, const void* kn, int64_t ldkn, const void* lat,
+cudaError_t launch_mla_rope_qk(bool f32, const SeqBatch& sb, void* q, int64_t ldq, const void* kn, int64_t ldkn, const void* lat,
                                int64_t ldlat, int R, void* k, int H, int dn, int dr, const RopeTable& rope, cudaStream_t st);
 
-// qf [n_tok, H, R + dr] = [q_nope W_uk | rotated q_rope] with w_uk [H * dn, R].
-cudaError_t launch_mla_absorb_q(bool f32, const SeqBatch& sb, const void* q, const void* w_uk, void* qf, int H, int dn,
+// qf [n_tok, H, R + dr] = [q_nope W_uk | rotated q_rope] with w_uk [H * dn, R]; rows of q are ldq apart.
+cudaError_t launch_mla_absorb_q(bool f32, const SeqBatch& sb, const void* q, int64_t ldq, const void* w_uk, void* qf, int H, int dn,
                                 int dr, int R, const RopeTable& rope, cudaStream_t st);
-// o [n_tok, H * dv] = o_lat [n_tok, H, R] W_uv with w_uv [H * dv, R].
-cudaError_t launch_mla_absorb_out(bool f32, const void* o_lat, const void* w_uv, void* o, int n_tok, int H, int dv, int R,
-                                  cudaStream_t st);
+// o [n_tok, H * dv] = o_lat [n_tok, H, R] W_uv with w_uv [H * dv, R], times sigmoid(gate [n_tok, ldg]) unless that is null.
+cudaError_t launch_mla_absorb_out(bool f32, const void* o_lat, const void* w_uv, const void* gate, int64_t ldg, void* o, int n_tok, int H,
+                                  int dv, int R, cudaStream_t st);
+// o [rows, N] *= sigmoid(gate [rows, ldg]) in place.
+cudaError_t launch_sigmoid_gate(bool f32, void* o, const void* gate, int64_t ldg, int rows, int N, cudaStream_t st);
 
-// Causal softmax attention of qf over the pages: row n attends to positions 0 .. pos(n) of its sequence; values are
+// Causal softmax attention of qf over the pages: row n attends to the last `window` positions up to pos(n) of its sequence; values are
 // the first R features of a cached row; `sink` (optional, [H]) adds exp(sink) to every denominator. n_splits > 1
 // cuts the keys into ranges merged by a second kernel (part_o [n_tok, H, S, R], part_ml [n_tok, H, S, 2] fp32).
 cudaError_t launch_latent_attention(bool f32, const SeqBatch& sb, const void* qf, const PagedRows& pages, int R,
-                                    const float* sink, float scale, int H, int n_splits, float* part_o, float* part_ml,
+                                    const float* sink, float scale, int window, int H, int n_splits, float* part_o, float* part_ml,
                                     void* o_lat, cudaStream_t st);
 
 // Experts of a token: table[token, :top] (each with weight 1 / top), or with `logits` [M, E] fp32 the `top` largest, whose
@@ -119,6 +123,12 @@ cudaError_t launch_moe_combine_rows(const __nv_bfloat16* ys, const int* row_of, 
 // ---- windowed attention (window_attention.cu) ------------------------------------------------------------------------
 struct WindowMask {
   int size, keep_first;   // i sees j when j <= i and (i - j < size or j < keep_first); no window: size 1 << 30
+  int pool;               // > 0 (then keep_first 0): i also sees the mean of every block of `pool` tokens that lies wholly before its window
+};
+struct ScoreArgs {
+  float scale;
+  float softcap;          // > 0: scores become softcap * tanh(score / softcap)
+  const float* sink;      // optional [H]: exp(sink) joins the denominator, no key and no value
 };
 // y [n_tok, ldy] = [q of H heads | k of G heads], D wide. q [n_tok, H, D] = unit RMS norm of the rotated (y + bias); the
 // cache row becomes [k likewise | k as projected, the values]; both also go to k, v [n_tok, G, D] unless null. `rope` holds
@@ -126,11 +136,12 @@ struct WindowMask {
 cudaError_t launch_qk_prepare(bool f32, const SeqBatch& sb, const void* y, int64_t ldy, const float* bias, int H, int G, int D,
                               bool unit_norm, float eps, const RopeTable& rope, const PagedRows& pages, void* q, void* k, void* v,
                               int* status, cudaStream_t st);
-// Softmax attention of q [n_tok, H, D] over the pages' rows [K (G D) | V (G DV)] of G kv heads, any sizes. n_splits > 1 cuts the
-// visible keys into ranges merged by a second kernel (part_o [n_tok, H, S, DV], part_ml [n_tok, H, S, 2] fp32).
-cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, int H, int G, int D, int DV,
-                                    WindowMask mask, float scale, int n_splits, float* part_o, float* part_ml, void* out,
-                                    cudaStream_t st);
+// Softmax attention of q [n_tok, H, D] over the pages' rows [K (G D) | V (G DV)] of G kv heads, any sizes; `pooled` [n_pages,
+// ceil(page_size / pool), width] holds the block means. n_splits > 1 cuts the visible keys into ranges merged by a second kernel
+// (part_o [n_tok, H, S, DV], part_ml [n_tok, H, S, 2] fp32).
+cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, const void* pooled, int H, int G,
+                                    int D, int DV, WindowMask mask, const ScoreArgs& score, int n_splits, float* part_o, float* part_ml,
+                                    void* out, cudaStream_t st);
 
 // ---- interleaved rotation, rotated values (rotated_kv.cu) ----------------------------------------------------------------
 // Columns of a projection row and their biases ([heads * width] fp32 or null).
@@ -148,6 +159,29 @@ cudaError_t launch_qkv_rotate(bool f32, const SeqBatch& sb, const QkvRows& in, c
 // out[n, h * dv + c] = scale sigmoid(g[n, h]) (o [n_tok, H, ldh] turned back by the row's position).
 cudaError_t launch_turn_back_gate(bool f32, const SeqBatch& sb, const void* o, int ldh, const void* g, int64_t ldg, const RopeTable& vrope,
                                   float scale, int H, int dv, void* out, int64_t ldo, cudaStream_t st);
+
+// ---- grouped-query operands with mixed values and block means (mixed_kv.cu) ------------------------------------------------
+struct MixedKv {
+  QkvRows in;              // biases unused
+  const float* q_factor;   // optional [n_pos]: q is multiplied by the factor of its position
+  int n_pos;
+  const void* v_first;     // optional [n_tok, ld_first]: v becomes (1 - lambda) v + lambda v_first
+  int64_t ld_first;
+  float lambda;
+  int H, G, dk, dv;
+  int dkp, dvp;            // widths of the dense operands, features past dk / dv are zero
+  void* pooled;            // optional [n_pages, ceil(page_size / pool), width]: means of whole blocks of `pool` cache rows
+  int pool;
+  const int* row0;         // optional [n_seq]: row of a sequence's first token in dense k, v (null: its packed row)
+};
+// q [n_tok, H, dkp], the cache row [K (G dk) | V (G dv)] and, unless null, dense k [rows, G, dkp], v [rows, G, dvp]. With one token per
+// sequence the mean of a block is written with its last row; otherwise launch_pool_rows follows.
+cudaError_t launch_mixed_kv(bool f32, const SeqBatch& sb, const MixedKv& a, const PagedRows& pages, void* q, void* k, void* v, int* status,
+                            cudaStream_t st);
+// Means of the blocks that the step's rows complete. With `pad` [n_seq] they also go to the pad[b] dense rows before row0[b] (zeros
+// past the whole blocks); n_rows bounds the work: blocks, or blocks and dense rows, over all sequences.
+cudaError_t launch_pool_rows(bool f32, const SeqBatch& sb, const MixedKv& a, const PagedRows& pages, const int* pad, int n_rows, void* k,
+                             void* v, int* status, cudaStream_t st);
 
 // ---- residual streams and row activations (stream_kernels.cu) ------------------------------------------------------------
 constexpr int kMaxStreams = 16;

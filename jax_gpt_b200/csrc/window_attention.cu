@@ -1,5 +1,7 @@
 // Grouped-query attention with a sliding window and kept first tokens on packed batches over paged key / value rows:
-//   position i sees j when j <= i and (i - j < size or j < keep_first).
+//   position i sees j when j <= i and (i - j < size or j < keep_first),
+// or instead of the first tokens one mean key and value for every block of tokens that lies wholly before the window. Scores may be
+// soft-capped, the denominator may hold a sink.
 //
 // qk_prepare turns a projection row [q heads | k heads] into attention operands (bias, half-split rotation, unit RMS norm
 // per head) and writes the cache row [K of every kv head | V of every kv head]; the projected keys double as values.
@@ -179,8 +181,8 @@ __device__ __forceinline__ void stage_row(const T* __restrict__ src, bool live, 
 
 template <typename T>
 __global__ void __launch_bounds__(kWaWarps * 32)
-window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows pages, int H, int G, int D, int DV,
-                   WindowMask mask, float scale, float* __restrict__ part_o, float* __restrict__ part_ml, T* __restrict__ out) {
+window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows pages, const T* __restrict__ pooled, int H, int G, int D, int DV,
+                   WindowMask mask, const ScoreArgs score, float* __restrict__ part_o, float* __restrict__ part_ml, T* __restrict__ out) {
   extern __shared__ float sm[];
   const int DS = D | 1;                    // odd stride: lanes read a column of keys without bank conflicts
   float* sk = sm;                          // [kWaK][DS]
@@ -203,29 +205,34 @@ window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows 
   if (r0 < 0) return;
   const int slot = sb.ids[b], start = sb.start[b];
   const int p_lo = start + r0 / rep, p_hi = start + (r0 + cnt - 1) / rep;
-  // visible key tiles: the kept first keys, then from the window of the first query to the last query
-  const int n_keep = (min(mask.keep_first, p_hi + 1) + kWaK - 1) / kWaK;
-  const int w0 = max(n_keep, max(0, p_lo - mask.size + 1) / kWaK), w1 = p_hi / kWaK + 1;
+  // visible key tiles: the kept first keys or the block means, then from the window of the first query to the last query
+  const bool blocks = mask.pool > 0;
+  const int kept = blocks ? blocks_seen(p_hi, mask.size, mask.pool) : min(mask.keep_first, p_hi + 1);
+  const int n_keep = (kept + kWaK - 1) / kWaK;
+  const int w0 = max(blocks ? 0 : n_keep, max(0, p_lo - mask.size + 1) / kWaK), w1 = p_hi / kWaK + 1;
   const int n_tiles = n_keep + max(0, w1 - w0), per = (n_tiles + S - 1) / S;
   const int i0 = split * per, i1 = min(n_tiles, i0 + per);
   auto head = [&](int q) { return (static_cast<int64_t>(sb.cu[b] + (r0 + q) / rep) * H + g * rep + (r0 + q) % rep); };
   for (int i = threadIdx.x; i < kWaQ * D; i += blockDim.x) sq[i] = i / D < cnt ? ldf(qx + head(i / D) * D + i % D) : 0.f;
   for (int i = threadIdx.x; i < kWaQ * DV; i += blockDim.x) so[i] = 0.f;
   float m[kWaMine], l[kWaMine];
-  int pos[kWaMine];                        // position of the pair's token; -1: no pair
+  int pos[kWaMine], first[kWaMine];        // position of the pair's token (-1: no pair), blocks that it sees
 #pragma unroll
   for (int j = 0; j < kWaMine; ++j) {
     const int q = warp + j * kWaWarps;
     m[j] = -INFINITY;
     l[j] = 0.f;
     pos[j] = q < cnt ? start + (r0 + q) / rep : -1;
+    first[j] = blocks ? blocks_seen(pos[j], mask.size, mask.pool) : 0;
   }
   for (int it = i0; it < i1; ++it) {
     const int k0 = (it < n_keep ? it : w0 + it - n_keep) * kWaK;
+    const bool means = blocks && it < n_keep;
     __syncthreads();
     for (int k = warp; k < kWaK; k += kWaWarps) {
-      const int64_t row = k0 + k <= p_hi ? page_row(pages, slot, k0 + k) : -1;
-      const T* base = static_cast<const T*>(pages.pool) + (row < 0 ? 0 : row) * pages.width;
+      const int64_t row = means ? (k0 + k < kept ? pooled_row(pages, mask.pool, slot, k0 + k) : -1)
+                                : (k0 + k <= p_hi ? page_row(pages, slot, k0 + k) : -1);
+      const T* base = (means ? pooled : static_cast<const T*>(pages.pool)) + (row < 0 ? 0 : row) * pages.width;
       stage_row(base + g * D, row >= 0, D, lane, sk + k * DS);
       stage_row(base + G * D + g * DV, row >= 0, DV, lane, sv + k * DV);
     }
@@ -245,8 +252,10 @@ window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows 
 #pragma unroll
     for (int j = 0; j < kWaMine; ++j) {
       const int kp = k0 + lane;
-      const bool seen = kp <= pos[j] && (pos[j] - kp < mask.size || kp < mask.keep_first);
-      const float sc = seen ? s[j] * scale : -INFINITY;
+      const bool seen = means ? kp < first[j] : kp <= pos[j] && (pos[j] - kp < mask.size || kp < mask.keep_first);
+      float sc = s[j] * score.scale;
+      if (score.softcap > 0.f) sc = score.softcap * tanhf(sc / score.softcap);
+      if (!seen) sc = -INFINITY;
       const float mn = fmaxf(m[j], warp_max(sc));
       const float ref = mn == -INFINITY ? 0.f : mn;   // nothing seen yet: every weight below is 0
       const float p = expf(sc - ref);
@@ -277,7 +286,13 @@ window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows 
     if (q >= cnt) continue;
     const int64_t nh = head(q);
     if (S == 1) {
-      const float w = 1.f / l[j];
+      float den = l[j], f = 1.f;
+      if (score.sink != nullptr) {
+        const float sk = score.sink[g * rep + (r0 + q) % rep], mm = fmaxf(m[j], sk);
+        f = expf(m[j] - mm);
+        den = den * f + expf(sk - mm);
+      }
+      const float w = f / den;
       for (int c = lane; c < DV; c += 32) stf(out + nh * DV + c, so[q * DV + c] * w);
     } else {
       for (int c = lane; c < DV; c += 32) part_o[(nh * S + split) * DV + c] = so[q * DV + c];
@@ -290,11 +305,12 @@ window_attn_kernel(const SeqBatch sb, const T* __restrict__ qx, const PagedRows 
 }
 
 template <typename T>
-__global__ void window_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int D, int S,
-                                    T* __restrict__ out) {
+__global__ void window_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const float* __restrict__ sink,
+                                    int H, int D, int S, T* __restrict__ out) {
   const int64_t nh = blockIdx.x;
-  float mm = -INFINITY, den = 0.f;
+  float mm = sink != nullptr ? sink[nh % H] : -INFINITY;
   for (int s = 0; s < S; ++s) mm = fmaxf(mm, part_ml[(nh * S + s) * 2]);
+  float den = sink != nullptr ? expf(sink[nh % H] - mm) : 0.f;
   for (int s = 0; s < S; ++s) den += part_ml[(nh * S + s) * 2 + 1] * expf(part_ml[(nh * S + s) * 2] - mm);
   for (int c = threadIdx.x; c < D; c += blockDim.x) {
     float v = 0.f;
@@ -307,15 +323,16 @@ __global__ void window_merge_kernel(const float* __restrict__ part_o, const floa
 }
 
 template <typename T>
-cudaError_t window_attention_t(const SeqBatch& sb, const T* q, const PagedRows& pages, int H, int G, int D, int DV,
-                               WindowMask mask, float scale, int n_splits, float* part_o, float* part_ml, T* out, cudaStream_t st) {
+cudaError_t window_attention_t(const SeqBatch& sb, const T* q, const PagedRows& pages, const T* pooled, int H, int G, int D, int DV,
+                               WindowMask mask, const ScoreArgs& score, int n_splits, float* part_o, float* part_ml, T* out,
+                               cudaStream_t st) {
   static int have = 0;
   const int smem = 4 * (kWaK * ((D | 1) + DV) + kWaQ * (D + DV) + kWaQ * kWaK);
   cudaError_t e = want_smem(window_attn_kernel<T>, smem, have);
   if (e != cudaSuccess) return e;
   const dim3 grid(static_cast<unsigned>(static_cast<int64_t>(sb.n_tok) * (H / G) / kWaQ + sb.n_seq), n_splits, G);
-  window_attn_kernel<T><<<grid, kWaWarps * 32, smem, st>>>(sb, q, pages, H, G, D, DV, mask, scale, part_o, part_ml, out);
-  if (n_splits > 1) window_merge_kernel<T><<<sb.n_tok * H, 128, 0, st>>>(part_o, part_ml, DV, n_splits, out);
+  window_attn_kernel<T><<<grid, kWaWarps * 32, smem, st>>>(sb, q, pages, pooled, H, G, D, DV, mask, score, part_o, part_ml, out);
+  if (n_splits > 1) window_merge_kernel<T><<<sb.n_tok * H, 128, 0, st>>>(part_o, part_ml, score.sink, H, DV, n_splits, out);
   return cudaGetLastError();
 }
 
@@ -349,16 +366,17 @@ cudaError_t launch_qk_prepare(bool f32, const SeqBatch& sb, const void* y, int64
   return cudaGetLastError();
 }
 
-cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, int H, int G, int D, int DV,
-                                    WindowMask mask, float scale, int n_splits, float* part_o, float* part_ml, void* out,
-                                    cudaStream_t st) {
-  if (G < 1 || H % G != 0 || pages.width != G * (D + DV) || mask.size < 1 || mask.keep_first < 0 || n_splits < 1 ||
-      (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
+cudaError_t launch_window_attention(bool f32, const SeqBatch& sb, const void* q, const PagedRows& pages, const void* pooled, int H, int G,
+                                    int D, int DV, WindowMask mask, const ScoreArgs& score, int n_splits, float* part_o, float* part_ml,
+                                    void* out, cudaStream_t st) {
+  if (G < 1 || H % G != 0 || pages.width != G * (D + DV) || mask.size < 1 || mask.keep_first < 0 || n_splits < 1 || mask.pool < 0 ||
+      (mask.pool > 0 && (pooled == nullptr || mask.keep_first > 0)) || (n_splits > 1 && (part_o == nullptr || part_ml == nullptr)))
     return cudaErrorInvalidValue;
-  return f32 ? window_attention_t<float>(sb, static_cast<const float*>(q), pages, H, G, D, DV, mask, scale, n_splits, part_o, part_ml,
-                                         static_cast<float*>(out), st)
-             : window_attention_t<__nv_bfloat16>(sb, static_cast<const __nv_bfloat16*>(q), pages, H, G, D, DV, mask, scale, n_splits,
-                                                 part_o, part_ml, static_cast<__nv_bfloat16*>(out), st);
+  using B = __nv_bfloat16;
+  return f32 ? window_attention_t<float>(sb, static_cast<const float*>(q), pages, static_cast<const float*>(pooled), H, G, D, DV, mask, score,
+                                         n_splits, part_o, part_ml, static_cast<float*>(out), st)
+             : window_attention_t<B>(sb, static_cast<const B*>(q), pages, static_cast<const B*>(pooled), H, G, D, DV, mask, score, n_splits,
+                                     part_o, part_ml, static_cast<B*>(out), st);
 }
 
 }  // namespace b200
