@@ -16,11 +16,12 @@ from .paged import PagedCache
 class HybridPagedCache:
     def __init__(self, widths: Sequence[int], state_shapes: Sequence[Tuple[int, ...]], ring_shapes: Sequence[Optional[Tuple[int, ...]]],
                  n_pages: int, page_size: int, max_seqs: int, max_pages_per_seq: int, dtype=torch.bfloat16, device="cpu",
-                 vec_shapes: Sequence[Optional[Tuple[int, ...]]] = ()):
+                 vec_shapes: Sequence[Optional[Tuple[int, ...]]] = (), blocks: Sequence[int] = ()):
         """``widths``: row width of every attention layer; ``state_shapes`` / ``ring_shapes`` / ``vec_shapes``: per recurrent
         layer the shape of one sequence's state, of its ring of past inputs (None: none) and of what else it carries (a normaliser and
-        a running maximum; None: nothing). All fp32."""
-        self.paged = PagedCache(len(widths), list(widths), n_pages, page_size, max_seqs, max_pages_per_seq, dtype, device)
+        a running maximum; None: nothing). All fp32. ``blocks``: per attention layer the size of token blocks whose mean rows are
+        kept (0: none)."""
+        self.paged = PagedCache(len(widths), list(widths), n_pages, page_size, max_seqs, max_pages_per_seq, dtype, device, blocks=blocks)
         self.states = [torch.zeros(max_seqs, *s, dtype=torch.float32, device=device) for s in state_shapes]
         self.rings = [None if s is None else torch.zeros(max_seqs, *s, dtype=torch.float32, device=device) for s in ring_shapes]
         self.vecs = [None if s is None else torch.zeros(max_seqs, *s, dtype=torch.float32, device=device) for s in vec_shapes]

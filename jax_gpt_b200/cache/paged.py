@@ -127,10 +127,13 @@ class _NativeTable:
 class PagedCache:
     """``pool``: (n_layers, n_pages, page_size, width), or with ``width`` a sequence of ``n_layers`` widths a list of
     (n_pages, page_size, width) pools, one per layer. ``block_table``: (max_seqs, max_pages_per_seq)
-    int32 page ids (-1 = unassigned). ``seq_lens``: (max_seqs,) int32 tokens stored per sequence."""
+    int32 page ids (-1 = unassigned). ``seq_lens``: (max_seqs,) int32 tokens stored per sequence. ``blocks``: per layer the size P of
+    blocks of tokens whose mean row is kept beside the rows (0: none); ``pooled[layer]`` (n_pages, ceil(page_size / P), width) holds
+    them, a block in the page of its last token, so that means come and go with the pages."""
 
     def __init__(self, n_layers: int, width: Union[int, Sequence[int]], n_pages: int, page_size: int = 64, max_seqs: int = 64,
-                 max_pages_per_seq: int = 64, dtype=torch.bfloat16, device="cpu", native: Optional[bool] = None):
+                 max_pages_per_seq: int = 64, dtype=torch.bfloat16, device="cpu", native: Optional[bool] = None,
+                 blocks: Sequence[int] = ()):
         self.page_size, self.n_layers, self.dtype = page_size, n_layers, dtype
         self.device = torch.device(device)
         if isinstance(width, int):
@@ -141,6 +144,9 @@ class PagedCache:
             assert len(self.widths) == n_layers, "one width per layer"
             self.pool = [torch.zeros(n_pages, page_size, w, dtype=dtype, device=device) for w in self.widths]
         self.width = width
+        self.blocks = list(blocks) or [0] * n_layers
+        self.pooled = [torch.zeros(n_pages, (page_size + P - 1) // P, w, dtype=dtype, device=device) if P else None
+                       for P, w in zip(self.blocks, self.widths)]
         on_gpu = self.device.type == "cuda"
         ops = None
         if native is not False:
@@ -239,6 +245,18 @@ class PagedCache:
         length = self._tab.length(seq_id) if length is None else length
         pages, offs = self.slots(seq_id, 0, length)
         return self.pool[layer][pages, offs]
+
+    def pooled_slots(self, layer: int, seq_id: int, first: int, n: int):
+        """(page ids, rows) of the means of blocks [first, first + n) of a sequence, as device tensors."""
+        P = self.blocks[layer]
+        blk = torch.arange(first, first + n, device=self.block_table.device)
+        page = (blk * P + P - 1) // self.page_size
+        return self.block_table[seq_id, page].long(), blk - page * self.page_size // P
+
+    def gather_pooled(self, layer: int, seq_id: int, n: int):
+        """Dense (n, width) view of a sequence's first block means (reference path and tests)."""
+        pages, rows = self.pooled_slots(layer, seq_id, 0, n)
+        return self.pooled[layer][pages, rows]
 
     def length(self, seq_id: int) -> int:
         return self._tab.length(seq_id)

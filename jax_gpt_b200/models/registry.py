@@ -40,6 +40,7 @@ FAMILIES: Dict[str, Family] = {f.name: f for f in (
     Family("vobunex", _BASE + "vobunex", "VobunexConfig", ("Vobunex",), from_dir=_FOLDER, engine="VobunexEngine"),
     Family("fovudra", _BASE + "fovudra", "FovudraConfig", ("Fovudra",), from_dir=_FOLDER, engine="FovudraEngine"),
     Family("munazen", _BASE + "munazen", "MunazenConfig", ("Munazen",), from_dir=_FOLDER, engine="MunazenEngine"),
+    Family("mopalorn", _BASE + "mopalorn", "MopalornConfig", ("Mopalorn",), from_dir=_FOLDER, engine="MopalornEngine"),
 )}
 
 

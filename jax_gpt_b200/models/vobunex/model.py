@@ -17,9 +17,8 @@ from typing import List, Optional
 import torch
 
 from ...cache.hybrid import HybridPagedCache
-from ...ops import attention as attn_ops
 from ...ops import latent_attention as LA
-from ...ops import mla_decode, ssm
+from ...ops import ssm
 from ...ops.gemm import linear_rows
 from ...ops.norm import LAYERNORM
 from ...ops.packed import PackedBatch, embed_bigram, norm_rows, seq_begin
@@ -51,44 +50,13 @@ def make_rope(config: VobunexConfig, n_pos: int, device="cpu") -> list:
     return out
 
 
-# ------------------------------------------------------------------------------------------------
-def _flash_ok(batch: PackedBatch, h, m: LatentAttention) -> bool:
-    """Whole prompts whose heads have the flash kernel's MLA shape."""
-    return (h.is_cuda and h.dtype == torch.bfloat16 and batch.fresh and not batch.single and m.dim + m.rot_dim == 192
-            and m.vdim == 128 and m.kv_rank % 8 == 0 and m.rot_dim % 8 == 0)
-
-
-def _paged_kernel_ok(batch: PackedBatch, h, m: LatentAttention, page_size: int) -> bool:
-    return (h.is_cuda and h.dtype == torch.bfloat16 and batch.single and m.kv_rank == 512 and m.rot_dim == 64 and page_size == 64)
-
-
 def latent_attention_mixer(h, mp, m: LatentAttention, batch: PackedBatch, cache: HybridPagedCache, layer: int, rope, eps, x):
     """Adds the mixer's output for the normed input ``h`` to the residual ``x``; ``layer`` counts attention layers."""
-    N, H, dn, dr, dv, R = h.shape[0], m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
-    flash = _flash_ok(batch, h, m)
+    flash = LA.flash_ok(batch, h, m.dim, m.rot_dim, m.vdim, m.kv_rank)
     y = linear_rows(h, mp["down"])
     cq, lat = LA.mla_prepare(batch, y, mp["q_norm"], mp["kv_norm"], eps, rope, cache.paged, layer, want_latent=flash)
-    q = linear_rows(cq, mp["uq"]).view(N, H, dn + dr)
-    if flash:
-        kv = linear_rows(lat[:, :R], mp["ukv"])                       # (N, H dn | H dv)
-        k = LA.mla_rope_qk(batch, q, kv[:, :H * dn], lat, R, rope)
-        v = kv[:, H * dn:]
-        o = torch.empty(N, H * dv, device=h.device, dtype=h.dtype)
-        same = len(set(batch.lens)) == 1
-        parts = [(0, N, batch.n_seq)] if same else [(sum(batch.lens[:b]), n, 1) for b, n in enumerate(batch.lens)]
-        for c0, n, B in parts:
-            T = n // B
-            as4 = lambda t, d: t[c0:c0 + n].unflatten(0, (B, T)).unflatten(-1, (H, d))
-            attn_ops.attn_fwd(q[c0:c0 + n].view(B, T, H, dn + dr), k[c0:c0 + n].view(B, T, H, dn + dr), as4(v, dv), True, m.scale,
-                              out=as4(o, dv), sink=mp["sink"])
-    else:
-        w_uk, w_uv = mp["ukv"][:H * dn], mp["ukv"][H * dn:]
-        qf = LA.mla_absorb_q(batch, q, w_uk, rope, dr)
-        if _paged_kernel_ok(batch, h, m, cache.page_size):
-            o_lat = mla_decode.mla_paged_decode(qf, cache.paged, layer, batch.ids, m.scale, sink=mp["sink"], max_len=batch.max_len)
-        else:
-            o_lat = LA.latent_attention(batch, qf, cache.paged, layer, R, m.scale, mp["sink"])
-        o = LA.mla_absorb_out(o_lat, w_uv)
+    q = linear_rows(cq, mp["uq"]).view(h.shape[0], m.heads, m.dim + m.rot_dim)
+    o = LA.attend(batch, q, lat, mp["ukv"], m.kv_rank, m.vdim, rope, cache.paged, layer, m.scale, mp["sink"])
     linear_rows(o, mp["o"], out=x, accumulate=True)
 
 

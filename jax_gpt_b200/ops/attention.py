@@ -44,10 +44,13 @@ def _as2d(t):
     return t.as_strided((B * T, H * D), (t.stride(1), 1))
 
 
-def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None, sink=None, window: int = 0, keep_first: int = 0):
+def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None, sink=None, window: int = 0, keep_first: int = 0,
+             softcap: float = 0.0, pool: int = 0, pool_rows: int = 0):
     """Raw CUDA forward. Returns (out [B,T,H,D] bf16, lse [B,H,T] fp32 in log2 units). ``sink`` (H,) fp32 adds
     exp(sink) to every softmax denominator of its head (and to lse). ``window`` > 0: query i sees keys j <= i with
-    i - j < window or j < keep_first; key tiles nobody sees are skipped."""
+    i - j < window or j < keep_first; key tiles nobody sees are skipped. ``softcap`` > 0 (without a window): scores become
+    softcap tanh(score / softcap). ``pool`` > 0 (with a window): k and v hold ``pool_rows`` (a multiple of 128) rows of means of
+    ``pool`` tokens in front of a sequence's T tokens; a mean is seen once its block has left the window."""
     B, T, H, D = q.shape
     Hkv, Dv = k.shape[2], v.shape[3]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
@@ -56,7 +59,7 @@ def attn_fwd(q, k, v, causal=True, scale=None, out=None, lse=None, sink=None, wi
     if lse is None:
         lse = torch.empty(B, H, T, device=q.device, dtype=torch.float32)
     _ext.ops().attn_fwd(_as2d(q), _as2d(k), _as2d(v), _as2d(out), lse, B, T, H, Hkv, D, scale, causal, Dv, sink, window,
-                          keep_first)
+                          keep_first, softcap, pool, pool_rows)
     return out, lse
 
 
@@ -146,19 +149,22 @@ def decode_widths_ok(H: int, Hkv: int, D: int, Dv: int) -> bool:
 
 def attention_decode_paged(q, pool, block_table, seq_ids, seq_lens, n_kv_heads: int, len_add: int = 1, scale=None,
                            scratch=None, out=None, max_len: Optional[int] = None, window: int = 0, keep_first: int = 0,
-                           v_dim: int = 0):
+                           v_dim: int = 0, softcap: float = 0.0, sink=None, pooled=None, pool_block: int = 0):
     """One query token per sequence over a PAGED cache (cache/paged.py): ``pool`` (n_pages, page_size, 2 * Hkv * D)
     holds K of every kv head then V per cached token, ``block_table`` (max_seqs, max_pages) the page ids,
     ``seq_ids`` (B,) the sequence of every query row, ``seq_lens`` (max_seqs,) the committed lengths, all on the
     device; ``len_add`` keys beyond the committed length are attended (1: the new token's row is written, the length
     not yet advanced). ``window`` > 0: only the last ``window`` keys and the first ``keep_first`` are seen.
-    q (B, H, D). Returns (B, H, D), or (B, H, v_dim) where the values have a width of their own."""
+    ``softcap`` > 0: scores become softcap tanh(score / softcap); ``sink`` (H,) fp32 joins the denominators; ``pooled`` (with a window):
+    means of blocks of ``pool_block`` cached rows, (n_pages, ceil(page_size / pool_block), width), seen where their block lies before the
+    window (not together with ``softcap``). q (B, H, D). Returns (B, H, D), or (B, H, v_dim) where the values have a width of their own."""
     B, H, D = q.shape
     Hkv, Dv = n_kv_heads, v_dim or q.shape[2]
     scale = scale if scale is not None else 1.0 / math.sqrt(D)
     cuda_ok = (q.is_cuda and q.dtype == torch.bfloat16 and pool.dtype == torch.bfloat16 and decode_widths_ok(H, Hkv, D, Dv)
-               and pool.shape[-1] == Hkv * (D + Dv))
+               and pool.shape[-1] == Hkv * (D + Dv) and not (softcap > 0 and pooled is not None))
     if not cuda_ok:
+        assert softcap == 0 and sink is None and pooled is None, "only the kernel takes capped scores, sinks and block means"
         outs = []
         ps = pool.shape[1]
         for b in range(B):
@@ -178,13 +184,14 @@ def attention_decode_paged(q, pool, block_table, seq_ids, seq_lens, n_kv_heads: 
         q2 = q2.contiguous()
     if scratch is None:
         n_keys = max_len or block_table.shape[1] * pool.shape[1]
-        S = decode_splits(B, Hkv, min(n_keys, window + keep_first) if window > 0 else n_keys)
+        blocks = (n_keys - window) // pool_block if pooled is not None and n_keys > window else 0
+        S = decode_splits(B, Hkv, min(n_keys, window + keep_first) + blocks if window > 0 else n_keys)
         scratch = (torch.empty(B, H, S, Dv, device=q.device, dtype=torch.float32),
                    torch.empty(B, H, S, 2, device=q.device, dtype=torch.float32))
     if out is None:
         out = torch.empty(B, H * Dv, device=q.device, dtype=torch.bfloat16)
     _ext.ops().attn_decode_paged(q2, pool, block_table, seq_ids, seq_lens, int(len_add), H, Hkv, scale, scratch[0],
-                                 scratch[1], out, window, keep_first)
+                                 scratch[1], out, window, keep_first, softcap, sink, pooled, pool_block)
     return out.view(B, H, Dv)
 
 

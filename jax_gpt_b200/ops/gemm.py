@@ -14,7 +14,7 @@ import torch
 
 from .. import _ext
 
-EPI_NONE, EPI_GELU, EPI_GELU_GRAD, EPI_RELU2, EPI_SILU = 0, 1, 2, 4, 5
+EPI_NONE, EPI_GELU, EPI_GELU_GRAD, EPI_RELU2, EPI_SILU, EPI_XIELU = 0, 1, 2, 4, 5, 6
 OUT_BF16, OUT_F32, OUT_F32_ATOMIC = 0, 1, 2
 
 
@@ -29,8 +29,15 @@ def gelu_tanh_grad(x: torch.Tensor) -> torch.Tensor:
     return 0.5 * (1 + t) + 0.5 * x * (1 - t * t) * k0 * (1 + 3 * k1 * x * x)
 
 
+def xielu(z: torch.Tensor, a: float, b: float) -> torch.Tensor:
+    """``a z^2 + z / 2`` for z > 0, ``b (exp(z) - 1 - z) + z / 2`` otherwise (fp32)."""
+    z = z.float()
+    n = z.clamp_max(0)
+    return torch.where(z > 0, a * z * z, b * (torch.expm1(n) - n)) + 0.5 * z
+
+
 def gemm_ref(a, b, *, a_mn_major=False, b_mn_major=False, out=None, bias=None, residual=None, aux=None,
-             epilogue=EPI_NONE, out_mode=OUT_BF16, alpha=1.0, split_k=1):
+             epilogue=EPI_NONE, out_mode=OUT_BF16, alpha=1.0, split_k=1, act_args=(0.0, 0.0)):
     """fp32 reference of :func:`gemm` with identical argument conventions."""
     A = a.float().t() if a_mn_major else a.float()
     Bm = b.float() if b_mn_major else b.float().t()
@@ -48,6 +55,8 @@ def gemm_ref(a, b, *, a_mn_major=False, b_mn_major=False, out=None, bias=None, r
         acc = acc.clamp_min(0).square()
     elif epilogue == EPI_SILU:
         acc = torch.nn.functional.silu(acc)
+    elif epilogue == EPI_XIELU:
+        acc = xielu(acc, *act_args)
     if residual is not None:
         acc = acc + residual.float()
     if out is None:
@@ -62,11 +71,12 @@ def gemm_ref(a, b, *, a_mn_major=False, b_mn_major=False, out=None, bias=None, r
 def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn_major: bool = False, b_mn_major: bool = False,
          out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
          residual: Optional[torch.Tensor] = None, aux: Optional[torch.Tensor] = None, epilogue: int = EPI_NONE,
-         out_mode: int = OUT_BF16, alpha: float = 1.0, split_k: int = 1) -> torch.Tensor:
-    """See module docstring. ``out_mode=OUT_F32_ATOMIC`` accumulates into ``out`` (fp32)."""
+         out_mode: int = OUT_BF16, alpha: float = 1.0, split_k: int = 1, act_args=(0.0, 0.0)) -> torch.Tensor:
+    """See module docstring. ``out_mode=OUT_F32_ATOMIC`` accumulates into ``out`` (fp32). ``act_args``: the two constants of
+    ``EPI_XIELU``."""
     if not a.is_cuda:
         return gemm_ref(a, b, a_mn_major=a_mn_major, b_mn_major=b_mn_major, out=out, bias=bias, residual=residual,
-                        aux=aux, epilogue=epilogue, out_mode=out_mode, alpha=alpha, split_k=split_k)
+                        aux=aux, epilogue=epilogue, out_mode=out_mode, alpha=alpha, split_k=split_k, act_args=act_args)
     M = a.shape[1] if a_mn_major else a.shape[0]
     N = b.shape[1] if b_mn_major else b.shape[0]
     if out is None:
@@ -74,7 +84,7 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_mn_major: bool = False, b_mn_maj
             out = torch.zeros(M, N, device=a.device, dtype=torch.float32)
         else:
             out = torch.empty(M, N, device=a.device, dtype=torch.bfloat16 if out_mode == OUT_BF16 else torch.float32)
-    _ext.ops().gemm(a, a_mn_major, b, b_mn_major, out, bias, residual, aux, epilogue, out_mode, alpha, split_k)
+    _ext.ops().gemm(a, a_mn_major, b, b_mn_major, out, bias, residual, aux, epilogue, out_mode, alpha, split_k, *act_args)
     return out
 
 
@@ -121,7 +131,7 @@ def linear_f32out(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
 
 
 ROWS_KERNEL_MAX = {torch.bfloat16: 32, torch.float32: 8}   # rows up to which linear layers run on the few-row kernel
-_ROW_ACTS = {None: (0, EPI_NONE), "relu2": (1, EPI_RELU2), "silu": (2, EPI_SILU)}   # few-row kernel, GEMM epilogue
+_ROW_ACTS = {None: (0, EPI_NONE), "relu2": (1, EPI_RELU2), "silu": (2, EPI_SILU), "xielu": (4, EPI_XIELU)}   # few-row kernel, GEMM epilogue
 _ROW_SILU_GLU = 3
 
 
@@ -130,9 +140,10 @@ def _few_rows(x) -> bool:
 
 
 def linear_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *, act: Optional[str] = None,
-                accumulate: bool = False, f32_out: bool = False) -> torch.Tensor:
+                accumulate: bool = False, f32_out: bool = False, act_args=(0.0, 0.0)) -> torch.Tensor:
     """Inference linear layer with ``w`` stored (out, in) as checkpoints have it: ``act(x @ w.T)``; ``act`` is None,
-    "relu2" (the square of relu) or "silu". ``accumulate`` adds into ``out`` (fp32: a 32-bit residual), ``f32_out`` returns fp32.
+    "relu2" (the square of relu), "silu" or "xielu" (its two constants are ``act_args``). ``accumulate`` adds into ``out`` (fp32: a
+    32-bit residual), ``f32_out`` returns fp32.
     x (M, in), bf16 or fp32, unit inner stride. On CUDA up to ``ROWS_KERNEL_MAX`` rows run on the few-row kernel
     (weights streamed once where the rows are 16-byte aligned), more rows on the tcgen05 GEMM in bf16 and on the library's fp32 GEMM in fp32."""
     M, N = x.shape[0], w.shape[0]
@@ -141,19 +152,21 @@ def linear_rows(x: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = 
         out = torch.empty(M, N, device=x.device, dtype=torch.float32 if f32_out else x.dtype)
     mode = 2 if accumulate else (1 if out.dtype == torch.float32 and x.dtype != torch.float32 else 0)
     if _few_rows(x):
-        _ext.ops().rows_linear(x, w, out, _ROW_ACTS[act][0], mode)
+        _ext.ops().rows_linear(x, w, out, _ROW_ACTS[act][0], mode, None, *act_args)
         return out
     if x.is_cuda and x.dtype == torch.bfloat16 and w.shape[1] % 8 == 0 and w.stride(0) % 8 == 0 and w.data_ptr() % 16 == 0:
         if x.stride(0) % 8 != 0 or x.data_ptr() % 16 != 0:
             x = x.contiguous()
         if act is None or mode == 0:
             return gemm(x, w, out=out, epilogue=_ROW_ACTS[act][1],
-                        out_mode=(OUT_BF16, OUT_F32, OUT_F32_ATOMIC)[mode])
+                        out_mode=(OUT_BF16, OUT_F32, OUT_F32_ATOMIC)[mode], act_args=act_args)
     y = x @ w.t() if mode == 0 else x.float() @ w.float().t()
     if act == "relu2":
         y = y.clamp_min(0).square()
     elif act == "silu":
         y = torch.nn.functional.silu(y)
+    elif act == "xielu":
+        y = xielu(y, *act_args)
     return out.add_(y) if accumulate else out.copy_(y)
 
 

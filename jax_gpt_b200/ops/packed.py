@@ -27,6 +27,7 @@ class PackedBatch:
     tok_seq: torch.Tensor = field(repr=False)
     start: torch.Tensor = field(repr=False)     # written by seq_begin
     prev_tok: torch.Tensor = field(repr=False)  # written by seq_begin: the token before each sequence's first row
+    made: dict = field(default_factory=dict, repr=False)
 
     @property
     def n_tok(self) -> int:
@@ -57,6 +58,12 @@ class PackedBatch:
         z = torch.zeros(2, B, dtype=torch.int32, device=device)
         return PackedBatch(list(seq_ids), list(lens), fresh, max_len, dev[:B].clone(), dev[B:2 * B + 1].clone(),
                            dev[2 * B + 1:2 * B + 1 + N].clone(), z[0].clone(), z[1].clone())
+
+    def memo(self, key, make):
+        """What ``make()`` derives from the batch's host description, made once."""
+        if key not in self.made:
+            self.made[key] = make()
+        return self.made[key]
 
     # ---- host views of the device description (restatements on CPU tensors) ----
     def rows(self):

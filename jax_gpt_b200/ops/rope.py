@@ -124,6 +124,13 @@ def rotate_interleaved(x: torch.Tensor, pos: torch.Tensor, tables) -> torch.Tens
     return torch.cat([turned, x[..., dims:]], dim=-1)
 
 
+def pair_order(width: int, dims: int) -> torch.Tensor:
+    """Order of ``width`` features that turns half-split pairs (i, i + dims / 2) into interleaved ones (2i, 2i + 1); the features
+    from ``dims`` on stay. Query and key weights reordered by it give the same scores."""
+    half = dims // 2
+    return torch.cat([torch.stack([torch.arange(half), torch.arange(half) + half], 1).flatten(), torch.arange(dims, width)])
+
+
 def rotate_half_split(x: torch.Tensor, pos: torch.Tensor, tables) -> torch.Tensor:
     """x (N, ..., d): of the first ``dims`` features, i and i + dims / 2 turn together by the angles of position ``pos[n]``."""
     cos, sin = tables

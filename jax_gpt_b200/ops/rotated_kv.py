@@ -13,20 +13,9 @@ from typing import Optional, Sequence, Tuple
 import torch
 
 from .. import _ext
-from . import attention as A
 from .packed import PackedBatch
 from .rope import rotate_interleaved
-from .window_attention import NO_WINDOW, flash_prompts, window_attention_any
-
-FLASH_WIDTHS = ((64, 64), (128, 128), (192, 128), (256, 256))     # (query and key, value) widths of the flash kernel
-
-
-def flash_widths(batch: PackedBatch, dtype, is_cuda: bool, dk: int, dv: int) -> Optional[Tuple[int, int]]:
-    """Operand widths of the flash kernel for whole prompts, None where it does not apply."""
-    if not is_cuda or dtype != torch.bfloat16 or not batch.fresh or batch.single:
-        return None
-    return next((w for w in FLASH_WIDTHS if w[0] >= dk and w[1] >= dv), None)
-
+from .window_attention import flash_widths, grouped_attention  # noqa: F401
 
 def qkv_rotate(batch: PackedBatch, y, cols: Sequence[int], bias, H: int, G: int, dk: int, dv: int, rope, vrope, cache, layer: int,
                dense: Optional[Tuple[int, int]]):
@@ -56,13 +45,7 @@ def qkv_rotate(batch: PackedBatch, y, cols: Sequence[int], bias, H: int, G: int,
 
 def causal_attention(batch: PackedBatch, q, k, v, cache, layer: int, G: int, dv: int, scale: float) -> torch.Tensor:
     """Output (N, H, >= dv) of the operands of ``qkv_rotate``: dense prompts, or q against the cached rows."""
-    N, H, D = q.shape
-    if k is not None:
-        return flash_prompts(batch, q, k, v, scale)
-    if (q.is_cuda and q.dtype == torch.bfloat16 and batch.single and A.decode_widths_ok(H, G, D, dv)):
-        return A.attention_decode_paged(q, cache.pool[layer], cache.block_table, batch.ids, cache.seq_lens, G, 0, scale,
-                                        max_len=batch.max_len, v_dim=dv)
-    return window_attention_any(batch, q, cache, layer, G, NO_WINDOW, 0, scale, v_dim=dv)
+    return grouped_attention(batch, q, k, v, cache, layer, G, dv, scale)
 
 
 def turn_back_gate(batch: PackedBatch, o, g, vrope, scale: float, out) -> None:
