@@ -9,12 +9,13 @@ def rms(x, eps):
     return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
 
 
-def turn_halves(x, base):
-    """x (T, ..., d): features i and i + d / 2 turn together by position * base^(-2 i / d)."""
+def turn_halves(x, base, pos=None):
+    """x (T, ..., d): features i and i + d / 2 turn together by position * base^(-2 i / d); positions 0, 1, .. or ``pos``."""
     T, d = x.shape[0], x.shape[-1]
+    pos = torch.arange(T) if pos is None else torch.tensor(pos)
     out = x.clone()
     for i in range(d // 2):
-        a = torch.arange(T, dtype=torch.float64) * base ** (-2.0 * i / d)
+        a = pos.double() * base ** (-2.0 * i / d)
         a = a.reshape([T] + [1] * (x.dim() - 2))
         u, v = x[..., i], x[..., i + d // 2]
         out[..., i] = u * torch.cos(a) - v * torch.sin(a)
@@ -94,7 +95,7 @@ def heads_of(h, m, w, p, first):
     raw = (h @ w[p + "v"].T).reshape(T, G, m["vdim"])
     v = raw
     if m.get("v_mix") and first is not None:
-        v = mixed_values(raw, first, w[p + "vmix"])
+        v = mixed_values(raw, first.reshape(raw.shape), w[p + "vmix"])
     of = torch.arange(H) // (H // G)
     return q, k[:, of], v[:, of], raw
 
