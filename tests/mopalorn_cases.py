@@ -295,8 +295,10 @@ def check_one_key_stands_out(device, tol, dtype=torch.float32, H=6, G=2, d=12, d
                 if P > 1 and qpos - target >= size and target // P < (qpos + 1) // P:
                     flips.append(("block", target // P))
                 for hide in flips:
-                    seen_both = ref(hide=hide)
-                    assert float((seen_both - want).abs().max()) > 3 * tol, ("the case does not show", size, P, qpos, target, hide)
+                    # (tokens of the block that are still in the window take most of the weight: there only fp32 shows it)
+                    beside = hide[0] == "block" and qpos - (target // P * P + P - 1) < size
+                    if not (beside and dtype == torch.bfloat16):
+                        assert float((ref(hide=hide) - want).abs().max()) > 3 * tol, ("the case does not show", size, P, qpos, target, hide)
                 for start in sorted({0, qpos, max(0, qpos - 3)}):           # as part of a prompt, a decode step, a short portion
                     put = lambda a, b: mixed_kv(begin(cache, 1, a, b - a, n + 9, device), rows(q[a:b], k[a:b], v[a:b]), cols, H, G, d, dv, cache, 1,
                                                 None, factors, vf[a:b].to(device), lam, window)
@@ -311,13 +313,14 @@ def check_one_key_stands_out(device, tol, dtype=torch.float32, H=6, G=2, d=12, d
                     assert float((got - want).abs().max()) < tol, (size, P, qpos, target, start)
 
 
-def check_one_latent_stands_out(device, tol, dtype=torch.float32, H=5, dn=6, dr=4, dv=7, R=9, n=75, ps=8, sizes=(20, 8, 1, 33, 75), rep=3.0):
+def check_one_latent_stands_out(device, tol, dtype=torch.float32, H=5, dn=6, dr=4, dv=7, R=9, n=75, ps=8, sizes=(20, 8, 1, 33, 75)):
     """Latent attention over a window with an output gate: a query that matches one chosen key far above the rest, on both sides of the
     window's edge, at page borders and at first positions; as part of a prompt, a decode step and a short portion."""
     from jax_gpt_b200.ops import latent_attention as LA
     from jax_gpt_b200.ops.rope import rope_tables
     g = torch.Generator().manual_seed(12)
     base, eps, scale = 300.0, 1e-4, 0.5
+    rep = 13.0 / (scale * (4 * dn ** 0.5 + dr))                 # the matching key scores about 13
     pairs = torch.tensor([x for i in range(dr // 2) for x in (i, i + dr // 2)])    # the kernels turn neighbours
     rnd = lambda t: t.to(dtype).double()
     y = torch.randn(n, R + dr, generator=g)
