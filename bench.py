@@ -187,9 +187,9 @@ def main():
                     help="2+ GPUs: skip the expert-parallel extras (fused EP-MoE layer, Qwen3.5-style MoE training step)")
     ap.add_argument("--extra-budget-s", type=float, default=420.0, help="wall-clock limit of the extras; past it the line is printed without them")
     ap.add_argument("--serve", action="store_true",
-                    help="instead of the training benchmark: prefill / decode throughput and kernel rooflines of Vobunex, Fovudra and Munazen beside the closest families")
+                    help="instead of the training benchmark: prefill / decode throughput and kernel rooflines of Vobunex, Fovudra, Munazen and Mopalorn beside the closest families")
     ap.add_argument("--serve-part", default="all", choices=["kernels", "models", "all"])
-    ap.add_argument("--serve-family", default="all", choices=["vobunex", "fovudra", "munazen", "all"])
+    ap.add_argument("--serve-family", default="all", choices=["vobunex", "fovudra", "munazen", "mopalorn", "all"])
     ap.add_argument("--extras-child", default="", help=argparse.SUPPRESS)   # internal: run only the extras, write them to this file
     args = ap.parse_args()
     if args.impl == "reference":

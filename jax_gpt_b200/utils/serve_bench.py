@@ -1,13 +1,13 @@
-"""Serving benchmark of Vobunex, Fovudra and Munazen beside the closest other families at equal widths (random weights, one GPU).
+"""Serving benchmark of Vobunex, Fovudra, Munazen and Mopalorn beside the closest other families at equal widths (random weights, one GPU).
 
-    python bench.py --serve [--serve-part kernels|models|all] [--serve-family vobunex|fovudra|munazen|all]
+    python bench.py --serve [--serve-part kernels|models|all] [--serve-family vobunex|fovudra|munazen|mopalorn|all]
 
 ``models``: prefill and decode tokens/s of whole models. The hybrid (Mamba-2 + latent attention) stands beside the
 Qwen3.5-style hybrid (Gated DeltaNet + gated attention), latent-attention-only layers beside the DeepSeek-V3 layers; same
 width, depth, expert count and expert width, each family on its own serving path (decode: CUDA-graph engines, the
 others' experts on the fused expert kernel). ``kernels``: device time and roofline fraction of every kernel of a layer
-beside the like kernel of the other family. Fovudra's and Munazen's
-tables are made in utils/serve_bench_fovudra.py and utils/serve_bench_munazen.py.
+beside the like kernel of the other family. The other families'
+tables are made in utils/serve_bench_fovudra.py, utils/serve_bench_munazen.py and utils/serve_bench_mopalorn.py.
 
 Timing: CUDA events. Kernels are timed inside a captured graph that writes a 256 MB buffer (larger than L2) before every
 launch; the time of the same graph without the launches is subtracted. The roofline of a kernel is the slower of its
@@ -430,9 +430,10 @@ def run(part: str = "all", family: str = "all") -> dict:
     torch.cuda.set_device(dev)
     out = {"data": "synthetic token ids, random weights", "dtype": "bf16 (fp32 residual, norms, states)"}
     from . import serve_bench_fovudra as fov
+    from . import serve_bench_mopalorn as mop
     from . import serve_bench_munazen as mun
     for name, kernels, models in (("vobunex", kernel_table, model_table), ("fovudra", fov.kernel_table, fov.model_table),
-                                  ("munazen", mun.kernel_table, mun.model_table)):
+                                  ("munazen", mun.kernel_table, mun.model_table), ("mopalorn", mop.kernel_table, mop.model_table)):
         if family not in (name, "all"):
             continue
         out[name] = {}

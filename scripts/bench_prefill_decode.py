@@ -119,7 +119,7 @@ def make_runner(args, device):
             logits, cache = forward(params, nxt[:, None], cfg, cache=cache, is_decode=True, ep_group=ep, tp_group=tp_group)
             return logits[:, -1].argmax(-1), cache
         return prefill, decode, cfg
-    if args.model in ("vobunex", "fovudra", "munazen"):
+    if args.model in ("vobunex", "fovudra", "munazen", "mopalorn"):
         if args.tp > 1 or args.dp > 1 or args.w8a8 or args.fp8:
             raise SystemExit(f"--tp / --dp / --w8a8 / --fp8 do not apply to --model {args.model}")
         from jax_gpt_b200.models.registry import FAMILIES, load_model
@@ -222,7 +222,7 @@ def find_max_batch(prefill, decode, cap):
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
-    ap.add_argument("--model", default="qwen35", choices=["qwen35", "deepseek_v3", "vobunex", "fovudra", "munazen"])
+    ap.add_argument("--model", default="qwen35", choices=["qwen35", "deepseek_v3", "vobunex", "fovudra", "munazen", "mopalorn"])
     ap.add_argument("--model-dir", default="", help="HF safetensors directory (random weights when empty)")
     ap.add_argument("--scenario", default="1k1k", choices=sorted(SCENARIOS))
     ap.add_argument("--tp", type=int, default=1)

@@ -86,11 +86,11 @@ def qwen_config(name: str):
 
 
 def step_engine_config(family: str, name: str):
-    """Preset of a family on the shared step engine (``--model vobunex`` / ``fovudra`` / ``munazen``)."""
+    """Preset of a family on the shared step engine (``--model vobunex`` / ``fovudra`` / ``munazen`` / ``mopalorn``)."""
     from jax_gpt_b200.models.registry import FAMILIES
     cls = FAMILIES[family].config_class()
     wide = dict(width=4096, heads=32, ff=1536, **({"kv_heads": 4} if family == "fovudra" else {}))
-    if family == "munazen":
+    if family in ("munazen", "mopalorn"):
         wide = dict(width=4096, heads=32, kv_heads=4)
     return {"tiny": cls.tiny, "serving": cls.serving, "serving_wide": lambda: cls.serving(**wide)}[name]()
 
