@@ -37,13 +37,16 @@ __device__ __forceinline__ void store_n(T* p, const float (&f)[V]) {
 template <typename T, int V, typename F>
 __device__ __forceinline__ void block_mean(const PagedRows& pages, int P, int slot, int blk, F put) {
   const float inv = 1.f / P;
+  const int first = blk * P, last = first + P - 1;
+  const bool one_page = first / pages.page_size == last / pages.page_size;   // then its rows follow one another
+  const int64_t row0 = page_row(pages, slot, first);
   for (int i = threadIdx.x * V; i < pages.width; i += blockDim.x * V) {
     float s[V];
 #pragma unroll
     for (int j = 0; j < V; ++j) s[j] = 0.f;
-#pragma unroll 4
+#pragma unroll 8
     for (int r = 0; r < P; ++r) {
-      const int64_t row = page_row(pages, slot, blk * P + r);
+      const int64_t row = one_page ? row0 + r : page_row(pages, slot, first + r);
       float f[V];
       load_n<T, V>(static_cast<const T*>(pages.pool) + (row < 0 ? 0 : row) * pages.width + i, f);
 #pragma unroll

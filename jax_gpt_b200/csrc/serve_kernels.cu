@@ -461,7 +461,9 @@ __device__ __forceinline__ float rotated(const RopeTable& r, int pos, int i, F a
   return (i & 1) == 0 ? at(i) * c - at(i + 1) * s : at(i) * c + at(i - 1) * s;
 }
 
-template <typename T>
+// kHold > 0: the first kHold features of every thread stay in registers (turned where they turn), so that one wait covers all loads; for
+// steps of a few tokens, where latency is all there is.
+template <typename T, int kHold>
 __global__ void mla_prepare_kernel(const SeqBatch sb, const T* __restrict__ y, int64_t ldy, int q_rank, int R, int dr,
                                    const float* __restrict__ q_gamma, const float* __restrict__ kv_gamma, float eps,
                                    const RopeTable rope, const PagedRows pages, T* __restrict__ cq, T* __restrict__ lat,
@@ -472,27 +474,39 @@ __global__ void mla_prepare_kernel(const SeqBatch sb, const T* __restrict__ y, i
   const int pos = sb.start[b] + n - sb.cu[b];
   const T* row = y + static_cast<int64_t>(n) * ldy;
   const T* kv = row + q_rank;
-  float sq = 0.f, sk = 0.f;
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = ldf(row + i); sq += v * v; }
-  for (int i = threadIdx.x; i < R; i += blockDim.x) { const float v = ldf(kv + i); sk += v * v; }
-  const float iq = q_rank > 0 ? 1.f / sqrtf(block_sum(sq, red) / q_rank + eps) : 0.f;
-  const float ik = 1.f / sqrtf(block_sum(sk, red) / R + eps);
-  for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
-    stf(cq + static_cast<int64_t>(n) * q_rank + i, ldf(row + i) * iq * q_gamma[i]);
   const int64_t dst = page_row(pages, sb.ids[b], pos);
   if (dst < 0 || pos >= rope.max_pos) {
     if (threadIdx.x == 0) report_status(status, kBadArgument, 302, b, pos);
     return;
   }
+  auto turned = [&](int i) { return rotated(rope, pos, i - R, [&](int j) { return ldf(kv + R + j); }); };
+  float held[kHold > 0 ? kHold : 1], gain[kHold > 0 ? kHold : 1];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int k = 0; k < kHold; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    held[k] = i < R ? ldf(kv + i) : (i < R + dr ? turned(i) : 0.f);
+    gain[k] = i < R ? kv_gamma[i] : 0.f;
+    if (i < R) sk += held[k] * held[k];
+  }
+  for (int i = threadIdx.x + kHold * blockDim.x; i < R; i += blockDim.x) { const float v = ldf(kv + i); sk += v * v; }
+  for (int i = threadIdx.x; i < q_rank; i += blockDim.x) { const float v = ldf(row + i); sq += v * v; }
+  const float iq = q_rank > 0 ? 1.f / sqrtf(block_sum(sq, red) / q_rank + eps) : 0.f;
+  const float ik = 1.f / sqrtf(block_sum(sk, red) / R + eps);
+  for (int i = threadIdx.x; i < q_rank; i += blockDim.x)
+    stf(cq + static_cast<int64_t>(n) * q_rank + i, ldf(row + i) * iq * q_gamma[i]);
   T* prow = static_cast<T*>(pages.pool) + dst * pages.width;
   T* lrow = lat != nullptr ? lat + static_cast<int64_t>(n) * (R + dr) : nullptr;
-  for (int i = threadIdx.x; i < R + dr; i += blockDim.x) {
-    float v;
-    if (i < R) v = ldf(kv + i) * ik * kv_gamma[i];
-    else v = rotated(rope, pos, i - R, [&](int j) { return ldf(kv + R + j); });
+  auto put = [&](int i, float v) {
     stf(prow + i, v);
     if (lrow != nullptr) stf(lrow + i, v);
+  };
+#pragma unroll
+  for (int k = 0; k < kHold; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i < R + dr) put(i, i < R ? held[k] * ik * gain[k] : held[k]);
   }
+  for (int i = threadIdx.x + kHold * blockDim.x; i < R + dr; i += blockDim.x) put(i, i < R ? ldf(kv + i) * ik * kv_gamma[i] : turned(i));
 }
 
 // One block per token: query heads rotated in place, keys assembled.
@@ -1183,13 +1197,12 @@ cudaError_t launch_mla_prepare(bool f32, const SeqBatch& sb, const void* y, int6
                                const float* q_gamma, const float* kv_gamma, float eps, const RopeTable& rope,
                                const PagedRows& pages, void* cq, void* lat, int* status, cudaStream_t st) {
   const int th = threads_for(q_rank + R + dr);
-  if (f32)
-    mla_prepare_kernel<float><<<sb.n_tok, th, 0, st>>>(sb, static_cast<const float*>(y), ldy, q_rank, R, dr, q_gamma, kv_gamma,
-                                                       eps, rope, pages, static_cast<float*>(cq), static_cast<float*>(lat), status);
-  else
-    mla_prepare_kernel<__nv_bfloat16><<<sb.n_tok, th, 0, st>>>(sb, static_cast<const __nv_bfloat16*>(y), ldy, q_rank, R, dr, q_gamma,
-                                                               kv_gamma, eps, rope, pages, static_cast<__nv_bfloat16*>(cq),
-                                                               static_cast<__nv_bfloat16*>(lat), status);
+#define B200_MLA(T, HOLD)                                                                                                                       \
+  mla_prepare_kernel<T, HOLD><<<sb.n_tok, th, 0, st>>>(sb, static_cast<const T*>(y), ldy, q_rank, R, dr, q_gamma, kv_gamma, eps, rope, pages, \
+                                                       static_cast<T*>(cq), static_cast<T*>(lat), status)
+  if (sb.n_tok <= 64) { if (f32) B200_MLA(float, 8); else B200_MLA(__nv_bfloat16, 8); }
+  else { if (f32) B200_MLA(float, 0); else B200_MLA(__nv_bfloat16, 0); }
+#undef B200_MLA
   return cudaGetLastError();
 }
 

@@ -7,6 +7,7 @@
     python -m jax_gpt_b200.utils.kernel_bench --op ssd_scan --B 2 --T 4096 --H 64
     python -m jax_gpt_b200.utils.kernel_bench --op gated_scan | decay_scan | channel_scan --B 2 --T 4096 --H 16
     python -m jax_gpt_b200.utils.kernel_bench --op gated_lru --B 2 --T 4096 --H 16
+    python -m jax_gpt_b200.utils.kernel_bench --op capped_attention | pooled_attention --B 2 --T 4096 --H 16
     python -m jax_gpt_b200.utils.kernel_bench --op gdn_prep_fwd | gdn_prep_bwd | gdn_prefill --B 1 --T 4096
 
 Each run does ``--warmup`` untimed launches, then times ``--iters`` launches with CUDA events on
@@ -216,6 +217,26 @@ def main(argv=None):
         fn = lambda: ssm.ssd_scan(batch, xbc, dt, db, al, dk, state, G)
         bytes_ = 2.0 * B * T * (C + H * 64 + H) + 4.0 * state.numel()
         flops = B * T / 128 * H * 2.0 * 128 * (128 * 128 + 3 * 128 * 64)
+    elif args.op in ("capped_attention", "pooled_attention"):
+        # --B sequences of --T tokens, --H query heads of 128 over --H / 8 kv heads: scores under a soft cap of 50, or a window of 1024
+        # and the means of blocks of 16 before it, with a sink
+        from ..cache.paged import PagedCache
+        from ..ops import window_attention as WA
+        from ..ops.mixed_kv import mixed_kv
+        from .serve_bench import _start_batch
+        B, T, H, G, W, P = args.B, args.T, args.H, max(1, args.H // 8), 1024, 16
+        pooled = args.op == "pooled_attention"
+        batch = _start_batch(list(range(B)), [T] * B, 0, dev, T)
+        per = (T + 63) // 64
+        cache = PagedCache(1, [2 * G * 128], B * per, 64, B, per, torch.bfloat16, dev, blocks=[P if pooled else 0])
+        for i in range(B):
+            cache.reserve(i, T)
+        y = torch.randn(B * T, (H + 2 * G) * 128, device=dev).to(torch.bfloat16)
+        q, k, v = mixed_kv(batch, y, (0, H * 128, (H + G) * 128), H, G, 128, 128, cache, 0, (128, 128), window=W)
+        sink = torch.randn(H, device=dev)
+        fn = lambda: WA.flash_prompts(batch, q, k, v, 0.09, W, sink=sink, pool=P) if pooled else WA.flash_prompts(batch, q, k, v, 0.09, softcap=50.0)
+        seen = sum(min(i + 1, W) + max(0, i - W + 1) // P for i in range(T)) if pooled else T * (T + 1) / 2
+        flops, bytes_ = B * H * seen * 4.0 * 128, 0.0
     elif args.op == "gated_lru":
         # --B sequences of --T tokens, --H gate blocks of 128 channels, four taps
         from ..ops.gated_lru import LruWeights, gated_lru

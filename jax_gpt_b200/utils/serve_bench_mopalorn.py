@@ -154,12 +154,12 @@ def kernel_table(dev, width: int = 2048, seqs: int = 2, seq_len: int = 4096, dec
         last = _start_batch(list(range(B)), [1] * B, ctx - 1, dev, ctx + 1)     # the step that completes a block
         put(d, "value mixing, cache write, a block's mean", tm(lambda: mix(last, yq1, vf1, block_pages, None, None), 2.0 * B * K * (2 * H + 5 * G + 2 * G * (pool + 1))), rot1,
             "bias, rotation of q k v, cache write")
-        xb, hb, yo = rn(B, D), rn(B, ff), torch.empty(B, ff, device=dev, dtype=BF)
-        lin = tm(lambda: linear_rows(xb, w_up), 2.0 * w_up.numel())
-        for name, fn, w in (("projection q latent gate", lambda: linear_rows(xb, w_in), w_in), ("projection q k v", lambda: linear_rows(xb, w_g), w_g),
-                            ("feed-forward up with its activation", lambda: linear_rows(xb, w_up, **xielu), w_up), ("feed-forward down", lambda: linear_rows(hb, w_dn), w_dn)):
-            put(d, name, tm(fn, 2.0 * w.numel()), lin, "the few-row kernel to the feed-forward's width, no activation")
-        del yo
+        xb, hb = rn(B, D), rn(B, ff)
+        for name, fn, w, x in (("projection q latent gate", lambda: linear_rows(xb, w_in), w_in, xb), ("projection q k v", lambda: linear_rows(xb, w_g), w_g, xb),
+                               ("feed-forward up with its activation", lambda: linear_rows(xb, w_up, **xielu), w_up, xb),
+                               ("feed-forward down", lambda: linear_rows(hb, w_dn), w_dn, hb)):
+            yo = torch.empty(B, w.shape[0], device=dev, dtype=BF)
+            put(d, name, tm(fn, 2.0 * w.numel()), tm(lambda: gemm(x, w, out=yo), 2.0 * w.numel()), "tcgen05 GEMM of the same size, no activation")
     _ext.check_status(dev)
     return out
 
