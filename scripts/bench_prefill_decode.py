@@ -10,7 +10,7 @@ that fits (doubling then bisection on out-of-memory, ``--max-batch`` caps it), t
 Timing is on the device with CUDA events, maximum over ranks (the reference uses host
 perf_counter and means only, scripts/bench_prefill_decode.py:246-264). ``--model`` selects the
 Qwen3.5 hybrid (``--config`` preset), the DeepSeek-V3 shape with its paged latent cache or Vobunex /
-Fovudra / Munazen on the shared step engine.
+Fovudra / Munazen / Mopalorn on the shared step engine.
 Results are printed and written as JSON to ``--out``.
 """
 from __future__ import annotations

@@ -134,7 +134,7 @@ def test_whole_prompts_with_many_blocks(d, dv, size, P, lens):
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 1e-4), (torch.bfloat16, 1.0)])
 def test_activation(dtype, tol):
     from jax_gpt_b200.ops.gemm import linear_rows
-    K.check_activation(linear_rows, DEV, dtype, tol, ((1, 64, 40), (3, 33, 9), (8, 256, 128), (20, 128, 72), (300, 256, 384), (1000, 512, 1024), (70, 21, 10)))
+    K.check_activation(linear_rows, DEV, dtype, tol, ((1, 64, 40), (3, 33, 9), (8, 256, 128), (20, 128, 72), (300, 256, 384), (1000, 512, 1024), (70, 21, 10), (100, 64, 77), (257, 128, 200)))
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
